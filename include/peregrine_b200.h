@@ -348,6 +348,8 @@ PG_API int32_t pg_embedding(pg_ctx *ctx, const float *d_table, const int32_t *d_
                             float *d_out);
 PG_API int32_t pg_argmax_advance(pg_ctx *ctx, const float *d_logits, int64_t B, int64_t V, int32_t *d_tokens,
                                  int32_t *d_pos, int64_t pos_limit);
+/* The same with one position per row: d_pos [B] (nullable). */
+PG_API int32_t pg_argmax_rows(pg_ctx *ctx, const float *d_logits, int64_t B, int64_t V, int32_t *d_tokens, int32_t *d_pos, int64_t pos_limit);
 /* ---- the same step with every linear sharded by output column over the ranks of a node (one process per GPU):
  *      whole KV heads with their query heads per rank (fuse_qkv's column order, src/models/llama/attention.rs:51-71,
  *      regrouped per rank), the same channel range of gate and up per rank (src/models/llama/decoder.rs:49-67), the

@@ -1,4 +1,5 @@
-"""ctypes binding of libperegrine_b200.so (the declarations of include/peregrine_b200.h).
+"""ctypes bindings of libperegrine_b200.so (the declarations of include/peregrine_b200.h) and of
+libperegrine_b200_lm.so (include/peregrine_b200_lm.h, with the shared part of the first header).
 
 There is no fallback of any kind: if the library is missing, cannot be loaded, or a call
 fails, an exception is raised.
@@ -10,6 +11,7 @@ import os
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "lib", "libperegrine_b200.so")
+LIB_LM_PATH = os.path.join(_HERE, "lib", "libperegrine_b200_lm.so")
 
 PG_OK = 0
 PG_ERR_INVALID = -1
@@ -118,6 +120,7 @@ SIGNATURES = {
     "pg_gqa_attention_decode_fused": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _vp]),
     "pg_embedding": (_i32, [_vp, _vp, _vp, _i64, _i64, _vp]),
     "pg_argmax_advance": (_i32, [_vp, _vp, _i64, _i64, _vp, _vp, _i64]),
+    "pg_argmax_rows": (_i32, [_vp, _vp, _i64, _i64, _vp, _vp, _i64]),
     "pg_matmul_f32": (_i32, [_vp, _vp, _vp, _i64, _i64, _i64, _vp]),
 }
 
@@ -141,38 +144,82 @@ TUNE_SIGNATURES = {
     "pg_huffman_last_sweeps": (_int, []),
 }
 
-_lib = None
+# ---- libperegrine_b200_lm.so ----
+F32, BF16 = 0, 1
+ACT_NONE, ACT_GELU_TANH_GLU, ACT_CLAMPED_SWISH_GLU = 0, 1, 2
 
 
-def load() -> C.CDLL:
-    """Loads the shared library (building it first if the sources are newer and nvcc exists)."""
-    global _lib
-    if _lib is not None:
-        return _lib
-    if not os.path.exists(LIB_PATH):
+class PgBatch(C.Structure):
+    _fields_ = [("rows", _i32), ("seqs", _i32), ("max_len", _i32), ("d_tokens", _vp), ("d_pos", _vp), ("d_row_seq", _vp), ("d_seq_row0", _vp),
+                ("d_seq_slot", _vp)]
+
+
+class PgDelta(C.Structure):
+    _fields_ = [("heads", _i32), ("kv_heads", _i32), ("dim", _i32), ("vdim", _i32), ("taps", _i32), ("eps", C.c_float), ("unit_eps", C.c_float),
+                ("d_conv", _vp), ("d_a_log", _vp), ("d_dt_bias", _vp), ("d_norm", _vp), ("d_work", _vp)]
+
+
+class PgAttention(C.Structure):
+    _fields_ = [("heads", _i32), ("kv_heads", _i32), ("dim", _i32), ("vdim", _i32), ("cap", _i32), ("eps", C.c_float), ("scale", C.c_float),
+                ("temp_coef", C.c_float), ("temp_every", C.c_float), ("sink", _i32), ("d_q_norm", _vp), ("d_k_norm", _vp), ("d_q", _vp), ("d_part", _vp),
+                ("d_tickets", _vp)]
+
+
+_pb, _pd, _pa = C.POINTER(PgBatch), C.POINTER(PgDelta), C.POINTER(PgAttention)
+_f = C.c_float
+LM_SIGNATURES = {
+    "pg_linear_wrap": (_i32, [_vp, _vp, _i64, _i64, _i64, C.POINTER(_vp)]),
+    "pg_linear_free": (_i32, [_vp, _vp]),
+    "pg_linear_run": (_i32, [_vp, _vp, _vp, _i32, _i64, _i32, _f, _vp, _i32, _i64]),
+    "pg_linear_run_routed": (_i32, [_vp, _vp, _vp, _vp, _i32, _i32, _i32, _f, _vp, _i32, _i64]),
+    "pg_route_create": (_i32, [_vp, _i64, _i64, _i64, _i64, C.POINTER(_vp)]),
+    "pg_route_free": (_i32, [_vp, _vp]),
+    "pg_route_max_rows": (_i64, [_vp]),
+    "pg_route_run": (_i32, [_vp, _vp, _i32, _vp, _i64, _i64, _vp, _i32, _i32]),
+    "pg_route_read": (_i32, [_vp, _vp, _vp, _vp]),
+    "pg_embed_norm": (_i32, [_vp, _pb, _vp, _vp, _i64, _vp, _f, _vp, _vp, _i32, _i64]),
+    "pg_norm_add": (_i32, [_vp, _vp, _i64, _vp, _vp, _vp, _i64, _i64, _f, _vp, _i32, _i64]),
+    "pg_routed_norm_add": (_i32, [_vp, _vp, _vp, _i64, _vp, _vp, _vp, _i64, _i64, _f, _vp, _i32, _i64]),
+    "pg_norm_rows": (_i32, [_vp, _vp, _vp, _i64, _i64, _vp, _f, _vp, _i32, _i64]),
+    "pg_delta_work_floats": (_i64, [_pd, _i64]),
+    "pg_delta_run": (_i32, [_vp, _pd, _pb, _vp, _i64, _vp, _vp, _vp, _i32, _i64]),
+    "pg_attention_part_floats": (_i64, [_vp, _pa, _i64]),
+    "pg_attention_run": (_i32, [_vp, _pa, _pb, _vp, _i64, _vp, _vp, _vp, _i32, _i64]),
+}
+# what both libraries carry (csrc/pg_core.cu, csrc/pg_sample.cu)
+CORE = [n for n in SIGNATURES if n.startswith(("pg_ctx_", "pg_graph_", "pg_mem_"))] + ["pg_last_error", "pg_version", "pg_launch_count",
+                                                                                      "pg_argmax_advance", "pg_argmax_rows"]
+COMPONENTS = {"int8": (LIB_PATH, {**SIGNATURES, **TUNE_SIGNATURES}), "lm": (LIB_LM_PATH, {**{n: SIGNATURES[n] for n in CORE}, **LM_SIGNATURES})}
+
+_libs = {}
+
+
+def load(component: str = "int8") -> C.CDLL:
+    """Loads a shared library, building it first if it does not exist yet."""
+    if component in _libs:
+        return _libs[component]
+    path, signatures = COMPONENTS[component]
+    if not os.path.exists(path):
         from . import build as _build
 
-        _build.build()
+        _build.build(component)
     try:
-        lib = C.CDLL(LIB_PATH)
+        lib = C.CDLL(path)
     except OSError as e:  # loud, never silent
-        raise ImportError(f"cannot load {LIB_PATH}: {e}. Build it with `python -m peregrine_b200.build`.") from e
-    for name, (res, args) in SIGNATURES.items():
+        raise ImportError(f"cannot load {path}: {e}. Build it with `python -m peregrine_b200.build`.") from e
+    for name, (res, args) in signatures.items():
         fn = getattr(lib, name)
         fn.restype = res
         fn.argtypes = args
-    for name, (res, args) in TUNE_SIGNATURES.items():
-        fn = getattr(lib, name)
-        fn.restype = res
-        fn.argtypes = args
-    _lib = lib
+    _libs[component] = lib
     return lib
 
 
-def check(code: int) -> None:
+def check(code: int, lib: C.CDLL = None) -> None:
+    """Raises the error of a call into `lib` (default: libperegrine_b200.so)."""
     if code == PG_OK:
         return
-    msg = load().pg_last_error().decode("utf-8", "replace")
+    msg = (lib or load()).pg_last_error().decode("utf-8", "replace")
     if code == PG_ERR_INVALID:
         raise InvalidArgument(code, msg)
     raise PeregrineError(code, msg)

@@ -432,6 +432,8 @@ int32_t pgk_gemm_i8_wstream(pg_ctx *ctx, const int8_t *d_a, const float *d_as, i
 // the same product with its outputs stored into every rank's exchange buffer and the exchange published by the kernel
 int32_t pgk_gemm_i8_wstream_peer(pg_ctx *ctx, const int8_t *d_a, const float *d_as, int64_t m, int64_t k, const int8_t *d_bt,
                                  const float *d_ws, int64_t n, const PgPeerOut &out);
+// pg_sample.cu
+int32_t pgk_argmax_peer(pg_ctx *ctx, const float *d_logits, int64_t B, int64_t V, int v0, const PgPeerOut &out);
 // pg_llama_attn.cu
 int pgk_gqa_stream_splits(const pg_ctx *ctx, int64_t B, int64_t Hkv, int64_t cap);
 bool pgk_gqa_stream_supports(int64_t G);

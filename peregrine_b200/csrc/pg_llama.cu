@@ -12,13 +12,14 @@
 //   gqa_decode_*_kernel        GQA attention of one new token against the cache
 //                              (src/attention.rs:141-265: dot * 1/sqrt(hd), softmax, weighted sum of V),
 //                              split over the context so that all SMs stream the cache, then combined
-//   embedding / argmax         src/nn.rs:217-227, examples/llama/main.rs:15-26 (first maximum wins)
+//   embedding                  src/nn.rs:217-227 (the greedy choice is in csrc/pg_sample.cu)
 //
 // Everything is batched over independent sequences (one row per sequence); the position lives in
 // device memory so that a whole step can be recorded once and replayed.  f32 sums here run in a
 // different order from the reference's sequential loops, so this layer is checked to a tolerance, not
 // bit for bit (the linears inside it stay bit-exact for the activations they are given).
 #include "pg_internal.cuh"
+#include "pg_launch.cuh"
 
 namespace {
 
@@ -350,81 +351,6 @@ __global__ void embedding_kernel(const float *__restrict__ table, const int *__r
     for (int i = threadIdx.x; i < (dim >> 2); i += blockDim.x) dst[i] = __ldg(src + i);
 }
 
-// a cluster of cs CTAs per row, each scanning V / cs logits; the first maximum wins (examples/llama/main.rs:15-26).
-// The first CTA of row 0 also advances the position.
-// PEER (po.world > 0): `logits` holds this rank's V columns of a vocabulary sharded by column; the row's local
-// (maximum, index + v0) pair goes to slot [b][rank] of every rank's exchange buffer instead of tokens[b], and
-// pick_embed_kernel chooses among the ranks' pairs.
-__global__ void __launch_bounds__(1024) argmax_kernel(const float *__restrict__ logits, int V, int *__restrict__ tokens, int *pos_ptr,
-                                                       int pos_limit, int v0, const PgPeerOut po)
-{
-    __shared__ float bv[32];
-    __shared__ int bi[32];
-    __shared__ float xv[8];
-    __shared__ int xi[8];
-    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-    asm volatile("griddepcontrol.wait;" ::: "memory");
-    const uint32_t cs = cl_size(), rank = cl_rank();
-    const int b = blockIdx.x / cs;
-    const float *row = logits + (int64_t)b * V;
-    const int seg = (V + (int)cs - 1) / (int)cs;
-    const int i0 = (int)rank * seg, i1 = min(V, i0 + seg);
-    float best = -INFINITY;
-    int idx = 0x7fffffff;
-    for (int i = i0 + threadIdx.x; i < i1; i += blockDim.x) {
-        const float v = pg_ld_fresh(row + i);
-        if (v > best || (v == best && i < idx)) {
-            best = v;
-            idx = i;
-        }
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-        const int oi = __shfl_xor_sync(0xffffffffu, idx, o);
-        if (ov > best || (ov == best && oi < idx)) {
-            best = ov;
-            idx = oi;
-        }
-    }
-    if ((threadIdx.x & 31) == 0) {
-        bv[threadIdx.x >> 5] = best;
-        bi[threadIdx.x >> 5] = idx;
-    }
-    __syncthreads();
-    if (threadIdx.x == 0) {
-        for (int w = 1; w < (int)(blockDim.x >> 5); w++)
-            if (bv[w] > best || (bv[w] == best && bi[w] < idx)) {
-                best = bv[w];
-                idx = bi[w];
-            }
-        if (cs > 1) {
-            cl_store_f32(xv + rank, 0, best);     // everything meets in the first CTA of the cluster
-            cl_store_s32(xi + rank, 0, idx);
-        }
-    }
-    if (cs > 1) cl_sync();
-    if (threadIdx.x == 0 && rank == 0) {
-        for (uint32_t c = 1; c < cs; c++)
-            if (xv[c] > best || (xv[c] == best && xi[c] < idx)) {
-                best = xv[c];
-                idx = xi[c];
-            }
-        if (po.world > 0) {
-            // an all-NaN (or empty) slice never wins: -inf with the slice's first index
-            pg_cell_store2(po, pg_cell_seq(po), b, 0, (idx == 0x7fffffff) ? -INFINITY : best,
-                           __int_as_float((idx == 0x7fffffff) ? v0 : idx + v0));
-        } else {
-            tokens[b] = (idx == 0x7fffffff) ? 0 : idx;   // all-NaN row: the reference keeps index 0
-            if (b == 0 && pos_ptr) {
-                const int p = pg_ld_fresh(pos_ptr);
-                if (pos_limit <= 0 || p < pos_limit) *pos_ptr = p + 1;   // never past the end of the cache
-            }
-        }
-    }
-    if (po.world > 0) pg_cell_finish(po, pg_cell_seq(po), threadIdx.x);
-}
-
 // One CTA per sequence: waits for every rank's (maximum, index) pair of the sharded vocabulary, takes the first
 // maximum in index order (ranks own ascending column ranges, so rank order is index order; strict '>' as in
 // examples/llama/main.rs:15-26), stores the token, advances the position (CTA 0) and gathers the token's embedding
@@ -586,55 +512,6 @@ __global__ void __launch_bounds__(1024) gqa_combine_quant_kernel(const float *__
     const float inv = __fdiv_rn(1.0f, scale);
     if (tid == 0 && rank == 0) q8_scales[b] = scale;
     q8[at] = (int8_t)pg_round_clamp_i8(__fmul_rn(o, inv));
-}
-
-template <typename K, typename... Args>
-int32_t launch_pdl_cluster(pg_ctx *ctx, K kern, dim3 grid, dim3 block, size_t smem, int cs, Args... args)
-{
-    cudaLaunchAttribute attr[2];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
-    attr[1].id = cudaLaunchAttributeClusterDimension;
-    attr[1].val.clusterDim.x = (unsigned)cs;
-    attr[1].val.clusterDim.y = 1;
-    attr[1].val.clusterDim.z = 1;
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = grid;
-    cfg.blockDim = block;
-    cfg.dynamicSmemBytes = smem;
-    cfg.stream = ctx->stream;
-    cfg.attrs = attr;
-    cfg.numAttrs = cs > 1 ? 2 : 1;
-    PG_CUDA(cudaLaunchKernelEx(&cfg, kern, args...));
-    PG_LAUNCHED();
-    return PG_OK;
-}
-
-// CTAs per row for the row kernels: as many (up to 8) as keep the grid within about two CTAs per SM, divide the row's
-// `units` evenly and leave each CTA at least `min_units`.
-int row_cluster(const pg_ctx *ctx, int64_t rows, int64_t units, int64_t min_units)
-{
-    int cs = 8;
-    while (cs > 1 && (rows * cs > 2 * (int64_t)ctx->sm_count || units % cs != 0 || units / cs < min_units)) cs >>= 1;
-    return cs;
-}
-
-template <typename K, typename... Args>
-int32_t launch_pdl(pg_ctx *ctx, K kern, dim3 grid, dim3 block, size_t smem, Args... args)
-{
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = grid;
-    cfg.blockDim = block;
-    cfg.dynamicSmemBytes = smem;
-    cfg.stream = ctx->stream;
-    cfg.attrs = attr;
-    cfg.numAttrs = 1;
-    PG_CUDA(cudaLaunchKernelEx(&cfg, kern, args...));
-    PG_LAUNCHED();
-    return PG_OK;
 }
 
 }  // namespace
@@ -851,19 +728,6 @@ PG_API int32_t pg_embedding(pg_ctx *ctx, const float *d_table, const int32_t *d_
     return launch_pdl(ctx, embedding_kernel, dim3((unsigned)B), dim3(256), 0, d_table, (const int *)d_tokens, (int)dim, d_out);
 }
 
-// tokens[b] = argmax(logits[b, :]) (first maximum); d_pos (nullable) is advanced by one, but never beyond pos_limit
-// (pass the KV capacity; 0 = no limit): a decode loop that runs off the end of its cache stops advancing instead of
-// writing behind it.
-PG_API int32_t pg_argmax_advance(pg_ctx *ctx, const float *d_logits, int64_t B, int64_t V, int32_t *d_tokens, int32_t *d_pos, int64_t pos_limit)
-{
-    PG_ENTER(ctx);
-    PG_REQUIRE(d_logits && d_tokens && V > 0 && V <= 0x7fffffff, "argmax: bad arguments");
-    if (B == 0) return PG_OK;
-    const int cs = row_cluster(ctx, B, V, 4096);
-    return launch_pdl_cluster(ctx, argmax_kernel, dim3((unsigned)(B * cs)), dim3(1024), 0, cs, d_logits, (int)V, (int *)d_tokens, (int *)d_pos,
-                              (int)pos_limit, 0, NO_PEER_OUT);
-}
-
 // Greedy choice over a vocabulary sharded by column: this rank's [B, V_local] logits cover columns [v0, v0 + V_local).
 // Its per-sequence (maximum, index) pair (8 bytes) goes to every rank's exchange buffer ([B][world][2] floats, the
 // index as its bit pattern); pg_pick_embed then chooses.
@@ -874,9 +738,7 @@ PG_API int32_t pg_argmax_exchange(pg_ctx *ctx, const float *d_logits_local, int6
                "argmax_exchange: bad arguments");
     PG_REQUIRE((size_t)B * ex->world * 2 * sizeof(float) <= ex->y_bytes, "argmax_exchange: the exchange buffer is smaller than [B][world][2] floats");
     if (B == 0) return PG_OK;
-    const int cs = row_cluster(ctx, B, V_local, 1024);
-    return launch_pdl_cluster(ctx, argmax_kernel, dim3((unsigned)(B * cs)), dim3(1024), 0, cs, d_logits_local, (int)V_local, (int *)nullptr,
-                              (int *)nullptr, 0, (int)v0, pg_peer_out(ex, (int64_t)ex->world * 2, (int64_t)ex->rank * 2));
+    return pgk_argmax_peer(ctx, d_logits_local, B, V_local, (int)v0, pg_peer_out(ex, (int64_t)ex->world * 2, (int64_t)ex->rank * 2));
 }
 
 // Waits (bounded) for every rank's pair, stores tokens[b] = the first maximum over the whole vocabulary, advances

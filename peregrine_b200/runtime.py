@@ -38,7 +38,7 @@ class GpuBuffer:
         self.dtype = np.dtype(dtype)
         self.count = int(count)
         out = C.c_void_p()
-        _lib.check(ctx.lib.pg_mem_alloc(ctx.handle, self.nbytes, C.byref(out)))
+        ctx.check(ctx.lib.pg_mem_alloc(ctx.handle, self.nbytes, C.byref(out)))
         self.ptr = out.value or 0
 
     @property
@@ -48,18 +48,18 @@ class GpuBuffer:
     def write(self, host: np.ndarray) -> None:
         host = np.ascontiguousarray(host, self.dtype)
         assert host.size == self.count
-        _lib.check(self.ctx.lib.pg_mem_upload(self.ctx.handle, self.ptr, _ptr(host), self.nbytes))
+        self.ctx.check(self.ctx.lib.pg_mem_upload(self.ctx.handle, self.ptr, _ptr(host), self.nbytes))
         # the source array may be a temporary: make the copy complete before it can be freed
         self.ctx.sync()
 
     def read(self) -> np.ndarray:
         out = np.empty(self.count, self.dtype)
-        _lib.check(self.ctx.lib.pg_mem_download(self.ctx.handle, _ptr(out), self.ptr, self.nbytes))
+        self.ctx.check(self.ctx.lib.pg_mem_download(self.ctx.handle, _ptr(out), self.ptr, self.nbytes))
         return out
 
     def free(self) -> None:
         if self.ptr:
-            _lib.check(self.ctx.lib.pg_mem_free(self.ctx.handle, self.ptr))
+            self.ctx.check(self.ctx.lib.pg_mem_free(self.ctx.handle, self.ptr))
             self.ptr = 0
 
     def __del__(self):
@@ -71,14 +71,18 @@ class GpuBuffer:
 
 class GpuContext:
     """One CUDA device + stream.  `stream` may be a raw cudaStream_t (int) to share, e.g.
-    `torch.cuda.current_stream().cuda_stream`."""
+    `torch.cuda.current_stream().cuda_stream`.  `component`: the library the context belongs to, "int8"
+    (the quantised path) or "lm" (the bf16 / f32 language models)."""
 
-    def __init__(self, device: int = 0, stream: Optional[int] = None):
-        self.lib = _lib.load()
+    def __init__(self, device: int = 0, stream: Optional[int] = None, component: str = "int8"):
+        self.lib = _lib.load(component)
         h = C.c_void_p()
-        _lib.check(self.lib.pg_ctx_create(int(device), C.c_void_p(stream or 0), C.byref(h)))
+        self.check(self.lib.pg_ctx_create(int(device), C.c_void_p(stream or 0), C.byref(h)))
         self.handle = h
         self.device = int(device)
+
+    def check(self, code: int) -> None:
+        _lib.check(code, self.lib)
 
     # GpuContext::alloc / upload / sync
     def alloc(self, count: int, dtype=np.float32) -> GpuBuffer:
@@ -91,7 +95,7 @@ class GpuContext:
         return buf
 
     def sync(self) -> None:
-        _lib.check(self.lib.pg_ctx_sync(self.handle))
+        self.check(self.lib.pg_ctx_sync(self.handle))
 
     @property
     def stream(self) -> int:
@@ -99,7 +103,7 @@ class GpuContext:
 
     def device_status(self) -> int:
         v = C.c_int32(0)
-        _lib.check(self.lib.pg_ctx_device_status(self.handle, C.byref(v)))
+        self.check(self.lib.pg_ctx_device_status(self.handle, C.byref(v)))
         return v.value
 
     # batched submission (CUDA graph): `with gpu.record() as g: ...` then `g.launch()`
@@ -129,20 +133,20 @@ class Graph:
 
     def __enter__(self):
         self._n0 = self.ctx.lib.pg_launch_count()
-        _lib.check(self.ctx.lib.pg_graph_begin(self.ctx.handle))
+        self.ctx.check(self.ctx.lib.pg_graph_begin(self.ctx.handle))
         return self
 
     def __exit__(self, exc_type, exc, tb):
         h = C.c_void_p()
         rc = self.ctx.lib.pg_graph_end(self.ctx.handle, C.byref(h))
         if exc_type is None:
-            _lib.check(rc)
+            self.ctx.check(rc)
             self.handle = h
             self.kernels = int(self.ctx.lib.pg_launch_count() - self._n0)
         return False
 
     def launch(self) -> None:
-        _lib.check(self.ctx.lib.pg_graph_launch(self.ctx.handle, self.handle))
+        self.ctx.check(self.ctx.lib.pg_graph_launch(self.ctx.handle, self.handle))
 
     def free(self) -> None:
         if self.handle is not None and self.ctx.handle:
