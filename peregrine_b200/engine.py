@@ -2,19 +2,19 @@
 makes of them, and greedy generation.
 
 A step runs the next tokens of one or more requests.  `Engine.step` takes exactly what it is given (a trace);
-`Engine.generate` schedules: waiting prompts are run in portions of at most `portion` tokens as slots come free, and all
-sequences whose prompt is done decode together.  Decoding is one recorded graph per number of sequences, replayed; the
-greedy choice, the next tokens and the positions stay on the device.
+`Engine.generate` schedules: waiting prompts get slots as they come free; while a prompt is unfinished, a step carries the
+next token of every running sequence and portions of prompts, at most `portion` tokens in all; otherwise all sequences
+decode together, as one recorded graph per number of sequences, replayed, in which the greedy choice, the next tokens and
+the positions stay on the device (peregrine_b200/slot_model.py).
 """
 from __future__ import annotations
 
-import ctypes as C
 from dataclasses import dataclass, field
 from typing import Dict, Hashable, List, Optional, Sequence, Tuple
 
 import numpy as np
 
-from .layers import Batch
+from .state import OutOfSlots
 
 
 class RequestError(ValueError):
@@ -42,54 +42,15 @@ class Generation:
         return len(self.out) >= self.max_new or (bool(self.out) and self.out[-1] in self.stop)
 
 
-class _Decode:
-    """The recorded decode step of `n` sequences."""
-
-    def __init__(self, model, n: int):
-        self.model, self.n = model, n
-        self.batch = Batch(model.d, [(0, 0, [0])] * n, list(range(n)), fixed=True)
-        self.graph = None
-        self.keys: Optional[Tuple] = None     # the sequences whose tokens and positions the device arrays hold
-
-    def load(self, entries) -> None:
-        n = self.n
-        host = np.zeros(6 * n + 1, np.int32)
-        host[:n] = [e[2] for e in entries]
-        host[n:2 * n] = [e[1] for e in entries]
-        host[2 * n:3 * n] = np.arange(n)
-        host[3 * n:4 * n + 1] = np.arange(n + 1)
-        host[4 * n + 1:5 * n + 1] = [e[0] for e in entries]
-        host[5 * n + 1:] = np.arange(n)
-        self.batch.write(host)
-
-    def enqueue(self) -> None:
-        m, b = self.model, self.batch
-        m.forward(b)
-        m.head_rows(b.d_wanted, self.n)
-        m.d.check(m.lib.pg_argmax_rows(m.gpu.handle, m.logits.data_ptr(), self.n, m.vocab, b.d_tokens, b.d_pos, m.capacity))
-
-    def run(self) -> None:
-        """One step from what the device arrays hold."""
-        m = self.model
-        if self.graph is None:
-            with m.gpu.record() as g:
-                self.enqueue()
-            self.graph = g
-        self.graph.launch()
-
-    def tokens(self) -> np.ndarray:
-        out = np.empty(self.n, np.int32)
-        m = self.model
-        m.gpu.check(m.lib.pg_mem_download(m.gpu.handle, out.ctypes.data, self.batch.d_tokens, out.nbytes))
-        return out
-
-
 class Engine:
     def __init__(self, model, portion: int = 0):
         self.model = model
-        self.portion = min(int(portion or model.step_rows), model.step_rows)
+        # a step has room for the next tokens of all slots and some of a prompt
+        self.portion = max(min(int(portion or model.step_rows), model.step_rows), min(model.pool.slots + 1, model.step_rows))
+        self._runs = 0
         self.live: Dict[Hashable, Live] = {}
-        self._decode: Dict[int, _Decode] = {}
+        self._decoders: Dict[int, object] = {}
+        self._loaded: Dict[int, tuple] = {}     # the sequences whose next tokens a decoder's device arrays hold
 
     # ---- requests ------------------------------------------------------------------------------------------------
     def _request(self, key) -> Live:
@@ -125,7 +86,9 @@ class Engine:
             self._check_tokens(key, known or Live(-1), tokens)
             if any(not 0 <= w < len(tokens) for w in want):
                 raise RequestError(f"request {key!r}: a wanted place outside its tokens")
-        out, parts = [], []
+        if len(seen - set(self.live)) > self.model.pool.free:
+            raise OutOfSlots(f"{len(seen - set(self.live))} new requests, {self.model.pool.free} free slots")
+        out = []
         # rows of one step are limited: what does not fit follows in further steps
         todo = [[key, self._request(key), list(tokens), sorted(set(want)), 0] for key, tokens, want in entries]
         got: Dict[Tuple[Hashable, int], np.ndarray] = {}
@@ -144,7 +107,7 @@ class Engine:
                         wanted.append(at + w - lo)
                         rows.append((item[0], w))
                 at += n
-            self._run([(item[1].slot, item[1].length, item[2][lo:lo + n]) for item, lo, n in parts], wanted, rows, got)
+            got.update(zip(rows, self.model.run([(item[1].slot, item[1].length, item[2][lo:lo + n]) for item, lo, n in parts], wanted)))
             for item, lo, n in parts:
                 item[1].length += n
                 item[4] = lo + n
@@ -153,27 +116,12 @@ class Engine:
             out += [got[(key, w)] for w in want]
         return np.stack(out) if out else np.zeros((0, self.model.vocab), np.float32)
 
-    def _run(self, entries, wanted, names, got) -> None:
-        m = self.model
-        batch = Batch(m.d, entries, wanted)
-        m.forward(batch)
-        for i in range(0, len(wanted), m.max_wanted):
-            n = min(m.max_wanted, len(wanted) - i)
-            m.head_rows(batch.d_wanted + 4 * i, n)
-            for name, row in zip(names[i:i + n], m.read_logits(n)):
-                got[name] = row.copy()
-        self.check_device()
-
-    def check_device(self) -> None:
-        status = self.model.gpu.device_status()
-        if status:
-            raise RuntimeError(f"a kernel reported status {status}")
-
     # ---- generation ----------------------------------------------------------------------------------------------
     def generate(self, prompts: Sequence[Sequence[int]], max_new: int, stop: Sequence[int] = ()) -> List[List[int]]:
         """Greedy continuation of every prompt (token ids): at most max_new tokens each, up to and including a stop token."""
         m = self.model
-        jobs = [Generation(list(p), int(max_new), frozenset(stop), key=("generate", id(self), i)) for i, p in enumerate(prompts)]
+        self._runs += 1
+        jobs = [Generation(list(p), int(max_new), frozenset(stop), key=("generate", self._runs, i)) for i, p in enumerate(prompts)]
         for j in jobs:
             self._check_tokens(j.key, Live(-1), j.prompt)
             # the last new token is not run
@@ -188,7 +136,7 @@ class Engine:
                     self._request(j.key)
                     prefilling.append(j)
                 if prefilling:
-                    self._prefill(prefilling)
+                    self._mixed_step(prefilling, running)
                 else:
                     self._decode_step(running)
                 for j in [j for j in prefilling if j.fed == len(j.prompt)]:
@@ -202,50 +150,43 @@ class Engine:
                 self.end(j.key)
         return [j.out for j in jobs]
 
-    def _prefill(self, jobs: List[Generation]) -> None:
-        """One step of prompt portions; prompts that end in it get their first token."""
-        m = self.model
-        room, parts, wanted, enders, at = self.portion, [], [], [], 0
-        for j in jobs:
-            n = min(room, len(j.prompt) - j.fed)
-            if n <= 0:
+    def _mixed_step(self, prefilling: List[Generation], running: List[Generation]) -> None:
+        """One step of the running sequences' next tokens and, in the room that is left, portions of prompts; prompts that
+        end in it get their first token."""
+        parts, wanted, enders, at = [], [], [], 0
+        for j, tokens in [(j, j.out[-1:]) for j in running] + [(j, j.prompt[j.fed:]) for j in prefilling]:
+            tokens = tokens[:self.portion - at]
+            if not tokens:
                 continue
             r = self.live[j.key]
-            parts.append((r.slot, r.length, j.prompt[j.fed:j.fed + n]))
-            r.length += n
-            j.fed += n
-            room -= n
-            at += n
+            parts.append((r.slot, r.length, tokens))
+            r.length += len(tokens)
+            at += len(tokens)
+            if j.fed < len(j.prompt):
+                j.fed += len(tokens)
             if j.fed == len(j.prompt):
                 wanted.append(at - 1)
                 enders.append(j)
-        batch = Batch(m.d, parts, wanted)
-        m.forward(batch)
-        if enders:
-            n = len(enders)
-            m.head_rows(batch.d_wanted, n)
-            # the choice goes to the head of the batch's own arrays, which the step is done with
-            m.d.check(m.lib.pg_argmax_rows(m.gpu.handle, m.logits.data_ptr(), n, m.vocab, batch.d_tokens, None, 0))
-            out = np.empty(n, np.int32)
-            m.gpu.check(m.lib.pg_mem_download(m.gpu.handle, out.ctypes.data, batch.d_tokens, out.nbytes))
-            for j, t in zip(enders, out):
-                j.out.append(int(t))
-        self.check_device()
+        for j, t in zip(enders, self.model.run_greedy(parts, wanted)):
+            j.out.append(t)
 
     def _decode_step(self, jobs: List[Generation]) -> None:
         n = len(jobs)
-        d = self._decode.get(n)
+        d = self._decoders.get(n)
         if d is None:
-            d = self._decode[n] = _Decode(self.model, n)
-        keys = tuple((j.key, len(j.out)) for j in jobs)
-        if d.keys != keys:
+            d = self._decoders[n] = self.model.decoder(n)
+        if self._loaded.get(n) != tuple((j.key, len(j.out)) for j in jobs):
             d.load([(self.live[j.key].slot, self.live[j.key].length, j.out[-1]) for j in jobs])
         d.run()
         for j, t in zip(jobs, d.tokens()):
             self.live[j.key].length += 1
-            j.out.append(int(t))
-        d.keys = tuple((j.key, len(j.out)) for j in jobs)
-        self.check_device()
+            j.out.append(t)
+        self._loaded[n] = tuple((j.key, len(j.out)) for j in jobs)
+
+    def close(self) -> None:
+        for d in self._decoders.values():
+            d.free()
+        self._decoders = {}
 
 
 class LockstepEngine:

@@ -41,12 +41,16 @@ class Device:
         self._buffers = {}
 
     def f32(self, a):
-        """Host array (f32, or bf16 bits as uint16) -> f32 on the device."""
+        """Host array (f32, or bf16 bits as uint16) or torch tensor -> f32 on the device."""
+        if isinstance(a, self.torch.Tensor):
+            return a.to(self.dev).float().contiguous()
         return self.bf16(a).float().contiguous() if a.dtype == np.uint16 else self.torch.from_numpy(np.array(a, np.float32)).to(self.dev)
 
     def bf16(self, a):
-        """Host array (bf16 bits as uint16, or f32) -> bf16 on the device."""
+        """Host array (bf16 bits as uint16, or f32) or torch tensor -> bf16 on the device."""
         t = self.torch
+        if isinstance(a, t.Tensor):
+            return a.to(self.dev).to(t.bfloat16)
         if a.dtype == np.uint16:
             return t.from_numpy(np.array(a).view(np.int16)).to(self.dev).view(t.bfloat16)
         return t.from_numpy(np.array(a, np.float32)).to(self.dev).to(t.bfloat16)

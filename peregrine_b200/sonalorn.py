@@ -16,10 +16,9 @@ import os
 from dataclasses import dataclass
 from typing import Iterator, List
 
-import numpy as np
-
 from .layers import BATCH_WORDS, Attention, Batch, DenseFF, Device, GatedDelta, Linear, MoeFF, up
 from .safetensors_file import SafetensorsFile
+from .slot_model import SlotModel
 from .state import SlotPool
 
 ARCHITECTURE = "Sonalorn"
@@ -66,7 +65,7 @@ class Below:
         return self.weights[self.prefix + name]
 
 
-class SonalornModel:
+class SonalornModel(SlotModel):
     """weights: mapping name -> host array (bf16 bits as uint16, or f32, which is rounded to bf16 where a product reads it).
     slots / capacity: sequences alive at once and positions of each; step_rows: most tokens of one step; max_wanted: most
     rows of logits of one `head` call."""
@@ -74,7 +73,7 @@ class SonalornModel:
     def __init__(self, cfg: SonalornConfig, weights, gpu, dtype: str = "bfloat16", slots: int = 1, capacity: int = 0, step_rows: int = 2048,
                  max_wanted: int = 64):
         self.cfg, self.gpu, self.lib = cfg, gpu, gpu.lib
-        self.dtype, self.vocab, self.step_rows = dtype, cfg.vocab, int(step_rows)
+        self.dtype, self.vocab, self.step_rows = dtype, cfg.vocab, max(int(step_rows), slots + 1)
         d = self.d = Device(gpu, dtype, self.step_rows)
         torch = self.torch = d.torch
         f32 = torch.float32
@@ -157,21 +156,12 @@ class SonalornModel:
                 L["ff"].run(batch, h, y, add(L["norm2"], L["ls2"]))
             yield f"l{i}"
 
-    def forward(self, batch: Batch) -> None:
-        for _ in self.step_ops(batch):
-            pass
-
     def head_rows(self, d_rows: int, n: int) -> None:
         """logits[:n] of the rows of the residual stream named by n int32 at the device address d_rows."""
         d, c = self.d, self.cfg
         d.check(self.lib.pg_norm_rows(self.gpu.handle, self.x.data_ptr(), d_rows, n, c.width, self.final_norm.data_ptr(), c.eps, self.picked.data_ptr(),
                                       d.code, self.ldh))
         self.head.run(self.picked, n, self.logits)
-
-    def read_logits(self, n: int) -> np.ndarray:
-        out = np.empty((n, self.logits.shape[1]), np.float32)
-        self.gpu.check(self.lib.pg_mem_download(self.gpu.handle, out.ctypes.data, self.logits.data_ptr(), out.nbytes))
-        return out
 
     def weight_bytes(self, tokens: int = 1) -> int:
         """bf16 weight bytes that a step of `tokens` tokens reads at most (every expert that can be chosen, once)."""
