@@ -98,7 +98,7 @@ PG_API int32_t pg_delta_run(pg_ctx *ctx, const pg_delta *p, const pg_batch *batc
  * proj row: [q H*D | k G*D | v G*V] (f32).  Caches [slot][G][cap][dp] and [slot][G][cap][vp] in the step's type, dp and
  * vp = D and V rounded up to 16. */
 typedef struct pg_attention {
-    int32_t heads, kv_heads, dim, vdim, cap;
+    int32_t heads, kv_heads, dim, vdim, cap, slots; /* slots: of the caches */
     float eps, scale;
     float temp_coef, temp_every; /* temp_every == 0: none; else q *= 1 + coef * ln(floor((p + 1) / every) + 1) */
     int32_t sink;                /* 1: one is added to the softmax denominator */

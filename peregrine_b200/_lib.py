@@ -160,7 +160,7 @@ class PgDelta(C.Structure):
 
 
 class PgAttention(C.Structure):
-    _fields_ = [("heads", _i32), ("kv_heads", _i32), ("dim", _i32), ("vdim", _i32), ("cap", _i32), ("eps", C.c_float), ("scale", C.c_float),
+    _fields_ = [("heads", _i32), ("kv_heads", _i32), ("dim", _i32), ("vdim", _i32), ("cap", _i32), ("slots", _i32), ("eps", C.c_float), ("scale", C.c_float),
                 ("temp_coef", C.c_float), ("temp_every", C.c_float), ("sink", _i32), ("d_q_norm", _vp), ("d_k_norm", _vp), ("d_q", _vp), ("d_part", _vp),
                 ("d_tickets", _vp)]
 

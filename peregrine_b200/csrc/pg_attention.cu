@@ -6,8 +6,10 @@
 //                                   the newest position also normalises and appends the key and the value.  Scores and
 //                                   sums run on mma.sync with the group's heads as the 16 rows; each warp streams keys
 //                                   through its own ring.  The last CTA of a (sequence, head) to finish merges the slices.
-//   bf16, longer portions           attn_prep_kernel (norms, temperature, append), then attn_prompt_kernel: rows of a tile
-//                                   are (token, head of the group) pairs, which share the keys and values
+//   bf16, longer portions           attn_prep_kernel (norms, temperature, append), then the tcgen05 kernel of
+//                                   csrc/pg_attention_tc.cu, or attn_prompt_kernel (mma.sync) for short portions and for
+//                                   head widths that the former does not take.  Rows of a tile are (token, head of the
+//                                   group) pairs, which share the keys and values.
 //   f32                             attn_prep_kernel, then attn_f32_kernel (one CTA per token and head, FFMA)
 //
 // The sink is a score of 0 without a value: the running maximum starts at 0 and exp(-max) joins the denominator.
@@ -16,17 +18,11 @@
 #include <algorithm>
 
 #include "pg_async.cuh"
-#include "pg_lm.cuh"
+#include "pg_attention.cuh"
 
 namespace {
 
 constexpr float LOG2E = 1.4426950408889634f;
-
-struct AttnShape {
-    int H, G, rep, D, V, dp, vp, cap, sink;
-    float eps, scale, coef, every;
-    const float *qn, *kn;
-};
 
 __device__ __forceinline__ float temperature(const AttnShape &s, int pos)
 {
@@ -34,18 +30,23 @@ __device__ __forceinline__ float temperature(const AttnShape &s, int pos)
     return 1.0f + s.coef * logf(floorf(__fdiv_rn((float)(pos + 1), s.every)) + 1.0f);
 }
 
-// One warp: dst = rms_norm(src[0 .. D)) * w * mul; columns D .. dp are zero.
+// One warp: dst = rms_norm(src[0 .. D)) * w * mul; columns D .. dp are zero (D <= 256).
 template <typename TA>
 __device__ __forceinline__ void head_norm(const float *src, const float *__restrict__ w, int D, int dp, float eps, float mul, TA *dst, int lane)
 {
-    float ss = 0.0f;
-    for (int i = lane; i < D; i += 32) {
-        const float x = __ldcg(src + i);
-        ss += x * x;
+    float x[8], ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+        x[i] = i * 32 + lane < D ? __ldcg(src + i * 32 + lane) : 0.0f;
+        ss += x[i] * x[i];
     }
     ss = pg_warp_sum(ss);
     const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss, (float)D) + eps));
-    for (int i = lane; i < dp; i += 32) pg_put(dst + i, i < D ? __ldcg(src + i) * inv * __ldg(w + i) * mul : 0.0f);
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+        const int c = i * 32 + lane;
+        if (c < dp) pg_put(dst + c, c < D ? x[i] * inv * __ldg(w + c) * mul : 0.0f);
+    }
 }
 
 // a CTA per token
@@ -333,19 +334,36 @@ __global__ void __launch_bounds__(WARPS * 32)
 }
 
 // ---- one token per sequence: grid (slices, G, rows), 4 warps ------------------------------------------------------
-constexpr int AS_WARPS = 4, AS_STAGES = 3;
+constexpr int AS_WARPS = 4, AS_STAGES = 3, AS_SLICES = 64;
 
 // part [rows][G][slices][16][vp + 2]: sums, then maximum (log 2 units) and denominator of each head
 template <int DC, int VC, bool FUSED>
 __global__ void __launch_bounds__(AS_WARPS * 32)
     attn_step_kernel(const AttnShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, const bf16 *__restrict__ q, bf16 *kc, bf16 *vc,
-                     float *part, int32_t *tickets, bf16 *__restrict__ out, int64_t ldo, int32_t *status)
+                     float *part, int32_t *tickets, bf16 *__restrict__ out, int64_t ldo, int32_t *status, unsigned long long limit_ns)
 {
     extern __shared__ __align__(128) unsigned char smem[];
+    __shared__ __align__(8) uint64_t bars[AS_WARPS * AS_STAGES];
+    __shared__ float weight[16][AS_SLICES];
+    __shared__ float denom[16];
     __shared__ int last_in;
-    pg_pdl_begin();
+    __shared__ volatile int abort_flag;
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     const int split = blockIdx.x, S = gridDim.x, ht = FUSED ? 0 : blockIdx.y / s.G, g = FUSED ? blockIdx.y : blockIdx.y % s.G, b = blockIdx.z;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane >> 2, t = lane & 3;
+    const int kstride = s.dp * 2 + 16, vstride = s.vp * 2 + 16, stage = 16 * (kstride + vstride);
+    const uint32_t ring = pg_smem(smem) + (uint32_t)warp * AS_STAGES * stage, bar = pg_smem(bars) + (uint32_t)warp * AS_STAGES * 8;
+    bf16 *qs = reinterpret_cast<bf16 *>(smem + AS_WARPS * AS_STAGES * stage);   // [16][dp + 8]
+    float *mg = reinterpret_cast<float *>(smem);                                // the merge reuses the rings
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < AS_WARPS * AS_STAGES; i++) pg_mbar_init(pg_smem(bars) + 8 * i, 1);
+        abort_flag = 0;
+        pg_mbar_fence();
+    }
+    const int heads = min(16, s.rep - ht * 16), h0 = g * s.rep + ht * 16;
+    for (int i = threadIdx.x; i < (16 - heads) * (s.dp + 8) / 2; i += AS_WARPS * 32) reinterpret_cast<uint32_t *>(qs + heads * (s.dp + 8))[i] = 0u;
+    __syncthreads();
+    asm volatile("griddepcontrol.wait;" ::: "memory");
     const int pos = __ldcg(bt.d_pos + b);
     const int64_t slot = __ldcg(bt.d_seq_slot + b);
     const int len = pos + 1;
@@ -353,7 +371,6 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
         if (threadIdx.x == 0) atomicExch(status, (int32_t)PG_ERR_INVALID);
         return;
     }
-    const int heads = min(16, s.rep - ht * 16), h0 = g * s.rep + ht * 16;
     const int chunk = ((len + S - 1) / S + 63) & ~63;
     const int t0 = split * chunk, t1 = min(len, t0 + chunk);
     const int used = (len + chunk - 1) / chunk;           // slices with keys; the others leave at once
@@ -361,55 +378,44 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
     const bool newest = FUSED && t1 == len;
     bf16 *kb = kc + (slot * s.G + g) * (int64_t)s.cap * s.dp, *vb = vc + (slot * s.G + g) * (int64_t)s.cap * s.vp;
     const int nk = s.dp / 16, nv = s.vp / 8;
-    const int kstride = s.dp * 2 + 16, vstride = s.vp * 2 + 16;
-    const int stage = 16 * (kstride + vstride);
-    const uint32_t ring = pg_smem(smem) + (uint32_t)warp * AS_STAGES * stage;
-    bf16 *qs = reinterpret_cast<bf16 *>(smem + AS_WARPS * AS_STAGES * stage);   // [16][dp + 8]
-    float *mg = reinterpret_cast<float *>(smem);                                // the merge reuses the rings
 
-    // the warp's 16-key tiles: t0 + 16 (warp + 4 i)
+    // the warp's 16-key tiles: t0 + 16 (warp + 4 i); lanes 0 .. 15 ask for a key each, lanes 16 .. 31 for a value each
+    // (rows behind the slice repeat its last one and are masked)
     const int ntiles = (t1 - t0 + 15) / 16, mine = ntiles > warp ? (ntiles - warp + AS_WARPS - 1) / AS_WARPS : 0;
     auto fetch = [&](int i) {
-        const int j0 = t0 + 16 * (warp + AS_WARPS * i);
-        const uint32_t kt = ring + (uint32_t)(i % AS_STAGES) * stage, vt = kt + 16 * kstride;
-        for (int x = lane; x < 16 * nk * 2; x += 32) {
-            const int k = x / (nk * 2), e = (x - k * nk * 2) * 8;
-            pg_cp16(tile_at(kt, kstride, k, e), kb + (int64_t)min(j0 + k, t1 - 1) * s.dp + e);
-        }
-        for (int x = lane; x < 16 * nv; x += 32) {
-            const int k = x / nv, e = (x - k * nv) * 8;
-            pg_cp16(tile_at(vt, vstride, k, e), vb + (int64_t)min(j0 + k, t1 - 1) * s.vp + e);
-        }
+        const uint32_t at = ring + (uint32_t)(i % AS_STAGES) * stage, on = bar + (uint32_t)(i % AS_STAGES) * 8;
+        const int64_t key = min(t0 + 16 * (warp + AS_WARPS * i) + (lane & 15), t1 - 1);
+        if (lane == 0) pg_mbar_expect(on, 16u * (uint32_t)(s.dp + s.vp) * 2u);
+        __syncwarp();
+        if (lane < 16)
+            pg_bulk_load(at + (uint32_t)lane * kstride, kb + key * s.dp, (uint32_t)s.dp * 2u, on);
+        else
+            pg_bulk_load(at + 16u * kstride + (uint32_t)(lane - 16) * vstride, vb + key * s.vp, (uint32_t)s.vp * 2u, on);
     };
     auto prime = [&]() {
-#pragma unroll
-        for (int i = 0; i < AS_STAGES - 1; i++) {
-            if (i < mine) fetch(i);
-            pg_cp_commit();
-        }
+        for (int i = 0; i < AS_STAGES && i < mine; i++) fetch(i);
     };
     if (!newest) prime();
     const float *row = proj + (int64_t)b * ldp;
-    for (int h = warp; h < 16; h += AS_WARPS) {
+    if (newest && warp == 2) {
+        head_norm(row + (int64_t)(s.H + g) * s.D, s.kn, s.D, s.dp, s.eps, 1.0f, kb + (int64_t)pos * s.dp, lane);
+        asm volatile("fence.proxy.async.global;" ::: "memory");
+    }
+    if (newest && warp == 3) {
+        const float *src = row + (int64_t)(s.H + s.G) * s.D + (int64_t)g * s.V;
+        for (int c = lane; c < s.vp; c += 32) pg_put(vb + (int64_t)pos * s.vp + c, c < s.V ? __ldcg(src + c) : 0.0f);
+        asm volatile("fence.proxy.async.global;" ::: "memory");
+    }
+    for (int h = warp; h < heads; h += AS_WARPS) {
         bf16 *dst = qs + h * (s.dp + 8);
-        if (h >= heads) {
-            for (int i = lane; i < s.dp; i += 32) pg_put(dst + i, 0.0f);
-        } else if (FUSED) {
+        if (FUSED) {
             head_norm(row + (int64_t)(h0 + h) * s.D, s.qn, s.D, s.dp, s.eps, temperature(s, pos), dst, lane);
         } else {
             for (int i = lane; i < s.dp; i += 32) dst[i] = __float2bfloat16_rn(pg_get(q + ((int64_t)b * s.H + h0 + h) * s.dp + i));
         }
     }
-    if (newest && warp == 0) head_norm(row + (int64_t)(s.H + g) * s.D, s.kn, s.D, s.dp, s.eps, 1.0f, kb + (int64_t)pos * s.dp, lane);
-    if (newest && warp == 1) {
-        const float *src = row + (int64_t)(s.H + s.G) * s.D + (int64_t)g * s.V;
-        for (int c = lane; c < s.vp; c += 32) pg_put(vb + (int64_t)pos * s.vp + c, c < s.V ? __ldcg(src + c) : 0.0f);
-    }
     __syncthreads();
-    if (newest) {
-        __threadfence_block();
-        prime();
-    }
+    if (newest) prime();                                  // the row that this CTA has just stored is among them
     uint32_t qf[DC][4];
     {
         const uint32_t qb = pg_smem(qs);
@@ -424,11 +430,11 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
         for (int j = 0; j < 4; j++) o[i][j] = 0.0f;
     const float sl = s.scale * LOG2E;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;
+    bool ok = true;
     for (int i = 0; i < mine; i++) {
-        if (i + AS_STAGES - 1 < mine) fetch(i + AS_STAGES - 1);
-        pg_cp_commit();
-        pg_cp_wait<AS_STAGES - 1>();
-        __syncwarp();
+        ok = pg_mbar_wait(bar + (uint32_t)(i % AS_STAGES) * 8, (uint32_t)(i / AS_STAGES) & 1u, &abort_flag, status, limit_ns);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
         const int j0 = t0 + 16 * (warp + AS_WARPS * i);
         const uint32_t kt = ring + (uint32_t)(i % AS_STAGES) * stage, vt = kt + 16 * kstride;
         float sc[2][4] = {};
@@ -463,18 +469,26 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
         }
         l0 = l0 * f0 + ((p[0] + p[1]) + (p[4] + p[5]));
         l1 = l1 * f1 + ((p[2] + p[3]) + (p[6] + p[7]));
+        if (__any_sync(0xffffffffu, f0 != 1.0f || f1 != 1.0f)) {
 #pragma unroll
-        for (int x = 0; x < VC; x++) {
-            o[x][0] *= f0;
-            o[x][1] *= f0;
-            o[x][2] *= f1;
-            o[x][3] *= f1;
+            for (int x = 0; x < VC; x++) {
+                o[x][0] *= f0;
+                o[x][1] *= f0;
+                o[x][2] *= f1;
+                o[x][3] *= f1;
+            }
         }
         const uint32_t pf[4] = {pg_pack_bf16(p[0], p[1]), pg_pack_bf16(p[2], p[3]), pg_pack_bf16(p[4], p[5]), pg_pack_bf16(p[6], p[7])};
         values16<VC>(o, nv, pf, vt, vstride, 0, lane);
         __syncwarp();                                     // every lane is done with the stage before it is filled again
+        if (i + AS_STAGES < mine) fetch(i + AS_STAGES);
     }
-    pg_cp_wait<0>();
+    if (!ok) {
+        // copies that are still in flight get a bounded time to land before their shared memory is used again
+        const unsigned long long w0 = pg_globaltimer_ns();
+        while (pg_globaltimer_ns() - w0 < 2000000ull) {
+        }
+    }
 #pragma unroll
     for (int x = 1; x < 4; x <<= 1) {
         l0 += __shfl_xor_sync(0xffffffffu, l0, x);
@@ -487,17 +501,13 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
 #pragma unroll
     for (int i = 0; i < VC; i++) {
         if (i < nv) {
-            w0[i * 8 + 2 * t] = o[i][0];
-            w0[i * 8 + 2 * t + 1] = o[i][1];
-            w1[i * 8 + 2 * t] = o[i][2];
-            w1[i * 8 + 2 * t + 1] = o[i][3];
+            *reinterpret_cast<float2 *>(w0 + i * 8 + 2 * t) = make_float2(o[i][0], o[i][1]);
+            if (heads > 8) *reinterpret_cast<float2 *>(w1 + i * 8 + 2 * t) = make_float2(o[i][2], o[i][3]);
         }
     }
     if (t == 0) {
-        w0[s.vp] = m0;
-        w0[s.vp + 1] = l0;
-        w1[s.vp] = m1;
-        w1[s.vp + 1] = l1;
+        *reinterpret_cast<float2 *>(w0 + s.vp) = make_float2(m0, l0);
+        *reinterpret_cast<float2 *>(w1 + s.vp) = make_float2(m1, l1);
     }
     __syncthreads();
     const int64_t unit = ((int64_t)b * gridDim.y + blockIdx.y);
@@ -525,10 +535,7 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
             if (c < s.V) pg_put(out + (int64_t)b * ldo + (int64_t)(h0 + h) * s.V + c, __fdiv_rn(a, l));
         } else {
             mine_part[(size_t)h * ms + c] = a;
-            if (c == 0) {
-                mine_part[(size_t)h * ms + s.vp] = m;
-                mine_part[(size_t)h * ms + s.vp + 1] = l;
-            }
+            if (c == 0) *reinterpret_cast<float2 *>(mine_part + (size_t)h * ms + s.vp) = make_float2(m, l);
         }
     }
     if (used == 1) return;
@@ -541,22 +548,38 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
     __syncthreads();
     if (!last_in) return;
     __threadfence();
-    const float *parts = part + unit * S * 16 * ms;
-    for (int x = threadIdx.x; x < nh; x += AS_WARPS * 32) {
-        const int h = x / s.vp, c = x - h * s.vp;
-        if (c >= s.V) continue;
-        float m = s.sink ? 0.0f : -INFINITY;
-        for (int k = 0; k < used; k++) m = fmaxf(m, __ldcg(parts + ((size_t)k * 16 + h) * ms + s.vp));
-        float a = 0.0f, l = s.sink ? exp2f(-m) : 0.0f;
-        for (int k = 0; k < used; k++) {
-            const float *at = parts + ((size_t)k * 16 + h) * ms;
-            const float f = exp2f(__ldcg(at + s.vp) - m);
-            a = fmaf(f, __ldcg(at + c), a);
-            l = fmaf(f, __ldcg(at + s.vp + 1), l);
-        }
-        pg_put(out + (int64_t)b * ldo + (int64_t)(h0 + h) * s.V + c, __fdiv_rn(a, l));
-    }
     if (threadIdx.x == 0) tickets[unit] = 0;
+    // a warp per head: the slices' weights; then all columns with their loads in flight together
+    const float *parts = part + unit * S * 16 * ms;
+    for (int h = warp; h < heads; h += AS_WARPS) {
+        float2 ml[AS_SLICES / 32];
+        float m = s.sink ? 0.0f : -INFINITY, l = 0.0f;
+#pragma unroll
+        for (int i = 0; i < AS_SLICES / 32; i++) {
+            const int k = i * 32 + lane;
+            ml[i] = k < used ? __ldcg(reinterpret_cast<const float2 *>(parts + ((size_t)k * 16 + h) * ms + s.vp)) : make_float2(-INFINITY, 0.0f);
+            m = fmaxf(m, ml[i].x);
+        }
+#pragma unroll
+        for (int o2 = 16; o2 > 0; o2 >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o2));
+#pragma unroll
+        for (int i = 0; i < AS_SLICES / 32; i++) {
+            const float f = exp2f(ml[i].x - m);
+            weight[h][i * 32 + lane] = f;
+            l = fmaf(f, ml[i].y, l);
+        }
+        l = pg_warp_sum(l) + (s.sink ? exp2f(-m) : 0.0f);
+        if (lane == 0) denom[h] = __fdiv_rn(1.0f, l);
+    }
+    __syncthreads();
+    for (int x = threadIdx.x; x < heads * s.V; x += AS_WARPS * 32) {
+        const int h = x / s.V, c = x - h * s.V;
+        const float *at = parts + (size_t)h * ms + c;
+        float a = 0.0f;
+#pragma unroll 8
+        for (int k = 0; k < used; k++) a = fmaf(weight[h][k], __ldcg(at + (size_t)k * 16 * ms), a);
+        pg_put(out + (int64_t)b * ldo + (int64_t)(h0 + h) * s.V + c, a * denom[h]);
+    }
 }
 
 AttnShape shape_of(const pg_attention *p)
@@ -575,7 +598,7 @@ int slices(const pg_ctx *ctx, int64_t units, int64_t cap)
 {
     int64_t S = std::max<int64_t>(1, 2 * (int64_t)ctx->sm_count / std::max<int64_t>(1, units));
     S = std::min<int64_t>(S, std::max<int64_t>(1, cap / 128));
-    return (int)std::min<int64_t>(S, 64);
+    return (int)std::min<int64_t>(S, AS_SLICES);
 }
 
 template <int DC, int VC>
@@ -598,11 +621,11 @@ int32_t run_step(pg_ctx *ctx, const AttnShape &s, const pg_batch *bt, const floa
     const int rings = AS_WARPS * AS_STAGES * stage;
     const int smem = std::max(rings + 16 * (s.dp + 8) * 2, AS_WARPS * 16 * (s.vp + 2) * 4);
     static std::atomic<uint64_t> set{0};
-    PG_CUDA(pg_max_smem_once(attn_step_kernel<DC, VC, FUSED>, 226 * 1024, ctx->device, set));
+    PG_CUDA(pg_max_smem_once(attn_step_kernel<DC, VC, FUSED>, 220 * 1024, ctx->device, set));
     const int ht = (s.rep + 15) / 16;
     const int S = slices(ctx, (int64_t)bt->rows * s.G * ht, s.cap);
     return launch_pdl(ctx, attn_step_kernel<DC, VC, FUSED>, dim3((unsigned)S, (unsigned)(s.G * ht), (unsigned)bt->rows), dim3(AS_WARPS * 32), (size_t)smem, s,
-                      *bt, proj, ldp, q, kc, vc, part, tickets, out, ldo, ctx->d_status);
+                      *bt, proj, ldp, q, kc, vc, part, tickets, out, ldo, ctx->d_status, ctx->wait_limit_ns);
 }
 
 }  // namespace
@@ -646,6 +669,7 @@ PG_API int32_t pg_attention_run(pg_ctx *ctx, const pg_attention *p, const pg_bat
         const int32_t rc = launch_pdl(ctx, attn_prep_kernel<bf16>, dim3((unsigned)M), dim3(256), 0, s, *batch, d_proj, ldp, q, kc, vc, ctx->d_status);
         if (rc != PG_OK) return rc;
     }
+    if (!step && pgk_attention_prompt_tc_supports(s, batch, p->slots, ldo, out)) return pgk_attention_prompt_tc(ctx, s, batch, p->slots, q, kc, vc, out, ldo);
 #define PG_AT(DC, VC)                                                                                                        \
     do {                                                                                                                     \
         if (fused) return run_step<DC, VC, true>(ctx, s, batch, d_proj, ldp, q, kc, vc, p->d_part, p->d_tickets, out, ldo);  \

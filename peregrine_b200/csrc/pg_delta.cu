@@ -7,9 +7,12 @@
 //
 //   one token per sequence   delta_step_kernel: convolution, unit norms, gates, the state update and the gated output
 //                            norm of one (head, sequence) in one CTA; the state is read and written once
-//   longer portions          delta_prep_kernel (convolution, unit norms, gates; a CTA per token), delta_scan_kernel (the
-//                            recurrence; a warp holds four columns of a head's state in registers), delta_out_kernel
-//                            (output norm and gate; also stores the convolution inputs that the next portion needs)
+//   longer portions          delta_prep_kernel (convolution, unit norms, gates; a CTA per four tokens), delta_scan_kernel
+//                            (the recurrence, four tokens at a time: their read-outs come from the state the first of them
+//                            finds, corrected by the pairs' products k_a . k_b and q_a . k_b, so that one round of
+//                            reductions serves four tokens; a warp holds eight columns of a head's state in registers),
+//                            delta_out_kernel (output norm and gate; also stores the convolution inputs that the next
+//                            portion needs)
 //
 // Convolution inputs are kept per slot in a ring of `taps` entries, position p in entry p mod taps: a single token
 // writes an entry that nobody reads any more, so heads that share channels need no order among their CTAs.
@@ -181,185 +184,372 @@ __global__ void __launch_bounds__(DS_T)
 }
 
 // ---- longer portions ---------------------------------------------------------------------------------------------
-// work rows: q [G D] | k [G D] | v [H V] | o [H V], and per token: kq [G] | beta [H] | decay [H]
+// work rows: q [G D] | k [G D] | v [H V] | o [H V] per token; coef: 32 floats per block of four tokens and head.  With the
+// decays g_a of a block's tokens, c_a = g_0 .. g_a and r_ab = g_{b+1} .. g_a:
+//   u_a = beta_a (v_a - c_a S^T k_a - sum_{b<a} r_ab (k_b . k_a) u_b)
+//   o_a = c_a S^T q_a + sum_{b<=a} r_ab (k_b . q_a) u_b
+//   S <- c_3 S + sum_b r_3b k_b u_b^T
+// coef: c [4] | beta [4] | r_3b [4] | r_ab (k_b . k_a) of the 6 pairs b < a | r_ab (k_b . q_a) of the 10 pairs b <= a
 struct DeltaWork {
-    float *q, *k, *v, *o, *kq, *beta, *dec;
+    float *q, *k, *v, *o, *coef;
 };
+constexpr int BT = 4;            // tokens of a block
+// blocks of a sequence are numbered from here on
+__device__ __forceinline__ int64_t first_block(int row0, int seq) { return row0 / BT + seq; }
 
+// grid (ceil(longest / 4), seqs).  TAPS: the number of taps, 0 = any
+template <int TAPS>
 __global__ void __launch_bounds__(256)
     delta_prep_kernel(const DeltaShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, const float *__restrict__ ring, const DeltaWork w)
 {
-    extern __shared__ __align__(16) float sm[];   // q and k channels
+    extern __shared__ __align__(16) float sm[];   // q and k channels [4][2 G D], then the pairs' products [G][16]
     pg_pdl_begin();
-    const int m = blockIdx.x, seq = __ldcg(bt.d_row_seq + m);
-    const int pos = __ldcg(bt.d_pos + m), t = m - __ldcg(bt.d_seq_row0 + seq);
-    const float *row = proj + (int64_t)m * ldp;
+    const int seq = blockIdx.y, row0 = __ldcg(bt.d_seq_row0 + seq), T = __ldcg(bt.d_seq_row0 + seq + 1) - row0;
+    const int t0 = blockIdx.x * BT, n = min(BT, T - t0), m0 = row0 + t0;
+    if (n <= 0) return;
+    const int pos0 = __ldcg(bt.d_pos + row0);
+    const float *row = proj + (int64_t)m0 * ldp;
     const float *rg = ring + (int64_t)__ldcg(bt.d_seq_slot + seq) * s.taps * s.C;
     const int qk = 2 * s.G * s.D;
+    float *dots = sm + (size_t)BT * qk;
     for (int c = threadIdx.x; c < s.C; c += 256) {
-        const float y = conv_at(s, row, ldp, rg, c, t, pos);
-        if (c < qk)
-            sm[c] = y;
-        else
-            w.v[(int64_t)m * s.H * s.V + c - qk] = y;
+        float y[BT];
+        if constexpr (TAPS > 0) {
+            float x[TAPS - 1 + BT], wt[TAPS];
+#pragma unroll
+            for (int j = 0; j < TAPS; j++) wt[j] = __ldg(s.conv + (int64_t)j * s.C + c);
+#pragma unroll
+            for (int j = 0; j < TAPS - 1 + BT; j++) {
+                const int t = t0 + j - (TAPS - 1);        // of the sequence's tokens in this step
+                x[j] = 0.0f;
+                if (t >= 0) {
+                    if (t < T) x[j] = __ldcg(row + (int64_t)(j - (TAPS - 1)) * ldp + c);
+                } else if (pos0 + t >= 0) {
+                    x[j] = __ldcg(rg + (int64_t)((pos0 + t) % TAPS) * s.C + c);
+                }
+            }
+#pragma unroll
+            for (int a = 0; a < BT; a++) {
+                float acc = 0.0f;
+#pragma unroll
+                for (int j = 0; j < TAPS; j++) acc = fmaf(wt[j], x[a + j], acc);
+                y[a] = pg_silu(acc);
+            }
+        } else {
+#pragma unroll
+            for (int a = 0; a < BT; a++) y[a] = a < n ? conv_at(s, row + (int64_t)a * ldp, ldp, rg, c, t0 + a, pos0 + t0 + a) : 0.0f;
+        }
+#pragma unroll
+        for (int a = 0; a < BT; a++) {
+            if (c < qk)
+                sm[(size_t)a * qk + c] = a < n ? y[a] : 0.0f;
+            else if (a < n)
+                w.v[(int64_t)(m0 + a) * s.H * s.V + c - qk] = y[a];
+        }
     }
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int g = warp; g < s.G; g += 8) {
-        const float *q = sm + g * s.D, *k = sm + (s.G + g) * s.D;
-        float a = 0.0f, b = 0.0f, d = 0.0f;
-        for (int i = lane; i < s.D; i += 32) {
-            a += q[i] * q[i];
-            b += k[i] * k[i];
-            d += q[i] * k[i];
+    for (int i = warp; i < BT * 2 * s.G; i += 8) {        // unit norms: (token, q or k, head)
+        const int a = i / (2 * s.G), hd = i - a * 2 * s.G;
+        float *x = sm + (size_t)a * qk + hd * s.D;
+        float ss = 0.0f;
+        for (int d = lane; d < s.D; d += 32) ss += x[d] * x[d];
+        ss = pg_warp_sum(ss);
+        const bool is_q = hd < s.G;
+        const float inv = __fdiv_rn(is_q ? s.qscale : 1.0f, sqrtf(ss + s.unit_eps));
+        float *dst = (is_q ? w.q : w.k) + ((int64_t)(m0 + a) * s.G + (is_q ? hd : hd - s.G)) * s.D;
+        for (int d = lane; d < s.D; d += 32) {
+            const float y = x[d] * inv;
+            x[d] = y;
+            if (a < n) dst[d] = y;
         }
-        a = pg_warp_sum(a);
-        b = pg_warp_sum(b);
-        d = pg_warp_sum(d);
-        const float iq = __fdiv_rn(s.qscale, sqrtf(a + s.unit_eps)), ik = __fdiv_rn(1.0f, sqrtf(b + s.unit_eps));
-        for (int i = lane; i < s.D; i += 32) {
-            w.q[((int64_t)m * s.G + g) * s.D + i] = q[i] * iq;
-            w.k[((int64_t)m * s.G + g) * s.D + i] = k[i] * ik;
-        }
-        if (lane == 0) w.kq[(int64_t)m * s.G + g] = d * iq * ik;
     }
-    const float *tail = row + s.C + (int64_t)s.H * s.V;
+    __syncthreads();
+    for (int g = warp; g < s.G; g += 8) {                 // the pairs' products
+        float p[16] = {};
+        for (int d = lane; d < s.D; d += 32) {
+            float q[BT], k[BT];
+#pragma unroll
+            for (int a = 0; a < BT; a++) {
+                q[a] = sm[(size_t)a * qk + g * s.D + d];
+                k[a] = sm[(size_t)a * qk + (s.G + g) * s.D + d];
+            }
+#pragma unroll
+            for (int a = 0, i = 0, j = 6; a < BT; a++)
+#pragma unroll
+                for (int b = 0; b <= a; b++) {
+                    if (b < a) p[i] = fmaf(k[b], k[a], p[i]), i++;
+                    p[j] = fmaf(k[b], q[a], p[j]), j++;
+                }
+        }
+#pragma unroll
+        for (int i = 0; i < 16; i++) {
+            p[i] = pg_warp_sum(p[i]);
+            if (lane == i) dots[g * 16 + i] = p[i];
+        }
+    }
+    __syncthreads();
     for (int h = threadIdx.x; h < s.H; h += 256) {
-        w.beta[(int64_t)m * s.H + h] = pg_sigmoid(__ldcg(tail + h));
-        w.dec[(int64_t)m * s.H + h] = expf(log_decay(__ldcg(tail + s.H + h), __ldg(s.a_log + h), __ldg(s.dt_bias + h)));
+        const float *dp = dots + h / (s.H / s.G) * 16;
+        const float al = __ldg(s.a_log + h), db = __ldg(s.dt_bias + h);
+        float g[BT], o[32];
+#pragma unroll
+        for (int a = 0; a < BT; a++) {
+            const float *tail = row + (int64_t)a * ldp + s.C + (int64_t)s.H * s.V;
+            g[a] = a < n ? expf(log_decay(__ldcg(tail + s.H + h), al, db)) : 1.0f;
+            o[4 + a] = a < n ? pg_sigmoid(__ldcg(tail + h)) : 0.0f;
+            o[a] = a ? o[a - 1] * g[a] : g[0];
+        }
+        o[11] = 1.0f;
+#pragma unroll
+        for (int b = BT - 2; b >= 0; b--) o[8 + b] = o[9 + b] * g[b + 1];
+#pragma unroll
+        for (int a = 0, i = 0, j = 6; a < BT; a++)
+#pragma unroll
+            for (int b = 0; b <= a; b++) {
+                float r = 1.0f;
+#pragma unroll
+                for (int x = b + 1; x <= a; x++) r *= g[x];
+                if (b < a) o[12 + i] = r * dp[i], i++;
+                o[12 + j] = r * dp[j], j++;
+            }
+        float4 *dst = reinterpret_cast<float4 *>(w.coef + ((first_block(row0, seq) + blockIdx.x) * s.H + h) * 32);
+        o[28] = o[29] = o[30] = o[31] = 0.0f;
+#pragma unroll
+        for (int i = 0; i < 8; i++) dst[i] = make_float4(o[4 * i], o[4 * i + 1], o[4 * i + 2], o[4 * i + 3]);
     }
 }
 
-// grid (ceil(V / 32), H, seqs), 8 warps.  Warp w: columns w * 4 .. w * 4 + 3 of the CTA's 32; of its lanes, eight share a
-// column: lane l = lane & 7 holds rows l * 4 + 32 i .. + 3 (i < NI) of column lane >> 3.
-template <int NI>
-__global__ void __launch_bounds__(256)
-    delta_scan_kernel(const DeltaShape s, const pg_batch bt, const DeltaWork w, float *state)
+typedef unsigned long long f32x2;    // two f32 in a register pair
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c)
 {
-    constexpr int DP = NI * 32;
-    constexpr int SC_TB = NI <= 4 ? 16 : 8;      // tokens per shared-memory tile
-    __shared__ __align__(16) float tk[2][SC_TB][DP], tq[2][SC_TB][DP];
-    __shared__ __align__(16) float tv[2][SC_TB][32];
-    __shared__ float ts[2][SC_TB][4];            // kq, beta, decay
+    f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b)
+{
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ f32x2 pack2(float lo, float hi)
+{
+    f32x2 d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ float sum2(f32x2 v)
+{
+    float lo, hi;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+    return lo + hi;
+}
+struct __align__(16) Quad {
+    f32x2 lo, hi;
+};
+
+// grid (ceil(V / 32), H, seqs), 4 warps.  Warp w: columns 8 w .. 8 w + 7 of the CTA's 32.  Eight lanes share two columns:
+// lane l = lane & 7 holds rows l * 4 + 32 i .. + 3 (i < NI) of columns 2 (lane >> 3) and 2 (lane >> 3) + 1, and does a block's
+// algebra for the column of its parity.
+template <int NI>
+struct ScanTile {
+    static constexpr int DP = NI * 32;
+    static constexpr int TB = NI <= 4 ? 16 : 8;           // tokens per tile
+    static constexpr int STAGES = 3;
+    struct Stage {
+        float k[TB][DP], q[TB][DP], v[TB][32], coef[TB / BT][32];
+    };
+};
+
+template <int NI>
+__global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaShape s, const pg_batch bt, const DeltaWork w, float *state)
+{
+    using C = ScanTile<NI>;
+    constexpr int DP = C::DP, TB = C::TB;
+    extern __shared__ __align__(16) unsigned char smem[];
+    typename C::Stage *stages = reinterpret_cast<typename C::Stage *>(smem);
     pg_pdl_begin();
     const int h = blockIdx.y, seq = blockIdx.z, g = h / (s.H / s.G), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int row0 = __ldcg(bt.d_seq_row0 + seq), T = __ldcg(bt.d_seq_row0 + seq + 1) - row0;
     if (T <= 0) return;
     const int pos0 = __ldcg(bt.d_pos + row0);
-    const int c0 = blockIdx.x * 32, mycol = warp * 4 + (lane >> 3), l = lane & 7;
-    const bool col_ok = c0 + mycol < s.V;
-    float *st = state + ((int64_t)__ldcg(bt.d_seq_slot + seq) * s.H + h) * (int64_t)s.D * s.vs + c0 + mycol;
-    float S[NI][4];
+    const int c0 = blockIdx.x * 32, col = warp * 8 + (lane >> 3) * 2, l = lane & 7, par = lane & 1;
+    const int64_t block0 = first_block(row0, seq);
+    float *st = state + ((int64_t)__ldcg(bt.d_seq_slot + seq) * s.H + h) * (int64_t)s.D * s.vs + c0 + col;
+    f32x2 S[2][NI][2];
 #pragma unroll
-    for (int i = 0; i < NI; i++)
-#pragma unroll
-        for (int j = 0; j < 4; j++) {
-            const int r = l * 4 + 32 * i + j;
-            S[i][j] = (pos0 > 0 && col_ok && r < s.D) ? __ldcg(st + (int64_t)r * s.vs) : 0.0f;
-        }
-    // a tile into shared memory; rows of q and k behind D and columns behind V are zero
-    auto fetch = [&](int buf, int t0) {
-        const int n = min(SC_TB, T - t0);
-        // (16-byte copies that bypass L1 where the shape allows them)
-        const bool vec = ((s.D | s.V) & 3) == 0;
-        for (int i = tid; i < SC_TB * DP / 4; i += 256) {
-            const int t = i / (DP / 4), d = (i - t * (DP / 4)) * 4;
-            const int64_t at = ((int64_t)(row0 + t0 + t) * s.G + g) * s.D + d;
-            if (vec && t < n && d < s.D) {
-                pg_cp16(pg_smem(&tk[buf][t][d]), w.k + at);
-                pg_cp16(pg_smem(&tq[buf][t][d]), w.q + at);
-            } else {
-#pragma unroll
-                for (int j = 0; j < 4; j++) {
-                    const bool in = t < n && d + j < s.D;
-                    tk[buf][t][d + j] = in ? __ldcg(w.k + at + j) : 0.0f;
-                    tq[buf][t][d + j] = in ? __ldcg(w.q + at + j) : 0.0f;
-                }
-            }
-        }
-        for (int i = tid; i < SC_TB * 8; i += 256) {
-            const int t = i / 8, c = (i & 7) * 4;
-            const float *v = w.v + (int64_t)(row0 + t0 + t) * s.H * s.V + (int64_t)h * s.V + c0 + c;
-            if (vec && t < n && c0 + c < s.V) {
-                pg_cp16(pg_smem(&tv[buf][t][c]), v);
-            } else {
-#pragma unroll
-                for (int j = 0; j < 4; j++) tv[buf][t][c + j] = (t < n && c0 + c + j < s.V) ? __ldcg(v + j) : 0.0f;
-            }
-        }
-        if (tid < n) {
-            const int64_t m = row0 + t0 + tid;
-            ts[buf][tid][0] = __ldcg(w.kq + m * s.G + g);
-            ts[buf][tid][1] = __ldcg(w.beta + m * s.H + h);
-            ts[buf][tid][2] = __ldcg(w.dec + m * s.H + h);
-        }
-        pg_cp_commit();
-    };
-    fetch(0, 0);
-    int buf = 0;
-    for (int t0 = 0; t0 < T; t0 += SC_TB, buf ^= 1) {
-        const int n = min(SC_TB, T - t0);
-        if (t0 + SC_TB < T) {
-            fetch(buf ^ 1, t0 + SC_TB);
-            pg_cp_wait<1>();
-        } else {
-            pg_cp_wait<0>();
-        }
-        __syncthreads();
-        float4 k[NI], q[NI];
-#pragma unroll
-        for (int i = 0; i < NI; i++) {
-            k[i] = *reinterpret_cast<const float4 *>(&tk[buf][0][l * 4 + 32 * i]);
-            q[i] = *reinterpret_cast<const float4 *>(&tq[buf][0][l * 4 + 32 * i]);
-        }
-        for (int t = 0; t < n; t++) {
-            // the next token's rows are asked for before this one's chain of dependent steps
-            float4 kn[NI], qn[NI];
-            const int tn = min(t + 1, SC_TB - 1);
-#pragma unroll
-            for (int i = 0; i < NI; i++) {
-                kn[i] = *reinterpret_cast<const float4 *>(&tk[buf][tn][l * 4 + 32 * i]);
-                qn[i] = *reinterpret_cast<const float4 *>(&tq[buf][tn][l * 4 + 32 * i]);
-            }
-            const float kq = ts[buf][t][0], beta = ts[buf][t][1], dec = ts[buf][t][2], v = tv[buf][t][mycol];
-            float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-            for (int i = 0; i < NI; i++) {
-                a[0] = fmaf(k[i].x, S[i][0], a[0]), a[1] = fmaf(k[i].y, S[i][1], a[1]), a[2] = fmaf(k[i].z, S[i][2], a[2]), a[3] = fmaf(k[i].w, S[i][3], a[3]);
-                b[0] = fmaf(q[i].x, S[i][0], b[0]), b[1] = fmaf(q[i].y, S[i][1], b[1]), b[2] = fmaf(q[i].z, S[i][2], b[2]), b[3] = fmaf(q[i].w, S[i][3], b[3]);
-            }
-            float sk = (a[0] + a[1]) + (a[2] + a[3]), sq = (b[0] + b[1]) + (b[2] + b[3]);
-#pragma unroll
-            for (int o = 1; o < 8; o <<= 1) {
-                sk += __shfl_xor_sync(0xffffffffu, sk, o);
-                sq += __shfl_xor_sync(0xffffffffu, sq, o);
-            }
-            const float u = beta * (v - dec * sk);
-#pragma unroll
-            for (int i = 0; i < NI; i++) {
-                S[i][0] = fmaf(k[i].x, u, dec * S[i][0]);
-                S[i][1] = fmaf(k[i].y, u, dec * S[i][1]);
-                S[i][2] = fmaf(k[i].z, u, dec * S[i][2]);
-                S[i][3] = fmaf(k[i].w, u, dec * S[i][3]);
-            }
-            if (l == 0 && col_ok) w.o[(int64_t)(row0 + t0 + t) * s.H * s.V + (int64_t)h * s.V + c0 + mycol] = dec * sq + kq * u;
-#pragma unroll
-            for (int i = 0; i < NI; i++) {
-                k[i] = kn[i];
-                q[i] = qn[i];
-            }
-        }
-        __syncthreads();
-    }
-    if (col_ok) {
+    for (int c = 0; c < 2; c++)
 #pragma unroll
         for (int i = 0; i < NI; i++)
 #pragma unroll
-            for (int j = 0; j < 4; j++) {
-                const int r = l * 4 + 32 * i + j;
-                if (r < s.D) st[(int64_t)r * s.vs] = S[i][j];
+            for (int j = 0; j < 2; j++) {
+                const int r = l * 4 + 32 * i + 2 * j;
+                const bool in = pos0 > 0 && c0 + col + c < s.V;
+                S[c][i][j] = pack2((in && r < s.D) ? __ldcg(st + (int64_t)r * s.vs + c) : 0.0f, (in && r + 1 < s.D) ? __ldcg(st + (int64_t)(r + 1) * s.vs + c) : 0.0f);
+            }
+    // A tile into shared memory; rows of q and k behind D, columns behind V and tokens behind T are zero.  (16-byte copies
+    // that bypass L1 where the shape allows them.)
+    const bool vec = ((s.D | s.V) & 3) == 0;
+    auto fetch = [&](int tile) {
+        typename C::Stage &e = stages[tile % C::STAGES];
+        const int t0 = tile * TB, n = min(TB, T - t0);
+        if (n > 0) {
+            for (int i = tid; i < TB * DP / 4; i += 128) {
+                const int t = i / (DP / 4), d = (i - t * (DP / 4)) * 4;
+                const int64_t at = ((int64_t)(row0 + t0 + t) * s.G + g) * s.D + d;
+                if (vec && t < n && d < s.D) {
+                    pg_cp16(pg_smem(&e.k[t][d]), w.k + at);
+                    pg_cp16(pg_smem(&e.q[t][d]), w.q + at);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 4; j++) {
+                        const bool in = t < n && d + j < s.D;
+                        e.k[t][d + j] = in ? __ldcg(w.k + at + j) : 0.0f;
+                        e.q[t][d + j] = in ? __ldcg(w.q + at + j) : 0.0f;
+                    }
+                }
+            }
+            for (int i = tid; i < TB * 8; i += 128) {
+                const int t = i / 8, c = (i & 7) * 4;
+                const float *v = w.v + (int64_t)(row0 + t0 + t) * s.H * s.V + (int64_t)h * s.V + c0 + c;
+                if (vec && t < n && c0 + c < s.V) {
+                    pg_cp16(pg_smem(&e.v[t][c]), v);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 4; j++) e.v[t][c + j] = (t < n && c0 + c + j < s.V) ? __ldcg(v + j) : 0.0f;
+                }
+            }
+            if (tid < TB / BT * 8) {
+                const int bi = tid / 8;
+                if (bi * BT < n) pg_cp16(pg_smem(&e.coef[bi][(tid & 7) * 4]), w.coef + ((block0 + t0 / BT + bi) * s.H + h) * 32 + (tid & 7) * 4);
+            }
+        }
+        pg_cp_commit();
+    };
+    const int tiles = (T + TB - 1) / TB;
+    fetch(0);
+    fetch(1);
+    for (int tile = 0; tile < tiles; tile++) {
+        fetch(tile + 2);                                  // its stage was left behind the last barrier
+        pg_cp_wait<2>();
+        __syncthreads();
+        const typename C::Stage &e = stages[tile % C::STAGES];
+        const int t0 = tile * TB, blocks = (min(TB, T - t0) + BT - 1) / BT;
+        for (int bi = 0; bi < blocks; bi++) {
+            const float(*kt)[DP] = &e.k[bi * BT], (*qt)[DP] = &e.q[bi * BT];
+            f32x2 ak[BT][2] = {}, aq[BT][2] = {};
+#pragma unroll
+            for (int i = 0; i < NI; i++) {
+#pragma unroll
+                for (int a = 0; a < BT; a++) {
+                    const Quad k = *reinterpret_cast<const Quad *>(&kt[a][l * 4 + 32 * i]), q = *reinterpret_cast<const Quad *>(&qt[a][l * 4 + 32 * i]);
+#pragma unroll
+                    for (int c = 0; c < 2; c++) {
+                        ak[a][c] = fma2(k.lo, S[c][i][0], ak[a][c]);
+                        ak[a][c] = fma2(k.hi, S[c][i][1], ak[a][c]);
+                        aq[a][c] = fma2(q.lo, S[c][i][0], aq[a][c]);
+                        aq[a][c] = fma2(q.hi, S[c][i][1], aq[a][c]);
+                    }
+                }
+            }
+            const float4 *cf = reinterpret_cast<const float4 *>(e.coef[bi]);
+            const float4 cc = cf[0], be = cf[1], r3 = cf[2], p0 = cf[3], p1 = cf[4], p2 = cf[5], p3 = cf[6];
+            float v[BT];
+#pragma unroll
+            for (int a = 0; a < BT; a++) v[a] = e.v[bi * BT + a][col + par];
+            // the column of this lane's parity, then the sums over the eight lanes
+            float sk[BT], sq[BT];
+#pragma unroll
+            for (int a = 0; a < BT; a++) {
+                const float k0 = sum2(ak[a][0]), k1 = sum2(ak[a][1]), q0 = sum2(aq[a][0]), q1 = sum2(aq[a][1]);
+                sk[a] = (par ? k1 : k0) + __shfl_xor_sync(0xffffffffu, par ? k0 : k1, 1);
+                sq[a] = (par ? q1 : q0) + __shfl_xor_sync(0xffffffffu, par ? q0 : q1, 1);
+            }
+#pragma unroll
+            for (int o = 2; o < 8; o <<= 1)
+#pragma unroll
+                for (int a = 0; a < BT; a++) {
+                    sk[a] += __shfl_xor_sync(0xffffffffu, sk[a], o);
+                    sq[a] += __shfl_xor_sync(0xffffffffu, sq[a], o);
+                }
+            // pairs: p0 = kk10 kk20 kk21 kk30, p1 = kk31 kk32 qk00 qk10, p2 = qk11 qk20 qk21 qk22, p3 = qk30 qk31 qk32 qk33
+            const float u0 = be.x * (v[0] - cc.x * sk[0]);
+            const float u1 = be.y * (v[1] - cc.y * sk[1] - p0.x * u0);
+            const float u2 = be.z * (v[2] - cc.z * sk[2] - p0.y * u0 - p0.z * u1);
+            const float u3 = be.w * (v[3] - cc.w * sk[3] - p0.w * u0 - p1.x * u1 - p1.y * u2);
+            const float o0 = cc.x * sq[0] + p1.z * u0;
+            const float o1 = cc.y * sq[1] + p1.w * u0 + p2.x * u1;
+            const float o2 = cc.z * sq[2] + p2.y * u0 + p2.z * u1 + p2.w * u2;
+            const float o3 = cc.w * sq[3] + p3.x * u0 + p3.y * u1 + p3.z * u2 + p3.w * u3;
+            // lane l stores token l >> 1 of its column
+            const int a = l >> 1, t = t0 + bi * BT + a;
+            if (t < T && c0 + col + par < s.V)
+                w.o[(int64_t)(row0 + t) * s.H * s.V + (int64_t)h * s.V + c0 + col + par] = a == 0 ? o0 : (a == 1 ? o1 : (a == 2 ? o2 : o3));
+            const float mine[BT] = {r3.x * u0, r3.y * u1, r3.z * u2, r3.w * u3};
+            f32x2 uw[BT][2];
+#pragma unroll
+            for (int b = 0; b < BT; b++) {
+                const float other = __shfl_xor_sync(0xffffffffu, mine[b], 1);
+                const float x0 = par ? other : mine[b], x1 = par ? mine[b] : other;
+                uw[b][0] = pack2(x0, x0);
+                uw[b][1] = pack2(x1, x1);
+            }
+            const f32x2 dec = pack2(cc.w, cc.w);
+#pragma unroll
+            for (int i = 0; i < NI; i++) {
+#pragma unroll
+                for (int c = 0; c < 2; c++) {
+                    S[c][i][0] = mul2(dec, S[c][i][0]);
+                    S[c][i][1] = mul2(dec, S[c][i][1]);
+                }
+#pragma unroll
+                for (int b = 0; b < BT; b++) {
+                    const Quad k = *reinterpret_cast<const Quad *>(&kt[b][l * 4 + 32 * i]);
+#pragma unroll
+                    for (int c = 0; c < 2; c++) {
+                        S[c][i][0] = fma2(k.lo, uw[b][c], S[c][i][0]);
+                        S[c][i][1] = fma2(k.hi, uw[b][c], S[c][i][1]);
+                    }
+                }
+            }
+        }
+        __syncthreads();
+    }
+    pg_cp_wait<0>();
+#pragma unroll
+    for (int c = 0; c < 2; c++) {
+        if (c0 + col + c >= s.V) continue;
+#pragma unroll
+        for (int i = 0; i < NI; i++)
+#pragma unroll
+            for (int j = 0; j < 2; j++) {
+                const int r = l * 4 + 32 * i + 2 * j;
+                float lo, hi;
+                asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(S[c][i][j]));
+                if (r < s.D) st[(int64_t)r * s.vs + c] = lo;
+                if (r + 1 < s.D) st[(int64_t)(r + 1) * s.vs + c] = hi;
             }
     }
+}
+
+template <int NI>
+int32_t run_scan(pg_ctx *ctx, const DeltaShape &s, const pg_batch *bt, const DeltaWork &w, float *state)
+{
+    constexpr int smem = ScanTile<NI>::STAGES * (int)sizeof(typename ScanTile<NI>::Stage);
+    static std::atomic<uint64_t> set{0};
+    PG_CUDA(pg_max_smem_once(delta_scan_kernel<NI>, smem, ctx->device, set));
+    return launch_pdl(ctx, delta_scan_kernel<NI>, dim3((unsigned)((s.V + 31) / 32), (unsigned)s.H, (unsigned)bt->seqs), dim3(128), (size_t)smem, s, *bt, w, state);
+}
+
+template <int TAPS>
+int32_t run_prep(pg_ctx *ctx, const DeltaShape &s, const pg_batch *bt, const float *proj, int64_t ldp, const float *ring, const DeltaWork &w)
+{
+    const size_t smem = ((size_t)BT * 2 * s.G * s.D + 16 * s.G) * 4;
+    PG_REQUIRE(smem <= 220 * 1024, "delta: too many query / key channels");
+    static std::atomic<uint64_t> set{0};
+    PG_CUDA(pg_max_smem_once(delta_prep_kernel<TAPS>, 220 * 1024, ctx->device, set));
+    return launch_pdl(ctx, delta_prep_kernel<TAPS>, dim3((unsigned)((bt->max_len + BT - 1) / BT), (unsigned)bt->seqs), dim3(256), smem, s, *bt, proj, ldp, ring, w);
 }
 
 // a CTA per token: o / rms(o) * norm * silu(gate) per head; the sequence's last taps - 1 tokens also store their
@@ -411,7 +601,8 @@ PG_API int64_t pg_delta_work_floats(const pg_delta *p, int64_t max_rows)
 {
     if (!p || max_rows < 0) return 0;
     const int64_t G = p->kv_heads, H = p->heads, D = p->dim, V = p->vdim;
-    return max_rows * (2 * G * D + 2 * H * V + G + 2 * H) + 32;
+    // (a block of four tokens per sequence may be a single token)
+    return max_rows * (2 * G * D + 2 * H * V) + (max_rows + 8) * H * 32 + 64;
 }
 
 PG_API int32_t pg_delta_run(pg_ctx *ctx, const pg_delta *p, const pg_batch *batch, const float *d_proj, int64_t ldp, float *d_ring, float *d_state,
@@ -440,28 +631,29 @@ PG_API int32_t pg_delta_run(pg_ctx *ctx, const pg_delta *p, const pg_batch *batc
     w.k = at, at += pg_up((int64_t)M * s.G * s.D, 4);
     w.v = at, at += pg_up((int64_t)M * s.H * s.V, 4);
     w.o = at, at += pg_up((int64_t)M * s.H * s.V, 4);
-    w.kq = at, at += pg_up((int64_t)M * s.G, 4);
-    w.beta = at, at += pg_up((int64_t)M * s.H, 4);
-    w.dec = at;
-    const size_t smem = (size_t)2 * s.G * s.D * 4;
-    PG_REQUIRE(smem <= 200 * 1024, "delta: too many query / key channels");
-    static std::atomic<uint64_t> set{0};
-    PG_CUDA(pg_max_smem_once(delta_prep_kernel, 200 * 1024, ctx->device, set));
-    int32_t rc = launch_pdl(ctx, delta_prep_kernel, dim3((unsigned)M), dim3(256), smem, s, *batch, d_proj, ldp, (const float *)d_ring, w);
-    if (rc != PG_OK) return rc;
-    const dim3 g((unsigned)((s.V + 31) / 32), (unsigned)s.H, (unsigned)batch->seqs);
-    if (s.D <= 32)
-        rc = launch_pdl(ctx, delta_scan_kernel<1>, g, dim3(256), 0, s, *batch, w, d_state);
-    else if (s.D <= 64)
-        rc = launch_pdl(ctx, delta_scan_kernel<2>, g, dim3(256), 0, s, *batch, w, d_state);
-    else if (s.D <= 96)
-        rc = launch_pdl(ctx, delta_scan_kernel<3>, g, dim3(256), 0, s, *batch, w, d_state);
-    else if (s.D <= 128)
-        rc = launch_pdl(ctx, delta_scan_kernel<4>, g, dim3(256), 0, s, *batch, w, d_state);
-    else if (s.D <= 192)
-        rc = launch_pdl(ctx, delta_scan_kernel<6>, g, dim3(256), 0, s, *batch, w, d_state);
+    w.coef = at;
+    int32_t rc;
+    if (s.taps == 2)
+        rc = run_prep<2>(ctx, s, batch, d_proj, ldp, d_ring, w);
+    else if (s.taps == 3)
+        rc = run_prep<3>(ctx, s, batch, d_proj, ldp, d_ring, w);
+    else if (s.taps == 4)
+        rc = run_prep<4>(ctx, s, batch, d_proj, ldp, d_ring, w);
     else
-        rc = launch_pdl(ctx, delta_scan_kernel<8>, g, dim3(256), 0, s, *batch, w, d_state);
+        rc = run_prep<0>(ctx, s, batch, d_proj, ldp, d_ring, w);
+    if (rc != PG_OK) return rc;
+    if (s.D <= 32)
+        rc = run_scan<1>(ctx, s, batch, w, d_state);
+    else if (s.D <= 64)
+        rc = run_scan<2>(ctx, s, batch, w, d_state);
+    else if (s.D <= 96)
+        rc = run_scan<3>(ctx, s, batch, w, d_state);
+    else if (s.D <= 128)
+        rc = run_scan<4>(ctx, s, batch, w, d_state);
+    else if (s.D <= 192)
+        rc = run_scan<6>(ctx, s, batch, w, d_state);
+    else
+        rc = run_scan<8>(ctx, s, batch, w, d_state);
     if (rc != PG_OK) return rc;
     if (dtype == PG_BF16)
         return launch_pdl(ctx, delta_out_kernel<bf16>, dim3((unsigned)M), dim3(256), 0, s, *batch, d_proj, ldp, w, d_ring, (bf16 *)d_out, ldo);

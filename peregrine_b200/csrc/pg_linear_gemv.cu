@@ -8,9 +8,9 @@
 //     rows and the eight up rows behind them, whose sums land in the same lanes, so the gate is applied in registers.
 //   * Products run on mma.sync m16n8k16 with a permuted K (a lane's 16 contiguous bytes of a weight row and of an
 //     activation row feed two MMAs).  The parts of a tile meet in shared memory, added in a fixed order.
-//   * K beyond 16 x 256 elements: clusters of 2, 4 or 8 CTAs work on the same tiles, each with its part of K; the other
-//     CTAs store their sums into cells of their own in the first CTA's shared memory, one cluster barrier per round, and
-//     the first CTA adds the cells in a fixed order.
+//   * K beyond 16 x 256 elements (SPLIT): sp CTAs take the same tiles, each with its part of K, and write their raw sums to
+//     slabs of their own; the last of them to finish (a ticket per group) adds the slabs in a fixed order and writes the
+//     outputs of all the group's tiles.  Nobody waits for anybody.
 //   * ROUTED: the rows come in blocks of 16 that share an expert; the tiles of all blocks form one list, of which a CTA
 //     takes a contiguous stretch.
 //
@@ -32,26 +32,23 @@ constexpr int GV_STRIDE = GV_KW_MAX * 2 + 64;             // bytes per ring row:
 constexpr int GV_SLOT = 8 * GV_STRIDE;
 constexpr int GV_RING = GV_WARPS * GV_SLOTS * GV_SLOT;
 
-// shared memory: ring | partial sums [2][16 warps][32 lanes][4 NT] | cells [2][groups][cs - 1][32][4 NT] | barriers
-template <int ACT, bool HI, bool ROUTED, bool CL, typename TY>
+// shared memory: ring | partial sums [2][16 warps][32 lanes][4 NT] | barriers
+// slabs (SPLIT): [sp][items][32 lanes][4 NT]
+template <int ACT, bool HI, bool ROUTED, bool SPLIT, typename TY>
 __global__ void __launch_bounds__(GV_THREADS, 1)
     linear_gemv_kernel(const bf16 *__restrict__ a, int M, const bf16 *__restrict__ w, int N, int K, int kw, int KW, int KH, float limit,
-                       TY *__restrict__ y, int64_t ldy, const PgRouted rt, int32_t *status, unsigned long long limit_ns)
+                       TY *__restrict__ y, int64_t ldy, const PgRouted rt, int sp, float *slabs, unsigned int *tickets, int32_t *status,
+                       unsigned long long limit_ns)
 {
     constexpr int NT = ACT == PG_ACT_NONE ? 1 : 2;
     constexpr int CELL = 4 * NT;                          // floats per lane
     extern __shared__ __align__(128) unsigned char smem[];
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, r = lane >> 2, t = lane & 3;
-    uint32_t my_rank = 0, cs = 1;
-    if (CL) {
-        my_rank = cl_rank();
-        cs = cl_size();
-    }
+    const int my_part = SPLIT ? (int)blockIdx.x % sp : 0;
     const int groups = GV_WARPS / kw, slot_idx = warp / kw, kpart = warp - slot_idx * kw;
     float *part = reinterpret_cast<float *>(smem + GV_RING);
-    float *cells = part + 2 * GV_WARPS * 32 * CELL;
-    unsigned char *tail = reinterpret_cast<unsigned char *>(cells + (CL ? 2 * groups * (int)(cs - 1) * 32 * CELL : 0));
+    unsigned char *tail = reinterpret_cast<unsigned char *>(part + 2 * GV_WARPS * 32 * CELL);
     const uint32_t bars = pg_smem(tail), my_bar = bars + (uint32_t)warp * (GV_SLOTS * 8);
     volatile int *abort_flag = reinterpret_cast<volatile int *>(tail + GV_WARPS * GV_SLOTS * 8);
     const uint32_t ring = pg_smem(smem) + (uint32_t)warp * (GV_SLOTS * GV_SLOT);
@@ -62,17 +59,16 @@ __global__ void __launch_bounds__(GV_THREADS, 1)
     }
     __syncthreads();
 
-    const int ka0 = CL ? (int)my_rank * KH : 0;
+    const int ka0 = my_part * KH;
     const int k0 = ka0 + kpart * KW;
-    const int klen = max(0, min(KW, (CL ? min(K, ka0 + KH) : K) - k0));   // a multiple of 32; 0 only in a short last range
+    const int klen = max(0, min(KW, min(K, ka0 + KH) - k0));   // a multiple of 32; 0 only in a short last range
     const int tiles = (N + 8 * NT - 1) / (8 * NT);
-    const int64_t unit = blockIdx.x / cs, units = gridDim.x / cs;
+    const int64_t unit = SPLIT ? blockIdx.x / sp : blockIdx.x, units = SPLIT ? gridDim.x / sp : gridDim.x;
     if (ROUTED) asm volatile("griddepcontrol.wait;" ::: "memory");
     const int nblk = ROUTED ? __ldcg(rt.blocks) : 1;
     const int64_t items = (int64_t)nblk * tiles, per = (items + units * groups - 1) / (units * groups);
     const int64_t first = (unit * groups + slot_idx) * per;
     const int mine = (int)max((int64_t)0, min(per, items - first));
-    const int rounds = (int)max((int64_t)0, min(per, items - unit * groups * per));   // of the CTA: those of its slot 0
     const int total = klen > 0 ? mine * NT : 0;
 
     // fill f: item f / NT, half f % NT
@@ -93,23 +89,38 @@ __global__ void __launch_bounds__(GV_THREADS, 1)
     for (int f = 0; f < GV_SLOTS; f++)
         if (f < total) issue(f);
     if (!ROUTED) asm volatile("griddepcontrol.wait;" ::: "memory");
-    if (CL) cl_sync();                                    // every CTA of the cluster runs before anyone stores into it
+
+    // outputs of a tile; lane: rows r and r + 8, columns 2t and 2t + 1
+    auto finish = [&](const float (&acc)[NT][4], int blk, int tile) {
+#pragma unroll
+        for (int h = 0; h < (HI ? 2 : 1); h++) {
+            const int m = (ROUTED ? blk * PG_ROUTE_SMALL : 0) + r + 8 * h;
+            if (ROUTED ? (__ldcg(rt.row_pair + m) < 0) : (m >= M)) continue;
+            const int n = tile * 8 + 2 * t, nmax = N / NT;
+            float v0 = acc[0][2 * h], v1 = acc[0][2 * h + 1];
+            if (ACT != PG_ACT_NONE) {
+                v0 = pg_glu<ACT>(v0, acc[NT - 1][2 * h], limit);
+                v1 = pg_glu<ACT>(v1, acc[NT - 1][2 * h + 1], limit);
+            }
+            if (n < nmax) pg_put(y + m * ldy + n, v0);
+            if (n + 1 < nmax) pg_put(y + m * ldy + n + 1, v1);
+        }
+    };
 
     uint4 lo[GV_KSTEPS], hi[GV_KSTEPS];
     const int steps = klen >> 5;
     int have = -1;                                        // the row block whose activations the registers hold
     bool ok = true;
     int f = 0;
-    for (int j = 0; j < (CL ? rounds : mine); j++) {
+    for (int j = 0; j < mine; j++) {
         float acc[NT][4];
 #pragma unroll
         for (int h = 0; h < NT; h++)
 #pragma unroll
             for (int i = 0; i < 4; i++) acc[h][i] = 0.0f;
-        const bool busy = j < mine;
         const int64_t it = first + j;
         const int blk = ROUTED ? (int)(it / tiles) : 0, tile = (int)(it - (int64_t)blk * tiles);
-        if (busy && klen > 0) {
+        if (klen > 0) {
             if (blk != have) {
                 have = blk;
                 int64_t r0 = r, r1 = r + 8;
@@ -148,7 +159,7 @@ __global__ void __launch_bounds__(GV_THREADS, 1)
                 }
             }
         }
-        if (busy && kw > 1) {
+        if (kw > 1) {
             float *mine_at = part + ((size_t)((j & 1) * GV_WARPS + warp) * 32 + lane) * CELL;
             if (kpart != 0) {
 #pragma unroll
@@ -168,43 +179,48 @@ __global__ void __launch_bounds__(GV_THREADS, 1)
                 }
             }
         }
-        if (CL) {
-            float *cell = cells + ((size_t)((j & 1) * groups + slot_idx) * (cs - 1) * 32 + lane) * CELL;   // + (rank - 1) * 32 * CELL
-            if (busy && my_rank != 0 && kpart == 0) {
-                float *dst = cell + (size_t)(my_rank - 1) * 32 * CELL;
+        if (SPLIT) {
+            if (kpart == 0) {
+                float4 *dst = reinterpret_cast<float4 *>(slabs + (((int64_t)my_part * items + it) * 32 + lane) * CELL);
+#pragma unroll
+                for (int h = 0; h < NT; h++) dst[h] = make_float4(acc[h][0], acc[h][1], acc[h][2], acc[h][3]);
+            }
+        } else if (kpart == 0 && ok) {
+            finish(acc, blk, tile);
+        }
+    }
+    if (SPLIT) {
+        __shared__ int last_in;
+        __threadfence();
+        __syncthreads();
+        if (threadIdx.x == 0) {
+            __threadfence();
+            last_in = atomicAdd(tickets + unit, 1u) == (unsigned)(sp - 1);
+            if (last_in) tickets[unit] = 0;
+        }
+        __syncthreads();
+        if (last_in) {
+            __threadfence();
+            const int64_t i0 = unit * groups * per, i1 = min(items, i0 + (int64_t)groups * per);
+            for (int64_t it = i0 + warp; it < i1; it += GV_WARPS) {
+                float acc[NT][4];
 #pragma unroll
                 for (int h = 0; h < NT; h++)
 #pragma unroll
-                    for (int i = 0; i < 4; i++) cl_store_f32(dst + h * 4 + i, 0, acc[h][i]);
-            }
-            cl_sync();
-            if (busy && my_rank == 0 && kpart == 0) {
-                for (uint32_t c = 0; c + 1 < cs; c++) {
+                    for (int i = 0; i < 4; i++) acc[h][i] = 0.0f;
+                for (int q = 0; q < sp; q++) {
+                    const float4 *src = reinterpret_cast<const float4 *>(slabs + (((int64_t)q * items + it) * 32 + lane) * CELL);
 #pragma unroll
                     for (int h = 0; h < NT; h++) {
-                        const float4 v = reinterpret_cast<const float4 *>(cell + (size_t)c * 32 * CELL)[h];
+                        const float4 v = __ldcg(src + h);
                         acc[h][0] += v.x;
                         acc[h][1] += v.y;
                         acc[h][2] += v.z;
                         acc[h][3] += v.w;
                     }
                 }
-            }
-        }
-        if (busy && kpart == 0 && ok && (!CL || my_rank == 0)) {
-            // lane: rows r and r + 8, columns 2t and 2t + 1 of the tile
-#pragma unroll
-            for (int h = 0; h < (HI ? 2 : 1); h++) {
-                const int m = (ROUTED ? blk * PG_ROUTE_SMALL : 0) + r + 8 * h;
-                if (ROUTED ? (__ldcg(rt.row_pair + m) < 0) : (m >= M)) continue;
-                const int n = tile * 8 + 2 * t, nmax = N / NT;
-                float v0 = acc[0][2 * h], v1 = acc[0][2 * h + 1];
-                if (ACT != PG_ACT_NONE) {
-                    v0 = pg_glu<ACT>(v0, acc[NT - 1][2 * h], limit);
-                    v1 = pg_glu<ACT>(v1, acc[NT - 1][2 * h + 1], limit);
-                }
-                if (n < nmax) pg_put(y + m * ldy + n, v0);
-                if (n + 1 < nmax) pg_put(y + m * ldy + n + 1, v1);
+                const int blk = ROUTED ? (int)(it / tiles) : 0;
+                finish(acc, blk, (int)(it - (int64_t)blk * tiles));
             }
         }
     }
@@ -216,70 +232,72 @@ __global__ void __launch_bounds__(GV_THREADS, 1)
     }
 }
 
-template <int ACT, bool HI, bool ROUTED, bool CL, typename TY>
-int32_t gv_launch(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int M, int kw, int KW, int KH, int grid, int cs, float limit, TY *y, int64_t ldy,
+constexpr size_t GV_TICKET_BYTES = 64 * 1024;   // the head of the context's split-K workspace: zero between calls
+
+template <int ACT, bool HI, bool ROUTED, bool SPLIT, typename TY>
+int32_t gv_launch(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int M, int kw, int KW, int KH, int grid, int sp, float limit, TY *y, int64_t ldy,
                   const PgRouted &rt)
 {
     constexpr int NT = ACT == PG_ACT_NONE ? 1 : 2;
-    auto kern = linear_gemv_kernel<ACT, HI, ROUTED, CL, TY>;
-    const int smem = GV_RING + (2 * GV_WARPS + (CL ? 2 * (GV_WARPS / kw) * (cs - 1) : 0)) * 32 * 4 * NT * 4 + GV_WARPS * GV_SLOTS * 8 + 16;
-    PG_REQUIRE(smem <= 227 * 1024, "linear: shared memory of the streaming form");
+    auto kern = linear_gemv_kernel<ACT, HI, ROUTED, SPLIT, TY>;
+    const int smem = GV_RING + 2 * GV_WARPS * 32 * 4 * NT * 4 + GV_WARPS * GV_SLOTS * 8 + 16;
+    static_assert(GV_RING + 2 * GV_WARPS * 32 * 8 * 4 + GV_WARPS * GV_SLOTS * 8 + 16 <= 226 * 1024, "shared memory of the streaming form");
     static std::atomic<uint64_t> smem_set{0};
-    PG_CUDA(pg_max_smem_once(kern, 227 * 1024, ctx->device, smem_set));
-    return launch_pdl_cluster(ctx, kern, dim3((unsigned)grid), dim3(GV_THREADS), (size_t)smem, cs, a, M, lin->w, (int)lin->n, (int)lin->k, kw, KW, KH,
-                              limit, y, ldy, rt, ctx->d_status, ctx->wait_limit_ns);
+    PG_CUDA(pg_max_smem_once(kern, 226 * 1024, ctx->device, smem_set));
+    unsigned int *tickets = reinterpret_cast<unsigned int *>(ctx->splitk);
+    float *slabs = SPLIT ? reinterpret_cast<float *>(reinterpret_cast<unsigned char *>(ctx->splitk) + GV_TICKET_BYTES) : nullptr;
+    return launch_pdl(ctx, kern, dim3((unsigned)grid), dim3(GV_THREADS), (size_t)smem, a, M, lin->w, (int)lin->n, (int)lin->k, kw, KW, KH, limit, y, ldy, rt,
+                      sp, slabs, tickets, ctx->d_status, ctx->wait_limit_ns);
 }
 
-inline int gv_cluster(int64_t k)
-{
-    for (int cs = 1; cs <= 8; cs *= 2)
-        if (k <= (int64_t)cs * GV_WARPS * GV_KW_MAX) return cs;
-    return 0;
-}
+// parts of K that CTAs share
+inline int gv_parts(int64_t k) { return (int)((k + GV_WARPS * GV_KW_MAX - 1) / (GV_WARPS * GV_KW_MAX)); }
 
 }  // namespace
 
-bool pgk_linear_gemv_supports(const pg_linear *lin, int64_t m) { return m >= 1 && m <= 16 && gv_cluster(lin->k) != 0 && lin->n < (1 << 30); }
+bool pgk_linear_gemv_supports(const pg_linear *lin, int64_t m) { return m >= 1 && m <= 16 && gv_parts(lin->k) <= 16 && lin->n < (1 << 30); }
 
 int32_t pgk_linear_gemv(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int64_t m, int act, float limit, void *y, int y_dtype, int64_t ldy,
                         const PgRouted *routed, int64_t max_blocks)
 {
     const int K = (int)lin->k, nt = act == PG_ACT_NONE ? 1 : 2;
     const int64_t items = ((lin->n + 8 * nt - 1) / (8 * nt)) * (routed ? max_blocks : 1);
-    const int cs = gv_cluster(K);
-    PG_REQUIRE(cs != 0, "linear: K too long for the streaming form");
-    const int KH = cs > 1 ? (int)pg_up((K + cs - 1) / cs, 32) : K;
-    const int64_t units = ctx->sm_count / cs;
-    // parts of K: as few as registers allow, more while every (tile, part) still finds a warp of its own
+    const int sp = gv_parts(K);
+    const int KH = sp > 1 ? (int)pg_up((K + sp - 1) / sp, 32) : K;
+    const int64_t units = ctx->sm_count / sp;
+    if (sp > 1) {
+        const int32_t rc = pg_splitk_reserve(ctx, GV_TICKET_BYTES + (size_t)sp * (size_t)items * 32 * 4 * nt * sizeof(float));
+        if (rc != PG_OK) return rc;
+    }
+    // parts of a CTA's K: as few as registers allow, more while every (tile, part) still finds a warp of its own
     int kw = 1;
     while (kw < GV_WARPS && (KH + kw - 1) / kw > GV_KW_MAX) kw *= 2;
     while (kw < GV_WARPS && KH / (kw * 2) >= 64 && items * (kw * 2) <= units * GV_WARPS) kw *= 2;
-    auto part = [&](int p) { return (int)pg_up((KH + p - 1) / p, 32); };
-    const int KW = part(kw);
+    const int KW = (int)pg_up((KH + kw - 1) / kw, 32);
     PG_REQUIRE(KW <= GV_KW_MAX, "linear: K part too long");
     const int groups = GV_WARPS / kw;
-    const int grid = (int)std::min<int64_t>(units, (items + groups - 1) / groups) * cs;
+    const int grid = (int)std::min<int64_t>(units, (items + groups - 1) / groups) * sp;
     static const PgRouted no_route = {};
     const PgRouted &rt = routed ? *routed : no_route;
     const bool hi = m > 8 || routed;
     const int M = (int)m;
-#define PG_GV(ACT, HI, RT, CL, TY) return gv_launch<ACT, HI, RT, CL, TY>(ctx, lin, a, M, kw, KW, KH, grid, cs, limit, (TY *)y, ldy, rt)
-#define PG_GV_CL(ACT, HI, RT, TY)          \
-    do {                                   \
-        if (cs > 1) PG_GV(ACT, HI, RT, true, TY); \
-        PG_GV(ACT, HI, RT, false, TY);     \
+#define PG_GV(ACT, HI, RT, SP, TY) return gv_launch<ACT, HI, RT, SP, TY>(ctx, lin, a, M, kw, KW, KH, grid, sp, limit, (TY *)y, ldy, rt)
+#define PG_GV_SP(ACT, HI, RT, TY)                 \
+    do {                                          \
+        if (sp > 1) PG_GV(ACT, HI, RT, true, TY); \
+        PG_GV(ACT, HI, RT, false, TY);            \
     } while (0)
 #define PG_GV_ACT(ACT, TY)                           \
     do {                                             \
-        if (routed) PG_GV_CL(ACT, true, true, TY);   \
-        if (hi) PG_GV_CL(ACT, true, false, TY);      \
-        PG_GV_CL(ACT, false, false, TY);             \
+        if (routed) PG_GV_SP(ACT, true, true, TY);   \
+        if (hi) PG_GV_SP(ACT, true, false, TY);      \
+        PG_GV_SP(ACT, false, false, TY);             \
     } while (0)
     if (act == PG_ACT_GELU_TANH_GLU) PG_GV_ACT(PG_ACT_GELU_TANH_GLU, bf16);
     if (act == PG_ACT_CLAMPED_SWISH_GLU) PG_GV_ACT(PG_ACT_CLAMPED_SWISH_GLU, bf16);
     if (y_dtype == PG_BF16) PG_GV_ACT(PG_ACT_NONE, bf16);
     PG_GV_ACT(PG_ACT_NONE, float);
 #undef PG_GV
-#undef PG_GV_CL
+#undef PG_GV_SP
 #undef PG_GV_ACT
 }

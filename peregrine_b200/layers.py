@@ -185,7 +185,7 @@ class Attention:
         temp = p.get("q_temp") or {}
         self.dp, self.vp = up(D, 16), up(V, 16)
         f32 = d.torch.float32
-        self.c = _lib.PgAttention(H, G, D, V, self.cap, float(eps), float(p["scale"]), float(temp.get("coef", 0.0)), float(temp.get("every", 0.0)), int(sink),
+        self.c = _lib.PgAttention(H, G, D, V, self.cap, 0, float(eps), float(p["scale"]), float(temp.get("coef", 0.0)), float(temp.get("every", 0.0)), int(sink),
                                   self.qn.data_ptr(), self.kn.data_ptr(), 0, 0, 0)
         d.buffer("attn.part", 1, max(1, d.lib.pg_attention_part_floats(d.gpu.handle, C.byref(self.c), max_seqs)), f32)
         d.buffer("attn.tickets", 1, max_seqs * G * ((H // G + 15) // 16), d.torch.int32)
@@ -206,6 +206,7 @@ class Attention:
         self.c.d_q = d.buffer("attn.q", self.H * self.dp).data_ptr()
         self.c.d_part = d.buffer("attn.part", 1, 1, d.torch.float32).data_ptr()
         self.c.d_tickets = d.buffer("attn.tickets", 1, 1, d.torch.int32).data_ptr()
+        self.c.slots = state["k"].shape[0]
         d.check(d.lib.pg_attention_run(d.gpu.handle, C.byref(self.c), C.byref(batch.c), proj.data_ptr(), proj.stride(0), state["k"].data_ptr(),
                                        state["v"].data_ptr(), mixed.data_ptr(), d.code, mixed.stride(0)))
         self.out.run(mixed, rows, y)
