@@ -336,7 +336,7 @@ __global__ void __launch_bounds__(WARPS * 32)
 // ---- one token per sequence: grid (slices, G, rows), 4 warps ------------------------------------------------------
 constexpr int AS_WARPS = 4, AS_STAGES = 3, AS_SLICES = 64;
 
-// part [rows][G][slices][16][vp + 2]: sums, then maximum (log 2 units) and denominator of each head
+// part [rows][G][slices][16][vp + 4]: sums, then maximum (log 2 units) and denominator of each head
 template <int DC, int VC, bool FUSED>
 __global__ void __launch_bounds__(AS_WARPS * 32)
     attn_step_kernel(const AttnShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, const bf16 *__restrict__ q, bf16 *kc, bf16 *vc,
@@ -354,6 +354,7 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
     const int kstride = s.dp * 2 + 16, vstride = s.vp * 2 + 16, stage = 16 * (kstride + vstride);
     const uint32_t ring = pg_smem(smem) + (uint32_t)warp * AS_STAGES * stage, bar = pg_smem(bars) + (uint32_t)warp * AS_STAGES * 8;
     bf16 *qs = reinterpret_cast<bf16 *>(smem + AS_WARPS * AS_STAGES * stage);   // [16][dp + 8]
+    bf16 *k_new = qs + 16 * (s.dp + 8), *v_new = k_new + s.dp;                  // the newest position's key and value
     float *mg = reinterpret_cast<float *>(smem);                                // the merge reuses the rings
     if (threadIdx.x == 0) {
         for (int i = 0; i < AS_WARPS * AS_STAGES; i++) pg_mbar_init(pg_smem(bars) + 8 * i, 1);
@@ -395,16 +396,12 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
     auto prime = [&]() {
         for (int i = 0; i < AS_STAGES && i < mine; i++) fetch(i);
     };
-    if (!newest) prime();
+    prime();
     const float *row = proj + (int64_t)b * ldp;
-    if (newest && warp == 2) {
-        head_norm(row + (int64_t)(s.H + g) * s.D, s.kn, s.D, s.dp, s.eps, 1.0f, kb + (int64_t)pos * s.dp, lane);
-        asm volatile("fence.proxy.async.global;" ::: "memory");
-    }
+    if (newest && warp == 2) head_norm(row + (int64_t)(s.H + g) * s.D, s.kn, s.D, s.dp, s.eps, 1.0f, k_new, lane);
     if (newest && warp == 3) {
         const float *src = row + (int64_t)(s.H + s.G) * s.D + (int64_t)g * s.V;
-        for (int c = lane; c < s.vp; c += 32) pg_put(vb + (int64_t)pos * s.vp + c, c < s.V ? __ldcg(src + c) : 0.0f);
-        asm volatile("fence.proxy.async.global;" ::: "memory");
+        for (int c = lane; c < s.vp; c += 32) pg_put(v_new + c, c < s.V ? __ldcg(src + c) : 0.0f);
     }
     for (int h = warp; h < heads; h += AS_WARPS) {
         bf16 *dst = qs + h * (s.dp + 8);
@@ -415,7 +412,16 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
         }
     }
     __syncthreads();
-    if (newest) prime();                                  // the row that this CTA has just stored is among them
+    if (newest) {
+        // appended for later steps; this step takes the row from shared memory (below)
+        for (int i = threadIdx.x; i < (s.dp + s.vp) / 2; i += AS_WARPS * 32) {
+            const uint32_t x = reinterpret_cast<const uint32_t *>(k_new)[i];
+            if (i < s.dp / 2)
+                reinterpret_cast<uint32_t *>(kb + (int64_t)pos * s.dp)[i] = x;
+            else
+                reinterpret_cast<uint32_t *>(vb + (int64_t)pos * s.vp)[i - s.dp / 2] = x;
+        }
+    }
     uint32_t qf[DC][4];
     {
         const uint32_t qb = pg_smem(qs);
@@ -437,6 +443,14 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
         if (!ok) break;
         const int j0 = t0 + 16 * (warp + AS_WARPS * i);
         const uint32_t kt = ring + (uint32_t)(i % AS_STAGES) * stage, vt = kt + 16 * kstride;
+        if (newest && j0 + 16 > pos) {
+            // the copies brought what the cache held at the newest position: put the new row in its place
+            unsigned char *at = smem + (size_t)warp * AS_STAGES * stage + (size_t)(i % AS_STAGES) * stage;
+            for (int x = lane; x < s.dp / 2; x += 32) reinterpret_cast<uint32_t *>(at + (pos - j0) * kstride)[x] = reinterpret_cast<const uint32_t *>(k_new)[x];
+            for (int x = lane; x < s.vp / 2; x += 32)
+                reinterpret_cast<uint32_t *>(at + 16 * kstride + (pos - j0) * vstride)[x] = reinterpret_cast<const uint32_t *>(v_new)[x];
+            __syncwarp();
+        }
         float sc[2][4] = {};
         scores16<DC>(qf, nk, kt, kstride, 0, lane, sc[0], sc[1]);
         float b0 = -INFINITY, b1 = -INFINITY;
@@ -495,8 +509,8 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
         l1 += __shfl_xor_sync(0xffffffffu, l1, x);
     }
     __syncthreads();                                      // the rings are free
-    // warps meet in shared memory: [warp][16][vp + 2]
-    const int ms = s.vp + 2;
+    // warps meet in shared memory: [warp][16][vp + 4]
+    const int ms = s.vp + 4;
     float *w0 = mg + ((size_t)warp * 16 + r) * ms, *w1 = w0 + 8 * ms;
 #pragma unroll
     for (int i = 0; i < VC; i++) {
@@ -512,29 +526,37 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
     __syncthreads();
     const int64_t unit = ((int64_t)b * gridDim.y + blockIdx.y);
     float *mine_part = part + (unit * S + split) * 16 * ms;
-    const int nh = heads * s.vp;
-    for (int x = threadIdx.x; x < nh; x += AS_WARPS * 32) {
-        const int h = x / s.vp, c = x - h * s.vp;
+    const int vq = s.vp / 4;
+    for (int x = threadIdx.x; x < heads * vq; x += AS_WARPS * 32) {
+        const int h = x / vq, c = (x - h * vq) * 4;
         float m = -INFINITY;
 #pragma unroll
         for (int w = 0; w < AS_WARPS; w++) m = fmaxf(m, mg[((size_t)w * 16 + h) * ms + s.vp]);
-        float a = 0.0f, l = 0.0f;
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+        float l = 0.0f;
 #pragma unroll
         for (int w = 0; w < AS_WARPS; w++) {
             const float *at = mg + ((size_t)w * 16 + h) * ms;
             const float f = exp2f(at[s.vp] - m);          // 0 for a warp without keys
-            a = fmaf(f, at[c], a);
+            const float4 v = *reinterpret_cast<const float4 *>(at + c);
+            a.x = fmaf(f, v.x, a.x), a.y = fmaf(f, v.y, a.y), a.z = fmaf(f, v.z, a.z), a.w = fmaf(f, v.w, a.w);
             l = fmaf(f, at[s.vp + 1], l);
         }
         if (used == 1) {
+            float f = 1.0f;
             if (s.sink) {
-                const float mm = fmaxf(m, 0.0f), f = exp2f(m - mm);
-                a *= f;
+                const float mm = fmaxf(m, 0.0f);
+                f = exp2f(m - mm);
                 l = l * f + exp2f(-mm);
             }
-            if (c < s.V) pg_put(out + (int64_t)b * ldo + (int64_t)(h0 + h) * s.V + c, __fdiv_rn(a, l));
+            f = __fdiv_rn(f, l);
+            bf16 *dst = out + (int64_t)b * ldo + (int64_t)(h0 + h) * s.V + c;
+            const float y[4] = {a.x * f, a.y * f, a.z * f, a.w * f};
+#pragma unroll
+            for (int i = 0; i < 4; i++)
+                if (c + i < s.V) pg_put(dst + i, y[i]);
         } else {
-            mine_part[(size_t)h * ms + c] = a;
+            *reinterpret_cast<float4 *>(mine_part + (size_t)h * ms + c) = a;
             if (c == 0) *reinterpret_cast<float2 *>(mine_part + (size_t)h * ms + s.vp) = make_float2(m, l);
         }
     }
@@ -572,13 +594,21 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
         if (lane == 0) denom[h] = __fdiv_rn(1.0f, l);
     }
     __syncthreads();
-    for (int x = threadIdx.x; x < heads * s.V; x += AS_WARPS * 32) {
-        const int h = x / s.V, c = x - h * s.V;
+    for (int x = threadIdx.x; x < heads * vq; x += AS_WARPS * 32) {
+        const int h = x / vq, c = (x - h * vq) * 4;
         const float *at = parts + (size_t)h * ms + c;
-        float a = 0.0f;
-#pragma unroll 8
-        for (int k = 0; k < used; k++) a = fmaf(weight[h][k], __ldcg(at + (size_t)k * 16 * ms), a);
-        pg_put(out + (int64_t)b * ldo + (int64_t)(h0 + h) * s.V + c, a * denom[h]);
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 16
+        for (int k = 0; k < used; k++) {
+            const float4 v = __ldcg(reinterpret_cast<const float4 *>(at + (size_t)k * 16 * ms));
+            const float f = weight[h][k];
+            a.x = fmaf(f, v.x, a.x), a.y = fmaf(f, v.y, a.y), a.z = fmaf(f, v.z, a.z), a.w = fmaf(f, v.w, a.w);
+        }
+        bf16 *dst = out + (int64_t)b * ldo + (int64_t)(h0 + h) * s.V + c;
+        const float f = denom[h], y[4] = {a.x * f, a.y * f, a.z * f, a.w * f};
+#pragma unroll
+        for (int i = 0; i < 4; i++)
+            if (c + i < s.V) pg_put(dst + i, y[i]);
     }
 }
 
@@ -619,7 +649,7 @@ int32_t run_step(pg_ctx *ctx, const AttnShape &s, const pg_batch *bt, const floa
 {
     const int stage = 16 * ((s.dp + s.vp) * 2 + 32);
     const int rings = AS_WARPS * AS_STAGES * stage;
-    const int smem = std::max(rings + 16 * (s.dp + 8) * 2, AS_WARPS * 16 * (s.vp + 2) * 4);
+    const int smem = std::max(rings + 16 * (s.dp + 8) * 2 + (s.dp + s.vp) * 2, AS_WARPS * 16 * (s.vp + 4) * 4);
     static std::atomic<uint64_t> set{0};
     PG_CUDA(pg_max_smem_once(attn_step_kernel<DC, VC, FUSED>, 220 * 1024, ctx->device, set));
     const int ht = (s.rep + 15) / 16;
@@ -639,7 +669,7 @@ PG_API int64_t pg_attention_part_floats(pg_ctx *ctx, const pg_attention *p, int6
     const int64_t per = (int64_t)s.G * ((s.rep + 15) / 16);
     int64_t most = 0;
     for (int64_t rows = 1; rows <= max_seqs; rows++) most = std::max(most, rows * per * slices(ctx, rows * per, s.cap));
-    return most * 16 * (s.vp + 2);
+    return most * 16 * (s.vp + 4);
 }
 
 PG_API int32_t pg_attention_run(pg_ctx *ctx, const pg_attention *p, const pg_batch *batch, const float *d_proj, int64_t ldp, void *d_kcache,

@@ -53,7 +53,8 @@ __device__ __forceinline__ float conv_at(const DeltaShape &s, const float *row, 
 constexpr int DS_T = 256;
 constexpr int DS_KEEP = 16;      // state rows per thread that stay in registers between the two passes
 
-template <typename TA>
+// TAPS: the number of taps, 0 = any
+template <int TAPS, typename TA>
 __global__ void __launch_bounds__(DS_T)
     delta_step_kernel(const DeltaShape s, const float *__restrict__ proj, int64_t ldp, const int32_t *__restrict__ positions,
                       const int32_t *__restrict__ slots, float *ring, float *state, TA *__restrict__ out, int64_t ldo)
@@ -73,7 +74,12 @@ __global__ void __launch_bounds__(DS_T)
     const int vq = s.vs / 4, cpt = min(vq, DS_T), groups = DS_T / cpt;
     float *pq = pk + (size_t)groups * s.vs;
 
-    // the state's rows are asked for first
+    // what the end of the kernel needs and the state's rows are asked for first
+    const float *tail = row + s.C + (int64_t)s.H * s.V;
+    const float in_b = __ldcg(tail + h), in_a = __ldcg(tail + s.H + h);
+    float in_gate[4];                                     // vdim <= 1024
+#pragma unroll
+    for (int i = 0; i < 4; i++) in_gate[i] = tid + i * DS_T < s.V ? __ldcg(row + s.C + (int64_t)h * s.V + tid + i * DS_T) : 0.0f;
     const int rgid = tid / cpt, cv = tid - rgid * cpt;    // row group, column quad (in steps of cpt quads)
     const bool live = rgid < groups;
     float4 keep[DS_KEEP];
@@ -89,17 +95,55 @@ __global__ void __launch_bounds__(DS_T)
     }
 
     const int cq = g * s.D, ck = s.G * s.D + g * s.D, cvv = 2 * s.G * s.D + h * s.V;
-    for (int i = tid; i < 2 * s.D + s.V; i += DS_T) {
-        const int c = i < s.D ? cq + i : (i < 2 * s.D ? ck + i - s.D : cvv + i - 2 * s.D);
-        const float y = conv_at(s, row, ldp, rg, c, 0, pos);
-        if (i < s.D)
-            sq[i] = y;
-        else if (i < 2 * s.D)
-            sk[i - s.D] = y;
-        else
-            sv[i - 2 * s.D] = y;
-        // the entry this position takes is older than anything a convolution still reads
-        if (i >= 2 * s.D || h % rep == 0) rg[(int64_t)(pos % s.taps) * s.C + c] = __ldcg(row + c);
+    const int now = pos % s.taps;
+    // two channels per round, all their loads in flight together
+    for (int i0 = tid; i0 < 2 * s.D + s.V; i0 += 2 * DS_T) {
+        int ch[2];
+        float y[2], in[2];
+#pragma unroll
+        for (int u = 0; u < 2; u++) {
+            const int i = i0 + u * DS_T;
+            ch[u] = i >= 2 * s.D + s.V ? -1 : i < s.D ? cq + i : (i < 2 * s.D ? ck + i - s.D : cvv + i - 2 * s.D);
+        }
+        if constexpr (TAPS > 0) {
+            float x[2][TAPS], wt[2][TAPS];
+#pragma unroll
+            for (int u = 0; u < 2; u++)
+#pragma unroll
+                for (int j = 0; j < TAPS; j++) {
+                    const int back = TAPS - 1 - j;
+                    const int at = now - back < 0 ? now - back + TAPS : now - back;
+                    x[u][j] = ch[u] < 0 || back > pos ? 0.0f : back == 0 ? __ldcg(row + ch[u]) : __ldcg(rg + (int64_t)at * s.C + ch[u]);
+                    wt[u][j] = ch[u] < 0 ? 0.0f : __ldg(s.conv + (int64_t)j * s.C + ch[u]);
+                }
+#pragma unroll
+            for (int u = 0; u < 2; u++) {
+                float acc = 0.0f;
+#pragma unroll
+                for (int j = 0; j < TAPS; j++) acc = fmaf(wt[u][j], x[u][j], acc);
+                y[u] = pg_silu(acc);
+                in[u] = x[u][TAPS - 1];
+            }
+        } else {
+#pragma unroll
+            for (int u = 0; u < 2; u++) {
+                y[u] = ch[u] < 0 ? 0.0f : conv_at(s, row, ldp, rg, ch[u], 0, pos);
+                in[u] = ch[u] < 0 ? 0.0f : __ldcg(row + ch[u]);
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < 2; u++) {
+            const int i = i0 + u * DS_T;
+            if (ch[u] < 0) continue;
+            if (i < s.D)
+                sq[i] = y[u];
+            else if (i < 2 * s.D)
+                sk[i - s.D] = y[u];
+            else
+                sv[i - 2 * s.D] = y[u];
+            // the entry this position takes is older than anything a convolution still reads
+            if (i >= 2 * s.D || h % rep == 0) rg[(int64_t)now * s.C + ch[u]] = in[u];
+        }
     }
     for (int i = s.V + tid; i < s.vs; i += DS_T) sv[i] = 0.0f;
     __syncthreads();
@@ -112,9 +156,8 @@ __global__ void __launch_bounds__(DS_T)
         const float inv = __fdiv_rn(tid < 32 ? s.qscale : 1.0f, sqrtf(ss + s.unit_eps));
         for (int i = lane; i < s.D; i += 32) x[i] *= inv;
     } else if (tid == 64) {
-        const float *tail = row + s.C + (int64_t)s.H * s.V;
-        bc[0] = pg_sigmoid(__ldcg(tail + h));
-        bc[1] = expf(log_decay(__ldcg(tail + s.H + h), __ldg(s.a_log + h), __ldg(s.dt_bias + h)));
+        bc[0] = pg_sigmoid(in_b);
+        bc[1] = expf(log_decay(in_a, __ldg(s.a_log + h), __ldg(s.dt_bias + h)));
     }
     __syncthreads();
     if (tid < 32) {
@@ -178,9 +221,11 @@ __global__ void __launch_bounds__(DS_T)
     for (int c = tid; c < s.V; c += DS_T) ss += so[c] * so[c];
     ss = pg_block_sum(ss, red);
     const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss, (float)s.V) + s.eps));
-    const float *gate = row + s.C + (int64_t)h * s.V;
-    for (int c = tid; c < s.V; c += DS_T)
-        pg_put(out + (int64_t)b * ldo + (int64_t)h * s.V + c, so[c] * inv * __ldg(s.norm + c) * pg_silu(__ldcg(gate + c)));
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const int c = tid + i * DS_T;
+        if (c < s.V) pg_put(out + (int64_t)b * ldo + (int64_t)h * s.V + c, so[c] * inv * __ldg(s.norm + c) * pg_silu(in_gate[i]));
+    }
 }
 
 // ---- longer portions ---------------------------------------------------------------------------------------------
@@ -197,8 +242,34 @@ constexpr int BT = 4;            // tokens of a block
 // blocks of a sequence are numbered from here on
 __device__ __forceinline__ int64_t first_block(int row0, int seq) { return row0 / BT + seq; }
 
-// grid (ceil(longest / 4), seqs).  TAPS: the number of taps, 0 = any
-template <int TAPS>
+template <int V>
+struct Lanes {
+    float v[V];
+};
+template <int V>
+__device__ __forceinline__ Lanes<V> load_lanes(const float *p)
+{
+    Lanes<V> r;
+    if constexpr (V == 4) {
+        const float4 q = __ldcg(reinterpret_cast<const float4 *>(p));
+        r.v[0] = q.x, r.v[1] = q.y, r.v[2] = q.z, r.v[3] = q.w;
+    } else {
+        r.v[0] = __ldcg(p);
+    }
+    return r;
+}
+template <int V>
+__device__ __forceinline__ void store_lanes(float *p, const Lanes<V> &r)
+{
+    if constexpr (V == 4)
+        *reinterpret_cast<float4 *>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+    else
+        *p = r.v[0];
+}
+
+// grid (ceil(longest / 4), seqs).  TAPS: the number of taps, 0 = any; V: channels per thread and round (4 where rows and
+// groups of channels start on 16-byte boundaries)
+template <int TAPS, int V>
 __global__ void __launch_bounds__(256)
     delta_prep_kernel(const DeltaShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, const float *__restrict__ ring, const DeltaWork w)
 {
@@ -212,39 +283,43 @@ __global__ void __launch_bounds__(256)
     const float *rg = ring + (int64_t)__ldcg(bt.d_seq_slot + seq) * s.taps * s.C;
     const int qk = 2 * s.G * s.D;
     float *dots = sm + (size_t)BT * qk;
-    for (int c = threadIdx.x; c < s.C; c += 256) {
-        float y[BT];
+    for (int c = threadIdx.x * V; c < s.C; c += 256 * V) {
+        Lanes<V> y[BT];
         if constexpr (TAPS > 0) {
-            float x[TAPS - 1 + BT], wt[TAPS];
-#pragma unroll
-            for (int j = 0; j < TAPS; j++) wt[j] = __ldg(s.conv + (int64_t)j * s.C + c);
+            Lanes<V> x[TAPS - 1 + BT], wt[TAPS];
 #pragma unroll
             for (int j = 0; j < TAPS - 1 + BT; j++) {
                 const int t = t0 + j - (TAPS - 1);        // of the sequence's tokens in this step
-                x[j] = 0.0f;
+                x[j] = Lanes<V>{};
                 if (t >= 0) {
-                    if (t < T) x[j] = __ldcg(row + (int64_t)(j - (TAPS - 1)) * ldp + c);
+                    if (t < T) x[j] = load_lanes<V>(row + (int64_t)(j - (TAPS - 1)) * ldp + c);
                 } else if (pos0 + t >= 0) {
-                    x[j] = __ldcg(rg + (int64_t)((pos0 + t) % TAPS) * s.C + c);
+                    x[j] = load_lanes<V>(rg + (int64_t)((pos0 + t) % TAPS) * s.C + c);
                 }
             }
 #pragma unroll
-            for (int a = 0; a < BT; a++) {
-                float acc = 0.0f;
+            for (int j = 0; j < TAPS; j++) wt[j] = load_lanes<V>(s.conv + (int64_t)j * s.C + c);
 #pragma unroll
-                for (int j = 0; j < TAPS; j++) acc = fmaf(wt[j], x[a + j], acc);
-                y[a] = pg_silu(acc);
-            }
+            for (int a = 0; a < BT; a++)
+#pragma unroll
+                for (int i = 0; i < V; i++) {
+                    float acc = 0.0f;
+#pragma unroll
+                    for (int j = 0; j < TAPS; j++) acc = fmaf(wt[j].v[i], x[a + j].v[i], acc);
+                    y[a].v[i] = pg_silu(acc);
+                }
         } else {
 #pragma unroll
-            for (int a = 0; a < BT; a++) y[a] = a < n ? conv_at(s, row + (int64_t)a * ldp, ldp, rg, c, t0 + a, pos0 + t0 + a) : 0.0f;
+            for (int a = 0; a < BT; a++)
+#pragma unroll
+                for (int i = 0; i < V; i++) y[a].v[i] = a < n ? conv_at(s, row + (int64_t)a * ldp, ldp, rg, c + i, t0 + a, pos0 + t0 + a) : 0.0f;
         }
 #pragma unroll
         for (int a = 0; a < BT; a++) {
             if (c < qk)
-                sm[(size_t)a * qk + c] = a < n ? y[a] : 0.0f;
+                store_lanes<V>(sm + (size_t)a * qk + c, a < n ? y[a] : Lanes<V>{});
             else if (a < n)
-                w.v[(int64_t)(m0 + a) * s.H * s.V + c - qk] = y[a];
+                store_lanes<V>(w.v + (int64_t)(m0 + a) * s.H * s.V + c - qk, y[a]);
         }
     }
     __syncthreads();
@@ -369,7 +444,8 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaShape s, con
     constexpr int DP = C::DP, TB = C::TB;
     extern __shared__ __align__(16) unsigned char smem[];
     typename C::Stage *stages = reinterpret_cast<typename C::Stage *>(smem);
-    pg_pdl_begin();
+    // (The successor is not let in early: its CTAs would sit on the SMs through this long kernel.)
+    asm volatile("griddepcontrol.wait;" ::: "memory");
     const int h = blockIdx.y, seq = blockIdx.z, g = h / (s.H / s.G), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int row0 = __ldcg(bt.d_seq_row0 + seq), T = __ldcg(bt.d_seq_row0 + seq + 1) - row0;
     if (T <= 0) return;
@@ -542,14 +618,22 @@ int32_t run_scan(pg_ctx *ctx, const DeltaShape &s, const pg_batch *bt, const Del
     return launch_pdl(ctx, delta_scan_kernel<NI>, dim3((unsigned)((s.V + 31) / 32), (unsigned)s.H, (unsigned)bt->seqs), dim3(128), (size_t)smem, s, *bt, w, state);
 }
 
-template <int TAPS>
-int32_t run_prep(pg_ctx *ctx, const DeltaShape &s, const pg_batch *bt, const float *proj, int64_t ldp, const float *ring, const DeltaWork &w)
+template <int TAPS, int V>
+int32_t run_prep_v(pg_ctx *ctx, const DeltaShape &s, const pg_batch *bt, const float *proj, int64_t ldp, const float *ring, const DeltaWork &w)
 {
     const size_t smem = ((size_t)BT * 2 * s.G * s.D + 16 * s.G) * 4;
     PG_REQUIRE(smem <= 220 * 1024, "delta: too many query / key channels");
     static std::atomic<uint64_t> set{0};
-    PG_CUDA(pg_max_smem_once(delta_prep_kernel<TAPS>, 220 * 1024, ctx->device, set));
-    return launch_pdl(ctx, delta_prep_kernel<TAPS>, dim3((unsigned)((bt->max_len + BT - 1) / BT), (unsigned)bt->seqs), dim3(256), smem, s, *bt, proj, ldp, ring, w);
+    PG_CUDA(pg_max_smem_once(delta_prep_kernel<TAPS, V>, 220 * 1024, ctx->device, set));
+    return launch_pdl(ctx, delta_prep_kernel<TAPS, V>, dim3((unsigned)((bt->max_len + BT - 1) / BT), (unsigned)bt->seqs), dim3(256), smem, s, *bt, proj, ldp, ring, w);
+}
+
+template <int TAPS>
+int32_t run_prep(pg_ctx *ctx, const DeltaShape &s, const pg_batch *bt, const float *proj, int64_t ldp, const float *ring, const DeltaWork &w)
+{
+    const bool vec = ((2 * s.G * s.D) & 3) == 0 && ((s.H * s.V) & 3) == 0 && ldp % 4 == 0 &&
+                     (((uintptr_t)proj | (uintptr_t)ring | (uintptr_t)s.conv | (uintptr_t)w.v) & 15) == 0;
+    return vec ? run_prep_v<TAPS, 4>(ctx, s, bt, proj, ldp, ring, w) : run_prep_v<TAPS, 1>(ctx, s, bt, proj, ldp, ring, w);
 }
 
 // a CTA per token: o / rms(o) * norm * silu(gate) per head; the sequence's last taps - 1 tokens also store their
@@ -557,22 +641,53 @@ int32_t run_prep(pg_ctx *ctx, const DeltaShape &s, const pg_batch *bt, const flo
 template <typename TA>
 __global__ void __launch_bounds__(256)
     delta_out_kernel(const DeltaShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, const DeltaWork w, float *ring, TA *__restrict__ out,
-                     int64_t ldo)
+                     int64_t ldo, bool vec)
 {
     pg_pdl_begin();
     const int m = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const float *row = proj + (int64_t)m * ldp;
-    for (int h = warp; h < s.H; h += 8) {
-        const float *o = w.o + (int64_t)m * s.H * s.V + (int64_t)h * s.V;
-        float ss = 0.0f;
-        for (int c = lane; c < s.V; c += 32) {
-            const float x = __ldcg(o + c);
-            ss += x * x;
+    if (vec) {                                            // V a multiple of 4, at most 128: a quad per lane
+        for (int h0 = warp; h0 < s.H; h0 += 16) {         // two heads at a time
+            float4 o[2], gt[2];
+#pragma unroll
+            for (int i = 0; i < 2; i++) {
+                const int h = h0 + 8 * i;
+                o[i] = gt[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (h < s.H && lane * 4 < s.V) {
+                    o[i] = __ldcg(reinterpret_cast<const float4 *>(w.o + ((int64_t)m * s.H + h) * s.V) + lane);
+                    gt[i] = __ldcg(reinterpret_cast<const float4 *>(row + s.C + (int64_t)h * s.V) + lane);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < 2; i++) {
+                const int h = h0 + 8 * i;
+                const float ss = pg_warp_sum(o[i].x * o[i].x + o[i].y * o[i].y + o[i].z * o[i].z + o[i].w * o[i].w);
+                const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss, (float)s.V) + s.eps));
+                if (h < s.H && lane * 4 < s.V) {
+                    const float4 nw = __ldg(reinterpret_cast<const float4 *>(s.norm) + lane);
+                    TA *dst = out + (int64_t)m * ldo + (int64_t)h * s.V + lane * 4;
+                    const float y[4] = {o[i].x * inv * nw.x * pg_silu(gt[i].x), o[i].y * inv * nw.y * pg_silu(gt[i].y),
+                                        o[i].z * inv * nw.z * pg_silu(gt[i].z), o[i].w * inv * nw.w * pg_silu(gt[i].w)};
+                    if constexpr (sizeof(TA) == 2)
+                        *reinterpret_cast<uint2 *>(dst) = make_uint2(pg_pack_bf16(y[0], y[1]), pg_pack_bf16(y[2], y[3]));
+                    else
+                        *reinterpret_cast<float4 *>(dst) = make_float4(y[0], y[1], y[2], y[3]);
+                }
+            }
         }
-        ss = pg_warp_sum(ss);
-        const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss, (float)s.V) + s.eps));
-        for (int c = lane; c < s.V; c += 32)
-            pg_put(out + (int64_t)m * ldo + (int64_t)h * s.V + c, __ldcg(o + c) * inv * __ldg(s.norm + c) * pg_silu(__ldcg(row + s.C + (int64_t)h * s.V + c)));
+    } else {
+        for (int h = warp; h < s.H; h += 8) {
+            const float *o = w.o + (int64_t)m * s.H * s.V + (int64_t)h * s.V;
+            float ss = 0.0f;
+            for (int c = lane; c < s.V; c += 32) {
+                const float x = __ldcg(o + c);
+                ss += x * x;
+            }
+            ss = pg_warp_sum(ss);
+            const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss, (float)s.V) + s.eps));
+            for (int c = lane; c < s.V; c += 32)
+                pg_put(out + (int64_t)m * ldo + (int64_t)h * s.V + c, __ldcg(o + c) * inv * __ldg(s.norm + c) * pg_silu(__ldcg(row + s.C + (int64_t)h * s.V + c)));
+        }
     }
     const int seq = __ldcg(bt.d_row_seq + m);
     if (m >= __ldcg(bt.d_seq_row0 + seq + 1) - (s.taps - 1)) {
@@ -621,9 +736,16 @@ PG_API int32_t pg_delta_run(pg_ctx *ctx, const pg_delta *p, const pg_batch *batc
         const size_t smem = (size_t)(2 * ((s.D + 3) & ~3) + 2 * s.vs + 2 * groups * s.vs) * 4;
         PG_REQUIRE(smem <= 48 * 1024, "delta: shared memory");
         const dim3 g((unsigned)s.H, (unsigned)M);
-        if (dtype == PG_BF16)
-            return launch_pdl(ctx, delta_step_kernel<bf16>, g, dim3(DS_T), smem, s, d_proj, ldp, batch->d_pos, batch->d_seq_slot, d_ring, d_state, (bf16 *)d_out, ldo);
-        return launch_pdl(ctx, delta_step_kernel<float>, g, dim3(DS_T), smem, s, d_proj, ldp, batch->d_pos, batch->d_seq_slot, d_ring, d_state, (float *)d_out, ldo);
+#define PG_DS_CASE(N)                                                                                                                                   \
+    return dtype == PG_BF16 ? launch_pdl(ctx, delta_step_kernel<N, bf16>, g, dim3(DS_T), smem, s, d_proj, ldp, batch->d_pos, batch->d_seq_slot, d_ring, \
+                                         d_state, (bf16 *)d_out, ldo)                                                                                   \
+                            : launch_pdl(ctx, delta_step_kernel<N, float>, g, dim3(DS_T), smem, s, d_proj, ldp, batch->d_pos, batch->d_seq_slot, d_ring, \
+                                         d_state, (float *)d_out, ldo)
+        if (s.taps == 2) PG_DS_CASE(2);
+        if (s.taps == 3) PG_DS_CASE(3);
+        if (s.taps == 4) PG_DS_CASE(4);
+        PG_DS_CASE(0);
+#undef PG_DS_CASE
     }
     DeltaWork w;
     float *at = p->d_work;
@@ -655,9 +777,11 @@ PG_API int32_t pg_delta_run(pg_ctx *ctx, const pg_delta *p, const pg_batch *batc
     else
         rc = run_scan<8>(ctx, s, batch, w, d_state);
     if (rc != PG_OK) return rc;
+    const bool vec = s.V % 4 == 0 && s.V <= 128 && s.C % 4 == 0 && ldp % 4 == 0 && ldo % 4 == 0 &&
+                     (((uintptr_t)d_proj | (uintptr_t)d_out | (uintptr_t)s.norm | (uintptr_t)w.o) & 15) == 0;
     if (dtype == PG_BF16)
-        return launch_pdl(ctx, delta_out_kernel<bf16>, dim3((unsigned)M), dim3(256), 0, s, *batch, d_proj, ldp, w, d_ring, (bf16 *)d_out, ldo);
-    return launch_pdl(ctx, delta_out_kernel<float>, dim3((unsigned)M), dim3(256), 0, s, *batch, d_proj, ldp, w, d_ring, (float *)d_out, ldo);
+        return launch_pdl(ctx, delta_out_kernel<bf16>, dim3((unsigned)M), dim3(256), 0, s, *batch, d_proj, ldp, w, d_ring, (bf16 *)d_out, ldo, vec);
+    return launch_pdl(ctx, delta_out_kernel<float>, dim3((unsigned)M), dim3(256), 0, s, *batch, d_proj, ldp, w, d_ring, (float *)d_out, ldo, vec);
 }
 
 }  // extern "C"

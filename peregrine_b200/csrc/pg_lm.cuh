@@ -80,8 +80,9 @@ __device__ __forceinline__ void pg_pdl_begin()
     asm volatile("griddepcontrol.wait;" ::: "memory");
 }
 
-__device__ __forceinline__ float pg_sigmoid(float z) { return __fdiv_rn(1.0f, 1.0f + expf(-z)); }
-__device__ __forceinline__ float pg_silu(float z) { return __fdiv_rn(z, 1.0f + expf(-z)); }
+// (the quick division is within two units in the last place, and 0 where the denominator is beyond 2^126)
+__device__ __forceinline__ float pg_sigmoid(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }
+__device__ __forceinline__ float pg_silu(float z) { return __fdividef(z, 1.0f + expf(-z)); }
 __device__ __forceinline__ float pg_gelu_tanh(float z)
 {
     const float c = 0.7978845608028654f;   // sqrt(2 / pi)

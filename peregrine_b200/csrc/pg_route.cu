@@ -19,110 +19,117 @@ struct Choice {
     int n, top, groups, keep;
 };
 
-__device__ __forceinline__ void warp_argmax(float &v, int &i)
+// f32 -> u32 of the same order (not-a-number becomes 0, below every number)
+__device__ __forceinline__ uint32_t order_key(float v)
 {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, v, o);
-        const int oi = __shfl_xor_sync(0xffffffffu, i, o);
-        if (ov > v || (ov == v && oi < i)) {
-            v = ov;
-            i = oi;
-        }
-    }
+    const uint32_t b = __float_as_uint(v);
+    return v != v ? 0u : (b & 0x80000000u) ? ~b : (b | 0x80000000u);
+}
+// the largest key of the warp and the lowest index that has it; key 0 means none
+__device__ __forceinline__ void warp_best(uint32_t &key, int &idx)
+{
+    const uint32_t k = __reduce_max_sync(0xffffffffu, key);
+    idx = (int)__reduce_min_sync(0xffffffffu, key == k && k != 0u ? (unsigned)idx : (unsigned)RT_MAX);
+    key = k;
 }
 
-// One warp, one token: z = its n logits; c (shared, n floats) and gs (shared, `groups` floats) are scratch of the warp.
-__device__ __forceinline__ void choose(const float *z, const float *__restrict__ correction, const Choice ch, float *c, float *gs, int32_t *ids,
-                                       float *weights, int lane)
+// One warp, one token: z = its n <= 32 NV logits; lane l keeps the choice scores of outputs l + 32 i in registers.
+// gs: shared, `groups` words, scratch of the warp.
+template <int NV>
+__device__ __forceinline__ void choose(const float *z, const float *__restrict__ correction, const Choice ch, uint32_t *gs, int32_t *ids, float *weights, int lane)
 {
-    float mx = -INFINITY;
-    for (int i = lane; i < ch.n; i += 32) mx = fmaxf(mx, __ldcg(z + i));
+    float e[NV], mx = -INFINITY, sum = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        e[i] = lane + 32 * i < ch.n ? __ldcg(z + lane + 32 * i) : -INFINITY;
+        mx = fmaxf(mx, e[i]);
+    }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-    float sum = 0.0f;
-    for (int i = lane; i < ch.n; i += 32) sum += expf(__ldcg(z + i) - mx);
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        e[i] = expf(e[i] - mx);
+        sum += e[i];
+    }
     sum = pg_warp_sum(sum);
-    for (int i = lane; i < ch.n; i += 32) c[i] = __fdiv_rn(expf(__ldcg(z + i) - mx), sum) + __ldg(correction + i);
-    __syncwarp();
+    uint32_t key[NV];
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        e[i] = __fdiv_rn(e[i], sum);
+        key[i] = lane + 32 * i < ch.n ? order_key(e[i] + __ldg(correction + lane + 32 * i)) : 0u;
+    }
     if (ch.groups > 1) {
         const int per = ch.n / ch.groups;
-        for (int g = lane; g < ch.groups; g += 32) {
-            float b = -INFINITY;
-            for (int i = 0; i < per; i++) b = fmaxf(b, c[g * per + i]);
-            gs[g] = b;
-        }
+        for (int g = lane; g < ch.groups; g += 32) gs[g] = 0u;
         __syncwarp();
-        // the best `keep` groups are marked with +inf, one after the other
+#pragma unroll
+        for (int i = 0; i < NV; i++)
+            if (lane + 32 * i < ch.n) atomicMax(gs + (lane + 32 * i) / per, key[i]);
+        __syncwarp();
+        // the best `keep` groups are marked with all ones (no score has that key), one after the other
         for (int k = 0; k < ch.keep; k++) {
-            float v = -INFINITY;
+            uint32_t best = 0u;
             int idx = RT_MAX;
             for (int g = lane; g < ch.groups; g += 32) {
-                const float x = gs[g];
-                if (x != INFINITY && (x > v || (x == v && g < idx))) {
-                    v = x;
-                    idx = g;
-                }
+                const uint32_t x = gs[g];
+                if (x != 0xffffffffu && x > best) best = x, idx = g;
             }
-            warp_argmax(v, idx);
-            __syncwarp();
-            if (lane == 0 && idx < ch.groups) gs[idx] = INFINITY;
+            warp_best(best, idx);
+            if (lane == 0 && idx < ch.groups) gs[idx] = 0xffffffffu;
             __syncwarp();
         }
-        for (int i = lane; i < ch.n; i += 32)
-            if (gs[i / per] != INFINITY) c[i] = -INFINITY;
-        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < NV; i++)
+            if (lane + 32 * i < ch.n && gs[(lane + 32 * i) / per] != 0xffffffffu) key[i] = 0u;
     }
     for (int k = 0; k < ch.top; k++) {
-        float v = -INFINITY;
+        uint32_t best = 0u;
         int idx = RT_MAX;
-        for (int i = lane; i < ch.n; i += 32) {
-            const float x = c[i];
-            if (x > v || (x == v && x != -INFINITY && i < idx)) {
-                v = x;
-                idx = i;
-            }
+        float w = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NV; i++)
+            if (key[i] > best) best = key[i], idx = lane + 32 * i, w = e[i];
+        warp_best(best, idx);
+        if (idx >= ch.n) {                                // not-a-number scores choose nothing: weight 0
+            if (lane == 0) ids[k] = ch.n - 1, weights[k] = 0.0f;
+            continue;
         }
-        warp_argmax(v, idx);
-        const bool found = idx < ch.n;                    // not-a-number scores choose nothing: weight 0
-        if (!found) idx = ch.n - 1;
-        __syncwarp();
-        if (lane == 0) {
+        if ((idx & 31) == lane) {
             ids[k] = idx;
-            weights[k] = found ? __fdiv_rn(expf(__ldcg(z + idx) - mx), sum) : 0.0f;
-            if (found) c[idx] = -INFINITY;
+            weights[k] = w;
+#pragma unroll
+            for (int i = 0; i < NV; i++)
+                if (lane + 32 * i == idx) key[i] = 0u;
         }
-        __syncwarp();
     }
+    __syncwarp();
 }
 
+template <int NV>
 __global__ void __launch_bounds__(512)
     route_small_kernel(const float *__restrict__ logits, int64_t ld, int m, int experts, const float *__restrict__ correction, const Choice ch,
                        int32_t *ids, float *weights, int32_t *pair_row, int32_t *row_pair, int32_t *block_expert, int32_t *blocks)
 {
-    extern __shared__ float sm[];      // [16][n + groups] scratch, then [m * top] ids
-    __shared__ int chunk[32];
+    extern __shared__ uint32_t sm[];   // groups [16][ch.groups] | ids [m * top] | rank of each pair [m * top] | count, then block, per expert
+    __shared__ int chunk[16];
+    uint32_t *gs = sm;
+    int32_t *sid = reinterpret_cast<int32_t *>(sm + 16 * ch.groups), *rank = sid + m * ch.top, *count = rank + m * ch.top;
+    for (int e = threadIdx.x; e < experts; e += 512) count[e] = 0;
     pg_pdl_begin();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    float *c = sm + (size_t)warp * (ch.n + ch.groups);
-    int32_t *sid = reinterpret_cast<int32_t *>(sm + 16 * (size_t)(ch.n + ch.groups));
-    if (warp < m) {
-        choose(logits + (int64_t)warp * ld, correction, ch, c, c + ch.n, sid + warp * ch.top, weights + warp * ch.top, lane);
-        for (int k = lane; k < ch.top; k += 32) {
-            const int id = sid[warp * ch.top + k];
-            ids[warp * ch.top + k] = id;
-            if (id >= experts) pair_row[warp * ch.top + k] = -1;
-        }
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, pairs = m * ch.top;
+    if (warp < m) choose<NV>(logits + (int64_t)warp * ld, correction, ch, gs + warp * ch.groups, sid + warp * ch.top, weights + warp * ch.top, lane);
+    __syncthreads();
+    for (int p = threadIdx.x; p < pairs; p += 512) {
+        const int id = sid[p];
+        ids[p] = id;
+        rank[p] = id < experts ? atomicAdd(count + id, 1) : -1;
     }
     __syncthreads();
-    const int pairs = m * ch.top;
     // a block of 16 rows per expert in use, in the order of the experts
     int base = 0;
     for (int e0 = 0; e0 < experts; e0 += 512) {
         const int e = e0 + threadIdx.x;
-        bool used = false;
-        if (e < experts)
-            for (int p = 0; p < pairs && !used; p++) used = sid[p] == e;
+        const bool used = e < experts && count[e] > 0;
         const unsigned ballot = __ballot_sync(0xffffffffu, used);
         if (lane == 0) chunk[warp] = __popc(ballot);
         __syncthreads();
@@ -133,38 +140,36 @@ __global__ void __launch_bounds__(512)
         }
         if (used) {
             block_expert[at] = e;
-            int r = 0;
-            for (int p = 0; p < pairs; p++)
-                if (sid[p] == e) {
-                    pair_row[p] = r < PG_ROUTE_SMALL ? at * PG_ROUTE_SMALL + r : -1;
-                    if (r < PG_ROUTE_SMALL) row_pair[at * PG_ROUTE_SMALL + r] = p;
-                    r++;
-                }
-            for (; r < PG_ROUTE_SMALL; r++) row_pair[at * PG_ROUTE_SMALL + r] = -1;
+            for (int r = count[e]; r < PG_ROUTE_SMALL; r++) row_pair[at * PG_ROUTE_SMALL + r] = -1;
+            count[e] = at;
         }
         base += all;
         __syncthreads();
     }
     if (threadIdx.x == 0) *blocks = base;
+    for (int p = threadIdx.x; p < pairs; p += 512) {
+        const int r = rank[p];
+        const int row = r >= 0 && r < PG_ROUTE_SMALL ? count[sid[p]] * PG_ROUTE_SMALL + r : -1;
+        pair_row[p] = row;
+        if (row >= 0) row_pair[row] = p;
+    }
 }
 
+template <int NV>
 __global__ void __launch_bounds__(128)
     route_choose_kernel(const float *__restrict__ logits, int64_t ld, int m, int experts, const float *__restrict__ correction, const Choice ch,
                         int32_t *ids, float *weights, int32_t *count)
 {
-    extern __shared__ float sm[];
+    extern __shared__ uint32_t sm[];
     pg_pdl_begin();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * 4 + warp;
     if (t >= m) return;
-    float *c = sm + (size_t)warp * (ch.n + ch.groups);
-    choose(logits + (int64_t)t * ld, correction, ch, c, c + ch.n, ids + (int64_t)t * ch.top, weights + (int64_t)t * ch.top, lane);
-    __syncwarp();
-    if (lane == 0)
-        for (int k = 0; k < ch.top; k++) {
-            const int id = ids[(int64_t)t * ch.top + k];
-            if (id < experts) atomicAdd(count + id, 1);
-        }
+    choose<NV>(logits + (int64_t)t * ld, correction, ch, sm + warp * ch.groups, ids + (int64_t)t * ch.top, weights + (int64_t)t * ch.top, lane);
+    for (int k = lane; k < ch.top; k += 32) {
+        const int id = __ldcg(ids + (int64_t)t * ch.top + k);
+        if (id < experts) atomicAdd(count + id, 1);
+    }
 }
 
 // count -> first row of every expert (in cursor), the experts of the row blocks, the number of row blocks; count back to 0
@@ -301,16 +306,35 @@ PG_API int32_t pg_route_run(pg_ctx *ctx, pg_route *route, int32_t dtype, const f
     route->block = small ? PG_ROUTE_SMALL : PG_ROUTE_BLOCK;
     if (m == 0) return PG_OK;
     const Choice ch = {n, (int)route->top, groups, keep};
+#define PG_RT_SMALL(NV)                                                                                                                                  \
+    do {                                                                                                                                                 \
+        static std::atomic<uint64_t> set{0};                                                                                                             \
+        PG_CUDA(pg_max_smem_once(route_small_kernel<NV>, 220 * 1024, ctx->device, set));                                                                 \
+        return launch_pdl(ctx, route_small_kernel<NV>, dim3(1), dim3(512), smem, d_logits, ld, (int)m, (int)route->experts, d_correction, ch, route->ids, \
+                          route->weights, route->pair_row, route->row_pair, route->block_expert, route->blocks);                                         \
+    } while (0)
+#define PG_RT_CHOOSE(NV)                                                                                                                                 \
+    launch_pdl(ctx, route_choose_kernel<NV>, dim3((unsigned)((m + 3) / 4)), dim3(128), (size_t)4 * groups * 4, d_logits, ld, (int)m, (int)route->experts, \
+               d_correction, ch, route->ids, route->weights, route->count)
     if (small) {
-        const size_t smem = (size_t)16 * (n + groups) * 4 + (size_t)m * route->top * 4;
-        PG_REQUIRE(smem <= 200 * 1024, "route: too many router outputs");
-        static std::atomic<uint64_t> set{0};
-        PG_CUDA(pg_max_smem_once(route_small_kernel, 200 * 1024, ctx->device, set));
-        return launch_pdl(ctx, route_small_kernel, dim3(1), dim3(512), smem, d_logits, ld, (int)m, (int)route->experts, d_correction, ch, route->ids,
-                          route->weights, route->pair_row, route->row_pair, route->block_expert, route->blocks);
+        const size_t smem = ((size_t)16 * groups + 2 * m * route->top + route->experts) * 4;
+        PG_REQUIRE(smem <= 220 * 1024, "route: too many choices for the one-CTA form");
+        if (n <= 32) PG_RT_SMALL(1);
+        if (n <= 128) PG_RT_SMALL(4);
+        if (n <= 256) PG_RT_SMALL(8);
+        PG_RT_SMALL(32);
     }
-    int32_t rc = launch_pdl(ctx, route_choose_kernel, dim3((unsigned)((m + 3) / 4)), dim3(128), (size_t)4 * (n + groups) * 4, d_logits, ld, (int)m,
-                            (int)route->experts, d_correction, ch, route->ids, route->weights, route->count);
+    int32_t rc;
+    if (n <= 32)
+        rc = PG_RT_CHOOSE(1);
+    else if (n <= 128)
+        rc = PG_RT_CHOOSE(4);
+    else if (n <= 256)
+        rc = PG_RT_CHOOSE(8);
+    else
+        rc = PG_RT_CHOOSE(32);
+#undef PG_RT_SMALL
+#undef PG_RT_CHOOSE
     if (rc != PG_OK) return rc;
     rc = launch_pdl(ctx, route_layout_kernel, dim3(1), dim3(1024), 0, (int)route->experts, route->count, route->cursor, route->block_expert, route->blocks);
     if (rc != PG_OK) return rc;
