@@ -444,8 +444,7 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaShape s, con
     constexpr int DP = C::DP, TB = C::TB;
     extern __shared__ __align__(16) unsigned char smem[];
     typename C::Stage *stages = reinterpret_cast<typename C::Stage *>(smem);
-    // (The successor is not let in early: its CTAs would sit on the SMs through this long kernel.)
-    asm volatile("griddepcontrol.wait;" ::: "memory");
+    // (launched whole, and the successor is not let in early either)
     const int h = blockIdx.y, seq = blockIdx.z, g = h / (s.H / s.G), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int row0 = __ldcg(bt.d_seq_row0 + seq), T = __ldcg(bt.d_seq_row0 + seq + 1) - row0;
     if (T <= 0) return;
@@ -615,7 +614,7 @@ int32_t run_scan(pg_ctx *ctx, const DeltaShape &s, const pg_batch *bt, const Del
     constexpr int smem = ScanTile<NI>::STAGES * (int)sizeof(typename ScanTile<NI>::Stage);
     static std::atomic<uint64_t> set{0};
     PG_CUDA(pg_max_smem_once(delta_scan_kernel<NI>, smem, ctx->device, set));
-    return launch_pdl(ctx, delta_scan_kernel<NI>, dim3((unsigned)((s.V + 31) / 32), (unsigned)s.H, (unsigned)bt->seqs), dim3(128), (size_t)smem, s, *bt, w, state);
+    return launch_whole(ctx, delta_scan_kernel<NI>, dim3((unsigned)((s.V + 31) / 32), (unsigned)s.H, (unsigned)bt->seqs), dim3(128), (size_t)smem, s, *bt, w, state);
 }
 
 template <int TAPS, int V>

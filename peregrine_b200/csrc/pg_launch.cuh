@@ -52,3 +52,18 @@ inline int32_t launch_pdl(pg_ctx *ctx, K kern, dim3 grid, dim3 block, size_t sme
     PG_LAUNCHED();
     return PG_OK;
 }
+
+// A launch that starts when everything before it has ended.  For long kernels with about one CTA per SM: started early,
+// their CTAs are placed around those of the predecessor, several on one SM and none on others, and stay there.
+template <typename K, typename... Args>
+inline int32_t launch_whole(pg_ctx *ctx, K kern, dim3 grid, dim3 block, size_t smem, Args... args)
+{
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = ctx->stream;
+    PG_CUDA(cudaLaunchKernelEx(&cfg, kern, args...));
+    PG_LAUNCHED();
+    return PG_OK;
+}

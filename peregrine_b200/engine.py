@@ -211,9 +211,10 @@ class LockstepEngine:
         for i in range(n + max_new - 1):
             if all(done):
                 break
-            m.set_position(i)
+            if i == 0:
+                m.set_position(0)          # every step advances it
             if i < n:
-                m.set_tokens([p[i] for p in rows])
+                m.set_tokens([p[i] for p in rows])     # (waits until torch's writes have landed)
                 m.embed()
             m.gpu.sync()
             if m.graph is None:

@@ -66,3 +66,37 @@ def test_from_gguf_decode_step(gpu, oracle_mt, kind):
     # K, V above were advanced by check_stages with the GPU's rows; the free-running oracle overwrites the same position
     assert np.abs(logits - ref).max() <= 2e-2 * np.abs(ref).max()
     model.free()
+
+
+def test_engine_generates_from_a_file(gpu, tmp_path):
+    """`load_engine` on a GGUF file: greedy continuations through the recorded step equal the same steps made by hand."""
+    from peregrine_b200 import llama_gguf
+    from peregrine_b200.registry import load_engine
+
+    g = rng(77)
+    blob, _ = make_model(g, layers=2, hidden=512, n_q=4, n_kv=1, ffn=768, vocab=512)
+    path = tmp_path / "model.gguf"
+    path.write_bytes(blob)
+    prompts = g.integers(0, 512, (2, 5)).tolist()
+    engine = load_engine(str(path), gpu=gpu, slots=3, capacity=32)
+    got = engine.generate(prompts, 6)
+    assert engine.generate(prompts, 6) == got              # from the start again, with the recorded step
+    stop = got[0][2]
+    short = engine.generate(prompts, 6, stop=[stop])
+    assert short[0] == got[0][:got[0].index(stop) + 1]
+    engine.model.free()
+    model, _ = llama_gguf.from_gguf(str(path), gpu, batch=3, capacity=32)
+    rows = prompts + [prompts[0]]
+    out = []
+    model.set_position(0)
+    for i in range(10):
+        if i < 5:
+            model.set_tokens([p[i] for p in rows])
+            model.embed()
+        model.enqueue_step()
+        gpu.sync()
+        if i >= 4:
+            out.append(model.tokens.cpu().tolist())
+    assert got == [[o[k] for o in out] for k in range(2)]
+    assert gpu.device_status() == 0
+    model.free()
