@@ -41,13 +41,21 @@ class SonalornConfig:
                 raise ValueError(f"layer {i}: unknown mixer type {L['type']!r}")
             if L.get("mlp") and L["mlp"]["kind"] not in ("dense", "moe"):
                 raise ValueError(f"layer {i}: unknown feed-forward kind {L['mlp']['kind']!r}")
-            j = L.get("weights_of")
-            if j is not None:
-                if not 0 <= j < len(cfg.layers) or cfg.layers[j].get("weights_of") is not None:
-                    raise ValueError(f"layer {i}: weights_of {j} names no layer with tensors")
-                if L["type"] != cfg.layers[j]["type"]:
-                    raise ValueError(f"layer {i}: another type than layer {j}, whose tensors it uses")
+            if L["type"] != cfg.layers[cfg.tensors_of(i)]["type"]:
+                raise ValueError(f"layer {i}: another type than layer {cfg.tensors_of(i)}, whose tensors it uses")
         return cfg
+
+    def tensors_of(self, i: int) -> int:
+        """The layer whose tensors layer i uses."""
+        j = i
+        for _ in self.layers:
+            k = self.layers[j].get("weights_of")
+            if k is None:
+                return j
+            if not 0 <= k < len(self.layers):
+                break
+            j = k
+        raise ValueError(f"layer {i}: weights_of leads to no layer with tensors")
 
     @staticmethod
     def load(path: str) -> "SonalornConfig":
@@ -113,7 +121,7 @@ class SonalornModel(SlotModel):
         self._own = list(own.values())
         self.layers = []
         for i, L in enumerate(cfg.layers):
-            shared = own[i if L.get("weights_of") is None else L["weights_of"]]
+            shared = own[cfg.tensors_of(i)]
             self.layers.append({**shared, "state": shared["mixer"].new_state(self.pool)})
         self.ldh = up(cfg.width, 64)
         self.x = torch.zeros(self.step_rows, cfg.width, dtype=f32, device=d.dev)

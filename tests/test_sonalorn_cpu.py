@@ -78,6 +78,9 @@ def test_safetensors_round_trip_and_damage(tmp_path):
 def test_config():
     c = SonalornConfig.from_dict(t.small_config())
     assert (c.vocab, c.width, c.max_positions, c.eps, len(c.layers)) == (83, 96, 300, 1e-5, 4)
+    d = t.small_config()
+    d["layers"].append(dict(d["layers"][1], weights_of=2))
+    assert [SonalornConfig.from_dict(d).tensors_of(i) for i in range(5)] == [0, 1, 1, 3, 1]
     for change in (lambda d: d["layers"][0].update(type="window"), lambda d: d["layers"][0]["mlp"].update(kind="none"),
                    lambda d: d["layers"][2].update(weights_of=2), lambda d: d["layers"][2].update(weights_of=0), lambda d: d["layers"][2].update(weights_of=9)):
         d = t.small_config()

@@ -449,19 +449,29 @@ def test_model_however_a_prompt_is_cut(lm, dtype, make):
     e.close()
 
 
+def ragged_config():
+    """Widths at which prompts run on the tcgen05 attention kernel and the delta rule in its 16-byte forms."""
+    return t.config(83, 128, [t.layer("attention", t.attention(4, 1, 64, 64, 0.2, (0.4, 50)), t.dense(72)),
+                              t.layer("delta", t.delta(4, 2, 64, 32, 4), None),
+                              t.layer("attention", t.attention(4, 2, 128, 64, 0.1), None)], max_positions=500)
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_unequal_requests_together_equal_each_alone(lm, dtype):
-    cfg = t.small_config()
+@pytest.mark.parametrize("make,lengths,cuts", [
+    (t.small_config, {"a": 90, "b": 7, "c": 41}, {"a": [30, 1, 1, 40, 18], "b": [2, 1, 1, 1, 2], "c": [1, 1, 30, 1, 8]}),
+    (ragged_config, {"a": 370, "b": 8, "c": 180}, {"a": [200, 1, 60, 1, 108], "b": [2, 1, 2, 1, 2], "c": [33, 1, 130, 1, 15]})])
+def test_unequal_requests_together_equal_each_alone(lm, dtype, make, lengths, cuts):
+    cfg = make()
     W = t.weights(cfg, 21)
+    oracle = so.Model(cfg, W)
     g = rng(22)
-    prompts = {k: g.integers(0, 83, n).tolist() for k, n in (("a", 90), ("b", 7), ("c", 41))}
+    prompts = {k: g.integers(0, 83, n).tolist() for k, n in lengths.items()}
     alone, together = {}, {k: [] for k in prompts}
-    e = make_engine(lm, cfg, W, dtype)
+    e = make_engine(lm, cfg, W, dtype, step_rows=400)
     for k, x in prompts.items():
         alone[k] = e.step([(k, x, list(range(len(x))))])
         e.end(k)
     # in mixed steps, each with slots that others have used
-    cuts = {"a": [30, 1, 1, 40, 18], "b": [2, 1, 1, 1, 2], "c": [1, 1, 30, 1, 8]}
     at = dict.fromkeys(prompts, 0)
     for i in range(5):
         entries = []
@@ -474,9 +484,12 @@ def test_unequal_requests_together_equal_each_alone(lm, dtype):
         for k, x, want in entries:
             together[k].append(out[o:o + len(want)])
             o += len(want)
-    for k in prompts:
+    for k, x in prompts.items():
+        assert at[k] == len(x)
         err = logit_error(np.concatenate(together[k]), alone[k].astype(np.float64))
         assert np.median(err) < MODEL_TOL[dtype] / 4 and (dtype == "bfloat16" or err.max() < 1e-4), k
+        err = logit_error(alone[k], oracle.forward(x, oracle.start()))
+        assert np.median(err) < MODEL_TOL[dtype] / 2, k
     e.close()
 
 
