@@ -161,16 +161,28 @@ class PgDelta(C.Structure):
 
 class PgAttention(C.Structure):
     _fields_ = [("heads", _i32), ("kv_heads", _i32), ("dim", _i32), ("vdim", _i32), ("cap", _i32), ("slots", _i32), ("eps", C.c_float), ("scale", C.c_float),
-                ("temp_coef", C.c_float), ("temp_every", C.c_float), ("sink", _i32), ("d_q_norm", _vp), ("d_k_norm", _vp), ("d_q", _vp), ("d_part", _vp),
-                ("d_tickets", _vp)]
+                ("temp_coef", C.c_float), ("temp_every", C.c_float), ("sink", _i32), ("chunk", _i32), ("positions", _i32), ("d_q_norm", _vp),
+                ("d_k_norm", _vp), ("d_slopes", _vp), ("d_q", _vp), ("d_part", _vp), ("d_tickets", _vp)]
 
 
-_pb, _pd, _pa = C.POINTER(PgBatch), C.POINTER(PgDelta), C.POINTER(PgAttention)
+class PgLatent(C.Structure):
+    _fields_ = [("heads", _i32), ("dim", _i32), ("rot_dim", _i32), ("vdim", _i32), ("kv_rank", _i32), ("cap", _i32), ("slots", _i32), ("own", _i32),
+                ("eps", C.c_float), ("scale", C.c_float), ("d_rot", _vp), ("d_norm", _vp), ("d_uk", _vp), ("d_uv", _vp), ("d_q", _vp), ("d_part", _vp),
+                ("part_floats", _i64)]
+
+
+class PgScan(C.Structure):
+    _fields_ = [("inner", _i32), ("state", _i32), ("dt_rank", _i32), ("taps", _i32), ("d_conv", _vp), ("d_conv_bias", _vp), ("d_a", _vp), ("d_d", _vp),
+                ("d_dt_bias", _vp), ("d_dt", _vp)]
+
+
+_pb, _pd, _pa, _pl, _ps = (C.POINTER(x) for x in (PgBatch, PgDelta, PgAttention, PgLatent, PgScan))
 _f = C.c_float
 LM_SIGNATURES = {
     "pg_linear_wrap": (_i32, [_vp, _vp, _i64, _i64, _i64, C.POINTER(_vp)]),
     "pg_linear_free": (_i32, [_vp, _vp]),
     "pg_linear_run": (_i32, [_vp, _vp, _vp, _i32, _i64, _i32, _f, _vp, _i32, _i64]),
+    "pg_linear_run_ld": (_i32, [_vp, _vp, _vp, _i64, _i32, _i64, _i32, _f, _vp, _i32, _i64]),
     "pg_linear_run_routed": (_i32, [_vp, _vp, _vp, _vp, _i32, _i32, _i32, _f, _vp, _i32, _i64]),
     "pg_route_create": (_i32, [_vp, _i64, _i64, _i64, _i64, C.POINTER(_vp)]),
     "pg_route_free": (_i32, [_vp, _vp]),
@@ -178,6 +190,8 @@ LM_SIGNATURES = {
     "pg_route_run": (_i32, [_vp, _vp, _i32, _vp, _i64, _i64, _vp, _i32, _i32]),
     "pg_route_read": (_i32, [_vp, _vp, _vp, _vp]),
     "pg_embed_norm": (_i32, [_vp, _pb, _vp, _vp, _i64, _vp, _f, _vp, _vp, _i32, _i64]),
+    "pg_embed_prenorm": (_i32, [_vp, _pb, _vp, _i64, _vp, _f, _vp, _vp, _i32, _i64]),
+    "pg_norm_add_prenorm": (_i32, [_vp, _vp, _i64, _vp, _vp, _vp, _i64, _i64, _f, _vp, _i32, _i64]),
     "pg_norm_add": (_i32, [_vp, _vp, _i64, _vp, _vp, _vp, _i64, _i64, _f, _vp, _i32, _i64]),
     "pg_routed_norm_add": (_i32, [_vp, _vp, _vp, _i64, _vp, _vp, _vp, _i64, _i64, _f, _vp, _i32, _i64]),
     "pg_norm_rows": (_i32, [_vp, _vp, _vp, _i64, _i64, _vp, _f, _vp, _i32, _i64]),
@@ -185,6 +199,14 @@ LM_SIGNATURES = {
     "pg_delta_run": (_i32, [_vp, _pd, _pb, _vp, _i64, _vp, _vp, _vp, _i32, _i64]),
     "pg_attention_part_floats": (_i64, [_vp, _pa, _i64]),
     "pg_attention_run": (_i32, [_vp, _pa, _pb, _vp, _i64, _vp, _vp, _vp, _i32, _i64]),
+    "pg_latent_part_floats": (_i64, [_vp, _pl, _i32, _i64, _i64]),
+    "pg_latent_run": (_i32, [_vp, _pl, _pb, _i64, _i64, _i64, _vp, _i64, _vp, _vp, _i32, _i64]),
+    "pg_latent_prompt_supports": (_i32, [_pl]),
+    "pg_latent_prompt_prep": (_i32, [_vp, _pl, _pb, _i64, _i64, _i64, _vp, _i64, _vp]),
+    "pg_latent_prompt": (_i32, [_vp, _pl, _pb, _i64, _i64, _i64, _i64, _vp, _i64, _vp, _vp, _i64, _vp, _i64]),
+    "pg_scan_conv": (_i32, [_vp, _ps, _pb, _vp, _i64, _vp, _vp, _i32, _i64]),
+    "pg_scan_step": (_i32, [_vp, _ps, _pb, _vp, _i64, _vp, _i64, _vp, _i64, _vp, _vp, _i32, _i64]),
+    "pg_scan_run": (_i32, [_vp, _ps, _pb, _vp, _i64, _vp, _vp, _i64, _vp, _i64, _vp, _i64, _vp, _vp, _i32, _i64]),
 }
 # what both libraries carry (csrc/pg_core.cu, csrc/pg_sample.cu)
 CORE = [n for n in SIGNATURES if n.startswith(("pg_ctx_", "pg_graph_", "pg_mem_"))] + ["pg_last_error", "pg_version", "pg_launch_count",

@@ -41,7 +41,7 @@ SOURCES = CORE + [
 
 SOURCES_LM = CORE + [
     "pg_linear.cu", "pg_linear_gemv.cu", "pg_linear_tc.cu", "pg_linear_f32.cu",
-    "pg_route.cu", "pg_rows.cu", "pg_delta.cu", "pg_attention.cu", "pg_attention_tc.cu",
+    "pg_route.cu", "pg_rows.cu", "pg_delta.cu", "pg_scan.cu", "pg_attention.cu", "pg_attention_tc.cu", "pg_latent.cu",
 ]
 
 # component -> (library, sources)

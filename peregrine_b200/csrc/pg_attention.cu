@@ -1,5 +1,6 @@
-// Causal attention with per-head query / key norms, a query temperature and a softmax sink, for prompts and decoding,
-// over a contiguous cache per slot and key/value head.
+// Causal attention for prompts and decoding over a cache per slot and key/value head.  Each of these may be there or not:
+// per-head query / key norms, a query temperature, a softmax sink, a bias that grows with the distance (slope per head), and
+// a mask of chunks (a position sees its own chunk only; the cache is then a ring of whole chunks).
 //
 //   bf16, one token per sequence    attn_step_kernel: streams the cache once.  A CTA has one slice of the context of one
 //                                   (sequence, key/value head); it normalises the group's queries itself, the CTA with
@@ -30,7 +31,7 @@ __device__ __forceinline__ float temperature(const AttnShape &s, int pos)
     return 1.0f + s.coef * logf(floorf(__fdiv_rn((float)(pos + 1), s.every)) + 1.0f);
 }
 
-// One warp: dst = rms_norm(src[0 .. D)) * w * mul; columns D .. dp are zero (D <= 256).
+// One warp: dst = rms_norm(src[0 .. D)) * w * mul, or src * mul where w is null; columns D .. dp are zero (D <= 256).
 template <typename TA>
 __device__ __forceinline__ void head_norm(const float *src, const float *__restrict__ w, int D, int dp, float eps, float mul, TA *dst, int lane)
 {
@@ -41,11 +42,11 @@ __device__ __forceinline__ void head_norm(const float *src, const float *__restr
         ss += x[i] * x[i];
     }
     ss = pg_warp_sum(ss);
-    const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss, (float)D) + eps));
+    const float inv = w ? __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss, (float)D) + eps)) : 1.0f;
 #pragma unroll
     for (int i = 0; i < 8; i++) {
         const int c = i * 32 + lane;
-        if (c < dp) pg_put(dst + c, c < D ? x[i] * inv * __ldg(w + c) * mul : 0.0f);
+        if (c < dp) pg_put(dst + c, c < D ? x[i] * inv * (w ? __ldg(w + c) : 1.0f) * mul : 0.0f);
     }
 }
 
@@ -58,22 +59,23 @@ __global__ void __launch_bounds__(256)
     const int m = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int pos = __ldcg(bt.d_pos + m);
     const int64_t slot = __ldcg(bt.d_seq_slot + __ldcg(bt.d_row_seq + m));
-    if ((unsigned)pos >= (unsigned)s.cap) {   // outside the cache: record it, touch nothing
+    if ((unsigned)pos >= (unsigned)s.limit) {   // outside the cache: record it, touch nothing
         if (threadIdx.x == 0) atomicExch(status, (int32_t)PG_ERR_INVALID);
         return;
     }
     const float *row = proj + (int64_t)m * ldp;
     const float mul = temperature(s, pos);
+    const int at = attn_row(s, pos);
     for (int i = warp; i < s.H + 2 * s.G; i += 8) {
         if (i < s.H) {
             head_norm(row + i * s.D, s.qn, s.D, s.dp, s.eps, mul, q + ((int64_t)m * s.H + i) * s.dp, lane);
         } else if (i < s.H + s.G) {
             const int g = i - s.H;
-            head_norm(row + i * s.D, s.kn, s.D, s.dp, s.eps, 1.0f, kc + ((slot * s.G + g) * s.cap + pos) * s.dp, lane);
+            head_norm(row + i * s.D, s.kn, s.D, s.dp, s.eps, 1.0f, kc + ((slot * s.G + g) * s.cap + at) * s.dp, lane);
         } else {
             const int g = i - s.H - s.G;
             const float *src = row + (int64_t)(s.H + s.G) * s.D + (int64_t)g * s.V;
-            TA *dst = vc + ((slot * s.G + g) * s.cap + pos) * s.vp;
+            TA *dst = vc + ((slot * s.G + g) * s.cap + at) * s.vp;
             for (int c = lane; c < s.vp; c += 32) pg_put(dst + c, c < s.V ? __ldcg(src + c) : 0.0f);
         }
     }
@@ -91,16 +93,19 @@ __global__ void __launch_bounds__(AF_T)
     const int h = blockIdx.x, m = blockIdx.y, g = h / s.rep, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int pos = __ldcg(bt.d_pos + m);
     const int64_t slot = __ldcg(bt.d_seq_slot + __ldcg(bt.d_row_seq + m));
-    if ((unsigned)pos >= (unsigned)s.cap) return;
+    if ((unsigned)pos >= (unsigned)s.limit) return;
     float *sq = sm, *sp = sm + s.dp;
     for (int i = tid; i < s.dp; i += AF_T) sq[i] = __ldcg(q + ((int64_t)m * s.H + h) * s.dp + i);
-    const float *kb = kc + (slot * s.G + g) * (int64_t)s.cap * s.dp, *vb = vc + (slot * s.G + g) * (int64_t)s.cap * s.vp;
+    const int low = attn_low(s, pos);
+    const int64_t first = (slot * s.G + g) * (int64_t)s.cap + attn_row(s, low) - low;   // row of position 0, as it were
+    const float *kb = kc + first * s.dp, *vb = vc + first * s.vp;
+    const float slope = s.slopes ? __ldg(s.slopes + h) : 0.0f;
     constexpr int NV = 8;                      // value columns per thread (vdim <= 1024)
     float acc[NV], mx = s.sink ? 0.0f : -INFINITY, l = s.sink ? 1.0f : 0.0f;
 #pragma unroll
     for (int i = 0; i < NV; i++) acc[i] = 0.0f;
     __syncthreads();
-    for (int j0 = 0; j0 <= pos; j0 += AF_T) {
+    for (int j0 = low; j0 <= pos; j0 += AF_T) {
         const int j = j0 + tid;
         float sc = -INFINITY;
         if (j <= pos) {
@@ -112,7 +117,7 @@ __global__ void __launch_bounds__(AF_T)
                 d[0] = fmaf(sq[i], a.x, d[0]), d[1] = fmaf(sq[i + 1], a.y, d[1]), d[2] = fmaf(sq[i + 2], a.z, d[2]), d[3] = fmaf(sq[i + 3], a.w, d[3]);
                 d[4] = fmaf(sq[i + 4], b.x, d[4]), d[5] = fmaf(sq[i + 5], b.y, d[5]), d[6] = fmaf(sq[i + 6], b.z, d[6]), d[7] = fmaf(sq[i + 7], b.w, d[7]);
             }
-            sc = (((d[0] + d[1]) + (d[2] + d[3])) + ((d[4] + d[5]) + (d[6] + d[7]))) * s.scale;
+            sc = (((d[0] + d[1]) + (d[2] + d[3])) + ((d[4] + d[5]) + (d[6] + d[7]))) * s.scale - slope * (float)(pos - j);
         }
         float bm = sc;
 #pragma unroll
@@ -200,8 +205,10 @@ __global__ void __launch_bounds__(WARPS * 32)
     const int64_t slot = __ldcg(bt.d_seq_slot + seq);
     const bf16 *kb = kc + (slot * s.G + g) * (int64_t)s.cap * s.dp, *vb = vc + (slot * s.G + g) * (int64_t)s.cap * s.vp;
     const int last = min(rr0 + WARPS * 16, total) - 1;
-    const int kmax = pos0 + last / s.rep + 1;             // keys the tile sees
-    if (kmax > s.cap) return;                             // recorded by attn_prep_kernel
+    const int kmax = pos0 + last / s.rep + 1;             // the tile sees keys kmin .. kmax - 1
+    if (kmax > s.limit) return;                           // recorded by attn_prep_kernel
+    const int kmin = attn_low(s, pos0 + rr0 / s.rep);
+    const int low_last = attn_low(s, kmax - 1);           // the first key of its last row
     const int nk = s.dp / 16, nv = s.vp / 8;
     const int kstride = s.dp * 2 + 16, vstride = s.vp * 2 + 16;
     const uint32_t ks = pg_smem(smem), vs = ks + 2 * AP_KEYS * kstride;
@@ -209,6 +216,8 @@ __global__ void __launch_bounds__(WARPS * 32)
     const int my0 = rr0 + warp * 16 + r, my1 = my0 + 8;
     const int c0 = min(my0, total - 1), c1 = min(my1, total - 1);
     const int lim0 = pos0 + c0 / s.rep, lim1 = pos0 + c1 / s.rep;    // last key of the lane's two rows
+    const int low0 = attn_low(s, lim0), low1 = attn_low(s, lim1);    // and the first
+    const float bias0 = s.slopes ? __ldg(s.slopes + g * s.rep + c0 % s.rep) * LOG2E : 0.0f, bias1 = s.slopes ? __ldg(s.slopes + g * s.rep + c1 % s.rep) * LOG2E : 0.0f;
     uint32_t qf[DC][4];
     {
         const bf16 *q0 = q + ((int64_t)(row0 + c0 / s.rep) * s.H + g * s.rep + c0 % s.rep) * s.dp + 2 * t;
@@ -224,14 +233,19 @@ __global__ void __launch_bounds__(WARPS * 32)
         }
     }
     auto fetch = [&](int buf, int j0) {
-        const int kw = s.dp / 8, vw = s.vp / 8;
+        const int kw = s.dp / 8, vw = s.vp / 8, e0 = attn_row(s, j0), left = kmax - 1 - j0;
+        auto row_of = [&](int k) {                        // (at most one turn of the ring: it holds more than a tile's keys)
+            int e = e0 + min(k, left);
+            while (e >= s.cap) e -= s.cap;
+            return (int64_t)e;
+        };
         for (int i = threadIdx.x; i < AP_KEYS * kw; i += WARPS * 32) {
             const int k = i / kw, e = (i - k * kw) * 8;
-            pg_cp16(tile_at(ks + buf * AP_KEYS * kstride, kstride, k, e), kb + (int64_t)min(j0 + k, kmax - 1) * s.dp + e);
+            pg_cp16(tile_at(ks + buf * AP_KEYS * kstride, kstride, k, e), kb + row_of(k) * s.dp + e);
         }
         for (int i = threadIdx.x; i < AP_KEYS * vw; i += WARPS * 32) {
             const int k = i / vw, e = (i - k * vw) * 8;
-            pg_cp16(tile_at(vs + buf * AP_KEYS * vstride, vstride, k, e), vb + (int64_t)min(j0 + k, kmax - 1) * s.vp + e);
+            pg_cp16(tile_at(vs + buf * AP_KEYS * vstride, vstride, k, e), vb + row_of(k) * s.vp + e);
         }
         pg_cp_commit();
     };
@@ -241,10 +255,11 @@ __global__ void __launch_bounds__(WARPS * 32)
 #pragma unroll
         for (int j = 0; j < 4; j++) o[i][j] = 0.0f;
     const float sl = s.scale * LOG2E;                     // scores in units of log 2
-    float m0 = s.sink ? 0.0f : -INFINITY, m1 = m0, l0 = 0.0f, l1 = 0.0f;
-    fetch(0, 0);
+    // (a row may see no key of a chunk in front of its own: the maxima start finite, so that exp2(-inf - m) is 0)
+    float m0 = s.sink ? 0.0f : -1e30f, m1 = m0, l0 = 0.0f, l1 = 0.0f;
+    fetch(0, kmin);
     int buf = 0;
-    for (int j0 = 0; j0 < kmax; j0 += AP_KEYS, buf ^= 1) {
+    for (int j0 = kmin; j0 < kmax; j0 += AP_KEYS, buf ^= 1) {
         if (j0 + AP_KEYS < kmax) {
             fetch(buf ^ 1, j0 + AP_KEYS);
             pg_cp_wait<1>();
@@ -261,14 +276,14 @@ __global__ void __launch_bounds__(WARPS * 32)
 #pragma unroll
         for (int n = 0; n < AP_KEYS / 16; n++) scores16<DC>(qf, nk, kt, kstride, n * 16, lane, sc[2 * n], sc[2 * n + 1]);
         float b0 = -INFINITY, b1 = -INFINITY;
-        const bool edge = j0 + AP_KEYS - 1 > pos0 + rr0 / s.rep;   // some row of the tile does not see all of these keys
+        const bool edge = j0 + AP_KEYS - 1 > pos0 + rr0 / s.rep || j0 < low_last;   // some row of the tile does not see all of these keys
 #pragma unroll
         for (int n = 0; n < AP_KEYS / 8; n++)
 #pragma unroll
             for (int j = 0; j < 2; j++) {
                 const int key = j0 + n * 8 + 2 * t + j;
-                sc[n][j] = (!edge || key <= lim0) ? sc[n][j] * sl : -INFINITY;
-                sc[n][2 + j] = (!edge || key <= lim1) ? sc[n][2 + j] * sl : -INFINITY;
+                sc[n][j] = (!edge || (key <= lim0 && key >= low0)) ? fmaf(bias0, (float)(key - lim0), sc[n][j] * sl) : -INFINITY;
+                sc[n][2 + j] = (!edge || (key <= lim1 && key >= low1)) ? fmaf(bias1, (float)(key - lim1), sc[n][2 + j] * sl) : -INFINITY;
                 b0 = fmaxf(b0, sc[n][j]);
                 b1 = fmaxf(b1, sc[n][2 + j]);
             }
@@ -277,7 +292,6 @@ __global__ void __launch_bounds__(WARPS * 32)
             b0 = fmaxf(b0, __shfl_xor_sync(0xffffffffu, b0, x));
             b1 = fmaxf(b1, __shfl_xor_sync(0xffffffffu, b1, x));
         }
-        // (the first keys are seen by every row, so the maxima are finite from the first tile on)
         const float n0 = fmaxf(m0, b0), n1 = fmaxf(m1, b1);
         const float f0 = exp2f(m0 - n0), f1 = exp2f(m1 - n1);
         m0 = n0;
@@ -367,8 +381,8 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
     asm volatile("griddepcontrol.wait;" ::: "memory");
     const int pos = __ldcg(bt.d_pos + b);
     const int64_t slot = __ldcg(bt.d_seq_slot + b);
-    const int len = pos + 1;
-    if ((unsigned)pos >= (unsigned)s.cap) {   // outside the cache: record it, touch nothing (all CTAs of the row leave)
+    const int low = attn_low(s, pos), len = pos + 1 - low;   // keys are counted from the first that is seen
+    if ((unsigned)pos >= (unsigned)s.limit) {   // outside the cache: record it, touch nothing (all CTAs of the row leave)
         if (threadIdx.x == 0) atomicExch(status, (int32_t)PG_ERR_INVALID);
         return;
     }
@@ -377,7 +391,8 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
     const int used = (len + chunk - 1) / chunk;           // slices with keys; the others leave at once
     if (t0 >= t1) return;
     const bool newest = FUSED && t1 == len;
-    bf16 *kb = kc + (slot * s.G + g) * (int64_t)s.cap * s.dp, *vb = vc + (slot * s.G + g) * (int64_t)s.cap * s.vp;
+    const int64_t first = (slot * s.G + g) * (int64_t)s.cap + attn_row(s, low);
+    bf16 *kb = kc + first * s.dp, *vb = vc + first * s.vp;
     const int nk = s.dp / 16, nv = s.vp / 8;
 
     // the warp's 16-key tiles: t0 + 16 (warp + 4 i); lanes 0 .. 15 ask for a key each, lanes 16 .. 31 for a value each
@@ -417,9 +432,9 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
         for (int i = threadIdx.x; i < (s.dp + s.vp) / 2; i += AS_WARPS * 32) {
             const uint32_t x = reinterpret_cast<const uint32_t *>(k_new)[i];
             if (i < s.dp / 2)
-                reinterpret_cast<uint32_t *>(kb + (int64_t)pos * s.dp)[i] = x;
+                reinterpret_cast<uint32_t *>(kb + (int64_t)(len - 1) * s.dp)[i] = x;
             else
-                reinterpret_cast<uint32_t *>(vb + (int64_t)pos * s.vp)[i - s.dp / 2] = x;
+                reinterpret_cast<uint32_t *>(vb + (int64_t)(len - 1) * s.vp)[i - s.dp / 2] = x;
         }
     }
     uint32_t qf[DC][4];
@@ -435,6 +450,7 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
 #pragma unroll
         for (int j = 0; j < 4; j++) o[i][j] = 0.0f;
     const float sl = s.scale * LOG2E;
+    const float bias0 = s.slopes && r < heads ? __ldg(s.slopes + h0 + r) * LOG2E : 0.0f, bias1 = s.slopes && r + 8 < heads ? __ldg(s.slopes + h0 + r + 8) * LOG2E : 0.0f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;
     bool ok = true;
     for (int i = 0; i < mine; i++) {
@@ -443,12 +459,12 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
         if (!ok) break;
         const int j0 = t0 + 16 * (warp + AS_WARPS * i);
         const uint32_t kt = ring + (uint32_t)(i % AS_STAGES) * stage, vt = kt + 16 * kstride;
-        if (newest && j0 + 16 > pos) {
+        if (newest && j0 + 16 >= len) {
             // the copies brought what the cache held at the newest position: put the new row in its place
             unsigned char *at = smem + (size_t)warp * AS_STAGES * stage + (size_t)(i % AS_STAGES) * stage;
-            for (int x = lane; x < s.dp / 2; x += 32) reinterpret_cast<uint32_t *>(at + (pos - j0) * kstride)[x] = reinterpret_cast<const uint32_t *>(k_new)[x];
+            for (int x = lane; x < s.dp / 2; x += 32) reinterpret_cast<uint32_t *>(at + (len - 1 - j0) * kstride)[x] = reinterpret_cast<const uint32_t *>(k_new)[x];
             for (int x = lane; x < s.vp / 2; x += 32)
-                reinterpret_cast<uint32_t *>(at + 16 * kstride + (pos - j0) * vstride)[x] = reinterpret_cast<const uint32_t *>(v_new)[x];
+                reinterpret_cast<uint32_t *>(at + 16 * kstride + (len - 1 - j0) * vstride)[x] = reinterpret_cast<const uint32_t *>(v_new)[x];
             __syncwarp();
         }
         float sc[2][4] = {};
@@ -458,9 +474,10 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
         for (int n = 0; n < 2; n++)
 #pragma unroll
             for (int j = 0; j < 2; j++) {
-                const bool in = j0 + n * 8 + 2 * t + j < t1;
-                sc[n][j] = in ? sc[n][j] * sl : -INFINITY;
-                sc[n][2 + j] = in ? sc[n][2 + j] * sl : -INFINITY;
+                const int key = j0 + n * 8 + 2 * t + j;
+                const float back = (float)(key - (len - 1));
+                sc[n][j] = key < t1 ? fmaf(bias0, back, sc[n][j] * sl) : -INFINITY;
+                sc[n][2 + j] = key < t1 ? fmaf(bias1, back, sc[n][2 + j] * sl) : -INFINITY;
                 b0 = fmaxf(b0, sc[n][j]);
                 b1 = fmaxf(b1, sc[n][2 + j]);
             }
@@ -617,15 +634,17 @@ AttnShape shape_of(const pg_attention *p)
     AttnShape s;
     s.H = p->heads, s.G = p->kv_heads, s.rep = p->heads / p->kv_heads, s.D = p->dim, s.V = p->vdim;
     s.dp = (int)pg_up(s.D, 16), s.vp = (int)pg_up(s.V, 16);
-    s.cap = p->cap, s.sink = p->sink;
+    s.cap = p->cap, s.sink = p->sink, s.chunk = p->chunk, s.limit = p->positions > 0 ? p->positions : p->cap;
+    s.slopes = p->d_slopes;
     s.eps = p->eps, s.scale = p->scale, s.coef = p->temp_coef, s.every = p->temp_every;
     s.qn = p->d_q_norm, s.kn = p->d_k_norm;
     return s;
 }
 
-// slices of the context: enough CTAs for about two per SM, none shorter than 128 positions of a full cache
-int slices(const pg_ctx *ctx, int64_t units, int64_t cap)
+// slices of the context: enough CTAs for about two per SM, none shorter than 128 positions of the longest context
+int slices(const pg_ctx *ctx, int64_t units, const AttnShape &s)
 {
+    const int64_t cap = s.chunk && s.chunk < s.cap ? s.chunk : s.cap;
     int64_t S = std::max<int64_t>(1, 2 * (int64_t)ctx->sm_count / std::max<int64_t>(1, units));
     S = std::min<int64_t>(S, std::max<int64_t>(1, cap / 128));
     return (int)std::min<int64_t>(S, AS_SLICES);
@@ -653,12 +672,19 @@ int32_t run_step(pg_ctx *ctx, const AttnShape &s, const pg_batch *bt, const floa
     static std::atomic<uint64_t> set{0};
     PG_CUDA(pg_max_smem_once(attn_step_kernel<DC, VC, FUSED>, 220 * 1024, ctx->device, set));
     const int ht = (s.rep + 15) / 16;
-    const int S = slices(ctx, (int64_t)bt->rows * s.G * ht, s.cap);
+    const int S = slices(ctx, (int64_t)bt->rows * s.G * ht, s);
     return launch_pdl(ctx, attn_step_kernel<DC, VC, FUSED>, dim3((unsigned)S, (unsigned)(s.G * ht), (unsigned)bt->rows), dim3(AS_WARPS * 32), (size_t)smem, s,
                       *bt, proj, ldp, q, kc, vc, part, tickets, out, ldo, ctx->d_status, ctx->wait_limit_ns);
 }
 
 }  // namespace
+
+int32_t pgk_attention_f32(pg_ctx *ctx, const AttnShape &s, const pg_batch *bt, const float *q, const float *kc, const float *vc, float *out, int64_t ldo)
+{
+    PG_REQUIRE(bt->rows <= 65535, "attention: too many rows for the f32 form");
+    PG_REQUIRE(s.V <= 8 * AF_T && (s.dp + AF_T) * 4 <= 48 * 1024, "attention: heads too wide for the f32 form");
+    return launch_pdl(ctx, attn_f32_kernel, dim3((unsigned)s.H, (unsigned)bt->rows), dim3(AF_T), (size_t)(s.dp + AF_T) * 4, s, *bt, q, kc, vc, out, ldo);
+}
 
 extern "C" {
 
@@ -668,7 +694,7 @@ PG_API int64_t pg_attention_part_floats(pg_ctx *ctx, const pg_attention *p, int6
     const AttnShape s = shape_of(p);
     const int64_t per = (int64_t)s.G * ((s.rep + 15) / 16);
     int64_t most = 0;
-    for (int64_t rows = 1; rows <= max_seqs; rows++) most = std::max(most, rows * per * slices(ctx, rows * per, s.cap));
+    for (int64_t rows = 1; rows <= max_seqs; rows++) most = std::max(most, rows * per * slices(ctx, rows * per, s));
     return most * 16 * (s.vp + 4);
 }
 
@@ -676,10 +702,14 @@ PG_API int32_t pg_attention_run(pg_ctx *ctx, const pg_attention *p, const pg_bat
                                 void *d_vcache, void *d_out, int32_t dtype, int64_t ldo)
 {
     PG_ENTER(ctx);
-    PG_REQUIRE(p && batch && d_proj && d_kcache && d_vcache && d_out && p->d_q && p->d_part && p->d_tickets && p->d_q_norm && p->d_k_norm,
+    PG_REQUIRE(p && batch && d_proj && d_kcache && d_vcache && d_out && p->d_q && p->d_part && p->d_tickets,
                "attention: null pointer");
     PG_REQUIRE(p->heads > 0 && p->kv_heads > 0 && p->heads % p->kv_heads == 0 && p->dim > 0 && p->dim <= 256 && p->vdim > 0 && p->vdim <= 256 && p->cap > 0,
                "attention: bad shape (heads %d / %d, dim %d and vdim %d at most 256)", p->heads, p->kv_heads, p->dim, p->vdim);
+    PG_REQUIRE(p->chunk >= 0 && (p->chunk == 0 ? p->positions <= p->cap : p->cap % p->chunk == 0),
+               "attention: a cache of %d rows for %d positions in chunks of %d", p->cap, p->positions, p->chunk);
+    PG_REQUIRE(p->chunk == 0 || p->positions <= p->cap || ((int64_t)(p->chunk + batch->max_len - 2) / p->chunk + 1) * p->chunk <= p->cap,
+               "attention: a step of %d tokens has more chunks of %d than the cache of %d rows", batch->max_len, p->chunk, p->cap);
     const AttnShape s = shape_of(p);
     PG_REQUIRE(ldp >= (int64_t)(s.H + s.G) * s.D + (int64_t)s.G * s.V && ldo >= (int64_t)s.H * s.V, "attention: rows too short");
     PG_REQUIRE(s.G <= 65535 && batch->rows >= 0 && batch->seqs <= 65535, "attention: too many heads or sequences");
@@ -689,9 +719,7 @@ PG_API int32_t pg_attention_run(pg_ctx *ctx, const pg_attention *p, const pg_bat
         int32_t rc = launch_pdl(ctx, attn_prep_kernel<float>, dim3((unsigned)M), dim3(256), 0, s, *batch, d_proj, ldp, (float *)p->d_q, (float *)d_kcache,
                                 (float *)d_vcache, ctx->d_status);
         if (rc != PG_OK) return rc;
-        PG_REQUIRE(M <= 65535, "attention: too many rows for the f32 form");
-        return launch_pdl(ctx, attn_f32_kernel, dim3((unsigned)s.H, (unsigned)M), dim3(AF_T), (size_t)(s.dp + AF_T) * 4, s, *batch, (const float *)p->d_q,
-                          (const float *)d_kcache, (const float *)d_vcache, (float *)d_out, ldo);
+        return pgk_attention_f32(ctx, s, batch, (const float *)p->d_q, (const float *)d_kcache, (const float *)d_vcache, (float *)d_out, ldo);
     }
     bf16 *q = (bf16 *)p->d_q, *kc = (bf16 *)d_kcache, *vc = (bf16 *)d_vcache, *out = (bf16 *)d_out;
     const bool step = batch->max_len == 1, fused = step && s.rep <= 16;

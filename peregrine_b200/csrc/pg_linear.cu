@@ -34,15 +34,22 @@ PG_API int32_t pg_linear_free(pg_ctx *ctx, pg_linear *lin)
 PG_API int32_t pg_linear_run(pg_ctx *ctx, pg_linear *lin, const void *d_a, int32_t dtype, int64_t m, int32_t act, float limit, void *d_y,
                              int32_t y_dtype, int64_t ldy)
 {
+    return pg_linear_run_ld(ctx, lin, d_a, lin ? lin->k : 0, dtype, m, act, limit, d_y, y_dtype, ldy);
+}
+
+PG_API int32_t pg_linear_run_ld(pg_ctx *ctx, pg_linear *lin, const void *d_a, int64_t lda, int32_t dtype, int64_t m, int32_t act, float limit, void *d_y,
+                                int32_t y_dtype, int64_t ldy)
+{
     PG_ENTER(ctx);
     PG_REQUIRE(lin && d_a && d_y && m >= 0, "linear: bad arguments");
+    PG_REQUIRE(lda >= lin->k && lda % 8 == 0, "linear: rows of a are %lld apart, K is %lld (and a multiple of 8 is wanted)", (long long)lda, (long long)lin->k);
     PG_REQUIRE(act >= PG_ACT_NONE && act <= PG_ACT_CLAMPED_SWISH_GLU && (act == PG_ACT_NONE || (lin->n % 16 == 0 && y_dtype == dtype)),
                "linear: bad activation");
     PG_REQUIRE(ldy >= (act == PG_ACT_NONE ? lin->n : lin->n / 2) && ((uintptr_t)d_a & 15) == 0, "linear: output rows too short or operand not aligned");
     if (m == 0) return PG_OK;
-    if (dtype == PG_F32) return pgk_linear_f32(ctx, lin, (const float *)d_a, m, act, limit, d_y, y_dtype, ldy, nullptr);
-    if (pgk_linear_gemv_supports(lin, m)) return pgk_linear_gemv(ctx, lin, (const bf16 *)d_a, m, act, limit, d_y, y_dtype, ldy, nullptr, 1);
-    return pgk_linear_tc(ctx, lin, (const bf16 *)d_a, m, act, limit, d_y, y_dtype, ldy, nullptr);
+    if (dtype == PG_F32) return pgk_linear_f32(ctx, lin, (const float *)d_a, lda, m, act, limit, d_y, y_dtype, ldy, nullptr);
+    if (pgk_linear_gemv_supports(lin, m)) return pgk_linear_gemv(ctx, lin, (const bf16 *)d_a, lda, m, act, limit, d_y, y_dtype, ldy, nullptr, 1);
+    return pgk_linear_tc(ctx, lin, (const bf16 *)d_a, lda, m, act, limit, d_y, y_dtype, ldy, nullptr);
 }
 
 PG_API int32_t pg_linear_run_routed(pg_ctx *ctx, pg_linear *lin, pg_route *route, const void *d_a, int32_t dtype, int32_t by_token, int32_t act,
@@ -58,7 +65,7 @@ PG_API int32_t pg_linear_run_routed(pg_ctx *ctx, pg_linear *lin, pg_route *route
     if (route->block == PG_ROUTE_SMALL) {
         PG_REQUIRE(dtype == PG_BF16 && pgk_linear_gemv_supports(lin, 1), "linear: the route was made for the streaming form");
         const int64_t pairs = route->m * route->top;
-        return pgk_linear_gemv(ctx, lin, (const bf16 *)d_a, route->m, act, limit, d_y, y_dtype, ldy, &rt, pairs < route->experts ? pairs : route->experts);
+        return pgk_linear_gemv(ctx, lin, (const bf16 *)d_a, lin->k, route->m, act, limit, d_y, y_dtype, ldy, &rt, pairs < route->experts ? pairs : route->experts);
     }
     // rows the route can have for this many tokens
     const int64_t pairs = route->m * route->top;
@@ -74,8 +81,8 @@ PG_API int32_t pg_linear_run_routed(pg_ctx *ctx, pg_linear *lin, pg_route *route
         if (rc != PG_OK) return rc;
         a = ctx->scratch;
     }
-    if (dtype == PG_F32) return pgk_linear_f32(ctx, lin, (const float *)a, rows, act, limit, d_y, y_dtype, ldy, &rt);
-    return pgk_linear_tc(ctx, lin, (const bf16 *)a, rows, act, limit, d_y, y_dtype, ldy, &rt);
+    if (dtype == PG_F32) return pgk_linear_f32(ctx, lin, (const float *)a, lin->k, rows, act, limit, d_y, y_dtype, ldy, &rt);
+    return pgk_linear_tc(ctx, lin, (const bf16 *)a, lin->k, rows, act, limit, d_y, y_dtype, ldy, &rt);
 }
 
 }  // extern "C"

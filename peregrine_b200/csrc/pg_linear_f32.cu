@@ -8,7 +8,7 @@ constexpr int FM = 64, FN = 64, FK = 16;
 
 template <int ACT, typename TY>
 __global__ void __launch_bounds__(256)
-    linear_f32_kernel(const float *__restrict__ a, const bf16 *__restrict__ w, int M, int N, int K, float limit, TY *__restrict__ y, int64_t ldy,
+    linear_f32_kernel(const float *__restrict__ a, int64_t lda, const bf16 *__restrict__ w, int M, int N, int K, float limit, TY *__restrict__ y, int64_t ldy,
                       const PgRouted rt)
 {
     __shared__ float sa[FK][FM + 4];
@@ -25,7 +25,7 @@ __global__ void __launch_bounds__(256)
     for (int k0 = 0; k0 < K; k0 += FK) {
         float4 va = make_float4(0.f, 0.f, 0.f, 0.f);
         uint2 vw = make_uint2(0u, 0u);
-        if (m0 + lr < M) va = __ldcg(reinterpret_cast<const float4 *>(a + (int64_t)(m0 + lr) * K + k0 + lk));
+        if (m0 + lr < M) va = __ldcg(reinterpret_cast<const float4 *>(a + (m0 + lr) * lda + k0 + lk));
         if (n0 + lr < N) vw = __ldg(reinterpret_cast<const uint2 *>(w + (int64_t)(n0 + lr) * K + k0 + lk));
         __syncthreads();
         sa[lk][lr] = va.x, sa[lk + 1][lr] = va.y, sa[lk + 2][lr] = va.z, sa[lk + 3][lr] = va.w;
@@ -70,7 +70,7 @@ __global__ void __launch_bounds__(256)
 
 }  // namespace
 
-int32_t pgk_linear_f32(pg_ctx *ctx, const pg_linear *lin, const float *a, int64_t m, int act, float limit, void *y, int y_dtype, int64_t ldy,
+int32_t pgk_linear_f32(pg_ctx *ctx, const pg_linear *lin, const float *a, int64_t lda, int64_t m, int act, float limit, void *y, int y_dtype, int64_t ldy,
                        const PgRouted *routed)
 {
     PG_REQUIRE(y_dtype == PG_F32, "linear: an f32 step has f32 outputs");
@@ -79,7 +79,7 @@ int32_t pgk_linear_f32(pg_ctx *ctx, const pg_linear *lin, const float *a, int64_
     const dim3 grid((unsigned)((m + FM - 1) / FM), (unsigned)((lin->n + FN - 1) / FN));
     PG_REQUIRE(grid.y <= 65535, "linear: too many output columns for the f32 form");
 #define PG_F32_CASE(A) \
-    return launch_pdl(ctx, linear_f32_kernel<A, float>, grid, dim3(256), 0, a, lin->w, (int)m, (int)lin->n, (int)lin->k, limit, (float *)y, ldy, rt)
+    return launch_pdl(ctx, linear_f32_kernel<A, float>, grid, dim3(256), 0, a, lda, lin->w, (int)m, (int)lin->n, (int)lin->k, limit, (float *)y, ldy, rt)
     if (act == PG_ACT_NONE) PG_F32_CASE(PG_ACT_NONE);
     if (act == PG_ACT_GELU_TANH_GLU) PG_F32_CASE(PG_ACT_GELU_TANH_GLU);
     PG_F32_CASE(PG_ACT_CLAMPED_SWISH_GLU);

@@ -36,7 +36,7 @@ constexpr int GV_RING = GV_WARPS * GV_SLOTS * GV_SLOT;
 // slabs (SPLIT): [sp][items][32 lanes][4 NT]
 template <int ACT, bool HI, bool ROUTED, bool SPLIT, typename TY>
 __global__ void __launch_bounds__(GV_THREADS, 1)
-    linear_gemv_kernel(const bf16 *__restrict__ a, int M, const bf16 *__restrict__ w, int N, int K, int kw, int KW, int KH, float limit,
+    linear_gemv_kernel(const bf16 *__restrict__ a, int64_t lda, int M, const bf16 *__restrict__ w, int N, int K, int kw, int KW, int KH, float limit,
                        TY *__restrict__ y, int64_t ldy, const PgRouted rt, int sp, float *slabs, unsigned int *tickets, int32_t *status,
                        unsigned long long limit_ns)
 {
@@ -132,7 +132,7 @@ __global__ void __launch_bounds__(GV_THREADS, 1)
                     r0 = rt.by_token ? p0 / rt.top : blk * PG_ROUTE_SMALL + r;
                     r1 = rt.by_token ? p1 / rt.top : blk * PG_ROUTE_SMALL + r + 8;
                 }
-                const bf16 *a0 = a + r0 * K + k0 + t * 8, *a1 = a + r1 * K + k0 + t * 8;
+                const bf16 *a0 = a + r0 * lda + k0 + t * 8, *a1 = a + r1 * lda + k0 + t * 8;
 #pragma unroll
                 for (int s = 0; s < GV_KSTEPS; s++) {
                     lo[s] = hi[s] = make_uint4(0u, 0u, 0u, 0u);
@@ -235,7 +235,7 @@ __global__ void __launch_bounds__(GV_THREADS, 1)
 constexpr size_t GV_TICKET_BYTES = 64 * 1024;   // the head of the context's split-K workspace: zero between calls
 
 template <int ACT, bool HI, bool ROUTED, bool SPLIT, typename TY>
-int32_t gv_launch(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int M, int kw, int KW, int KH, int grid, int sp, float limit, TY *y, int64_t ldy,
+int32_t gv_launch(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int64_t lda, int M, int kw, int KW, int KH, int grid, int sp, float limit, TY *y, int64_t ldy,
                   const PgRouted &rt)
 {
     constexpr int NT = ACT == PG_ACT_NONE ? 1 : 2;
@@ -246,7 +246,7 @@ int32_t gv_launch(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int M, int k
     PG_CUDA(pg_max_smem_once(kern, 226 * 1024, ctx->device, smem_set));
     unsigned int *tickets = reinterpret_cast<unsigned int *>(ctx->splitk);
     float *slabs = SPLIT ? reinterpret_cast<float *>(reinterpret_cast<unsigned char *>(ctx->splitk) + GV_TICKET_BYTES) : nullptr;
-    return launch_pdl(ctx, kern, dim3((unsigned)grid), dim3(GV_THREADS), (size_t)smem, a, M, lin->w, (int)lin->n, (int)lin->k, kw, KW, KH, limit, y, ldy, rt,
+    return launch_pdl(ctx, kern, dim3((unsigned)grid), dim3(GV_THREADS), (size_t)smem, a, lda, M, lin->w, (int)lin->n, (int)lin->k, kw, KW, KH, limit, y, ldy, rt,
                       sp, slabs, tickets, ctx->d_status, ctx->wait_limit_ns);
 }
 
@@ -257,7 +257,7 @@ inline int gv_parts(int64_t k) { return (int)((k + GV_WARPS * GV_KW_MAX - 1) / (
 
 bool pgk_linear_gemv_supports(const pg_linear *lin, int64_t m) { return m >= 1 && m <= 16 && gv_parts(lin->k) <= 16 && lin->n < (1 << 30); }
 
-int32_t pgk_linear_gemv(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int64_t m, int act, float limit, void *y, int y_dtype, int64_t ldy,
+int32_t pgk_linear_gemv(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int64_t lda, int64_t m, int act, float limit, void *y, int y_dtype, int64_t ldy,
                         const PgRouted *routed, int64_t max_blocks)
 {
     const int K = (int)lin->k, nt = act == PG_ACT_NONE ? 1 : 2;
@@ -281,7 +281,7 @@ int32_t pgk_linear_gemv(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int64_
     const PgRouted &rt = routed ? *routed : no_route;
     const bool hi = m > 8 || routed;
     const int M = (int)m;
-#define PG_GV(ACT, HI, RT, SP, TY) return gv_launch<ACT, HI, RT, SP, TY>(ctx, lin, a, M, kw, KW, KH, grid, sp, limit, (TY *)y, ldy, rt)
+#define PG_GV(ACT, HI, RT, SP, TY) return gv_launch<ACT, HI, RT, SP, TY>(ctx, lin, a, lda, M, kw, KW, KH, grid, sp, limit, (TY *)y, ldy, rt)
 #define PG_GV_SP(ACT, HI, RT, TY)                 \
     do {                                          \
         if (sp > 1) PG_GV(ACT, HI, RT, true, TY); \

@@ -248,24 +248,24 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
 }
 
 // ---------------------------------------------------------------- host side ----
-// [rows, k] bf16 row-major; box = 64 elements of K x box_rows rows
-int32_t encode_kmajor(CUtensorMap *map, const void *ptr, int64_t rows, int64_t k, int box_rows)
+// [rows, k] bf16, rows ld elements apart; box = 64 elements of K x box_rows rows
+int32_t encode_kmajor(CUtensorMap *map, const void *ptr, int64_t rows, int64_t k, int64_t ld, int box_rows)
 {
-    const cuuint64_t dims[2] = {(cuuint64_t)k, (cuuint64_t)rows}, strides[1] = {(cuuint64_t)k * 2};
+    const cuuint64_t dims[2] = {(cuuint64_t)k, (cuuint64_t)rows}, strides[1] = {(cuuint64_t)ld * 2};
     const cuuint32_t box[2] = {(cuuint32_t)BK, (cuuint32_t)box_rows};
     return pg_encode_bf16(map, ptr, 2, dims, strides, box);
 }
 
 template <int BN, int ACT, typename TY>
-int32_t launch(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t m, float limit, TY *y, int64_t ldy, const PgRouted &rt)
+int32_t launch(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t lda, int64_t m, float limit, TY *y, int64_t ldy, const PgRouted &rt)
 {
     using C = Cfg<BN>;
     CUtensorMap ta;
-    int32_t rc = encode_kmajor(&ta, a, m, lin->k, BM);
+    int32_t rc = encode_kmajor(&ta, a, m, lin->k, lda, BM);
     if (rc) return rc;
     const int at = BN == 128 || BN == 32 ? 0 : 1;
     if (lin->tmap_rows[at] != BN) {
-        rc = encode_kmajor(reinterpret_cast<CUtensorMap *>(lin->tmap[at]), lin->w, lin->experts * lin->n, lin->k, BN);
+        rc = encode_kmajor(reinterpret_cast<CUtensorMap *>(lin->tmap[at]), lin->w, lin->experts * lin->n, lin->k, lin->k, BN);
         if (rc) return rc;
         lin->tmap_rows[at] = BN;
     }
@@ -279,22 +279,22 @@ int32_t launch(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t m, float limi
 }
 
 template <int ACT, typename TY>
-int32_t dispatch(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t m, float limit, TY *y, int64_t ldy, const PgRouted &rt)
+int32_t dispatch(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t lda, int64_t m, float limit, TY *y, int64_t ldy, const PgRouted &rt)
 {
     // the widest tile that still gives every SM one
     const int64_t tiles_m = (m + BM - 1) / BM;
     int bn = 32;
     for (int cand = 64; cand <= 256; cand *= 2)
         if (tiles_m * ((lin->n + cand - 1) / cand) >= ctx->sm_count) bn = cand;
-    if (bn == 256) return launch<256, ACT, TY>(ctx, lin, a, m, limit, y, ldy, rt);
-    if (bn == 128) return launch<128, ACT, TY>(ctx, lin, a, m, limit, y, ldy, rt);
-    if (bn == 64) return launch<64, ACT, TY>(ctx, lin, a, m, limit, y, ldy, rt);
-    return launch<32, ACT, TY>(ctx, lin, a, m, limit, y, ldy, rt);
+    if (bn == 256) return launch<256, ACT, TY>(ctx, lin, a, lda, m, limit, y, ldy, rt);
+    if (bn == 128) return launch<128, ACT, TY>(ctx, lin, a, lda, m, limit, y, ldy, rt);
+    if (bn == 64) return launch<64, ACT, TY>(ctx, lin, a, lda, m, limit, y, ldy, rt);
+    return launch<32, ACT, TY>(ctx, lin, a, lda, m, limit, y, ldy, rt);
 }
 
 }  // namespace
 
-int32_t pgk_linear_tc(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t m, int act, float limit, void *y, int y_dtype, int64_t ldy,
+int32_t pgk_linear_tc(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t lda, int64_t m, int act, float limit, void *y, int y_dtype, int64_t ldy,
                       const PgRouted *routed)
 {
     static const PgRouted no_route = {};
@@ -302,8 +302,8 @@ int32_t pgk_linear_tc(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t m, int
     PG_REQUIRE(m < (1ll << 31) - 256 && lin->experts * lin->n < (1ll << 31) - 256, "linear: too many rows");
     PG_REQUIRE(act == PG_ACT_NONE || lin->n % 16 == 0, "linear: a gated product has a multiple of 16 columns");
     PG_REQUIRE(y_dtype == PG_F32 || (ldy % 8 == 0 && ((uintptr_t)y & 15) == 0), "linear: bf16 output rows start on 16-byte boundaries");
-    if (act == PG_ACT_GELU_TANH_GLU) return dispatch<PG_ACT_GELU_TANH_GLU, bf16>(ctx, lin, a, m, limit, (bf16 *)y, ldy, rt);
-    if (act == PG_ACT_CLAMPED_SWISH_GLU) return dispatch<PG_ACT_CLAMPED_SWISH_GLU, bf16>(ctx, lin, a, m, limit, (bf16 *)y, ldy, rt);
-    if (y_dtype == PG_BF16) return dispatch<PG_ACT_NONE, bf16>(ctx, lin, a, m, limit, (bf16 *)y, ldy, rt);
-    return dispatch<PG_ACT_NONE, float>(ctx, lin, a, m, limit, (float *)y, ldy, rt);
+    if (act == PG_ACT_GELU_TANH_GLU) return dispatch<PG_ACT_GELU_TANH_GLU, bf16>(ctx, lin, a, lda, m, limit, (bf16 *)y, ldy, rt);
+    if (act == PG_ACT_CLAMPED_SWISH_GLU) return dispatch<PG_ACT_CLAMPED_SWISH_GLU, bf16>(ctx, lin, a, lda, m, limit, (bf16 *)y, ldy, rt);
+    if (y_dtype == PG_BF16) return dispatch<PG_ACT_NONE, bf16>(ctx, lin, a, lda, m, limit, (bf16 *)y, ldy, rt);
+    return dispatch<PG_ACT_NONE, float>(ctx, lin, a, lda, m, limit, (float *)y, ldy, rt);
 }

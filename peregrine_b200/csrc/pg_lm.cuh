@@ -46,13 +46,13 @@ struct PgRouted {
 
 // pg_linear_gemv.cu: m <= 16 rows (or row blocks of 16) against streamed weights
 bool pgk_linear_gemv_supports(const pg_linear *lin, int64_t m);
-int32_t pgk_linear_gemv(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int64_t m, int act, float limit, void *y, int y_dtype, int64_t ldy,
+int32_t pgk_linear_gemv(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int64_t lda, int64_t m, int act, float limit, void *y, int y_dtype, int64_t ldy,
                         const PgRouted *routed, int64_t max_blocks);
 // pg_linear_tc.cu
-int32_t pgk_linear_tc(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t m, int act, float limit, void *y, int y_dtype, int64_t ldy,
+int32_t pgk_linear_tc(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t lda, int64_t m, int act, float limit, void *y, int y_dtype, int64_t ldy,
                       const PgRouted *routed);
 // pg_linear_f32.cu
-int32_t pgk_linear_f32(pg_ctx *ctx, const pg_linear *lin, const float *a, int64_t m, int act, float limit, void *y, int y_dtype, int64_t ldy,
+int32_t pgk_linear_f32(pg_ctx *ctx, const pg_linear *lin, const float *a, int64_t lda, int64_t m, int act, float limit, void *y, int y_dtype, int64_t ldy,
                        const PgRouted *routed);
 // pg_route.cu: rows of h in the order of the route (many-token form)
 int32_t pgk_route_gather(pg_ctx *ctx, const pg_route *route, const void *h, size_t row_bytes, void *out);

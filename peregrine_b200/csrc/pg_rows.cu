@@ -1,12 +1,14 @@
 // Row kernels of the f32 residual stream: a row is normalised (x / sqrt(mean(x^2) + eps) * w) and
 //
-//   EMBED   becomes the residual row, from the token's and the position's embedding
+//   EMBED   becomes the residual row, from the token's and, if there are any, the position's embedding (and is not
+//           normalised where the model has no norm there)
 //   ADD     is added to the residual row, scaled per channel (norm on a sublayer's output)
 //   ROUTED  the same, the row being the weighted sum of the token's expert outputs (identity experts: the residual row)
 //   PICK    is written out for the product behind it (the rows whose logits are wanted)
 //
-// and, except for PICK, the new residual row is written again in the type of the products that read it.  A cluster of
-// up to 8 CTAs shares a row when there are few rows.  The row lives in shared memory between the two passes.
+// and, except for PICK, the new residual row is written again in the type of the products that read it, normalised once
+// more with the weights of the next sublayer's norm where the model has one in front of it.  A cluster of up to 8 CTAs
+// shares a row when there are few rows.  The row lives in shared memory between the passes.
 #include "pg_lm.cuh"
 
 namespace {
@@ -24,7 +26,8 @@ struct RowArgs {
     const float *weights;
     int top, experts;
     float *x;
-    const float *w, *scale;
+    const float *w, *scale;     // EMBED: w null, no norm; scale null, 1
+    const float *next;          // weights of the norm in front of the next sublayer, or null
     float eps;
     int width;
     void *h;
@@ -61,7 +64,7 @@ __global__ void __launch_bounds__(RW_T) row_norm_kernel(const RowArgs a)
 {
     extern __shared__ __align__(16) float row[];   // this CTA's segment
     __shared__ float red[32];
-    __shared__ float xs[8];
+    __shared__ float xs[8], xs2[8];
     const uint32_t cs = cl_size(), rank = cl_rank();
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     if (cs > 1) cl_sync();   // every CTA of the cluster runs before anyone stores into it
@@ -74,17 +77,19 @@ __global__ void __launch_bounds__(RW_T) row_norm_kernel(const RowArgs a)
     const bf16 *tok = nullptr, *ptab = nullptr;
     if (SRC == SRC_EMBED) {
         tok = a.table + (int64_t)__ldcg(a.tokens + r) * a.width;
-        ptab = a.pos_table + (int64_t)__ldcg(a.pos + r) * a.width;
+        if (a.pos_table) ptab = a.pos_table + (int64_t)__ldcg(a.pos + r) * a.width;
     }
     float ss = 0.0f;
     for (int u = u0 + threadIdx.x; u < u1; u += RW_T) {
         float v[V];
         if (SRC == SRC_EMBED) {
-            float p[V];
             load_v<bf16, V>(tok + (int64_t)u * V, v);
-            load_v<bf16, V>(ptab + (int64_t)u * V, p);
+            if (ptab) {
+                float p[V];
+                load_v<bf16, V>(ptab + (int64_t)u * V, p);
 #pragma unroll
-            for (int i = 0; i < V; i++) v[i] += p[i];
+                for (int i = 0; i < V; i++) v[i] += p[i];
+            }
         } else if (SRC == SRC_ADD) {
             load_v<float, V>(a.y + r * a.ldy + (int64_t)u * V, v);
         } else if (SRC == SRC_PICK) {
@@ -112,8 +117,12 @@ __global__ void __launch_bounds__(RW_T) row_norm_kernel(const RowArgs a)
 #pragma unroll
         for (int i = 0; i < V; i++) ss += v[i] * v[i];
     }
-    ss = cl_allreduce<false>(pg_block_sum(ss, red), xs, cs, rank);
-    const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss, (float)a.width) + a.eps));
+    const bool plain = SRC == SRC_EMBED && !a.w;
+    float inv = 1.0f, ss2 = 0.0f;
+    if (!plain) {
+        ss = cl_allreduce<false>(pg_block_sum(ss, red), xs, cs, rank);
+        inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss, (float)a.width) + a.eps));
+    }
     TA *h = reinterpret_cast<TA *>(a.h) + r * a.ldh;
     for (int u = u0 + threadIdx.x; u < u1; u += RW_T) {
         float v[V];
@@ -123,12 +132,30 @@ __global__ void __launch_bounds__(RW_T) row_norm_kernel(const RowArgs a)
             float b[V];
             load_v<float, V>(x + (int64_t)u * V, b);
 #pragma unroll
-            for (int i = 0; i < V; i++) v[i] = b[i] + v[i] * inv * __ldg(a.w + u * V + i) * __ldg(a.scale + u * V + i);
-        } else {
+            for (int i = 0; i < V; i++) {
+                const float n = v[i] * inv * __ldg(a.w + u * V + i);
+                v[i] = b[i] + (a.scale ? n * __ldg(a.scale + u * V + i) : n);
+            }
+        } else if (!plain) {
 #pragma unroll
             for (int i = 0; i < V; i++) v[i] = v[i] * inv * __ldg(a.w + u * V + i);
         }
         if (SRC != SRC_PICK) store_v<float, V>(x + (int64_t)u * V, v);
+        if (SRC == SRC_PICK || !a.next) {
+            store_v<TA, V>(h + (int64_t)u * V, v);
+        } else {
+            store_v<float, V>(row + (size_t)(u - u0) * V, v);   // (read back by the same thread)
+#pragma unroll
+            for (int i = 0; i < V; i++) ss2 += v[i] * v[i];
+        }
+    }
+    if (SRC == SRC_PICK || !a.next) return;
+    ss2 = cl_allreduce<false>(pg_block_sum(ss2, red), xs2, cs, rank);
+    const float inv2 = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss2, (float)a.width) + a.eps));
+    for (int u = u0 + threadIdx.x; u < u1; u += RW_T) {
+        float v[V];
+#pragma unroll
+        for (int i = 0; i < V; i++) v[i] = row[(size_t)(u - u0) * V + i] * inv2 * __ldg(a.next + u * V + i);
         store_v<TA, V>(h + (int64_t)u * V, v);
     }
 }
@@ -136,7 +163,7 @@ __global__ void __launch_bounds__(RW_T) row_norm_kernel(const RowArgs a)
 template <int SRC>
 int32_t run_rows(pg_ctx *ctx, const RowArgs &a, int64_t rows, int32_t dtype, bool vec)
 {
-    PG_REQUIRE(a.width > 0 && a.width <= 32768 && a.ldh >= a.width && a.h && a.x && a.w, "row norm: bad arguments");
+    PG_REQUIRE(a.width > 0 && a.width <= 32768 && a.ldh >= a.width && a.h && a.x && (a.w || SRC == SRC_EMBED), "row norm: bad arguments");
     if (rows == 0) return PG_OK;
     vec = vec && a.width % 4 == 0 && a.ldh % 4 == 0;
     const int V = vec ? 4 : 1;
@@ -176,6 +203,29 @@ PG_API int32_t pg_embed_norm(pg_ctx *ctx, const pg_batch *batch, const void *d_t
     a.pos_table = (const bf16 *)d_pos_table_bf16;
     a.x = d_x, a.w = d_w, a.eps = eps, a.width = (int)width, a.h = d_h, a.ldh = ldh;
     return run_rows<SRC_EMBED>(ctx, a, batch->rows, dtype, true);
+}
+
+PG_API int32_t pg_embed_prenorm(pg_ctx *ctx, const pg_batch *batch, const void *d_table_bf16, int64_t width, const float *d_next, float eps, float *d_x,
+                                void *d_h, int32_t dtype, int64_t ldh)
+{
+    PG_ENTER(ctx);
+    PG_REQUIRE(batch && d_table_bf16 && d_next && batch->d_tokens, "embed_prenorm: null pointer");
+    RowArgs a = {};
+    a.tokens = batch->d_tokens;
+    a.table = (const bf16 *)d_table_bf16;
+    a.x = d_x, a.next = d_next, a.eps = eps, a.width = (int)width, a.h = d_h, a.ldh = ldh;
+    return run_rows<SRC_EMBED>(ctx, a, batch->rows, dtype, true);
+}
+
+PG_API int32_t pg_norm_add_prenorm(pg_ctx *ctx, const float *d_y, int64_t ldy, float *d_x, const float *d_w, const float *d_next, int64_t rows,
+                                   int64_t width, float eps, void *d_h, int32_t dtype, int64_t ldh)
+{
+    PG_ENTER(ctx);
+    PG_REQUIRE(d_y && d_w && ldy >= width, "norm_add_prenorm: bad arguments");
+    RowArgs a = {};
+    a.y = d_y, a.ldy = ldy, a.next = d_next;
+    a.x = d_x, a.w = d_w, a.eps = eps, a.width = (int)width, a.h = d_h, a.ldh = ldh;
+    return run_rows<SRC_ADD>(ctx, a, rows, dtype, ldy % 4 == 0);
 }
 
 PG_API int32_t pg_norm_add(pg_ctx *ctx, const float *d_y, int64_t ldy, float *d_x, const float *d_w, const float *d_scale, int64_t rows, int64_t width,

@@ -30,13 +30,24 @@ def file_model(architecture: str):
     return put
 
 
-@folder_model("Sonalorn")
-def _sonalorn(path, gpu=None, dtype="bfloat16", slots=1, capacity=0, step_rows=2048, portion=0, **_):
+def _slot_engine(model, path, gpu=None, dtype="bfloat16", slots=1, capacity=0, step_rows=2048, portion=0, **_):
     from .engine import Engine
+
+    return Engine(model.load(path, gpu or GpuContext(component="lm"), dtype=dtype, slots=slots, capacity=capacity, step_rows=step_rows), portion=portion)
+
+
+@folder_model("Sonalorn")
+def _sonalorn(path, **options):
     from .sonalorn import SonalornModel
 
-    gpu = gpu or GpuContext(component="lm")
-    return Engine(SonalornModel.load(path, gpu, dtype=dtype, slots=slots, capacity=capacity, step_rows=step_rows), portion=portion)
+    return _slot_engine(SonalornModel, path, **options)
+
+
+@folder_model("Bubotar")
+def _bubotar(path, **options):
+    from .bubotar import BubotarModel
+
+    return _slot_engine(BubotarModel, path, **options)
 
 
 @file_model("llama")

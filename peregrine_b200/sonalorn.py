@@ -11,15 +11,11 @@ are in peregrine_b200/layers.py.
 from __future__ import annotations
 
 import ctypes as C
-import json
-import os
 from dataclasses import dataclass
 from typing import Iterator, List
 
-from .layers import BATCH_WORDS, Attention, Batch, DenseFF, Device, GatedDelta, Linear, MoeFF, up
-from .safetensors_file import SafetensorsFile
-from .slot_model import SlotModel
-from .state import SlotPool
+from .layers import Attention, Batch, DenseFF, GatedDelta, MoeFF
+from .slot_model import Below, ResidualModel
 
 ARCHITECTURE = "Sonalorn"
 
@@ -57,85 +53,31 @@ class SonalornConfig:
             j = k
         raise ValueError(f"layer {i}: weights_of leads to no layer with tensors")
 
-    @staticmethod
-    def load(path: str) -> "SonalornConfig":
-        with open(os.path.join(path, "config.json")) as f:
-            return SonalornConfig.from_dict(json.load(f))
 
+class SonalornModel(ResidualModel):
+    Config = SonalornConfig
 
-class Below:
-    """The tensors whose names start with a prefix, by the rest of their names."""
-
-    def __init__(self, weights, prefix: str):
-        self.weights, self.prefix = weights, prefix
-
-    def __getitem__(self, name: str):
-        return self.weights[self.prefix + name]
-
-
-class SonalornModel(SlotModel):
-    """weights: mapping name -> host array (bf16 bits as uint16, or f32, which is rounded to bf16 where a product reads it).
-    slots / capacity: sequences alive at once and positions of each; step_rows: most tokens of one step; max_wanted: most
-    rows of logits of one `head` call."""
-
-    def __init__(self, cfg: SonalornConfig, weights, gpu, dtype: str = "bfloat16", slots: int = 1, capacity: int = 0, step_rows: int = 2048,
-                 max_wanted: int = 64):
-        self.cfg, self.gpu, self.lib = cfg, gpu, gpu.lib
-        self.dtype, self.vocab, self.step_rows = dtype, cfg.vocab, max(int(step_rows), slots + 1)
-        d = self.d = Device(gpu, dtype, self.step_rows)
-        torch = self.torch = d.torch
-        f32 = torch.float32
-
-        def matrix(name, rows):
-            t = d.bf16(weights[name]).contiguous()
-            if tuple(t.shape) != (rows, cfg.width):
-                raise ValueError(f"{name} is {list(t.shape)}, the configuration says [{rows}, {cfg.width}]")
-            return t
-
-        def vector(name):
-            t = d.f32(weights[name])
-            if tuple(t.shape) != (cfg.width,):
-                raise ValueError(f"{name} is {list(t.shape)}, the configuration says [{cfg.width}]")
-            return t
-
-        self.embed, self.pos = matrix("embed", cfg.vocab), matrix("pos", cfg.max_positions)
-        self.embed_norm, self.final_norm = vector("embed.norm"), vector("final.norm")
-        self.head = Linear(d, matrix("head", cfg.vocab))
-        self.capacity = min(int(capacity or cfg.max_positions), cfg.max_positions)
-        self.pool = SlotPool(slots, self.capacity, d.dev)
+    def build(self, weights) -> None:
+        cfg, d = self.cfg, self.d
+        self.pos, self.embed_norm = self.matrix("pos", cfg.max_positions), self.vector("embed.norm")
 
         def tensors(i, L):
-            W = Below(weights, f"l{i}.")
             mix = Below(weights, f"l{i}.mix.")
-            out = {"norm1": vector(f"l{i}.norm1"), "ls1": vector(f"l{i}.ls1"), "ff": None}
+            out = {"norm1": self.vector(f"l{i}.norm1"), "ls1": self.vector(f"l{i}.ls1"), "ff": None}
             if L["type"] == "delta":
                 out["mixer"] = GatedDelta(d, L["mixer"], mix, cfg.width, cfg.eps)
             else:
-                out["mixer"] = Attention(d, L["mixer"], mix, cfg.width, cfg.eps, self.capacity, slots)
+                out["mixer"] = Attention(d, L["mixer"], mix, cfg.width, cfg.eps, self.capacity, self.slots)
             if L.get("mlp"):
                 out["ff"] = (DenseFF if L["mlp"]["kind"] == "dense" else MoeFF)(d, L["mlp"], Below(weights, f"l{i}.mlp."), cfg.width)
-                out["norm2"], out["ls2"] = d.f32(W["norm2"]), d.f32(W["ls2"])
+                out["norm2"], out["ls2"] = self.vector(f"l{i}.norm2"), self.vector(f"l{i}.ls2")
             return out
 
         own = {i: tensors(i, L) for i, L in enumerate(cfg.layers) if L.get("weights_of") is None}
         self._own = list(own.values())
-        self.layers = []
-        for i, L in enumerate(cfg.layers):
+        for i in range(len(cfg.layers)):
             shared = own[cfg.tensors_of(i)]
             self.layers.append({**shared, "state": shared["mixer"].new_state(self.pool)})
-        self.ldh = up(cfg.width, 64)
-        self.x = torch.zeros(self.step_rows, cfg.width, dtype=f32, device=d.dev)
-        self.h = torch.zeros(self.step_rows, self.ldh, dtype=d.act, device=d.dev)
-        self.y = torch.zeros(self.step_rows, up(cfg.width, 4), dtype=f32, device=d.dev)
-        self.max_wanted = max(int(max_wanted), slots)
-        self.picked = torch.zeros(self.max_wanted, self.ldh, dtype=d.act, device=d.dev)
-        self.logits = torch.zeros(self.max_wanted, cfg.vocab, dtype=f32, device=d.dev)
-        d.buffer("batch", 1, BATCH_WORDS(d.rows), torch.int32)
-        torch.cuda.synchronize()   # torch filled the buffers on its own stream; the kernels use the context's
-
-    @staticmethod
-    def load(path: str, gpu, **kw) -> "SonalornModel":
-        return SonalornModel(SonalornConfig.load(path), SafetensorsFile(os.path.join(path, "model.safetensors")), gpu, **kw)
 
     # ---- one step ------------------------------------------------------------------------------------------------
     def step_ops(self, batch: Batch) -> Iterator[str]:
@@ -163,31 +105,3 @@ class SonalornModel(SlotModel):
             if L["ff"] is not None:
                 L["ff"].run(batch, h, y, add(L["norm2"], L["ls2"]))
             yield f"l{i}"
-
-    def head_rows(self, d_rows: int, n: int) -> None:
-        """logits[:n] of the rows of the residual stream named by n int32 at the device address d_rows."""
-        d, c = self.d, self.cfg
-        d.check(self.lib.pg_norm_rows(self.gpu.handle, self.x.data_ptr(), d_rows, n, c.width, self.final_norm.data_ptr(), c.eps, self.picked.data_ptr(),
-                                      d.code, self.ldh))
-        self.head.run(self.picked, n, self.logits)
-
-    def weight_bytes(self, tokens: int = 1) -> int:
-        """bf16 weight bytes that a step of `tokens` tokens reads at most (every expert that can be chosen, once)."""
-        total = self.head.bytes()
-        for L in self.layers:
-            total += L["mixer"].proj.bytes() + L["mixer"].out.bytes()
-            f = L["ff"]
-            if isinstance(f, DenseFF):
-                total += f.gate_up.bytes() + f.down.bytes()
-            elif f is not None:
-                used = min(f.E, tokens * f.top)
-                total += f.router.bytes() + (f.gate_up.bytes() + f.down.bytes()) * used // f.E
-        return total
-
-    def free(self) -> None:
-        for L in self._own:
-            L["mixer"].free()
-            if L["ff"] is not None:
-                L["ff"].free()
-        self.head.free()
-        self._own, self.layers = [], []
