@@ -12,6 +12,7 @@ Metric: achieved HBM bandwidth in GB/s = algorithmic bytes of the sweep / time, 
     python bench.py --gpus N --steps K --warmup W            this library
     python bench.py --impl reference ...                     the reference's CPU algorithm (C port)
     python bench.py --workload sonalorn                      the Sonalorn layers and kernels (bench_lm.py)
+    python bench.py --workload bubotar                       the Bubotar layers and kernels beside Sonalorn's (bench_lm.py)
 
 With N > 1 (one process per GPU, torchrun) the weights are sharded by output column over the ranks: one
 sweep, every rank quantises the (replicated) activations and computes its columns, and the products' own
@@ -846,9 +847,9 @@ def main():
     ap.add_argument("--collective", default="peer", choices=["peer", "nccl"],
                     help="N > 1, sharded: slices stored into every rank by the products' own epilogues, recorded in the step graph "
                          "(default), or eager NCCL all-gathers")
-    ap.add_argument("--workload", default="sweep", choices=["sweep", "sonalorn"],
-                    help="sonalorn: the Sonalorn layers and their kernels beside the Llama step's (bench_lm.py), one GPU")
-    ap.add_argument("--parts", default="", help="--workload sonalorn: which of dense,moe,kernels,llama (default: all)")
+    ap.add_argument("--workload", default="sweep", choices=["sweep", "sonalorn", "bubotar"],
+                    help="sonalorn / bubotar: the layers of that model and their kernels beside the closest other model (bench_lm.py), one GPU")
+    ap.add_argument("--parts", default="", help="--workload sonalorn: which of dense,moe,kernels,llama; bubotar: of bubotar,bubotar_kernels,dense,kernels (default: all)")
     args = ap.parse_args()
     # stdout carries the one JSON line and nothing else: libraries that print there (NCCL's version banner) are sent to
     # stderr by pointing file descriptor 1 at it; the line itself goes to a duplicate of the original stdout
@@ -856,7 +857,7 @@ def main():
     sys.stdout.flush()
     RESULT_OUT = os.fdopen(os.dup(1), "w")
     os.dup2(2, 1)
-    if args.workload == "sonalorn":
+    if args.workload != "sweep":
         import bench_lm
 
         bench_lm.run(args, RESULT_OUT, ClockSampler)

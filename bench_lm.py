@@ -1,11 +1,16 @@
-"""`bench.py --workload sonalorn`: throughput of Sonalorn layers at sizes that resemble a real model's (random weights), and
-of their kernels one by one, beside the Llama int8 decode step and its kernels at equal size.
+"""`bench.py --workload sonalorn` and `--workload bubotar`: throughput of a model's layers at sizes that resemble a real model's
+(random weights), and of their kernels one by one, beside the closest other model at equal size: for Sonalorn the Llama int8
+decode step and its kernels, for Bubotar Sonalorn's `dense` and its kernels.
 
-Models (bf16, 128256 tokens of vocabulary for `dense`, like the Llama step):
+Sonalorn models (bf16, 128256 tokens of vocabulary for `dense`, like the Llama step):
     dense  8 layers of width 4096: three delta layers (32 heads on 16 query/key heads, 128 x 128 states, 4 taps) to one
            attention layer (32 heads on 8, 128 wide), feed-forward 14336
     moe    8 layers of width 2048: delta 16 / 8 heads, attention 16 / 4 heads, 64 experts of 1024 and 16 identity experts,
            top 8 of the best 4 of 8 groups
+Bubotar model (the same vocabulary and width 4096):
+    bubotar  8 layers: scan (8192 channels, 16 states, rank 256, 4 taps) without a feed-forward, latent attention (32 heads of
+           128 + 64, values of 128, latents of 512), scan, attention (32 heads on 8, 128 wide, chunks of 4096); then the same,
+           the second latent layer with the first one's latents; feed-forward 14336 behind the attention layers
 Decoding: batch 1 and 16 behind a context of 2048, one recorded graph per step.  Prompts: 4096 tokens in one step.
 
 Every kernel is timed on its own memory: a graph of enough launches over different weights, states or caches that one
@@ -36,6 +41,32 @@ def sonalorn_config(kind: str, layers: int = 8, vocab: int = 128256, max_positio
             "layers": [{"type": "attention" if i % 4 == 3 else "delta", "mixer": attn if i % 4 == 3 else delta, "mlp": mlp} for i in range(layers)]}
 
 
+def bubotar_config(layers: int = 8, vocab: int = 128256) -> dict:
+    latent = {"heads": 32, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5, "rot": {"base": 10000.0, "dims": 64}}
+    attn = {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 4096}}
+    scan = {"inner": 8192, "state": 16, "dt_rank": 256, "conv": 4}
+    mlp = {"kind": "dense", "ff": 14336, "limit": 7.0}
+    four = [("mamba1", scan, None), ("latent_attention", latent, mlp), ("mamba1", scan, None), ("attention", attn, mlp)]
+    out = [{"type": k, "mixer": dict(p), "mlp": m} for i in range(layers) for k, p, m in [four[i % 4]]]
+    for i, L in enumerate(out):
+        if L["type"] == "latent_attention" and i > 1:
+            L["mixer"]["kv_from"] = 1
+    return {"architecture": "Bubotar", "vocab": vocab, "width": 4096, "norm": {"eps": 1e-5}, "logit_scale": 1.0, "layers": out}
+
+
+def bubotar_mixer_shape(kind: str, p: dict, N: int, name: str):
+    if kind == "mamba1":
+        I, S, R = p["inner"], p["state"], p["dt_rank"]
+        return {"in": (2 * I, N), "conv": (I, p["conv"]), "conv.b": (I,), "x": (R + 2 * S, I), "dt": (I, R), "dt.b": (I,), "A_log": (I, S), "D": (I,),
+                "o": (N, I)}[name]
+    H, D, V = p["heads"], p["dim"], p["vdim"]
+    if kind == "attention":
+        G = p["kv_heads"]
+        return {"q": (H * D, N), "k": (G * D, N), "v": (G * V, N), "o": (N, H * V)}[name]
+    K, R = p["kv_rank"], p["rot_dim"]
+    return {"q": (H * (D + R), N), "dkv": (K + R, N), "dkv.norm": (K,), "uk": (H * D, K), "uv": (H * V, K), "g": (H * V, N), "o": (N, H * V)}[name]
+
+
 class RandomWeights:
     """Draws a tensor on the device when the model asks for it."""
 
@@ -58,6 +89,8 @@ class RandomWeights:
         p = L["mixer"]
         if rest.startswith("mix."):
             rest = rest[4:]
+            if c["architecture"] == "Bubotar":
+                return bubotar_mixer_shape(L["type"], p, N, rest)
             G, H, D, V = p["kv_heads"], p["heads"], p["dim"], p["vdim"]
             if L["type"] == "delta":
                 return {"q": (G * D, N), "k": (G * D, N), "v": (H * V, N), "g": (H * V, N), "b": (H, N), "a": (H, N), "o": (N, H * V),
@@ -78,7 +111,7 @@ class RandomWeights:
         if len(s) == 1:
             if name.endswith("correction"):
                 return t.zeros(s, device=self.dev)
-            return t.full(s, -2.0 if name.endswith(("A_log", "dt_bias")) else 1.0, device=self.dev)
+            return t.full(s, -2.0 if name.endswith(("A_log", "dt_bias", "dt.b")) else 1.0, device=self.dev)
         return (t.randn(*s, generator=self.gen, device=self.dev, dtype=t.bfloat16) * (1.0 if name in ("embed", "pos") else s[1] ** -0.5)).to(t.bfloat16)
 
 
@@ -113,12 +146,13 @@ class Timer:
 
 
 def model_figures(torch, gpu, kind: str, hbm: float, tflops: float, layers: int = 8) -> dict:
-    from peregrine_b200.sonalorn import SonalornConfig, SonalornModel
+    from peregrine_b200.bubotar import BubotarModel
+    from peregrine_b200.sonalorn import SonalornModel
 
-    cfg = sonalorn_config(kind, layers)
+    Model, cfg = (BubotarModel, bubotar_config(layers)) if kind == "bubotar" else (SonalornModel, sonalorn_config(kind, layers))
     dev = torch.device("cuda", gpu.device)
     ctx0, T, steps = 2048, 4096, 64
-    m = SonalornModel(SonalornConfig.from_dict(cfg), RandomWeights(torch, cfg, dev), gpu, slots=16, capacity=T + 128, step_rows=T)
+    m = Model(Model.Config.from_dict(cfg), RandomWeights(torch, cfg, dev), gpu, slots=16, capacity=T + 128, step_rows=T)
     for L in m.layers:
         for v in L["state"].values():
             v.normal_()
@@ -141,7 +175,13 @@ def model_figures(torch, gpu, kind: str, hbm: float, tflops: float, layers: int 
         flops += 2.0 * T * (mx.proj.n * mx.proj.k + mx.out.n * mx.out.k)
         if hasattr(mx, "dp"):
             flops += 2.0 * T * T / 2 * mx.H * (mx.D + mx.V)
-        if hasattr(f, "route"):
+        if hasattr(mx, "unfold"):
+            flops += 2.0 * T * T / 2 * mx.H * (mx.D + mx.R + mx.V) + 2.0 * T * mx.unfold.n * mx.unfold.k
+        if hasattr(mx, "dtp"):
+            flops += 2.0 * T * (mx.low.n * mx.low.k + mx.dt.n * mx.dt.k)
+        if f is None:
+            pass
+        elif hasattr(f, "route"):
             flops += 2.0 * T * f.top * f.E / (f.E + f.I) * (f.gate_up.n * f.gate_up.k + f.down.n * f.down.k)
         else:
             flops += 2.0 * T * (f.gate_up.n * f.gate_up.k + f.down.n * f.down.k)
@@ -173,12 +213,15 @@ def model_figures(torch, gpu, kind: str, hbm: float, tflops: float, layers: int 
             d.tokens()
         e2e = (time.perf_counter() - t0) / steps
         kv = sum(B * mx.G * (ctx0 + steps / 2) * (mx.dp + mx.vp) * 2 for mx in (L["mixer"] for L in m.layers) if hasattr(mx, "dp"))
-        st = sum(2 * B * mx.H * mx.D * mx.V * 4 for mx in (L["mixer"] for L in m.layers) if not hasattr(mx, "dp"))
+        kv += sum(B * (ctx0 + steps / 2) * mx.ck * 2 for mx in (L["mixer"] for L in m.layers) if hasattr(mx, "ck"))
+        st = sum(2 * B * L["state"]["state"][0].numel() * 4 for L in m.layers if "state" in L["state"])
         moe_rows = 0.0
         nbytes = kv + st + m.head.bytes()
         for L in m.layers:
             mx, f = L["mixer"], L["ff"]
-            nbytes += mx.proj.bytes() + mx.out.bytes()
+            nbytes += mx.bytes()
+            if f is None:
+                continue
             if hasattr(f, "route"):
                 used = len(set(f.chosen(B)[0].ravel().tolist()) & set(range(f.E)))
                 moe_rows += used
@@ -332,6 +375,156 @@ def kernel_figures(torch, gpu, hbm: float, tflops: float) -> dict:
     return out
 
 
+def bubotar_kernel_figures(torch, gpu, hbm: float, tflops: float) -> dict:
+    """The kernels of Bubotar's layers at the sizes of `bubotar`."""
+    from peregrine_b200 import _lib
+    from peregrine_b200.layers import Attention, Batch, Device, LatentAttention, Linear, SelectiveScan, halving_slopes
+    from peregrine_b200.slot_model import Below
+    from peregrine_b200.state import SlotPool
+
+    dev = torch.device("cuda", gpu.device)
+    time_us = Timer(gpu, torch)
+    T, N, ctx0 = 4096, 4096, 2048
+    d = Device(gpu, "bfloat16", T)
+    out = {}
+
+    def note(name, us, nbytes=None, flops=None):
+        e = out[name] = {"us": us}
+        if nbytes:
+            e.update(gbs=nbytes / us * 1e-3, frac_of_hbm=nbytes / us * 1e-3 / hbm)
+        if flops:
+            e.update(tflops=flops / us * 1e-6, frac_of_bf16_peak=flops / us * 1e-6 / tflops)
+
+    rnd = lambda *s: torch.randn(*s, device=dev, dtype=torch.bfloat16) * s[-1] ** -0.5
+    for name, n, k, gated in (("scan_in", 16384, N, False), ("scan_low", 288, 8192, False), ("scan_dt", 8192, 256, False), ("latent_proj", 10816, N, False),
+                              ("latent_unfold", 8192, 512, False), ("o", N, 4096, False), ("scan_o", N, 8192, False), ("gate_up", 28672, N, True),
+                              ("down", N, 14336, False)):
+        ls = [Linear(d, (rnd(n // 2, k), rnd(n // 2, k)) if gated else rnd(n, k), gated=gated) for _ in range(min(80, max(2, int(400e6 / (n * k * 2)) + 1)))]
+        for M in (1, 16, 64, T):
+            a = torch.randn(M, k, device=dev).to(torch.bfloat16)
+            narrow = gated or name == "latent_unfold"
+            y = torch.zeros(M, n // 2 if gated else n, device=dev, dtype=torch.bfloat16 if narrow else torch.float32)
+            torch.cuda.synchronize()
+            act = _lib.ACT_CLAMPED_SWISH_GLU if gated else _lib.ACT_NONE
+            us = time_us([(lambda l=l: l.run(a, M, y, act, 7.0)) for l in (ls if M <= 64 else ls[:2])], reps=10)
+            note(f"product.{name}.m{M}", us, nbytes=(n * k + M * k) * 2 + y.numel() * y.element_size(), flops=2.0 * M * n * k if M > 64 else None)
+        for l in ls:
+            l.free()
+        del ls
+
+    cfg = bubotar_config()
+    W = RandomWeights(torch, cfg, dev)
+    cap = T + 64
+    pool = SlotPool(16, cap, dev)
+    steps = {B: Batch(d, [(s, ctx0, [1]) for s in range(B)], fixed=True) for B in (1, 16)}
+    long = Batch(d, [(0, 0, [1] * T)], fixed=True)
+    part = Batch(d, [(0, ctx0, [1] * 16)], fixed=True)
+    ptr = lambda t: t.data_ptr()
+    f32 = torch.float32
+
+    # scan
+    mx = [SelectiveScan(d, cfg["layers"][0]["mixer"], Below(W, "l0.mix."), N) for _ in range(4)]
+    states = [m.new_state(pool) for m in mx]
+    proj, mixed = torch.randn(T, mx[0].proj.n, device=dev), d.buffer("mixed", mx[0].out.k)
+    x, low = d.buffer("scan.x", mx[0].low.k), d.buffer("scan.low", mx[0].low.n, dtype=f32)
+    dt, bc = d.buffer("scan.dt", mx[0].I, dtype=f32), d.buffer("scan.bc", mx[0].low_bc.n, dtype=f32)
+    for v in (low, dt, bc, x):
+        v.normal_()
+    torch.cuda.synchronize()
+    ck, lib, gh, I, S = d.check, d.lib, gpu.handle, mx[0].I, mx[0].ss
+
+    def conv(m, s, b):
+        ck(lib.pg_scan_conv(gh, C.byref(m.c), C.byref(b.c), ptr(proj), proj.stride(0), ptr(s["ring"]), ptr(x), d.code, x.stride(0)))
+
+    def step(m, s, b):
+        ck(lib.pg_scan_step(gh, C.byref(m.c), C.byref(b.c), ptr(proj), proj.stride(0), ptr(x), x.stride(0), ptr(low), low.stride(0), ptr(s["state"]), ptr(mixed),
+                            d.code, mixed.stride(0)))
+
+    def scan(m, s, b):
+        ck(lib.pg_scan_run(gh, C.byref(m.c), C.byref(b.c), ptr(proj), proj.stride(0), ptr(s["ring"]), ptr(x), x.stride(0), ptr(dt), dt.stride(0), ptr(bc),
+                           bc.stride(0), ptr(s["state"]), ptr(mixed), d.code, mixed.stride(0)))
+    pairs = list(zip(mx, states)) * 3
+    for B, b in steps.items():
+        note(f"scan.conv.b{B}", time_us([(lambda m=m, s=s: conv(m, s, b)) for m, s in pairs]), nbytes=B * I * (4 * 4 + 4 + 2))
+        note(f"scan.step.b{B}", time_us([(lambda m=m, s=s: step(m, s, b)) for m, s in pairs]), nbytes=B * I * (2 * S * 4 + 8) + I * (256 * 2 + S * 4))
+    note(f"scan.conv.t{T}", time_us([(lambda m=m, s=s: conv(m, s, long)) for m, s in pairs[:2]], reps=5), nbytes=T * I * 6)
+    # an exponential per channel, state and token, on a unit of 16 per SM and clock, bounds the recurrence
+    us = time_us([(lambda m=m, s=s: scan(m, s, long)) for m, s in pairs[:2]], reps=5)
+    note(f"scan.run.t{T}", us, nbytes=T * I * (4 + 2 + 4 + 2))
+    out[f"scan.run.t{T}"]["frac_of_exponentials_at_1965_mhz"] = T * I * S / (148 * 16 * 1965.0) / us
+    for m in mx:
+        m.free()
+    del mx, states, pairs, proj
+    # latent attention
+    mx = [LatentAttention(d, cfg["layers"][1]["mixer"], Below(W, "l1.mix."), N, 1e-5, cap, 16) for _ in range(6)]
+    states = [m.new_state(pool) for m in mx]
+    for s in states:
+        s["latent"].normal_()
+    m0 = mx[0]
+    proj, mixed = torch.randn(T, m0.proj.n, device=dev), d.buffer("mixed", m0.out.k)
+    for m in mx:
+        m.c.d_q, m.c.d_part, m.c.part_floats, m.c.slots = ptr(d.buffer("latent.q", m.H * m.qd)), ptr(d.buffer("latent.part", 1, 1, f32)), m.part_rows, 16
+    kv = d.buffer("latent.kv", m0.unfold.n, cap)
+    torch.cuda.synchronize()
+
+    def short(m, s, b, n, longest):
+        ck(lib.pg_latent_run(gh, C.byref(m.c), C.byref(b.c), m.LONG, n, longest, ptr(proj), proj.stride(0), ptr(s["latent"]), ptr(mixed), d.code, mixed.stride(0)))
+
+    def prep(m, s):
+        ck(lib.pg_latent_prompt_prep(gh, C.byref(m.c), C.byref(long.c), 0, T, 0, ptr(proj), proj.stride(0), ptr(s["latent"])))
+
+    def attend(m, s):
+        ck(lib.pg_latent_prompt(gh, C.byref(m.c), C.byref(long.c), 0, T, T, 0, ptr(proj), proj.stride(0), ptr(s["latent"]), ptr(kv), kv.stride(0), ptr(mixed),
+                                mixed.stride(0)))
+
+    def whole(m, s):
+        prep(m, s)
+        m.unfold.run_ld(ptr(s["latent"][0]), m.ck, T, kv)
+        attend(m, s)
+    pairs = list(zip(mx, states))
+    wb = 2 * m0.H * 128 * 512 * 2
+    for B, b in steps.items():
+        note(f"latent.step.b{B}", time_us([(lambda m=m, s=s: short(m, s, b, B, 1)) for m, s in pairs]), nbytes=B * (ctx0 + 1) * m0.ck * 2 + wb,
+             flops=2.0 * B * m0.H * ((ctx0 + 1) * (m0.ck + 512) + 2 * 128 * 512))
+    note("latent.portion.t16", time_us([(lambda m=m, s=s: short(m, s, part, 16, 16)) for m, s in pairs]), nbytes=(ctx0 + 16) * m0.ck * 2 + wb,
+         flops=2.0 * 16 * m0.H * ((ctx0 + 8) * (m0.ck + 512) + 2 * 128 * 512))
+    fl = 2.0 * T * T / 2 * m0.H * (m0.D + m0.R + m0.V)
+    note(f"latent.prompt.prep.t{T}", time_us([(lambda m=m, s=s: prep(m, s)) for m, s in pairs[:2]], reps=5), nbytes=T * (m0.H * 192 * 6 + 576 * 6))
+    note(f"latent.prompt.attend.t{T}", time_us([(lambda m=m, s=s: attend(m, s)) for m, s in pairs[:2]], reps=5), flops=fl)
+    note(f"latent.prompt.t{T}", time_us([(lambda m=m, s=s: whole(m, s)) for m, s in pairs[:2]], reps=5), flops=fl + 2.0 * T * 8192 * 512)
+    for m in mx:
+        m.free()
+    del mx, states, pairs, proj
+    # chunked attention
+    proj = torch.randn(T, 6144, device=dev)
+    for size in (4096, 1024):
+        p = dict(cfg["layers"][3]["mixer"], mask={"size": size})
+        att = Attention(d, p, Below(W, "l3.mix."), N, 1e-5, cap, 16, sink=False, norms=False, slopes=halving_slopes(32), chunk=size)
+        states = [att.new_state(pool) for _ in range(4)]
+        for s in states:
+            s["k"].normal_(), s["v"].normal_()
+        mixed = d.buffer("mixed", att.out.k)
+        att.c.d_q, att.c.d_part = ptr(d.buffer("attn.q", att.H * att.dp)), ptr(d.buffer("attn.part", 1, 1, f32))
+        att.c.d_tickets, att.c.slots = ptr(d.buffer("attn.tickets", 1, 1, torch.int32)), 16
+        torch.cuda.synchronize()
+
+        def run(s, b):
+            ck(lib.pg_attention_run(gh, C.byref(att.c), C.byref(b.c), ptr(proj), proj.stride(0), ptr(s["k"]), ptr(s["v"]), ptr(mixed), d.code, mixed.stride(0)))
+        if size > ctx0:
+            for B, b in steps.items():
+                note(f"attention.chunk{size}.step.b{B}", time_us([(lambda s=s: run(s, b)) for s in states]), nbytes=B * 8 * (ctx0 + 1) * 256 * 2)
+        note(f"attention.chunk{size}.prompt.t{T}", time_us([(lambda s=s: run(s, long)) for s in states[:2]], reps=5), flops=4.0 * T * size / 2 * 32 * 128)
+        att.free()
+        del states
+    xs, y, one = torch.randn(T, N, device=dev), torch.randn(T, N, device=dev), torch.ones(N, device=dev)
+    h = torch.zeros(T, N, device=dev, dtype=torch.bfloat16)
+    torch.cuda.synchronize()
+    for M in (1, 16, T):
+        f = lambda: ck(lib.pg_norm_add_prenorm(gh, ptr(y), N, ptr(xs), ptr(one), ptr(one), M, N, 1e-5, ptr(h), d.code, N))
+        note(f"norm_add_prenorm.m{M}", time_us([f] * 8), nbytes=M * N * 14)
+    return out
+
+
 def llama_kernel_figures(torch, hbm: float, tflops: float) -> dict:
     """The like kernels of the Llama int8 path at equal size."""
     from peregrine_b200 import _lib
@@ -399,12 +592,16 @@ def run(args, result_out, clocks) -> None:
     except (OSError, ValueError):
         pass
     hbm, tflops = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
-    out = {"workload": "sonalorn", "data": "synthetic", "dtype": "bf16", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "source": "measured" if peaks else "fallback"}}
+    out = {"workload": args.workload, "data": "synthetic", "dtype": "bf16", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "source": "measured" if peaks else "fallback"}}
     gpu = GpuContext(component="lm")
     sampler = clocks(gpu.device)
     sampler.mark()
-    parts = args.parts.split(",") if args.parts else ["dense", "moe", "kernels", "llama"]
-    for kind in ("dense", "moe"):
+    usual = ["bubotar", "bubotar_kernels", "dense", "kernels"] if args.workload == "bubotar" else ["dense", "moe", "kernels", "llama"]
+    parts = args.parts.split(",") if args.parts else usual
+    if "bubotar_kernels" in parts:
+        out["bubotar_kernels"] = bubotar_kernel_figures(torch, gpu, hbm, tflops)
+        torch.cuda.empty_cache()
+    for kind in ("bubotar", "dense", "moe"):
         if kind in parts:
             out[kind] = model_figures(torch, gpu, kind, hbm, tflops)
             torch.cuda.empty_cache()
