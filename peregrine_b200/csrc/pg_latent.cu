@@ -6,7 +6,7 @@
 //
 //   bf16, short      latent_query_kernel   q' per head on mma.sync, the queries' rotation, and the new positions' cache rows
 //                    latent_attn_kernel    a CTA has a slice of the context and 16 or 32 (token, head) rows, which share the
-//                                          keys; the warps divide the keys for the scores and the columns for the sums
+//                                          keys; the warps divide keys and columns between them
 //                    latent_value_kernel   adds up the slices, W_uv per head on mma.sync, output gate
 //   bf16, longer     latent_prep_kernel (rotation, cache rows); then the caller unfolds keys and values of the whole context
 //                    by a product, and the tcgen05 kernel of csrc/pg_attention_tc.cu reads them
@@ -23,6 +23,13 @@
 namespace {
 
 constexpr float LOG2E = 1.4426950408889634f;
+
+__device__ __forceinline__ float pg_ex2(float x)
+{
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 
 struct LatentShape {
     int H, D, R, V, C;           // heads, unrotated and rotated query widths, value width, latent width
@@ -57,41 +64,56 @@ __device__ __forceinline__ void rotate(const LatentShape &s, const float *src, i
     }
 }
 
-// One warp: the cache row of a token, [c | 0 | rotated key part | 0].
+// One warp: the cache row of a token, [c | 0 | rotated key part | 0] (kv_rank <= 512).
 template <typename TA>
 __device__ __forceinline__ void append(const LatentShape &s, const float *kv, int pos, TA *dst, int lane)
 {
-    float ss = 0.0f;
-    for (int i = lane; i < s.C; i += 32) {
-        const float x = __ldcg(kv + i);
-        ss += x * x;
-    }
-    const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(pg_warp_sum(ss), (float)s.C) + s.eps));
-    for (int i = lane; i < s.cp; i += 32) pg_put(dst + i, i < s.C ? __ldcg(kv + i) * inv * __ldg(s.c_norm + i) : 0.0f);
+    float x[16], ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < 16; i++) x[i] = i * 32 + lane < s.C ? __ldcg(kv + i * 32 + lane) : 0.0f;
     rotate(s, kv + s.C, pos, dst + s.cp, s.rp, lane);
+#pragma unroll
+    for (int i = 0; i < 16; i++) ss += x[i] * x[i];
+    const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(pg_warp_sum(ss), (float)s.C) + s.eps));
+#pragma unroll
+    for (int i = 0; i < 16; i++) {
+        const int c = i * 32 + lane;
+        if (c < s.cp) pg_put(dst + c, c < s.C ? x[i] * inv * __ldg(s.c_norm + c) : 0.0f);
+    }
 }
 
 // D[16 x 8] of one warp: rows of `a` (shared memory, ld elements apart) times eight rows of w (global), K a multiple of 32.
-// A lane's 16 contiguous bytes of both feed two MMAs: K is permuted alike on both sides.
-__device__ __forceinline__ void product16x8(float (&d)[4], uint32_t a, int ld, const bf16 *__restrict__ w, int64_t ldw, int K, int lane)
-{
-    const int r = lane >> 2, t = lane & 3;
-    const uint32_t a0 = a + (uint32_t)(r * ld + t * 8) * 2, a1 = a0 + (uint32_t)(8 * ld) * 2;
-    const uint4 *b = reinterpret_cast<const uint4 *>(w + r * ldw + t * 8);
-    for (int k = 0; k < K; k += 128) {
-        uint4 x[4];
+// A lane's 16 contiguous bytes of both feed two MMAs: K is permuted alike on both sides.  `ask` brings the first PRE pieces
+// of the weights, which do not depend on the kernel before.
+template <int PRE>
+struct Weights8 {
+    uint4 x[PRE];
+    const uint4 *at;
+    int pieces;
+    __device__ __forceinline__ void ask(const bf16 *__restrict__ w, int64_t ldw, int K, int lane)
+    {
+        at = reinterpret_cast<const uint4 *>(w + (lane >> 2) * ldw + (lane & 3) * 8);
+        pieces = K / 32;
 #pragma unroll
-        for (int i = 0; i < 4; i++) x[i] = k + i * 32 < K ? __ldg(b + (k + i * 32) / 8) : make_uint4(0u, 0u, 0u, 0u);
-#pragma unroll
-        for (int i = 0; i < 4; i++) {
-            if (k + i * 32 < K) {
-                const uint4 lo = pg_lds128(a0 + (k + i * 32) * 2), hi = pg_lds128(a1 + (k + i * 32) * 2);
-                pg_mma_bf16(d, lo.x, hi.x, lo.y, hi.y, x[i].x, x[i].y);
-                pg_mma_bf16(d, lo.z, hi.z, lo.w, hi.w, x[i].z, x[i].w);
-            }
-        }
+        for (int i = 0; i < PRE; i++) x[i] = i < pieces ? __ldg(at + 4 * i) : make_uint4(0u, 0u, 0u, 0u);
     }
-}
+    __device__ __forceinline__ void times(float (&d)[4], uint32_t a, int ld, int lane)
+    {
+        const uint32_t a0 = a + (uint32_t)((lane >> 2) * ld + (lane & 3) * 8) * 2, a1 = a0 + (uint32_t)(8 * ld) * 2;
+        float e[4] = {};                                  // two sums: shorter chains
+        auto step = [&](const uint4 &v, int i) {
+            const uint4 lo = pg_lds128(a0 + i * 64), hi = pg_lds128(a1 + i * 64);
+            pg_mma_bf16(d, lo.x, hi.x, lo.y, hi.y, v.x, v.y);
+            pg_mma_bf16(e, lo.z, hi.z, lo.w, hi.w, v.z, v.w);
+        };
+#pragma unroll
+        for (int i = 0; i < PRE; i++)
+            if (i < pieces) step(x[i], i);
+        for (int i = PRE; i < pieces; i++) step(__ldg(at + 4 * i), i);
+#pragma unroll
+        for (int i = 0; i < 4; i++) d[i] += e[i];
+    }
+};
 
 // ---- short portions, bf16 ------------------------------------------------------------------------------------------
 // grid (H + own, column parts, tiles of 16 rows).  qx [rows][H][ck]: q', rotated part
@@ -99,14 +121,18 @@ constexpr int LQ_T = 256;
 __global__ void __launch_bounds__(LQ_T)
     latent_query_kernel(const LatentShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, bf16 *__restrict__ qx, bf16 *cache, int32_t *status)
 {
-    extern __shared__ __align__(16) unsigned char smem[];   // [16][dk + 8]
-    pg_pdl_begin();
+    constexpr int NW = LQ_T / 32;
+    extern __shared__ __align__(128) unsigned char smem[];   // [16][dk + 8]
     const int h = blockIdx.x, m0 = blockIdx.z * 16, n = min(16, bt.rows - m0), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int c_step = gridDim.y * NW * 8;
+    int c = (blockIdx.y * NW + warp) * 8;
+    Weights8<4> w;
+    if (h < s.H && c < s.cp) w.ask(s.uk + ((int64_t)h * s.cp + c) * s.dk, s.dk, s.dk, lane);
+    pg_pdl_begin();
     bf16 *sa = reinterpret_cast<bf16 *>(smem);
     const int ld = s.dk + 8;
     if (h == s.H) {
-        if (blockIdx.y != 0) return;
-        for (int i = warp; i < n; i += LQ_T / 32) {
+        for (int i = blockIdx.y * NW + warp; i < n; i += gridDim.y * NW) {
             const int m = m0 + i, pos = __ldcg(bt.d_pos + m), seq = __ldcg(bt.d_row_seq + m);
             if (seq_len(bt, seq) >= s.long_from) continue;
             if ((unsigned)pos >= (unsigned)s.cap) {   // outside the cache: record it, touch nothing
@@ -117,29 +143,30 @@ __global__ void __launch_bounds__(LQ_T)
         }
         return;
     }
-    for (int i = threadIdx.x; i < 16 * s.dk; i += LQ_T) {
-        const int r = i / s.dk, c = i - r * s.dk;
-        sa[r * ld + c] = __float2bfloat16_rn(r < n && c < s.D ? __ldcg(proj + (int64_t)(m0 + r) * ldp + h * (s.D + s.R) + c) : 0.0f);
+    for (int i = warp; i < 16; i += NW) {
+        const float *src = proj + (int64_t)(m0 + i) * ldp + h * (s.D + s.R);
+#pragma unroll 4
+        for (int k = lane; k < s.dk; k += 32) sa[i * ld + k] = __float2bfloat16_rn(i < n && k < s.D ? __ldcg(src + k) : 0.0f);
     }
-    if (blockIdx.y == 0) {
-        for (int i = warp; i < n; i += LQ_T / 32) {
-            const int m = m0 + i, pos = __ldcg(bt.d_pos + m);
-            if ((unsigned)pos >= (unsigned)s.cap) {
-                if (lane == 0) atomicExch(status, (int32_t)PG_ERR_INVALID);
-                continue;
-            }
-            rotate(s, proj + (int64_t)m * ldp + h * (s.D + s.R) + s.D, pos, qx + ((int64_t)m * s.H + h) * s.ck + s.cp, s.rp, lane);
+    for (int i = blockIdx.y * NW + warp; i < n; i += gridDim.y * NW) {
+        const int m = m0 + i, pos = __ldcg(bt.d_pos + m);
+        if ((unsigned)pos >= (unsigned)s.cap) {
+            if (lane == 0) atomicExch(status, (int32_t)PG_ERR_INVALID);
+            continue;
         }
+        rotate(s, proj + (int64_t)m * ldp + h * (s.D + s.R) + s.D, pos, qx + ((int64_t)m * s.H + h) * s.ck + s.cp, s.rp, lane);
     }
     __syncthreads();
     const int r = lane >> 2, t = lane & 3;
-    for (int c = (blockIdx.y * (LQ_T / 32) + warp) * 8; c < s.cp; c += gridDim.y * (LQ_T / 32) * 8) {
+    while (c < s.cp) {
         float d[4] = {};
-        product16x8(d, pg_smem(sa), ld, s.uk + ((int64_t)h * s.cp + c) * s.dk, s.dk, s.dk, lane);
+        w.times(d, pg_smem(sa), ld, lane);
 #pragma unroll
         for (int half = 0; half < 2; half++)
             if (r + 8 * half < n)
                 *reinterpret_cast<uint32_t *>(qx + ((int64_t)(m0 + r + 8 * half) * s.H + h) * s.ck + c + 2 * t) = pg_pack_bf16(d[2 * half], d[2 * half + 1]);
+        c += c_step;
+        if (c < s.cp) w.ask(s.uk + ((int64_t)h * s.cp + c) * s.dk, s.dk, s.dk, lane);
     }
 }
 
@@ -163,22 +190,27 @@ __device__ __forceinline__ int64_t first_tile(const LatentShape &s, int row0, in
 
 constexpr int LA_KEYS = 64;
 constexpr int LA_PS = LA_KEYS + 8;      // row stride of the weights in shared memory
+constexpr int LA_QSTEPS = 18;           // 16-column steps of half a key that a warp's query fragments cover (ck up to 576)
 
-// grid (slices, row tiles, seqs), 4 RT warps.  Shared memory: ring of `stages` tiles of keys [64][ck + 8] | queries [16 RT][ck + 8]
-// | weights [16 RT][LA_PS].  part [tile][slice][16 RT][cp + 4]: sums, then maximum (log 2 units) and denominator of each row.
-template <int RT>
-__global__ void __launch_bounds__(RT * 128)
-    latent_attn_kernel(const LatentShape s, const pg_batch bt, const bf16 *__restrict__ qx, const bf16 *__restrict__ cache, float *__restrict__ part, int per_seq, int stages,
-                       int32_t *status, unsigned long long limit_ns)
+// grid (slices, row tiles, seqs), 8 RT warps.  A warp has 16 keys of a tile, 16 rows and half of the key's columns for the
+// scores -- two warps exchange their halves' sums, and each goes on with eight keys -- and 64 / RT columns of all rows for the
+// sums.  QREG: the warp's part of the queries stays in registers.
+// Shared memory: ring of `stages` tiles of keys [64][ck + 8] | queries [16 RT][ck + 8] | weights [16 RT][LA_PS] | halves' sums
+// [8 RT warps][32 lanes][4].  part [tile][slice][16 RT][cp + 4]: sums, then maximum (log 2 units) and denominator of each row.
+template <int RT, bool QREG>
+__global__ void __launch_bounds__(RT * 256, 1)
+    latent_attn_kernel(const LatentShape s, const pg_batch bt, const bf16 *__restrict__ qx, const bf16 *__restrict__ cache, float *__restrict__ part, int per_seq,
+                       int stages, int32_t *status, unsigned long long limit_ns)
 {
-    constexpr int NW = 4 * RT, ROWS = 16 * RT, VT = 512 / NW / 8;   // 8-column tiles of a warp (kv_rank up to 512)
+    constexpr int NW = 8 * RT, ROWS = 16 * RT, VT = 512 / NW / 8;   // 8-column tiles of a warp (kv_rank up to 512)
     extern __shared__ __align__(128) unsigned char smem[];
     __shared__ __align__(8) uint64_t bars[4];
-    __shared__ float red[RT][4][16];
+    __shared__ __align__(16) float red[RT][16][8];
     __shared__ volatile int abort_flag;
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     const int split = blockIdx.x, S = gridDim.x, tile = blockIdx.y, seq = blockIdx.z;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane >> 2, t = lane & 3, kq = warp & 3, rt = warp >> 2;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane >> 2, t = lane & 3;
+    const int kh = warp & 1, kq = (warp >> 1) & 3, rt = warp >> 3;   // half of the columns, group of keys, row tile
     if (threadIdx.x == 0) {
         for (int i = 0; i < 4; i++) pg_mbar_init(pg_smem(bars) + 8 * i, 1);
         abort_flag = 0;
@@ -187,36 +219,44 @@ __global__ void __launch_bounds__(RT * 128)
     __syncthreads();
     asm volatile("griddepcontrol.wait;" ::: "memory");
     const int row0 = __ldcg(bt.d_seq_row0 + seq), T = seq_len(bt, seq), total = T * s.H, rr0 = tile * ROWS;
+    const int64_t slot = __ldcg(bt.d_seq_slot + seq);
     if (T >= s.long_from || rr0 >= total) return;
     const int pos0 = __ldcg(bt.d_pos + row0);
-    const int64_t slot = __ldcg(bt.d_seq_slot + seq);
     const Slices sl = slices_of(s, pos0, T, tile, ROWS, S);
     const int t0 = split * sl.chunk, t1 = min(sl.kmax, t0 + sl.chunk);
     if (t0 >= t1 || sl.kmax > s.cap) return;              // (positions outside the cache are recorded by latent_query_kernel)
     const int stride = s.ck * 2 + 16, stage = LA_KEYS * stride;
-    const uint32_t ring = pg_smem(smem), qs = ring + stages * stage, ps = qs + ROWS * stride;
+    const uint32_t ring = pg_smem(smem), qs = ring + stages * stage, ps = qs + ROWS * stride, xs = ps + ROWS * LA_PS * 2;
     const uint32_t bar = pg_smem(bars);
     const bf16 *keys = cache + slot * (int64_t)s.cap * s.ck;
     const int ntiles = (t1 - t0 + LA_KEYS - 1) / LA_KEYS;
-    // the first warp asks for a tile's rows, two per lane (rows behind the slice repeat its last one and are masked)
+    // every warp asks for some of a tile's rows (rows behind the slice repeat its last one and are masked)
     auto fetch = [&](int i) {
         const uint32_t at = ring + (uint32_t)(i % stages) * stage, on = bar + (uint32_t)(i % stages) * 8;
-        if (lane == 0) pg_mbar_expect(on, (uint32_t)LA_KEYS * s.ck * 2u);
-        __syncwarp();
-#pragma unroll
-        for (int x = lane; x < LA_KEYS; x += 32)
+        if (threadIdx.x == 0) pg_mbar_expect(on, (uint32_t)LA_KEYS * s.ck * 2u);
+        if (lane < LA_KEYS / NW) {
+            const int x = warp * (LA_KEYS / NW) + lane;
             pg_bulk_load(at + (uint32_t)x * stride, keys + (int64_t)min(t0 + i * LA_KEYS + x, t1 - 1) * s.ck, (uint32_t)s.ck * 2u, on);
+        }
     };
-    if (warp == 0)
-        for (int i = 0; i < stages && i < ntiles; i++) fetch(i);
-    for (int i = threadIdx.x; i < ROWS * (s.ck / 8); i += NW * 32) {
-        const int x = i / (s.ck / 8), e = (i - x * (s.ck / 8)) * 8;
-        pg_cp16(qs + (uint32_t)(x * stride + e * 2), qx + ((int64_t)row0 * s.H + min(rr0 + x, total - 1)) * s.ck + e);
+    for (int i = 0; i < stages && i < ntiles; i++) fetch(i);
+    for (int x = warp; x < ROWS; x += NW) {
+        const bf16 *src = qx + ((int64_t)row0 * s.H + min(rr0 + x, total - 1)) * s.ck;
+        for (int e = lane * 8; e < s.ck; e += 256) pg_cp16(qs + (uint32_t)(x * stride + e * 2), src + e);
     }
     pg_cp_commit();
     pg_cp_wait<0>();
     __syncthreads();
 
+    const int steps = s.ck / 16, half = (steps + 1) / 2, s0 = kh * half, sn = min(half, steps - s0);   // this warp's steps of the columns
+    const uint32_t q_at = qs + (uint32_t)((rt * 16 + (lane & 15)) * stride + (lane >> 4) * 16 + s0 * 32);
+    const uint32_t k_at = (uint32_t)((kq * 16 + (lane & 7) + ((lane >> 4) << 3)) * stride + ((lane >> 3) & 1) * 16 + s0 * 32);
+    uint32_t qf[QREG ? LA_QSTEPS : 1][4];
+    if (QREG) {
+#pragma unroll
+        for (int i = 0; i < LA_QSTEPS; i++)
+            if (i < sn) pg_ldsm4(qf[QREG ? i : 0], q_at + i * 32);
+    }
     const int cw = ((s.cp + NW - 1) / NW + 15) & ~15, c0 = warp * cw, nv = max(0, min(cw, s.cp - c0)) / 8;   // this warp's columns of the sums
     const int lim0 = pos0 + min(rr0 + rt * 16 + r, total - 1) / s.H, lim1 = pos0 + min(rr0 + rt * 16 + r + 8, total - 1) / s.H;
     const float scale = s.scale * LOG2E;
@@ -229,84 +269,87 @@ __global__ void __launch_bounds__(RT * 128)
 #pragma unroll
             for (int j = 0; j < 4; j++) o[x][i][j] = 0.0f;
     }
-    const uint32_t q_at = qs + (uint32_t)((rt * 16 + (lane & 15)) * stride + (lane >> 4) * 16);
-    const uint32_t k_at = (uint32_t)((kq * 16 + (lane & 7) + ((lane >> 4) << 3)) * stride + ((lane >> 3) & 1) * 16);
     const uint32_t v_at = (uint32_t)(((lane & 7) + ((lane >> 3) & 1) * 8) * stride + ((lane >> 4) * 8 + c0) * 2);
+    const uint32_t mine = xs + (uint32_t)(warp * 32 + lane) * 16, theirs = xs + (uint32_t)((warp ^ 1) * 32 + lane) * 16;
     bool ok = true;
     for (int it = 0; it < ntiles; it++) {
         ok = pg_mbar_wait(bar + (uint32_t)(it % stages) * 8, (uint32_t)(it / stages) & 1u, &abort_flag, status, limit_ns);
+        const uint32_t kt = ring + (uint32_t)(it % stages) * stage;
+        float sc[2][4] = {};
+        if (QREG) {
+#pragma unroll
+            for (int i = 0; i < LA_QSTEPS; i++) {
+                if (i < sn) {
+                    uint32_t b[4];
+                    pg_ldsm4(b, kt + k_at + i * 32);
+                    pg_mma_bf16(sc[0], qf[QREG ? i : 0][0], qf[QREG ? i : 0][1], qf[QREG ? i : 0][2], qf[QREG ? i : 0][3], b[0], b[1]);
+                    pg_mma_bf16(sc[1], qf[QREG ? i : 0][0], qf[QREG ? i : 0][1], qf[QREG ? i : 0][2], qf[QREG ? i : 0][3], b[2], b[3]);
+                }
+            }
+        } else {
+            for (int i = 0; i < sn; i++) {
+                uint32_t a[4], b[4];
+                pg_ldsm4(a, q_at + i * 32);
+                pg_ldsm4(b, kt + k_at + i * 32);
+                pg_mma_bf16(sc[0], a[0], a[1], a[2], a[3], b[0], b[1]);
+                pg_mma_bf16(sc[1], a[0], a[1], a[2], a[3], b[2], b[3]);
+            }
+        }
+        // eight keys each: the other half's sums of them from the neighbour
+        {
+            const float (&give)[4] = kh ? sc[0] : sc[1];
+            asm volatile("st.shared.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(mine), "f"(give[0]), "f"(give[1]), "f"(give[2]), "f"(give[3]) : "memory");
+        }
+        // also: every warp is done with the tile before, so its slot can be filled again
         if (!__syncthreads_and(ok)) {
             ok = false;
             break;
         }
-        const uint32_t kt = ring + (uint32_t)(it % stages) * stage;
-        float sc[2][2][4] = {};                           // two sums per tile of eight keys: shorter chains
-        for (int i = 0; i < s.ck / 16; i += 2) {
+        if (it > 0 && it - 1 + stages < ntiles) fetch(it - 1 + stages);
+        float sv[4];
+        {
+            const uint4 g = pg_lds128(theirs);
+            const float got[4] = {__uint_as_float(g.x), __uint_as_float(g.y), __uint_as_float(g.z), __uint_as_float(g.w)};
+            const int j0 = t0 + it * LA_KEYS + kq * 16 + kh * 8 + 2 * t;
 #pragma unroll
-            for (int u = 0; u < 2; u++) {
-                if (i + u < s.ck / 16) {
-                    uint32_t a[4], b[4];
-                    pg_ldsm4(a, q_at + (i + u) * 32);
-                    pg_ldsm4(b, kt + k_at + (i + u) * 32);
-                    pg_mma_bf16(sc[u][0], a[0], a[1], a[2], a[3], b[0], b[1]);
-                    pg_mma_bf16(sc[u][1], a[0], a[1], a[2], a[3], b[2], b[3]);
-                }
+            for (int j = 0; j < 4; j++) {
+                const int key = j0 + (j & 1);
+                const bool in = key < t1 && key <= (j < 2 ? lim0 : lim1);
+                sv[j] = in ? ((kh ? sc[1][j] : sc[0][j]) + got[j]) * scale : -INFINITY;
             }
         }
-        const int j0 = t0 + it * LA_KEYS + kq * 16;
-        float b0 = -INFINITY, b1 = -INFINITY;
-#pragma unroll
-        for (int n = 0; n < 2; n++)
-#pragma unroll
-            for (int j = 0; j < 2; j++) {
-                const int key = j0 + n * 8 + 2 * t + j;
-                sc[0][n][j] = key < t1 && key <= lim0 ? (sc[0][n][j] + sc[1][n][j]) * scale : -INFINITY;
-                sc[0][n][2 + j] = key < t1 && key <= lim1 ? (sc[0][n][2 + j] + sc[1][n][2 + j]) * scale : -INFINITY;
-                b0 = fmaxf(b0, sc[0][n][j]);
-                b1 = fmaxf(b1, sc[0][n][2 + j]);
-            }
+        float b0 = fmaxf(sv[0], sv[1]), b1 = fmaxf(sv[2], sv[3]);
 #pragma unroll
         for (int x = 1; x < 4; x <<= 1) {
             b0 = fmaxf(b0, __shfl_xor_sync(0xffffffffu, b0, x));
             b1 = fmaxf(b1, __shfl_xor_sync(0xffffffffu, b1, x));
         }
         if (t == 0) {
-            red[rt][kq][r] = b0;
-            red[rt][kq][r + 8] = b1;
+            red[rt][r][kq * 2 + kh] = b0;
+            red[rt][r + 8][kq * 2 + kh] = b1;
         }
-        __syncthreads();                                  // the maxima are there, and every warp is done with the tile before
-        if (warp == 0 && it > 0 && it - 1 + stages < ntiles) fetch(it - 1 + stages);
+        __syncthreads();                                  // the maxima are there
         float f[RT][2];
         bool moved = false;
 #pragma unroll
         for (int x = 0; x < RT; x++)
 #pragma unroll
             for (int e = 0; e < 2; e++) {
-                const int at = r + 8 * e;
-                const float top = fmaxf(m[x][e], fmaxf(fmaxf(red[x][0][at], red[x][1][at]), fmaxf(red[x][2][at], red[x][3][at])));
-                f[x][e] = exp2f(m[x][e] - top);
+                const float4 u = *reinterpret_cast<const float4 *>(red[x][r + 8 * e]), v = *reinterpret_cast<const float4 *>(red[x][r + 8 * e] + 4);
+                const float top = fmaxf(m[x][e], fmaxf(fmaxf(fmaxf(u.x, u.y), fmaxf(u.z, u.w)), fmaxf(fmaxf(v.x, v.y), fmaxf(v.z, v.w))));
+                f[x][e] = pg_ex2(m[x][e] - top);
+                moved |= top > m[x][e];
                 m[x][e] = top;
-                moved |= f[x][e] != 1.0f;
             }
         float m0 = m[0][0], m1 = m[0][1], f0 = f[0][0], f1 = f[0][1];
         if (RT == 2 && rt == 1) m0 = m[RT - 1][0], m1 = m[RT - 1][1], f0 = f[RT - 1][0], f1 = f[RT - 1][1];
-        float p[8];
-#pragma unroll
-        for (int n = 0; n < 2; n++)
-#pragma unroll
-            for (int j = 0; j < 2; j++) {
-                p[4 * n + j] = exp2f(sc[0][n][j] - m0);
-                p[4 * n + 2 + j] = exp2f(sc[0][n][2 + j] - m1);
-            }
-        l0 = l0 * f0 + ((p[0] + p[1]) + (p[4] + p[5]));
-        l1 = l1 * f1 + ((p[2] + p[3]) + (p[6] + p[7]));
+        const float p0 = pg_ex2(sv[0] - m0), p1 = pg_ex2(sv[1] - m0), p2 = pg_ex2(sv[2] - m1), p3 = pg_ex2(sv[3] - m1);
+        l0 = fmaf(l0, f0, p0 + p1);
+        l1 = fmaf(l1, f1, p2 + p3);
         {
-            const uint32_t at = ps + (uint32_t)((rt * 16 + r) * LA_PS + kq * 16 + 2 * t) * 2;
-#pragma unroll
-            for (int n = 0; n < 2; n++) {
-                asm volatile("st.shared.u32 [%0], %1;" ::"r"(at + n * 16), "r"(pg_pack_bf16(p[4 * n], p[4 * n + 1])) : "memory");
-                asm volatile("st.shared.u32 [%0], %1;" ::"r"(at + 8 * LA_PS * 2 + n * 16), "r"(pg_pack_bf16(p[4 * n + 2], p[4 * n + 3])) : "memory");
-            }
+            const uint32_t at = ps + (uint32_t)((rt * 16 + r) * LA_PS + kq * 16 + kh * 8 + 2 * t) * 2;
+            asm volatile("st.shared.u32 [%0], %1;" ::"r"(at), "r"(pg_pack_bf16(p0, p1)) : "memory");
+            asm volatile("st.shared.u32 [%0], %1;" ::"r"(at + 8 * LA_PS * 2), "r"(pg_pack_bf16(p2, p3)) : "memory");
         }
         __syncthreads();                                  // the weights are there
         if (__any_sync(0xffffffffu, moved)) {
@@ -353,8 +396,8 @@ __global__ void __launch_bounds__(RT * 128)
     }
     __syncthreads();
     if (t == 0) {
-        red[rt][kq][r] = l0;
-        red[rt][kq][r + 8] = l1;
+        red[rt][r][kq * 2 + kh] = l0;
+        red[rt][r + 8][kq * 2 + kh] = l1;
     }
     __syncthreads();
     const int ms = s.cp + 4;
@@ -368,32 +411,36 @@ __global__ void __launch_bounds__(RT * 128)
             for (int i = 0; i < VT; i++)
                 if (i < nv) *reinterpret_cast<float2 *>(row + c0 + i * 8 + 2 * t) = make_float2(o[x][i][2 * e], o[x][i][2 * e + 1]);
             if (warp == 0 && t == 0) {
-                const float l = (red[x][0][r + 8 * e] + red[x][1][r + 8 * e]) + (red[x][2][r + 8 * e] + red[x][3][r + 8 * e]);
-                *reinterpret_cast<float2 *>(row + s.cp) = make_float2(m[x][e], l);
+                const float *g = red[x][r + 8 * e];
+                *reinterpret_cast<float2 *>(row + s.cp) = make_float2(m[x][e], ((g[0] + g[1]) + (g[2] + g[3])) + ((g[4] + g[5]) + (g[6] + g[7])));
             }
         }
 }
 
-// grid (H, tiles of 16 rows): adds the slices of its rows, then W_uv of its head, then the gate
-constexpr int LV_T = 512;
+// grid (H, parts of 64 columns, groups of `group` <= 16 rows): adds the slices of its rows, then W_uv of its head, then the gate
+constexpr int LV_T = 256;
 constexpr int LV_SLICES = 64;
 __global__ void __launch_bounds__(LV_T)
-    latent_value_kernel(const LatentShape s, const pg_batch bt, const float *__restrict__ part, int per_seq, int S, int rows, const float *__restrict__ proj,
-                        int64_t ldp, bf16 *__restrict__ out, int64_t ldo)
+    latent_value_kernel(const LatentShape s, const pg_batch bt, const float *__restrict__ part, int per_seq, int S, int rows, int group,
+                        const float *__restrict__ proj, int64_t ldp, bf16 *__restrict__ out, int64_t ldo)
 {
-    extern __shared__ __align__(16) unsigned char smem[];   // [16][cp + 8]
+    extern __shared__ __align__(128) unsigned char smem[];   // [16][cp + 8]
     __shared__ float weight[16][LV_SLICES];
     __shared__ int64_t base[16];
     __shared__ int used[16];
+    const int h = blockIdx.x, m0 = blockIdx.z * group, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int c = blockIdx.y * 64 + warp * 8;
+    Weights8<16> w;
+    // (rows of W_uv behind the head's last one belong to the next head or are padding; their products are dropped)
+    if (c < s.V) w.ask(s.uv + ((int64_t)h * s.V + c) * s.cp, s.cp, s.cp, lane);
     pg_pdl_begin();
-    const int h = blockIdx.x, m0 = blockIdx.y * 16, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     bf16 *sa = reinterpret_cast<bf16 *>(smem);
     const int ld = s.cp + 8, ms = s.cp + 4;
-    {
+    for (int x = warp; x < 16; x += LV_T / 32) {
         // a warp per row: where its slices are, and their weights
-        const int m = m0 + warp;
+        const int m = m0 + x;
         int n = 0;
-        if (m < bt.rows) {
+        if (x < group && m < bt.rows) {
             const int seq = __ldcg(bt.d_row_seq + m), row0 = __ldcg(bt.d_seq_row0 + seq), T = seq_len(bt, seq);
             const int pos0 = __ldcg(bt.d_pos + row0), rr = (m - row0) * s.H + h, tile = rr / rows;
             const Slices sl = slices_of(s, pos0, T, tile, rows, S);
@@ -409,7 +456,7 @@ __global__ void __launch_bounds__(LV_T)
                     top = fmaxf(top, ml[i].x);
                 }
 #pragma unroll
-                for (int x = 16; x > 0; x >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, x));
+                for (int y = 16; y > 0; y >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, y));
 #pragma unroll
                 for (int i = 0; i < LV_SLICES / 32; i++) {
                     ml[i].x = exp2f(ml[i].x - top);
@@ -417,42 +464,47 @@ __global__ void __launch_bounds__(LV_T)
                 }
                 const float inv = __fdiv_rn(1.0f, pg_warp_sum(l));
 #pragma unroll
-                for (int i = 0; i < LV_SLICES / 32; i++) weight[warp][i * 32 + lane] = ml[i].x * inv;
-                if (lane == 0) base[warp] = at;
+                for (int i = 0; i < LV_SLICES / 32; i++) weight[x][i * 32 + lane] = ml[i].x * inv;
+                if (lane == 0) base[x] = at;
             }
         }
-        if (lane == 0) used[warp] = n;
+        if (lane == 0) used[x] = n;
     }
     __syncthreads();
     const int quads = s.cp / 4;
     for (int i = threadIdx.x; i < 16 * quads; i += LV_T) {
-        const int x = i / quads, c = (i - x * quads) * 4, n = used[x];
+        const int x = i / quads, k4 = (i - x * quads) * 4, n = used[x];
         float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-        const float *src = part + (n ? base[x] : 0) + c;
-#pragma unroll 8
+        const float *src = part + (n ? base[x] : 0) + k4;
+#pragma unroll 12
         for (int k = 0; k < n; k++) {
             const float4 v = __ldcg(reinterpret_cast<const float4 *>(src + (int64_t)k * rows * ms));
             const float f = weight[x][k];
             a.x = fmaf(f, v.x, a.x), a.y = fmaf(f, v.y, a.y), a.z = fmaf(f, v.z, a.z), a.w = fmaf(f, v.w, a.w);
         }
-        *reinterpret_cast<uint2 *>(sa + x * ld + c) = make_uint2(pg_pack_bf16(a.x, a.y), pg_pack_bf16(a.z, a.w));
+        *reinterpret_cast<uint2 *>(sa + x * ld + k4) = make_uint2(pg_pack_bf16(a.x, a.y), pg_pack_bf16(a.z, a.w));
     }
-    __syncthreads();
     const int r = lane >> 2, t = lane & 3;
-    for (int c = warp * 8; c < s.V; c += LV_T / 32 * 8) {
-        float d[4] = {};
-        // (rows of W_uv behind the head's last one belong to the next head or are padding; their products are dropped)
-        product16x8(d, pg_smem(sa), ld, s.uv + ((int64_t)h * s.V + c) * s.cp, s.cp, s.cp, lane);
+    float gate[2][2];
 #pragma unroll
-        for (int half = 0; half < 2; half++) {
-            const int x = r + 8 * half, m = m0 + x;
-            if (used[x] == 0) continue;
+    for (int half = 0; half < 2; half++)
 #pragma unroll
-            for (int j = 0; j < 2; j++) {
-                const int col = c + 2 * t + j;
-                if (col < s.V)
-                    pg_put(out + (int64_t)m * ldo + h * s.V + col, d[2 * half + j] * pg_sigmoid(__ldcg(proj + (int64_t)m * ldp + s.at_gate + h * s.V + col)));
-            }
+        for (int j = 0; j < 2; j++) {
+            const int col = c + 2 * t + j;
+            gate[half][j] = used[r + 8 * half] && col < s.V ? __ldcg(proj + (int64_t)(m0 + r + 8 * half) * ldp + s.at_gate + h * s.V + col) : 0.0f;
+        }
+    __syncthreads();
+    if (c >= s.V) return;
+    float d[4] = {};
+    w.times(d, pg_smem(sa), ld, lane);
+#pragma unroll
+    for (int half = 0; half < 2; half++) {
+        const int x = r + 8 * half, m = m0 + x;
+        if (used[x] == 0) continue;
+#pragma unroll
+        for (int j = 0; j < 2; j++) {
+            const int col = c + 2 * t + j;
+            if (col < s.V) pg_put(out + (int64_t)m * ldo + h * s.V + col, d[2 * half + j] * pg_sigmoid(gate[half][j]));
         }
     }
 }
@@ -554,7 +606,7 @@ LatentShape shape_of(const pg_latent *p)
 
 constexpr int LA_SMEM = 220 * 1024;
 int attn_rows(const LatentShape &s) { return s.H > 16 ? 32 : 16; }
-int attn_smem(const LatentShape &s, int stages) { return (stages * LA_KEYS + attn_rows(s)) * (s.ck * 2 + 16) + attn_rows(s) * LA_PS * 2; }
+int attn_smem(const LatentShape &s, int stages) { return (stages * LA_KEYS + attn_rows(s)) * (s.ck * 2 + 16) + attn_rows(s) * (LA_PS * 2 + 256); }
 
 // slices of the context: about one CTA per SM, none shorter than 64 positions of a full cache
 int slices(const pg_ctx *ctx, int64_t units, int64_t cap)
@@ -562,6 +614,18 @@ int slices(const pg_ctx *ctx, int64_t units, int64_t cap)
     int64_t S = std::max<int64_t>(1, (int64_t)ctx->sm_count / std::max<int64_t>(1, units));
     S = std::min<int64_t>(S, std::max<int64_t>(1, cap / LA_KEYS));
     return (int)std::min<int64_t>(S, LV_SLICES);
+}
+
+template <int RT>
+int32_t launch_attn(pg_ctx *ctx, const LatentShape &s, const pg_batch *batch, dim3 grid, const bf16 *q, const bf16 *cache, float *part, int per_seq, int stages)
+{
+    auto go = [&](auto kern, std::atomic<uint64_t> &set) -> int32_t {
+        PG_CUDA(pg_max_smem_once(kern, LA_SMEM, ctx->device, set));
+        return launch_pdl(ctx, kern, grid, dim3(RT * 256), (size_t)attn_smem(s, stages), s, *batch, q, cache, part, per_seq, stages, ctx->d_status,
+                          ctx->wait_limit_ns);
+    };
+    static std::atomic<uint64_t> set[2] = {};
+    return s.ck <= LA_QSTEPS * 32 ? go(latent_attn_kernel<RT, true>, set[0]) : go(latent_attn_kernel<RT, false>, set[1]);
 }
 
 int32_t check(const pg_latent *p, const pg_batch *batch, int64_t ldp, int64_t ldo)
@@ -636,20 +700,16 @@ PG_API int32_t pg_latent_run(pg_ctx *ctx, const pg_latent *p, const pg_batch *ba
     int stages = 4;
     while (stages > 2 && attn_smem(s, stages) > LA_SMEM) stages--;
     const dim3 grid((unsigned)S, (unsigned)tiles, (unsigned)batch->seqs);
-    if (rows == 32) {
-        static std::atomic<uint64_t> set{0};
-        PG_CUDA(pg_max_smem_once(latent_attn_kernel<2>, LA_SMEM, ctx->device, set));
-        rc = launch_pdl(ctx, latent_attn_kernel<2>, grid, dim3(256), (size_t)attn_smem(s, stages), s, *batch, (const bf16 *)q, (const bf16 *)cache, p->d_part,
-                        per_seq, stages, ctx->d_status, ctx->wait_limit_ns);
-    } else {
-        static std::atomic<uint64_t> set{0};
-        PG_CUDA(pg_max_smem_once(latent_attn_kernel<1>, LA_SMEM, ctx->device, set));
-        rc = launch_pdl(ctx, latent_attn_kernel<1>, grid, dim3(128), (size_t)attn_smem(s, stages), s, *batch, (const bf16 *)q, (const bf16 *)cache, p->d_part,
-                        per_seq, stages, ctx->d_status, ctx->wait_limit_ns);
-    }
+    rc = rows == 32 ? launch_attn<2>(ctx, s, batch, grid, q, cache, p->d_part, per_seq, stages) : launch_attn<1>(ctx, s, batch, grid, q, cache, p->d_part, per_seq, stages);
     if (rc != PG_OK) return rc;
-    return launch_pdl(ctx, latent_value_kernel, dim3((unsigned)s.H, row_tiles), dim3(LV_T), (size_t)(16 * (s.cp + 8) * 2), s, *batch, (const float *)p->d_part, per_seq, S,
-                      rows, d_proj, ldp, (bf16 *)d_out, ldo);
+    // groups of rows small enough for about one CTA per SM
+    const unsigned parts64 = (unsigned)((s.V + 63) / 64);
+    int group = 16;
+    while (group > 1 && (int64_t)s.H * parts64 * ((batch->rows + group - 1) / group) < ctx->sm_count * 3 / 4) group /= 2;
+    const int64_t groups = (batch->rows + group - 1) / group;
+    PG_REQUIRE(groups <= 65535 && parts64 <= 65535, "latent attention: too many rows");
+    return launch_pdl(ctx, latent_value_kernel, dim3((unsigned)s.H, parts64, (unsigned)groups), dim3(LV_T), (size_t)(16 * (s.cp + 8) * 2), s, *batch,
+                      (const float *)p->d_part, per_seq, S, rows, group, d_proj, ldp, (bf16 *)d_out, ldo);
 }
 
 PG_API int32_t pg_latent_prompt_supports(const pg_latent *p)

@@ -1,4 +1,5 @@
 // Products with bf16 weights: the handle and the choice of kernel (include/peregrine_b200_lm.h).
+#include <algorithm>
 #include <new>
 
 #include "pg_lm.cuh"
@@ -14,6 +15,9 @@ PG_API int32_t pg_linear_wrap(pg_ctx *ctx, const void *d_w_bf16, int64_t n, int6
     PG_REQUIRE(k % 64 == 0 && ((uintptr_t)d_w_bf16 & 15) == 0, "linear_wrap: K must be a multiple of 64 (K = %lld) and the weights 16-byte aligned",
                (long long)k);
     PG_REQUIRE(n < (1 << 30) && k < (1 << 30), "linear_wrap: shape too large");
+    // now, since the workspace cannot grow while a step is being recorded
+    const int32_t rc = pg_splitk_reserve(ctx, std::max(pgk_linear_gemv_workspace(n, k), PG_LM_TICKET_BYTES + (size_t)ctx->sm_count * 128 * 128 * sizeof(float)));
+    if (rc != PG_OK) return rc;
     pg_linear *l = new (std::nothrow) pg_linear();
     if (!l) PG_FAIL(PG_ERR_NOMEM, "out of host memory");
     l->w = (const bf16 *)d_w_bf16;

@@ -232,7 +232,6 @@ __global__ void __launch_bounds__(GV_THREADS, 1)
     }
 }
 
-constexpr size_t GV_TICKET_BYTES = 64 * 1024;   // the head of the context's split-K workspace: zero between calls
 
 template <int ACT, bool HI, bool ROUTED, bool SPLIT, typename TY>
 int32_t gv_launch(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int64_t lda, int M, int kw, int KW, int KH, int grid, int sp, float limit, TY *y, int64_t ldy,
@@ -245,7 +244,7 @@ int32_t gv_launch(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int64_t lda,
     static std::atomic<uint64_t> smem_set{0};
     PG_CUDA(pg_max_smem_once(kern, 226 * 1024, ctx->device, smem_set));
     unsigned int *tickets = reinterpret_cast<unsigned int *>(ctx->splitk);
-    float *slabs = SPLIT ? reinterpret_cast<float *>(reinterpret_cast<unsigned char *>(ctx->splitk) + GV_TICKET_BYTES) : nullptr;
+    float *slabs = SPLIT ? reinterpret_cast<float *>(reinterpret_cast<unsigned char *>(ctx->splitk) + PG_LM_TICKET_BYTES) : nullptr;
     return launch_pdl(ctx, kern, dim3((unsigned)grid), dim3(GV_THREADS), (size_t)smem, a, lda, M, lin->w, (int)lin->n, (int)lin->k, kw, KW, KH, limit, y, ldy, rt,
                       sp, slabs, tickets, ctx->d_status, ctx->wait_limit_ns);
 }
@@ -254,6 +253,12 @@ int32_t gv_launch(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int64_t lda,
 inline int gv_parts(int64_t k) { return (int)((k + GV_WARPS * GV_KW_MAX - 1) / (GV_WARPS * GV_KW_MAX)); }
 
 }  // namespace
+
+size_t pgk_linear_gemv_workspace(int64_t n, int64_t k)
+{
+    // plain and gated forms alike: 64 floats of slab per eight columns and part
+    return gv_parts(k) > 1 ? PG_LM_TICKET_BYTES + (size_t)gv_parts(k) * (size_t)(n + 16) * 64 : 0;
+}
 
 bool pgk_linear_gemv_supports(const pg_linear *lin, int64_t m) { return m >= 1 && m <= 16 && gv_parts(lin->k) <= 16 && lin->n < (1 << 30); }
 
@@ -266,7 +271,7 @@ int32_t pgk_linear_gemv(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int64_
     const int KH = sp > 1 ? (int)pg_up((K + sp - 1) / sp, 32) : K;
     const int64_t units = ctx->sm_count / sp;
     if (sp > 1) {
-        const int32_t rc = pg_splitk_reserve(ctx, GV_TICKET_BYTES + (size_t)sp * (size_t)items * 32 * 4 * nt * sizeof(float));
+        const int32_t rc = pg_splitk_reserve(ctx, PG_LM_TICKET_BYTES + (size_t)sp * (size_t)items * 32 * 4 * nt * sizeof(float));
         if (rc != PG_OK) return rc;
     }
     // parts of a CTA's K: as few as registers allow, more while every (tile, part) still finds a warp of its own

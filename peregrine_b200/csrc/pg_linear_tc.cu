@@ -1,9 +1,11 @@
 // Prefill-size product y = a W^T, bf16 operands and f32 sums, on the 5th-generation tensor cores: the structure of
 // gemm_i8_tcgen05_kernel (one persistent CTA per SM; TMA producer warp, one issuing lane, four epilogue warps, two TMEM
-// accumulators) for kind::f16, with two more things in it:
+// accumulators) for kind::f16, with three more things in it:
 //
 //   * gated products: W's rows alternate eight gate / eight up rows, so a lane's 32 accumulator columns hold complete
 //     pairs and the epilogue writes the gated bf16 activations (half the columns, a quarter of the bytes of the raw sums);
+//   * products with fewer tiles than SMs: K is divided over `sp` CTAs.  Each writes its raw sums to a slab; the last warp of a
+//     32-row band to finish (a ticket per band) adds the slabs in a fixed order and writes the outputs.  Nobody waits;
 //   * routed products: an A tile of 128 rows belongs to one expert, whose weights start at row expert * N of the
 //     stacked [experts * N][K] matrix.  Number and experts of the tiles are read on the device.
 //
@@ -32,6 +34,13 @@ struct Cfg {
     static constexpr int STAGES = ROOM / STAGE > 10 ? 10 : ROOM / STAGE;
     static constexpr int TMEM_COLS = (2 * BN < 32) ? 32 : 2 * BN;
     static constexpr size_t SMEM = (size_t)STAGES * STAGE + 1024 + 256 + 4 * PG_EPI_WARP_BYTES;
+};
+
+// How K is divided: parts of `blocks` 64-element blocks; slab of (unit, quarter): [BN][32 rows]
+struct KParts {
+    int parts, blocks;
+    float *slabs;
+    unsigned int *tickets;   // one per (tile, quarter), zero between calls
 };
 
 // Writes a lane's row of a block of 32 accumulator columns; n0: first column, N: columns of the product.
@@ -77,7 +86,7 @@ __device__ __forceinline__ void store_row(TY *y, int64_t ldy, int row, int n0, i
 template <int BN, int ACT, typename TY>
 __global__ void __launch_bounds__(TC_THREADS, 1)
     linear_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_b, int M, int N, int K, float limit,
-                     TY *__restrict__ y, int64_t ldy, const PgRouted rt, int32_t *status, unsigned long long limit_ns)
+                     TY *__restrict__ y, int64_t ldy, const PgRouted rt, const KParts kp, int32_t *status, unsigned long long limit_ns)
 {
     using C = Cfg<BN>;
     constexpr int STAGES = C::STAGES;
@@ -119,8 +128,10 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
     if (routed) asm volatile("griddepcontrol.wait;" ::: "memory");   // the list of tiles comes from the preceding kernels
     const int tiles_m = routed ? __ldcg(rt.blocks) : (M + BM - 1) / BM;
     const int tiles_n = (N + BN - 1) / BN;
-    const int total = tiles_m * tiles_n;
+    const int sp = kp.parts, total = tiles_m * tiles_n * sp;   // unit u: part u % sp of tile u / sp
     const int kblocks = K / BK;
+    auto k_first = [&](int u) { return (u % sp) * kp.blocks; };
+    auto k_end = [&](int u) { return min(kblocks, (u % sp + 1) * kp.blocks); };
     const int rows = routed ? tiles_m * BM : M;
 
     if (warp == 0) {
@@ -132,20 +143,21 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
             int early = 0;
             if (!routed) {
                 if ((int)blockIdx.x < total) {
-                    const int n0 = ((int)blockIdx.x / tiles_m) * BN;
-                    early = kblocks < STAGES ? kblocks : STAGES;
+                    const int n0 = ((int)blockIdx.x / sp / tiles_m) * BN, first = k_first(blockIdx.x);
+                    early = min(k_end(blockIdx.x) - first, STAGES);
                     for (int i = 0; i < early; i++) {
                         pg_mbar_expect(bar_full + 8 * i, C::STAGE);
-                        tma_load_2d(base + i * C::STAGE + C::STAGE_A, &tmap_b, bar_full + 8 * i, i * BK, n0);
+                        tma_load_2d(base + i * C::STAGE + C::STAGE_A, &tmap_b, bar_full + 8 * i, (first + i) * BK, n0);
                     }
                 }
                 asm volatile("griddepcontrol.wait;" ::: "memory");
             }
             for (int u = blockIdx.x; ok && u < total; u += gridDim.x) {
-                const int m0 = (u % tiles_m) * BM;
-                const int n0 = (u / tiles_m) * BN;
-                const int b0 = routed ? __ldcg(rt.block_expert + u % tiles_m) * N + n0 : n0;
-                for (int kb = 0; kb < kblocks; kb++) {
+                const int tile = u / sp;
+                const int m0 = (tile % tiles_m) * BM;
+                const int n0 = (tile / tiles_m) * BN;
+                const int b0 = routed ? __ldcg(rt.block_expert + tile % tiles_m) * N + n0 : n0;
+                for (int kb = k_first(u), end = k_end(u); kb < end; kb++) {
                     if (!(ok = pg_mbar_wait(bar_empty + 8 * stage, phase ^ 1, abort_flag, status, limit_ns))) break;
                     const uint32_t sa = base + stage * C::STAGE;
                     if (early > 0) {
@@ -178,14 +190,15 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
                 if (!(ok = pg_mbar_wait(bar_tempty + 8 * acc, acc_phase ^ 1, abort_flag, status, limit_ns))) break;
                 tc_fence_after();
                 const uint32_t d_tmem = tmem_base + acc * BN;
-                for (int kb = 0; kb < kblocks; kb++) {
+                const int first = k_first(u), end = k_end(u);
+                for (int kb = first; kb < end; kb++) {
                     if (!(ok = pg_mbar_wait(bar_full + 8 * stage, phase, abort_flag, status, limit_ns))) break;
                     tc_fence_after();
                     const uint32_t sa = base + stage * C::STAGE;
                     const uint64_t da = make_smem_desc(sa), db = make_smem_desc(sa + C::STAGE_A);
 #pragma unroll
                     for (int j = 0; j < BKB / UMMA_KB; j++)
-                        umma_f16(d_tmem, da + (uint64_t)(j * (UMMA_KB >> 4)), db + (uint64_t)(j * (UMMA_KB >> 4)), idesc, (kb | j) != 0 ? 1u : 0u);
+                        umma_f16(d_tmem, da + (uint64_t)(j * (UMMA_KB >> 4)), db + (uint64_t)(j * (UMMA_KB >> 4)), idesc, kb != first || j != 0 ? 1u : 0u);
                     umma_commit(bar_empty + 8 * stage);   // stage reusable once these MMAs have read it
                     if (++stage == STAGES) {
                         stage = 0;
@@ -208,8 +221,9 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
         const bool vec_ok = ACT == PG_ACT_NONE && sizeof(TY) == 4 && ((N & 3) == 0) && ((ldy & 3) == 0) && (((uintptr_t)y & 15) == 0);
         bool ok = true;
         for (int u = blockIdx.x; ok && u < total; u += gridDim.x) {
-            const int m0 = (u % tiles_m) * BM;
-            const int n0 = (u / tiles_m) * BN;
+            const int tile = u / sp;
+            const int m0 = (tile % tiles_m) * BM;
+            const int n0 = (tile / tiles_m) * BN;
             ok = pg_mbar_wait(bar_tfull + 8 * acc, acc_phase, abort_flag, status, limit_ns);
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) break;
@@ -217,20 +231,56 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
             const int row_base = m0 + q * 32, row = row_base + lane;
             const uint32_t taddr = tmem_base + ((uint32_t)(q * 32) << 16) + acc * BN;
             const uint32_t stage_buf = base + (uint32_t)((size_t)STAGES * C::STAGE) + 256u + (uint32_t)q * PG_EPI_WARP_BYTES;
-#pragma unroll 1
-            for (int c = 0; c < BN; c += 32) {
-                if (row_base >= rows || n0 + c >= N) break;   // uniform over the warp
-                uint32_t v[32];
-                tmem_ld32(taddr + c, v);
+            auto put = [&](const uint32_t (&v)[32], int c) {
                 if (vec_ok)
                     pg_store_block_32x32(reinterpret_cast<uint32_t *>(y) + (int64_t)row_base * ldy + n0 + c, ldy, rows - row_base, N - (n0 + c), stage_buf,
                                          lane, v);
                 else if (row < rows)
                     store_row<ACT, TY>(y, ldy, row, n0 + c, N, v, limit);
+            };
+#pragma unroll 1
+            for (int c = 0; c < BN; c += 32) {
+                if (row_base >= rows || n0 + c >= N) break;   // uniform over the warp
+                uint32_t v[32];
+                tmem_ld32(taddr + c, v);
+                if (sp > 1) {
+                    float *slab = kp.slabs + (((int64_t)u * 4 + q) * BN + c) * 32 + lane;
+#pragma unroll
+                    for (int j = 0; j < 32; j++) __stcg(slab + j * 32, __uint_as_float(v[j]));
+                } else {
+                    put(v, c);
+                }
             }
             tc_fence_before();
             __syncwarp();
             if (lane == 0) pg_mbar_arrive(bar_tempty + 8 * acc);
+            if (sp > 1 && row_base < rows) {
+                unsigned int *ticket = kp.tickets + tile * 4 + q;
+                __threadfence();
+                __syncwarp();
+                const unsigned int before = __shfl_sync(0xffffffffu, lane == 0 ? atomicAdd(ticket, 1u) : 0u, 0);
+                if (before == (unsigned)(sp - 1)) {
+                    __threadfence();
+                    if (lane == 0) *ticket = 0;
+#pragma unroll 1
+                    for (int c = 0; c < BN; c += 32) {
+                        if (n0 + c >= N) break;
+                        const float *slab = kp.slabs + (((int64_t)tile * sp * 4 + q) * BN + c) * 32 + lane;
+                        float sum[32];
+#pragma unroll
+                        for (int j = 0; j < 32; j++) sum[j] = __ldcg(slab + j * 32);
+                        for (int p = 1; p < sp; p++) {
+                            const float *at = slab + (int64_t)p * 4 * BN * 32;
+#pragma unroll
+                            for (int j = 0; j < 32; j++) sum[j] += __ldcg(at + j * 32);
+                        }
+                        uint32_t v[32];
+#pragma unroll
+                        for (int j = 0; j < 32; j++) v[j] = __float_as_uint(sum[j]);
+                        put(v, c);
+                    }
+                }
+            }
             if (++acc == 2) {
                 acc = 0;
                 acc_phase ^= 1;
@@ -257,7 +307,8 @@ int32_t encode_kmajor(CUtensorMap *map, const void *ptr, int64_t rows, int64_t k
 }
 
 template <int BN, int ACT, typename TY>
-int32_t launch(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t lda, int64_t m, float limit, TY *y, int64_t ldy, const PgRouted &rt)
+int32_t launch(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t lda, int64_t m, float limit, TY *y, int64_t ldy, const PgRouted &rt,
+               KParts kp)
 {
     using C = Cfg<BN>;
     CUtensorMap ta;
@@ -272,9 +323,11 @@ int32_t launch(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t lda, int64_t 
     auto kern = linear_tc_kernel<BN, ACT, TY>;
     static std::atomic<uint64_t> smem_set{0};
     PG_CUDA(pg_max_smem_once(kern, (int)C::SMEM, ctx->device, smem_set));
-    const int64_t tiles = ((m + BM - 1) / BM) * ((lin->n + BN - 1) / BN);
+    const int64_t tiles = ((m + BM - 1) / BM) * ((lin->n + BN - 1) / BN) * kp.parts;
+    kp.tickets = reinterpret_cast<unsigned int *>(ctx->splitk);
+    kp.slabs = reinterpret_cast<float *>(reinterpret_cast<unsigned char *>(ctx->splitk) + PG_LM_TICKET_BYTES);
     return launch_pdl(ctx, kern, dim3((unsigned)std::min<int64_t>(tiles, ctx->sm_count)), dim3(TC_THREADS), C::SMEM, ta,
-                      *reinterpret_cast<CUtensorMap *>(lin->tmap[at]), (int)m, (int)lin->n, (int)lin->k, limit, y, ldy, rt, ctx->d_status,
+                      *reinterpret_cast<CUtensorMap *>(lin->tmap[at]), (int)m, (int)lin->n, (int)lin->k, limit, y, ldy, rt, kp, ctx->d_status,
                       ctx->wait_limit_ns);
 }
 
@@ -283,13 +336,32 @@ int32_t dispatch(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t lda, int64_
 {
     // the widest tile that still gives every SM one
     const int64_t tiles_m = (m + BM - 1) / BM;
+    auto tiles = [&](int w) { return tiles_m * ((lin->n + w - 1) / w); };
     int bn = 32;
     for (int cand = 64; cand <= 256; cand *= 2)
-        if (tiles_m * ((lin->n + cand - 1) / cand) >= ctx->sm_count) bn = cand;
-    if (bn == 256) return launch<256, ACT, TY>(ctx, lin, a, lda, m, limit, y, ldy, rt);
-    if (bn == 128) return launch<128, ACT, TY>(ctx, lin, a, lda, m, limit, y, ldy, rt);
-    if (bn == 64) return launch<64, ACT, TY>(ctx, lin, a, lda, m, limit, y, ldy, rt);
-    return launch<32, ACT, TY>(ctx, lin, a, lda, m, limit, y, ldy, rt);
+        if (tiles(cand) >= ctx->sm_count) bn = cand;
+    const int kblocks = (int)(lin->k / BK);
+    KParts kp = {1, kblocks, nullptr, nullptr};
+    if (bn < 128 && rt.blocks == nullptr) {
+        // narrow tiles read the rows of a over and over: K in parts of at least four blocks instead, if that fills the GPU too
+        for (int cand = lin->n > 64 ? 128 : lin->n > 32 ? 64 : 32; cand >= 32; cand /= 2) {
+            const int64_t most = std::min<int64_t>(ctx->sm_count / std::max<int64_t>(1, tiles(cand)), kblocks / 4);
+            if (most < 2 || tiles(cand) * most < ctx->sm_count * 3 / 4) continue;
+            bn = cand;
+            kp.blocks = (kblocks + (int)most - 1) / (int)most;
+            kp.parts = (kblocks + kp.blocks - 1) / kp.blocks;
+            break;
+        }
+        const size_t need = PG_LM_TICKET_BYTES + (size_t)tiles(bn) * kp.parts * BM * bn * sizeof(float);
+        if (kp.parts > 1 && need > ctx->splitk_bytes) {
+            const int32_t rc = pg_splitk_reserve(ctx, need);
+            if (rc != PG_OK) return rc;
+        }
+    }
+    if (bn == 256) return launch<256, ACT, TY>(ctx, lin, a, lda, m, limit, y, ldy, rt, kp);
+    if (bn == 128) return launch<128, ACT, TY>(ctx, lin, a, lda, m, limit, y, ldy, rt, kp);
+    if (bn == 64) return launch<64, ACT, TY>(ctx, lin, a, lda, m, limit, y, ldy, rt, kp);
+    return launch<32, ACT, TY>(ctx, lin, a, lda, m, limit, y, ldy, rt, kp);
 }
 
 }  // namespace

@@ -44,6 +44,11 @@ struct PgRouted {
     int top, by_token;
 };
 
+// The context's split-K workspace: tickets, zero between calls, then slabs.
+constexpr size_t PG_LM_TICKET_BYTES = 64 * 1024;
+// what pg_linear_wrap reserves for the streaming form of a matrix, and for the tensor-core form (a tile of 128 x 128 per SM)
+size_t pgk_linear_gemv_workspace(int64_t n, int64_t k);
+
 // pg_linear_gemv.cu: m <= 16 rows (or row blocks of 16) against streamed weights
 bool pgk_linear_gemv_supports(const pg_linear *lin, int64_t m);
 int32_t pgk_linear_gemv(pg_ctx *ctx, const pg_linear *lin, const bf16 *a, int64_t lda, int64_t m, int act, float limit, void *y, int y_dtype, int64_t ldy,

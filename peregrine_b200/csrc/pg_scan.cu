@@ -7,8 +7,8 @@
 //   scan_step_kernel    one token per sequence: W_dt, softplus, update, read-out and gate in one launch; the state is read and
 //                       written once
 //   scan_run_kernel     portions: a CTA has 32 channels of a sequence, four lanes per channel, whose states stay in registers;
-//                       step sizes, inputs, B and C come in tiles of tokens through shared memory, the next tile's loads in
-//                       flight meanwhile.  It also stores the convolution inputs that the next portion needs.
+//                       step sizes, inputs, B and C come in tiles of tokens through shared memory, brought and finished by
+//                       four more warps.  It also stores the convolution inputs that the next portion needs.
 //
 // Convolution inputs are kept per slot in a ring of `taps` entries, position p in entry p mod taps: a single token writes an
 // entry that nobody reads any more.  A sequence starts at position 0: what its slot holds is then taken as zero.
@@ -24,13 +24,27 @@ struct ScanShape {
     const bf16 *dt;
 };
 
-__device__ __forceinline__ float softplus(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
-
 __device__ __forceinline__ float ex2(float x)
 {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
+}
+
+// ln(1 + e^x) = max(x, 0) + ln(1 + e) with e = e^-|x| in (0, 1], and ln(1 + e) = 2 artanh(e / (2 + e)) by its power series:
+// the argument is at most 1/3, and what is left out is below 2^-26 of the sum.
+__device__ __forceinline__ float softplus(float x)
+{
+    const float e = ex2(-1.4426950408889634f * fabsf(x)), z = __fdividef(e, 2.0f + e), w = z * z;
+    float p = 1.0f / 15.0f;
+    p = fmaf(p, w, 1.0f / 13.0f);
+    p = fmaf(p, w, 1.0f / 11.0f);
+    p = fmaf(p, w, 1.0f / 9.0f);
+    p = fmaf(p, w, 1.0f / 7.0f);
+    p = fmaf(p, w, 1.0f / 5.0f);
+    p = fmaf(p, w, 1.0f / 3.0f);
+    p = fmaf(p, w, 1.0f);
+    return fmaf(2.0f * z, p, fmaxf(x, 0.0f));
 }
 
 template <int V>
@@ -120,19 +134,69 @@ __global__ void __launch_bounds__(SC_T)
 }
 
 // ---- the recurrence ------------------------------------------------------------------------------------------------
-constexpr int SR_T = 128, SR_CH = 32;   // channels of a CTA: four lanes each, quads q, q + 4, .. of a channel's states
+constexpr int SR_CH = 32, SR_T = 128;   // channels of a CTA: four lanes each, quads q, q + 4, .. of a channel's states
 
-// A quad of states takes a token; returns its part of the read-out.
-__device__ __forceinline__ float update(float4 &S, const float4 &a, float dt, float du, const float4 &b, const float4 &c)
+// a pair of f32 in one register pair, and the pairwise instructions
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pair(float lo, float hi)
 {
-    S.x = fmaf(ex2(dt * a.x), S.x, du * b.x);
-    S.y = fmaf(ex2(dt * a.y), S.y, du * b.y);
-    S.z = fmaf(ex2(dt * a.z), S.z, du * b.z);
-    S.w = fmaf(ex2(dt * a.w), S.w, du * b.w);
-    return fmaf(S.x, c.x, S.y * c.y) + fmaf(S.z, c.z, S.w * c.w);
+    f32x2 v;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(lo), "f"(hi));
+    return v;
+}
+__device__ __forceinline__ float2 halves(f32x2 v)
+{
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b)
+{
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c)
+{
+    f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+struct Quad {
+    f32x2 lo, hi;
+};
+__device__ __forceinline__ Quad quad(const float4 &v) { return {pair(v.x, v.y), pair(v.z, v.w)}; }
+__device__ __forceinline__ float4 quad4(const Quad &v)
+{
+    const float2 a = halves(v.lo), b = halves(v.hi);
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ Quad load_quad(const float *p)   // shared memory
+{
+    const ulonglong2 v = *reinterpret_cast<const ulonglong2 *>(p);
+    return {v.x, v.y};
+}
+__device__ __forceinline__ f32x2 ex2_pair(f32x2 v)
+{
+    const float2 h = halves(v);
+    return pair(ex2(h.x), ex2(h.y));
+}
+
+// A quad of states takes a token (dt and dt x in both halves); returns its part of the read-out.
+__device__ __forceinline__ f32x2 update(Quad &S, const Quad &a, f32x2 dt, f32x2 du, const Quad &b, const Quad &c)
+{
+    S.lo = fma2(ex2_pair(mul2(dt, a.lo)), S.lo, mul2(du, b.lo));
+    S.hi = fma2(ex2_pair(mul2(dt, a.hi)), S.hi, mul2(du, b.hi));
+    return fma2(S.lo, c.lo, mul2(S.hi, c.hi));
+}
+__device__ __forceinline__ float sum2(f32x2 v)
+{
+    const float2 h = halves(v);
+    return h.x + h.y;
 }
 
 // grid (ceil(inner / 32), ceil(rows / R)).  NC: quads of states per lane
+constexpr int SS_W = 8;                  // 16-byte pieces of a row of W_dt that a lane asks for ahead (rank up to 256)
 template <int NC, int R, typename TA>
 __global__ void __launch_bounds__(SR_T)
     scan_step_kernel(const ScanShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, const TA *__restrict__ x, int64_t ldx,
@@ -146,51 +210,61 @@ __global__ void __launch_bounds__(SR_T)
     float *sdt = sm, *sbc = sm + R * s.dtp;
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     // weights do not depend on the kernel before
-    float4 a[NC];
+    const uint4 *wrow = reinterpret_cast<const uint4 *>(s.dt + (int64_t)c * s.dtp) + q;
+    const int pieces = live ? s.dtp / 32 : 0;
+    uint4 w[SS_W];
+#pragma unroll
+    for (int k = 0; k < SS_W; k++) w[k] = k < pieces ? __ldg(wrow + 4 * k) : make_uint4(0u, 0u, 0u, 0u);
+    Quad a[NC];
 #pragma unroll
     for (int i = 0; i < NC; i++)
-        a[i] = live && q + 4 * i < quads ? __ldg(reinterpret_cast<const float4 *>(s.a + (int64_t)c * s.ss) + q + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        a[i] = quad(live && q + 4 * i < quads ? __ldg(reinterpret_cast<const float4 *>(s.a + (int64_t)c * s.ss) + q + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f));
     const float dt_bias = live ? __ldg(s.dt_bias + c) : 0.0f, skip = live ? __ldg(s.d + c) : 0.0f;
     asm volatile("griddepcontrol.wait;" ::: "memory");
-    float4 S[R][NC];
     int64_t at[R];
-    float xv[R], z[R];
+    bool old[R];
 #pragma unroll
     for (int r = 0; r < R; r++) {
         const int m = m0 + r;
         const bool on = live && m < bt.rows;
         at[r] = on ? ((int64_t)__ldcg(bt.d_seq_slot + __ldcg(bt.d_row_seq + m)) * s.inner + c) * s.ss : -1;
-        const bool old = on && __ldcg(bt.d_pos + m) > 0;
+        old[r] = on && __ldcg(bt.d_pos + m) > 0;
+    }
+#pragma unroll
+    for (int r = 0; r < R; r++) {
+        const bool on = m0 + r < bt.rows;
+        const float *src = low + (int64_t)(m0 + r) * ldl;
+        for (int k = tid; k < s.dtp; k += SR_T) sdt[r * s.dtp + k] = on ? __ldcg(src + k) : 0.0f;
+        for (int k = tid; k < 2 * NP; k += SR_T) {
+            const int which = k / NP, n = k - which * NP;
+            sbc[r * 2 * NP + k] = on && n < s.N ? __ldcg(src + s.dtp + which * s.N + n) : 0.0f;
+        }
+    }
+    Quad S[R][NC];
+    float xv[R], z[R];
+#pragma unroll
+    for (int r = 0; r < R; r++) {
 #pragma unroll
         for (int i = 0; i < NC; i++)
-            S[r][i] = old && q + 4 * i < quads ? __ldcg(reinterpret_cast<const float4 *>(state + at[r]) + q + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
-        xv[r] = on ? pg_get(x + (int64_t)m * ldx + c) : 0.0f;
-        z[r] = on ? __ldcg(proj + (int64_t)m * ldp + s.inner + c) : 0.0f;
-    }
-    for (int i = tid; i < R * s.dtp; i += SR_T) {
-        const int r = i / s.dtp, k = i - r * s.dtp;
-        sdt[i] = m0 + r < bt.rows ? __ldcg(low + (int64_t)(m0 + r) * ldl + k) : 0.0f;
-    }
-    for (int i = tid; i < R * 2 * NP; i += SR_T) {
-        const int r = i / (2 * NP), k = i - r * 2 * NP, which = k / NP, n = k - which * NP;
-        sbc[i] = m0 + r < bt.rows && n < s.N ? __ldcg(low + (int64_t)(m0 + r) * ldl + s.dtp + which * s.N + n) : 0.0f;
+            S[r][i] = quad(old[r] && q + 4 * i < quads ? __ldcg(reinterpret_cast<const float4 *>(state + at[r]) + q + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f));
+        xv[r] = at[r] >= 0 ? pg_get(x + (int64_t)(m0 + r) * ldx + c) : 0.0f;
+        z[r] = at[r] >= 0 ? __ldcg(proj + (int64_t)(m0 + r) * ldp + s.inner + c) : 0.0f;
     }
     __syncthreads();
     float acc[R] = {};
-    if (live) {
-        const uint4 *w = reinterpret_cast<const uint4 *>(s.dt + (int64_t)c * s.dtp) + q;
-#pragma unroll 2
-        for (int k = 0; k < s.dtp / 32; k++) {
-            const uint4 b = __ldg(w + 4 * k);
+    auto dot = [&](const uint4 &b, int k) {
 #pragma unroll
-            for (int r = 0; r < R; r++) {
-                const float4 *v = reinterpret_cast<const float4 *>(sdt + r * s.dtp + k * 32 + q * 8);
-                const float4 u0 = v[0], u1 = v[1];
-                acc[r] += (fmaf(pg_bf16_lo(b.x), u0.x, pg_bf16_hi(b.x) * u0.y) + fmaf(pg_bf16_lo(b.y), u0.z, pg_bf16_hi(b.y) * u0.w)) +
-                          (fmaf(pg_bf16_lo(b.z), u1.x, pg_bf16_hi(b.z) * u1.y) + fmaf(pg_bf16_lo(b.w), u1.z, pg_bf16_hi(b.w) * u1.w));
-            }
+        for (int r = 0; r < R; r++) {
+            const float4 *v = reinterpret_cast<const float4 *>(sdt + r * s.dtp + k * 32 + q * 8);
+            const float4 u0 = v[0], u1 = v[1];
+            acc[r] += (fmaf(pg_bf16_lo(b.x), u0.x, pg_bf16_hi(b.x) * u0.y) + fmaf(pg_bf16_lo(b.y), u0.z, pg_bf16_hi(b.y) * u0.w)) +
+                      (fmaf(pg_bf16_lo(b.z), u1.x, pg_bf16_hi(b.z) * u1.y) + fmaf(pg_bf16_lo(b.w), u1.z, pg_bf16_hi(b.w) * u1.w));
         }
-    }
+    };
+#pragma unroll
+    for (int k = 0; k < SS_W; k++)
+        if (k < pieces) dot(w[k], k);
+    for (int k = SS_W; k < pieces; k++) dot(__ldg(wrow + 4 * k), k);
 #pragma unroll
     for (int r = 0; r < R; r++) {
         acc[r] += __shfl_xor_sync(0xffffffffu, acc[r], 1);
@@ -199,9 +273,9 @@ __global__ void __launch_bounds__(SR_T)
         float y = 0.0f;
 #pragma unroll
         for (int i = 0; i < NC; i++) {
-            const float4 *b = reinterpret_cast<const float4 *>(sbc + r * 2 * NP) + q + 4 * i;
-            y += update(S[r][i], a[i], dt, du, b[0], b[NP / 4]);
-            if (at[r] >= 0 && q + 4 * i < quads) reinterpret_cast<float4 *>(state + at[r])[q + 4 * i] = S[r][i];
+            const float *b = sbc + r * 2 * NP + (q + 4 * i) * 4;
+            y += sum2(update(S[r][i], a[i], pair(dt, dt), pair(du, du), load_quad(b), load_quad(b + NP)));
+            if (at[r] >= 0 && q + 4 * i < quads) reinterpret_cast<float4 *>(state + at[r])[q + 4 * i] = quad4(S[r][i]);
         }
         y += __shfl_xor_sync(0xffffffffu, y, 1);
         y += __shfl_xor_sync(0xffffffffu, y, 2);
@@ -209,102 +283,133 @@ __global__ void __launch_bounds__(SR_T)
     }
 }
 
-// grid (ceil(inner / 32), seqs)
-constexpr int SR_TOKENS = 16;
+// grid (ceil(inner / 32), seqs), eight warps.  Tiles of TT tokens, two buffers: while warps 0 .. 3 run tile i through the
+// states, warps 4 .. 7 finish the outputs of tile i - 1, turn the raw step sizes of tile i + 1 into what the recurrence
+// takes, and ask for the inputs of tile i + 2.
 template <int NC, typename TA>
-__global__ void __launch_bounds__(SR_T)
+__global__ void __launch_bounds__(2 * SR_T)
     scan_run_kernel(const ScanShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, float *ring, const TA *__restrict__ x, int64_t ldx,
                     const float *__restrict__ dt, int64_t ldt, const float *__restrict__ bc, int64_t ldb, float *state, TA *__restrict__ out, int64_t ldo)
 {
-    constexpr int NP = 16 * NC, TT = SR_TOKENS, PER = TT * SR_CH / SR_T, PERB = TT * 2 * NP / SR_T;
-    __shared__ __align__(16) float sdt[TT][SR_CH], sdu[TT][SR_CH], sy[TT][SR_CH];
-    __shared__ __align__(16) float sbc[TT][2][NP];
+    constexpr int NP = 16 * NC, TT = NC > 4 ? 4 : 16, PER = TT * SR_CH / SR_T, PERB = TT * 2 * NP / SR_T;
+    __shared__ __align__(16) float4 sd[2][TT][SR_CH];      // dt, dt, dt x, dt x
+    __shared__ __align__(16) float sbc[2][TT][2][NP];
+    __shared__ float sy[2][TT][SR_CH];
     pg_pdl_begin();
-    const int tid = threadIdx.x, q = tid & 3, cl = tid >> 2, c0 = blockIdx.x * SR_CH, c = c0 + cl;
+    const bool aux = threadIdx.x >= SR_T;
+    const int tid = threadIdx.x & (SR_T - 1), c0 = blockIdx.x * SR_CH;
     const int seq = blockIdx.y, row0 = __ldcg(bt.d_seq_row0 + seq), T = __ldcg(bt.d_seq_row0 + seq + 1) - row0;
     if (T <= 0) return;
-    const int pos0 = __ldcg(bt.d_pos + row0), quads = s.ss / 4;
+    const int pos0 = __ldcg(bt.d_pos + row0), tiles = (T + TT - 1) / TT;
     const int64_t slot = __ldcg(bt.d_seq_slot + seq);
+    if (aux) {
+        // tokens tid / 32 + 4 i of channel tid % 32
+        const int ec = c0 + (tid & 31), et = tid >> 5;
+        const bool on = ec < s.inner;
+        const float dt_bias = on ? __ldg(s.dt_bias + ec) : 0.0f, skip = on ? __ldg(s.d + ec) : 0.0f;
+        float rdt[PER], rx[PER], rz[PER], rbc[PERB], x1[PER], z1[PER], x2[PER], z2[PER];
+        // (a tile's B and C lie in a fixed order of tokens and states: element tid + i SR_T)
+        auto fetch = [&](int t0) {
+#pragma unroll
+            for (int i = 0; i < PER; i++) {
+                const int t = t0 + et + i * (SR_T / 32);
+                const bool in = on && t < T;
+                const int64_t m = row0 + t;
+                rdt[i] = in ? __ldcg(dt + m * ldt + ec) : 0.0f;
+                rx[i] = in ? pg_get(x + m * ldx + ec) : 0.0f;
+                rz[i] = in ? __ldcg(proj + m * ldp + s.inner + ec) : 0.0f;
+            }
+#pragma unroll
+            for (int i = 0; i < PERB; i++) {
+                const int e = tid + i * SR_T, t = t0 + e / (2 * NP), k = e % (2 * NP), which = k / NP, n = k - which * NP;
+                rbc[i] = t < T && n < s.N ? __ldcg(bc + (int64_t)(row0 + t) * ldb + which * s.N + n) : 0.0f;
+            }
+        };
+        auto convert = [&](int tile) {
+            const int b = tile & 1;
+#pragma unroll
+            for (int i = 0; i < PER; i++) {
+                const int t = et + i * (SR_T / 32);
+                // (tokens behind the end leave the state alone: exp(0) S + 0)
+                const float d = on && tile * TT + t < T ? softplus(rdt[i] + dt_bias) : 0.0f, u = d * rx[i];
+                sd[b][t][tid & 31] = make_float4(d, d, u, u);
+                x2[i] = rx[i];
+                z2[i] = rz[i];
+            }
+#pragma unroll
+            for (int i = 0; i < PERB; i++) (&sbc[b][0][0][0])[tid + i * SR_T] = rbc[i];
+        };
+        auto finish = [&](int tile) {
+#pragma unroll
+            for (int i = 0; i < PER; i++) {
+                const int t = et + i * (SR_T / 32);
+                if (on && tile * TT + t < T)
+                    pg_put(out + (int64_t)(row0 + tile * TT + t) * ldo + ec, fmaf(skip, x1[i], sy[tile & 1][t][tid & 31]) * pg_silu(z1[i]));
+            }
+        };
+        auto shift = [&]() {
+#pragma unroll
+            for (int i = 0; i < PER; i++) x1[i] = x2[i], z1[i] = z2[i];
+        };
+        fetch(0);
+        convert(0);
+        fetch(TT);
+        for (int i = 0; i < tiles; i++) {
+            __syncthreads();                              // tile i may be run; tile i - 1 has been
+            if (i > 0) finish(i - 1);
+            shift();
+            if (i + 1 < tiles) {
+                convert(i + 1);
+                fetch((i + 2) * TT);
+            }
+        }
+        __syncthreads();
+        finish(tiles - 1);
+        // the inputs that the next portion's convolution reads (scan_conv_kernel is done with the old ones)
+        if (on)
+            for (int t = max(0, T - s.taps) + et; t < T; t += SR_T / 32)
+                ring[(slot * s.taps + (pos0 + t) % s.taps) * s.inner + ec] = __ldcg(proj + (int64_t)(row0 + t) * ldp + ec);
+        return;
+    }
+    const int q = tid & 3, cl = tid >> 2, c = c0 + cl, quads = s.ss / 4;
     const bool live = c < s.inner;
     float4 *st = reinterpret_cast<float4 *>(state + (slot * s.inner + c) * s.ss);
-    float4 a[NC], S[NC];
+    Quad a[NC], S[NC];
 #pragma unroll
     for (int i = 0; i < NC; i++) {
         const bool on = live && q + 4 * i < quads;
-        a[i] = on ? __ldg(reinterpret_cast<const float4 *>(s.a + (int64_t)c * s.ss) + q + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
-        S[i] = on && pos0 > 0 ? __ldcg(st + q + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        a[i] = quad(on ? __ldg(reinterpret_cast<const float4 *>(s.a + (int64_t)c * s.ss) + q + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f));
+        S[i] = quad(on && pos0 > 0 ? __ldcg(st + q + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f));
     }
-    // elements of a tile that this thread brings and finishes: tokens tid / 32 + 4 i of channel tid % 32
-    const int ec = c0 + (tid & 31), et = tid >> 5;
-    const bool elive = ec < s.inner;
-    const float dt_bias = elive ? __ldg(s.dt_bias + ec) : 0.0f, skip = elive ? __ldg(s.d + ec) : 0.0f;
-    float rdt[PER], rx[PER], rz[PER], rbc[PERB];
-    auto fetch = [&](int t0) {
-#pragma unroll
-        for (int i = 0; i < PER; i++) {
-            const int t = t0 + et + i * (SR_T / 32);
-            const bool on = elive && t < T;
-            const int64_t m = row0 + t;
-            rdt[i] = on ? __ldcg(dt + m * ldt + ec) : 0.0f;
-            rx[i] = on ? pg_get(x + m * ldx + ec) : 0.0f;
-            rz[i] = on ? __ldcg(proj + m * ldp + s.inner + ec) : 0.0f;
-        }
-#pragma unroll
-        for (int i = 0; i < PERB; i++) {
-            const int e = tid + i * SR_T, t = t0 + e / (2 * NP), k = e % (2 * NP), which = k / NP, n = k - which * NP;
-            rbc[i] = t < T && n < s.N ? __ldcg(bc + (int64_t)(row0 + t) * ldb + which * s.N + n) : 0.0f;
-        }
-    };
-    fetch(0);
-    for (int t0 = 0; t0 < T; t0 += TT) {
-        float kx[PER], kz[PER];
-#pragma unroll
-        for (int i = 0; i < PER; i++) {
-            const int t = et + i * (SR_T / 32);
-            // (tokens behind the end leave the state alone: exp(0) S + 0)
-            const float d = elive && t0 + t < T ? softplus(rdt[i] + dt_bias) : 0.0f;
-            sdt[t][tid & 31] = d;
-            sdu[t][tid & 31] = d * rx[i];
-            kx[i] = rx[i];
-            kz[i] = rz[i];
-        }
-#pragma unroll
-        for (int i = 0; i < PERB; i++) (&sbc[0][0][0])[tid + i * SR_T] = rbc[i];
+    for (int i = 0; i < tiles; i++) {
         __syncthreads();
-        if (t0 + TT < T) fetch(t0 + TT);
+        const int b = i & 1;
 #pragma unroll
         for (int t = 0; t < TT; t += 4) {
             float y[4];
 #pragma unroll
             for (int u = 0; u < 4; u++) {
-                const float d = sdt[t + u][cl], du = sdu[t + u][cl];
-                y[u] = 0.0f;
+                const Quad d = load_quad(reinterpret_cast<const float *>(&sd[b][t + u][cl]));
+                f32x2 part = 0;
 #pragma unroll
-                for (int i = 0; i < NC; i++)
-                    y[u] += update(S[i], a[i], d, du, reinterpret_cast<const float4 *>(sbc[t + u][0])[q + 4 * i],
-                                   reinterpret_cast<const float4 *>(sbc[t + u][1])[q + 4 * i]);
+                for (int n = 0; n < NC; n++) {
+                    const f32x2 v = update(S[n], a[n], d.lo, d.hi, load_quad(&sbc[b][t + u][0][(q + 4 * n) * 4]), load_quad(&sbc[b][t + u][1][(q + 4 * n) * 4]));
+                    part = n == 0 ? v : fma2(pair(1.0f, 1.0f), v, part);
+                }
+                y[u] = sum2(part);
             }
             // four tokens' sums over four lanes: lane q ends with token q's
             const bool odd = q & 1, up = q & 2;
             const float g0 = __shfl_xor_sync(0xffffffffu, odd ? y[0] : y[1], 1), g1 = __shfl_xor_sync(0xffffffffu, odd ? y[2] : y[3], 1);
             const float k0 = (odd ? y[1] : y[0]) + g0, k1 = (odd ? y[3] : y[2]) + g1;
             const float g2 = __shfl_xor_sync(0xffffffffu, up ? k0 : k1, 2);
-            sy[t + q][cl] = (up ? k1 : k0) + g2;
-        }
-        __syncthreads();
-#pragma unroll
-        for (int i = 0; i < PER; i++) {
-            const int t = et + i * (SR_T / 32);
-            if (elive && t0 + t < T) pg_put(out + (int64_t)(row0 + t0 + t) * ldo + ec, fmaf(skip, kx[i], sy[t][tid & 31]) * pg_silu(kz[i]));
+            sy[b][t + q][cl] = (up ? k1 : k0) + g2;
         }
     }
+    __syncthreads();
 #pragma unroll
     for (int i = 0; i < NC; i++)
-        if (live && q + 4 * i < quads) st[q + 4 * i] = S[i];
-    // the inputs that the next portion's convolution reads (scan_conv_kernel is done with the old ones)
-    if (elive)
-        for (int t = max(0, T - s.taps) + et; t < T; t += SR_T / 32)
-            ring[(slot * s.taps + (pos0 + t) % s.taps) * s.inner + ec] = __ldcg(proj + (int64_t)(row0 + t) * ldp + ec);
+        if (live && q + 4 * i < quads) st[q + 4 * i] = quad4(S[i]);
 }
 
 ScanShape shape_of(const pg_scan *p)
@@ -362,7 +467,7 @@ int32_t run_scan(pg_ctx *ctx, const ScanShape &s, const pg_batch *bt, const floa
                  int64_t ldt, const float *bc, int64_t ldb, float *state, TA *out, int64_t ldo)
 {
     const dim3 grid((unsigned)((s.inner + SR_CH - 1) / SR_CH), (unsigned)bt->seqs);
-#define PG_SR(NC) return launch_whole(ctx, scan_run_kernel<NC, TA>, grid, dim3(SR_T), 0, s, *bt, proj, ldp, ring, x, ldx, dt, ldt, bc, ldb, state, out, ldo)
+#define PG_SR(NC) return launch_whole(ctx, scan_run_kernel<NC, TA>, grid, dim3(2 * SR_T), 0, s, *bt, proj, ldp, ring, x, ldx, dt, ldt, bc, ldb, state, out, ldo)
     if (s.N <= 16) PG_SR(1);
     if (s.N <= 32) PG_SR(2);
     if (s.N <= 64) PG_SR(4);
