@@ -615,11 +615,15 @@ __global__ void __launch_bounds__(AS_WARPS * 32)
         const int h = x / vq, c = (x - h * vq) * 4;
         const float *at = parts + (size_t)h * ms + c;
         float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 16
-        for (int k = 0; k < used; k++) {
-            const float4 v = __ldcg(reinterpret_cast<const float4 *>(at + (size_t)k * 16 * ms));
-            const float f = weight[h][k];
-            a.x = fmaf(f, v.x, a.x), a.y = fmaf(f, v.y, a.y), a.z = fmaf(f, v.z, a.z), a.w = fmaf(f, v.w, a.w);
+        for (int k0 = 0; k0 < used; k0 += 8) {            // eight loads in flight; behind the last slice its weight is 0
+            float4 v[8];
+#pragma unroll
+            for (int k = 0; k < 8; k++) v[k] = __ldcg(reinterpret_cast<const float4 *>(at + (size_t)min(k0 + k, used - 1) * 16 * ms));
+#pragma unroll
+            for (int k = 0; k < 8; k++) {
+                const float f = k0 + k < used ? weight[h][k0 + k] : 0.0f;
+                a.x = fmaf(f, v[k].x, a.x), a.y = fmaf(f, v[k].y, a.y), a.z = fmaf(f, v[k].z, a.z), a.w = fmaf(f, v[k].w, a.w);
+            }
         }
         bf16 *dst = out + (int64_t)b * ldo + (int64_t)(h0 + h) * s.V + c;
         const float f = denom[h], y[4] = {a.x * f, a.y * f, a.z * f, a.w * f};

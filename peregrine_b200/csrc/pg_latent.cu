@@ -106,9 +106,9 @@ struct Weights8 {
             pg_mma_bf16(d, lo.x, hi.x, lo.y, hi.y, v.x, v.y);
             pg_mma_bf16(e, lo.z, hi.z, lo.w, hi.w, v.z, v.w);
         };
+        // (all in one stretch: behind the last piece the weights are zero)
 #pragma unroll
-        for (int i = 0; i < PRE; i++)
-            if (i < pieces) step(x[i], i);
+        for (int i = 0; i < PRE; i++) step(x[i], i < pieces ? i : 0);
         for (int i = PRE; i < pieces; i++) step(__ldg(at + 4 * i), i);
 #pragma unroll
         for (int i = 0; i < 4; i++) d[i] += e[i];
@@ -190,14 +190,15 @@ __device__ __forceinline__ int64_t first_tile(const LatentShape &s, int row0, in
 
 constexpr int LA_KEYS = 64;
 constexpr int LA_PS = LA_KEYS + 8;      // row stride of the weights in shared memory
-constexpr int LA_QSTEPS = 18;           // 16-column steps of half a key that a warp's query fragments cover (ck up to 576)
 
 // grid (slices, row tiles, seqs), 8 RT warps.  A warp has 16 keys of a tile, 16 rows and half of the key's columns for the
 // scores -- two warps exchange their halves' sums, and each goes on with eight keys -- and 64 / RT columns of all rows for the
-// sums.  QREG: the warp's part of the queries stays in registers.
+// sums.  KS: 16-column steps of half a key; the warp's part of the queries stays in registers (KS = 0: any number, queries from
+// shared memory).  The unrolled loops have no branches: behind the true width they repeat a step with zero queries, or make
+// columns that nobody reads.
 // Shared memory: ring of `stages` tiles of keys [64][ck + 8] | queries [16 RT][ck + 8] | weights [16 RT][LA_PS] | halves' sums
 // [8 RT warps][32 lanes][4].  part [tile][slice][16 RT][cp + 4]: sums, then maximum (log 2 units) and denominator of each row.
-template <int RT, bool QREG>
+template <int RT, int KS>
 __global__ void __launch_bounds__(RT * 256, 1)
     latent_attn_kernel(const LatentShape s, const pg_batch bt, const bf16 *__restrict__ qx, const bf16 *__restrict__ cache, float *__restrict__ part, int per_seq,
                        int stages, int32_t *status, unsigned long long limit_ns)
@@ -251,11 +252,11 @@ __global__ void __launch_bounds__(RT * 256, 1)
     const int steps = s.ck / 16, half = (steps + 1) / 2, s0 = kh * half, sn = min(half, steps - s0);   // this warp's steps of the columns
     const uint32_t q_at = qs + (uint32_t)((rt * 16 + (lane & 15)) * stride + (lane >> 4) * 16 + s0 * 32);
     const uint32_t k_at = (uint32_t)((kq * 16 + (lane & 7) + ((lane >> 4) << 3)) * stride + ((lane >> 3) & 1) * 16 + s0 * 32);
-    uint32_t qf[QREG ? LA_QSTEPS : 1][4];
-    if (QREG) {
+    uint32_t qf[KS ? KS : 1][4];
 #pragma unroll
-        for (int i = 0; i < LA_QSTEPS; i++)
-            if (i < sn) pg_ldsm4(qf[QREG ? i : 0], q_at + i * 32);
+    for (int i = 0; i < KS; i++) {
+        qf[i][0] = qf[i][1] = qf[i][2] = qf[i][3] = 0u;
+        if (i < sn) pg_ldsm4(qf[i], q_at + i * 32);
     }
     const int cw = ((s.cp + NW - 1) / NW + 15) & ~15, c0 = warp * cw, nv = max(0, min(cw, s.cp - c0)) / 8;   // this warp's columns of the sums
     const int lim0 = pos0 + min(rr0 + rt * 16 + r, total - 1) / s.H, lim1 = pos0 + min(rr0 + rt * 16 + r + 8, total - 1) / s.H;
@@ -276,15 +277,13 @@ __global__ void __launch_bounds__(RT * 256, 1)
         ok = pg_mbar_wait(bar + (uint32_t)(it % stages) * 8, (uint32_t)(it / stages) & 1u, &abort_flag, status, limit_ns);
         const uint32_t kt = ring + (uint32_t)(it % stages) * stage;
         float sc[2][4] = {};
-        if (QREG) {
+        if (KS) {
 #pragma unroll
-            for (int i = 0; i < LA_QSTEPS; i++) {
-                if (i < sn) {
-                    uint32_t b[4];
-                    pg_ldsm4(b, kt + k_at + i * 32);
-                    pg_mma_bf16(sc[0], qf[QREG ? i : 0][0], qf[QREG ? i : 0][1], qf[QREG ? i : 0][2], qf[QREG ? i : 0][3], b[0], b[1]);
-                    pg_mma_bf16(sc[1], qf[QREG ? i : 0][0], qf[QREG ? i : 0][1], qf[QREG ? i : 0][2], qf[QREG ? i : 0][3], b[2], b[3]);
-                }
+            for (int i = 0; i < KS; i++) {
+                uint32_t b[4];
+                pg_ldsm4(b, kt + k_at + (i < sn ? i : 0) * 32);
+                pg_mma_bf16(sc[0], qf[i][0], qf[i][1], qf[i][2], qf[i][3], b[0], b[1]);
+                pg_mma_bf16(sc[1], qf[i][0], qf[i][1], qf[i][2], qf[i][3], b[2], b[3]);
             }
         } else {
             for (int i = 0; i < sn; i++) {
@@ -352,6 +351,7 @@ __global__ void __launch_bounds__(RT * 256, 1)
             asm volatile("st.shared.u32 [%0], %1;" ::"r"(at + 8 * LA_PS * 2), "r"(pg_pack_bf16(p2, p3)) : "memory");
         }
         __syncthreads();                                  // the weights are there
+        if (nv == 0) continue;
         if (__any_sync(0xffffffffu, moved)) {
 #pragma unroll
             for (int x = 0; x < RT; x++)
@@ -370,14 +370,12 @@ __global__ void __launch_bounds__(RT * 256, 1)
             for (int x = 0; x < RT; x++) pg_ldsm4(a[x], ps + (uint32_t)((x * 16 + (lane & 15)) * LA_PS + kk * 16 + (lane >> 4) * 8) * 2);
 #pragma unroll
             for (int i = 0; i < VT; i += 2) {
-                if (i < nv) {
-                    uint32_t b[4];
-                    pg_ldsm4_t(b, kt + v_at + (uint32_t)(kk * 16 * stride + i * 16));
+                uint32_t b[4];
+                pg_ldsm4_t(b, kt + v_at + (uint32_t)(kk * 16 * stride + (i < nv ? i : 0) * 16));
 #pragma unroll
-                    for (int x = 0; x < RT; x++) {
-                        pg_mma_bf16(o[x][i], a[x][0], a[x][1], a[x][2], a[x][3], b[0], b[1]);
-                        pg_mma_bf16(o[x][i + 1], a[x][0], a[x][1], a[x][2], a[x][3], b[2], b[3]);
-                    }
+                for (int x = 0; x < RT; x++) {
+                    pg_mma_bf16(o[x][i], a[x][0], a[x][1], a[x][2], a[x][3], b[0], b[1]);
+                    pg_mma_bf16(o[x][i + 1], a[x][0], a[x][1], a[x][2], a[x][3], b[2], b[3]);
                 }
             }
         }
@@ -476,11 +474,15 @@ __global__ void __launch_bounds__(LV_T)
         const int x = i / quads, k4 = (i - x * quads) * 4, n = used[x];
         float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
         const float *src = part + (n ? base[x] : 0) + k4;
-#pragma unroll 12
-        for (int k = 0; k < n; k++) {
-            const float4 v = __ldcg(reinterpret_cast<const float4 *>(src + (int64_t)k * rows * ms));
-            const float f = weight[x][k];
-            a.x = fmaf(f, v.x, a.x), a.y = fmaf(f, v.y, a.y), a.z = fmaf(f, v.z, a.z), a.w = fmaf(f, v.w, a.w);
+        for (int k0 = 0; k0 < n; k0 += 12) {              // twelve loads in flight; behind the last slice its weight is 0
+            float4 v[12];
+#pragma unroll
+            for (int k = 0; k < 12; k++) v[k] = __ldcg(reinterpret_cast<const float4 *>(src + (int64_t)min(k0 + k, n - 1) * rows * ms));
+#pragma unroll
+            for (int k = 0; k < 12; k++) {
+                const float f = k0 + k < n ? weight[x][k0 + k] : 0.0f;
+                a.x = fmaf(f, v[k].x, a.x), a.y = fmaf(f, v[k].y, a.y), a.z = fmaf(f, v[k].z, a.z), a.w = fmaf(f, v[k].w, a.w);
+            }
         }
         *reinterpret_cast<uint2 *>(sa + x * ld + k4) = make_uint2(pg_pack_bf16(a.x, a.y), pg_pack_bf16(a.z, a.w));
     }
@@ -624,8 +626,12 @@ int32_t launch_attn(pg_ctx *ctx, const LatentShape &s, const pg_batch *batch, di
         return launch_pdl(ctx, kern, grid, dim3(RT * 256), (size_t)attn_smem(s, stages), s, *batch, q, cache, part, per_seq, stages, ctx->d_status,
                           ctx->wait_limit_ns);
     };
-    static std::atomic<uint64_t> set[2] = {};
-    return s.ck <= LA_QSTEPS * 32 ? go(latent_attn_kernel<RT, true>, set[0]) : go(latent_attn_kernel<RT, false>, set[1]);
+    static std::atomic<uint64_t> set[5] = {};
+    if (s.ck <= 96) return go(latent_attn_kernel<RT, 3>, set[0]);
+    if (s.ck <= 160) return go(latent_attn_kernel<RT, 5>, set[1]);
+    if (s.ck <= 320) return go(latent_attn_kernel<RT, 10>, set[2]);
+    if (s.ck <= 576) return go(latent_attn_kernel<RT, 18>, set[3]);
+    return go(latent_attn_kernel<RT, 0>, set[4]);
 }
 
 int32_t check(const pg_latent *p, const pg_batch *batch, int64_t ldp, int64_t ldo)

@@ -261,9 +261,9 @@ __global__ void __launch_bounds__(SR_T)
                       (fmaf(pg_bf16_lo(b.z), u1.x, pg_bf16_hi(b.z) * u1.y) + fmaf(pg_bf16_lo(b.w), u1.z, pg_bf16_hi(b.w) * u1.w));
         }
     };
+    // (all in one stretch: behind the rank's last piece the weights are zero)
 #pragma unroll
-    for (int k = 0; k < SS_W; k++)
-        if (k < pieces) dot(w[k], k);
+    for (int k = 0; k < SS_W; k++) dot(w[k], k < pieces ? k : 0);
     for (int k = SS_W; k < pieces; k++) dot(__ldg(wrow + 4 * k), k);
 #pragma unroll
     for (int r = 0; r < R; r++) {
@@ -282,6 +282,22 @@ __global__ void __launch_bounds__(SR_T)
         if (q == 0 && at[r] >= 0) pg_put(out + (int64_t)(m0 + r) * ldo + c, fmaf(skip, xv[r], y) * pg_silu(z[r]));
     }
 }
+
+// an element of a step's type before its conversion
+template <typename TA>
+struct Raw;
+template <>
+struct Raw<float> {
+    float v;
+    __device__ __forceinline__ void load(const float *p, bool in) { v = in ? __ldcg(p) : 0.0f; }
+    __device__ __forceinline__ float value() const { return v; }
+};
+template <>
+struct Raw<bf16> {
+    unsigned short v;
+    __device__ __forceinline__ void load(const bf16 *p, bool in) { v = in ? __ldcg(reinterpret_cast<const unsigned short *>(p)) : (unsigned short)0; }
+    __device__ __forceinline__ float value() const { return __uint_as_float((uint32_t)v << 16); }
+};
 
 // grid (ceil(inner / 32), seqs), eight warps.  Tiles of TT tokens, two buffers: while warps 0 .. 3 run tile i through the
 // states, warps 4 .. 7 finish the outputs of tile i - 1, turn the raw step sizes of tile i + 1 into what the recurrence
@@ -307,7 +323,8 @@ __global__ void __launch_bounds__(2 * SR_T)
         const int ec = c0 + (tid & 31), et = tid >> 5;
         const bool on = ec < s.inner;
         const float dt_bias = on ? __ldg(s.dt_bias + ec) : 0.0f, skip = on ? __ldg(s.d + ec) : 0.0f;
-        float rdt[PER], rx[PER], rz[PER], rbc[PERB], x1[PER], z1[PER], x2[PER], z2[PER];
+        float rdt[PER], rz[PER], rbc[PERB], x1[PER], z1[PER], x2[PER], z2[PER];
+        Raw<TA> rx[PER];                                  // (as loaded: nothing waits for a load before its tile is converted)
         // (a tile's B and C lie in a fixed order of tokens and states: element tid + i SR_T)
         auto fetch = [&](int t0) {
 #pragma unroll
@@ -316,7 +333,7 @@ __global__ void __launch_bounds__(2 * SR_T)
                 const bool in = on && t < T;
                 const int64_t m = row0 + t;
                 rdt[i] = in ? __ldcg(dt + m * ldt + ec) : 0.0f;
-                rx[i] = in ? pg_get(x + m * ldx + ec) : 0.0f;
+                rx[i].load(x + m * ldx + ec, in);
                 rz[i] = in ? __ldcg(proj + m * ldp + s.inner + ec) : 0.0f;
             }
 #pragma unroll
@@ -331,9 +348,9 @@ __global__ void __launch_bounds__(2 * SR_T)
             for (int i = 0; i < PER; i++) {
                 const int t = et + i * (SR_T / 32);
                 // (tokens behind the end leave the state alone: exp(0) S + 0)
-                const float d = on && tile * TT + t < T ? softplus(rdt[i] + dt_bias) : 0.0f, u = d * rx[i];
+                const float d = on && tile * TT + t < T ? softplus(rdt[i] + dt_bias) : 0.0f, xi = rx[i].value(), u = d * xi;
                 sd[b][t][tid & 31] = make_float4(d, d, u, u);
-                x2[i] = rx[i];
+                x2[i] = xi;
                 z2[i] = rz[i];
             }
 #pragma unroll
