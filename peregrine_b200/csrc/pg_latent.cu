@@ -5,8 +5,8 @@
 // W_uv (sum p c): attention of all heads over one key of kv_rank + rot_dim, whose first kv_rank columns are the value.
 //
 //   bf16, short      latent_query_kernel   q' per head on mma.sync, the queries' rotation, and the new positions' cache rows
-//                    latent_attn_kernel    a CTA has a slice of the context and 16 or 32 (token, head) rows, which share the
-//                                          keys; the warps divide keys and columns between them
+//                    latent_attn_kernel    a CTA has a slice of the context and 32 (token, head) rows, which share the keys;
+//                                          both products on the 5th-generation tensor cores
 //                    latent_value_kernel   adds up the slices, W_uv per head on mma.sync, output gate
 //   bf16, longer     latent_prep_kernel (rotation, cache rows); then the caller unfolds keys and values of the whole context
 //                    by a product, and the tcgen05 kernel of csrc/pg_attention_tc.cu reads them
@@ -17,8 +17,8 @@
 
 #include <algorithm>
 
-#include "pg_async.cuh"
 #include "pg_attention.cuh"
+#include "pg_tcgen05.cuh"
 
 namespace {
 
@@ -121,40 +121,62 @@ constexpr int LQ_T = 256;
 __global__ void __launch_bounds__(LQ_T)
     latent_query_kernel(const LatentShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, bf16 *__restrict__ qx, bf16 *cache, int32_t *status)
 {
-    constexpr int NW = LQ_T / 32;
+    constexpr int NW = LQ_T / 32, AHEAD = 4;
     extern __shared__ __align__(128) unsigned char smem[];   // [16][dk + 8]
     const int h = blockIdx.x, m0 = blockIdx.z * 16, n = min(16, bt.rows - m0), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int c_step = gridDim.y * NW * 8;
     int c = (blockIdx.y * NW + warp) * 8;
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    // weights and the batch's arrays do not depend on the kernel before
     Weights8<4> w;
     if (h < s.H && c < s.cp) w.ask(s.uk + ((int64_t)h * s.cp + c) * s.dk, s.dk, s.dk, lane);
-    pg_pdl_begin();
+    const int mine = blockIdx.y * NW + warp;                 // the first row that this warp rotates (or appends)
+    const int pos_first = mine < n ? __ldcg(bt.d_pos + m0 + mine) : 0;
     bf16 *sa = reinterpret_cast<bf16 *>(smem);
     const int ld = s.dk + 8;
     if (h == s.H) {
-        for (int i = blockIdx.y * NW + warp; i < n; i += gridDim.y * NW) {
-            const int m = m0 + i, pos = __ldcg(bt.d_pos + m), seq = __ldcg(bt.d_row_seq + m);
-            if (seq_len(bt, seq) >= s.long_from) continue;
+        const int seq_first = mine < n ? __ldcg(bt.d_row_seq + m0 + mine) : 0;
+        const int64_t slot_first = __ldcg(bt.d_seq_slot + seq_first);
+        const bool skip_first = seq_len(bt, seq_first) >= s.long_from;
+        asm volatile("griddepcontrol.wait;" ::: "memory");
+        for (int i = mine; i < n; i += gridDim.y * NW) {
+            const int m = m0 + i, pos = i == mine ? pos_first : __ldcg(bt.d_pos + m), seq = i == mine ? seq_first : __ldcg(bt.d_row_seq + m);
+            if (i == mine ? skip_first : seq_len(bt, seq) >= s.long_from) continue;
             if ((unsigned)pos >= (unsigned)s.cap) {   // outside the cache: record it, touch nothing
                 if (lane == 0) atomicExch(status, (int32_t)PG_ERR_INVALID);
                 continue;
             }
-            append(s, proj + (int64_t)m * ldp + s.at_kv, pos, cache + ((int64_t)__ldcg(bt.d_seq_slot + seq) * s.cap + pos) * s.ck, lane);
+            append(s, proj + (int64_t)m * ldp + s.at_kv, pos, cache + ((i == mine ? slot_first : (int64_t)__ldcg(bt.d_seq_slot + seq)) * s.cap + pos) * s.ck, lane);
         }
         return;
     }
-    for (int i = warp; i < 16; i += NW) {
-        const float *src = proj + (int64_t)(m0 + i) * ldp + h * (s.D + s.R);
-#pragma unroll 4
-        for (int k = lane; k < s.dk; k += 32) sa[i * ld + k] = __float2bfloat16_rn(i < n && k < s.D ? __ldcg(src + k) : 0.0f);
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    // all first loads in flight together: two rows of the unrotated part, one of the rotated
+    const float *src0 = proj + (int64_t)(m0 + warp) * ldp + h * (s.D + s.R), *src1 = src0 + 8 * ldp;
+    float v0[AHEAD], v1[AHEAD];
+#pragma unroll
+    for (int k = 0; k < AHEAD; k++) {
+        v0[k] = warp < n && k * 32 + lane < s.D ? __ldcg(src0 + k * 32 + lane) : 0.0f;
+        v1[k] = warp + 8 < n && k * 32 + lane < s.D ? __ldcg(src1 + k * 32 + lane) : 0.0f;
     }
-    for (int i = blockIdx.y * NW + warp; i < n; i += gridDim.y * NW) {
-        const int m = m0 + i, pos = __ldcg(bt.d_pos + m);
+    for (int i = mine; i < n; i += gridDim.y * NW) {
+        const int m = m0 + i, pos = i == mine ? pos_first : __ldcg(bt.d_pos + m);
         if ((unsigned)pos >= (unsigned)s.cap) {
             if (lane == 0) atomicExch(status, (int32_t)PG_ERR_INVALID);
             continue;
         }
         rotate(s, proj + (int64_t)m * ldp + h * (s.D + s.R) + s.D, pos, qx + ((int64_t)m * s.H + h) * s.ck + s.cp, s.rp, lane);
+    }
+#pragma unroll
+    for (int k = 0; k < AHEAD; k++) {
+        if (k * 32 < s.dk) {
+            sa[warp * ld + k * 32 + lane] = __float2bfloat16_rn(v0[k]);
+            sa[(warp + 8) * ld + k * 32 + lane] = __float2bfloat16_rn(v1[k]);
+        }
+    }
+    for (int k = AHEAD * 32 + lane; k < s.dk; k += 32) {
+        sa[warp * ld + k] = __float2bfloat16_rn(warp < n && k < s.D ? __ldcg(src0 + k) : 0.0f);
+        sa[(warp + 8) * ld + k] = __float2bfloat16_rn(warp + 8 < n && k < s.D ? __ldcg(src1 + k) : 0.0f);
     }
     __syncthreads();
     const int r = lane >> 2, t = lane & 3;
@@ -170,7 +192,7 @@ __global__ void __launch_bounds__(LQ_T)
     }
 }
 
-// The slices of a tile of rows: as many as the launch has, of a multiple of 64 keys each.
+// The slices of a tile of rows: as many as the launch has, of a multiple of 128 keys each.
 struct Slices {
     int kmax, chunk, used;
 };
@@ -178,7 +200,7 @@ __device__ __forceinline__ Slices slices_of(const LatentShape &s, int pos0, int 
 {
     Slices v;
     v.kmax = pos0 + (min((tile + 1) * rows, T * s.H) - 1) / s.H + 1;
-    v.chunk = ((v.kmax + S - 1) / S + 63) & ~63;
+    v.chunk = ((v.kmax + S - 1) / S + 127) & ~127;
     v.used = (v.kmax + v.chunk - 1) / v.chunk;
     return v;
 }
@@ -188,305 +210,329 @@ __device__ __forceinline__ int64_t first_tile(const LatentShape &s, int row0, in
     return per_seq ? (int64_t)seq * per_seq : (int64_t)row0 * s.H / rows + seq;
 }
 
-constexpr int LA_KEYS = 64;
-constexpr int LA_PS = LA_KEYS + 8;      // row stride of the weights in shared memory
-
-// grid (slices, row tiles, seqs), 8 RT warps.  A warp has 16 keys of a tile, 16 rows and half of the key's columns for the
-// scores -- two warps exchange their halves' sums, and each goes on with eight keys -- and 64 / RT columns of all rows for the
-// sums.  KS: 16-column steps of half a key; the warp's part of the queries stays in registers (KS = 0: any number, queries from
-// shared memory).  The unrolled loops have no branches: behind the true width they repeat a step with zero queries, or make
-// columns that nobody reads.
-// Shared memory: ring of `stages` tiles of keys [64][ck + 8] | queries [16 RT][ck + 8] | weights [16 RT][LA_PS] | halves' sums
-// [8 RT warps][32 lanes][4].  part [tile][slice][16 RT][cp + 4]: sums, then maximum (log 2 units) and denominator of each row.
-template <int RT, int KS>
-__global__ void __launch_bounds__(RT * 256, 1)
-    latent_attn_kernel(const LatentShape s, const pg_batch bt, const bf16 *__restrict__ qx, const bf16 *__restrict__ cache, float *__restrict__ part, int per_seq,
-                       int stages, int32_t *status, unsigned long long limit_ns)
+// Whether a condition holds in the first four warps, which all arrive here.
+__device__ __forceinline__ bool all_four(bool ok)
 {
-    constexpr int NW = 8 * RT, ROWS = 16 * RT, VT = 512 / NW / 8;   // 8-column tiles of a warp (kv_rank up to 512)
-    extern __shared__ __align__(128) unsigned char smem[];
-    __shared__ __align__(8) uint64_t bars[4];
-    __shared__ __align__(16) float red[RT][16][8];
+    uint32_t r;
+    asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.u32 p, %1, 0;\n\tbar.red.and.pred q, 1, 128, p;\n\tselp.u32 %0, 1, 0, q;\n\t}" : "=r"(r) : "r"((uint32_t)ok) : "memory");
+    return r != 0;
+}
+
+constexpr int LA_KEYS = 128, LA_ROWS = 32;
+constexpr int LA_BLOCK = LA_KEYS * 128;                   // bytes of 128 keys x 64 columns
+constexpr int LA_QBLOCK = LA_ROWS * 128;
+constexpr int LA_THREADS = 192;
+
+// grid (slices, tiles of 32 rows, seqs).  Everything stands on its head, so that the many keys and the many columns are the 128
+// rows of the tensor cores' tiles and the 32 (token, head) rows are their columns:
+//   S^T [128 keys x 32] = K Q^T                    K: a tile of keys, [block of 64 columns][128 keys][64], swizzled by the copies
+//   O^T [kv_rank x 32] += V^T P^T                  V: the first kv_rank columns of the same tile, read along its other side
+//   warp 4     TMA: the blocks of a key tile one by one -- those that this step does not write before griddepcontrol.wait --
+//              and the queries; a block is asked for again as soon as the products that read it have run
+//   warp 5     issues the products: S^T block by block as they arrive, O^T by groups of 128 columns
+//   warps 0-3  a thread owns a key (S^T) and a column of every group (O^T).  The rows' maxima over the keys are found by
+//              exchanging halves of the rows between lanes, 31 shuffles for 32 rows; they are only replaced, and O^T rescaled,
+//              when a row falls behind by more than 2^8.
+// Shared memory: key blocks | query blocks [64 columns][32 rows] | P [2][32 rows][64 keys].  TMEM: S^T 32 columns, O^T 32 for each
+// group.  part [tile][slice][32][cp + 4]: sums, then maximum (log 2 units) and denominator of each row.
+__global__ void __launch_bounds__(LA_THREADS, 1)
+    latent_attn_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_q, const LatentShape s, const pg_batch bt,
+                       float *__restrict__ part, int per_seq, int32_t *status, unsigned long long limit_ns)
+{
+    constexpr int MAXB = 10, TMEM_COLS = 256;
+    extern __shared__ uint8_t smem_raw[];
+    __shared__ __align__(8) uint64_t bars[2 * MAXB + 4];
+    __shared__ uint32_t tmem_slot;
     __shared__ volatile int abort_flag;
-    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-    const int split = blockIdx.x, S = gridDim.x, tile = blockIdx.y, seq = blockIdx.z;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane >> 2, t = lane & 3;
-    const int kh = warp & 1, kq = (warp >> 1) & 3, rt = warp >> 3;   // half of the columns, group of keys, row tile
+    __shared__ __align__(16) float red[LA_ROWS][4];          // a row's maximum, or sum, of each warp
+    __shared__ __align__(16) float now[4][LA_ROWS];          // the rows' maxima in use, per warp
+    __shared__ int lims[LA_ROWS];
+    const int nb = (s.ck + 63) / 64, ng = (s.cp + 127) / 128;   // blocks of a key, groups of 128 value columns
+    const uint32_t keys_at = (pg_smem(smem_raw) + 1023u) & ~1023u, q_at = keys_at + nb * LA_BLOCK, p_at = q_at + nb * LA_QBLOCK;
+    const uint32_t bar_full = pg_smem(bars), bar_empty = bar_full + 8 * MAXB, bar_q = bar_empty + 8 * MAXB, bar_s = bar_q + 8, bar_p = bar_s + 8, bar_o = bar_p + 8;
+    const int split = blockIdx.x, S = gridDim.x, tile = blockIdx.y, seq = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    // the batch's arrays do not depend on the kernel before
+    const int row0 = __ldcg(bt.d_seq_row0 + seq), T = seq_len(bt, seq), total = T * s.H, rr0 = tile * LA_ROWS;
+    const int slot = __ldcg(bt.d_seq_slot + seq);
+    if (T >= s.long_from || rr0 >= total) return;
+    const int pos0 = __ldcg(bt.d_pos + row0);
+    const Slices sl = slices_of(s, pos0, T, tile, LA_ROWS, S);
+    const int t0 = split * sl.chunk, t1 = min(sl.kmax, t0 + sl.chunk);
+    if (t0 >= t1 || sl.kmax > s.cap) return;              // (positions outside the cache are recorded by latent_query_kernel)
+    const int ntiles = (t1 - t0 + LA_KEYS - 1) / LA_KEYS;
     if (threadIdx.x == 0) {
-        for (int i = 0; i < 4; i++) pg_mbar_init(pg_smem(bars) + 8 * i, 1);
+        for (int i = 0; i < nb; i++) {
+            pg_mbar_init(bar_full + 8 * i, 1);
+            pg_mbar_init(bar_empty + 8 * i, 1);
+        }
+        pg_mbar_init(bar_q, 1);
+        pg_mbar_init(bar_s, 1);
+        pg_mbar_init(bar_p, 4);                           // one arrival per softmax warp
+        pg_mbar_init(bar_o, 1);
         abort_flag = 0;
         pg_mbar_fence();
     }
-    __syncthreads();
-    asm volatile("griddepcontrol.wait;" ::: "memory");
-    const int row0 = __ldcg(bt.d_seq_row0 + seq), T = seq_len(bt, seq), total = T * s.H, rr0 = tile * ROWS;
-    const int64_t slot = __ldcg(bt.d_seq_slot + seq);
-    if (T >= s.long_from || rr0 >= total) return;
-    const int pos0 = __ldcg(bt.d_pos + row0);
-    const Slices sl = slices_of(s, pos0, T, tile, ROWS, S);
-    const int t0 = split * sl.chunk, t1 = min(sl.kmax, t0 + sl.chunk);
-    if (t0 >= t1 || sl.kmax > s.cap) return;              // (positions outside the cache are recorded by latent_query_kernel)
-    const int stride = s.ck * 2 + 16, stage = LA_KEYS * stride;
-    const uint32_t ring = pg_smem(smem), qs = ring + stages * stage, ps = qs + ROWS * stride, xs = ps + ROWS * LA_PS * 2;
-    const uint32_t bar = pg_smem(bars);
-    const bf16 *keys = cache + slot * (int64_t)s.cap * s.ck;
-    const int ntiles = (t1 - t0 + LA_KEYS - 1) / LA_KEYS;
-    // every warp asks for some of a tile's rows (rows behind the slice repeat its last one and are masked)
-    auto fetch = [&](int i) {
-        const uint32_t at = ring + (uint32_t)(i % stages) * stage, on = bar + (uint32_t)(i % stages) * 8;
-        if (threadIdx.x == 0) pg_mbar_expect(on, (uint32_t)LA_KEYS * s.ck * 2u);
-        if (lane < LA_KEYS / NW) {
-            const int x = warp * (LA_KEYS / NW) + lane;
-            pg_bulk_load(at + (uint32_t)x * stride, keys + (int64_t)min(t0 + i * LA_KEYS + x, t1 - 1) * s.ck, (uint32_t)s.ck * 2u, on);
-        }
-    };
-    for (int i = 0; i < stages && i < ntiles; i++) fetch(i);
-    for (int x = warp; x < ROWS; x += NW) {
-        const bf16 *src = qx + ((int64_t)row0 * s.H + min(rr0 + x, total - 1)) * s.ck;
-        for (int e = lane * 8; e < s.ck; e += 256) pg_cp16(qs + (uint32_t)(x * stride + e * 2), src + e);
+    if (threadIdx.x < LA_ROWS) lims[threadIdx.x] = pos0 + min(rr0 + (int)threadIdx.x, total - 1) / s.H;
+    if (warp == 5) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(pg_smem(&tmem_slot)), "r"(TMEM_COLS) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
-    pg_cp_commit();
-    pg_cp_wait<0>();
+    tc_fence_before();
     __syncthreads();
+    tc_fence_after();
+    // (not before the CTA has its TMEM: nothing behind this kernel can then hold what it needs)
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    const uint32_t tmem_s = tmem_slot, tmem_o = tmem_s + 32;
 
-    const int steps = s.ck / 16, half = (steps + 1) / 2, s0 = kh * half, sn = min(half, steps - s0);   // this warp's steps of the columns
-    const uint32_t q_at = qs + (uint32_t)((rt * 16 + (lane & 15)) * stride + (lane >> 4) * 16 + s0 * 32);
-    const uint32_t k_at = (uint32_t)((kq * 16 + (lane & 7) + ((lane >> 4) << 3)) * stride + ((lane >> 3) & 1) * 16 + s0 * 32);
-    uint32_t qf[KS ? KS : 1][4];
-#pragma unroll
-    for (int i = 0; i < KS; i++) {
-        qf[i][0] = qf[i][1] = qf[i][2] = qf[i][3] = 0u;
-        if (i < sn) pg_ldsm4(qf[i], q_at + i * 32);
-    }
-    const int cw = ((s.cp + NW - 1) / NW + 15) & ~15, c0 = warp * cw, nv = max(0, min(cw, s.cp - c0)) / 8;   // this warp's columns of the sums
-    const int lim0 = pos0 + min(rr0 + rt * 16 + r, total - 1) / s.H, lim1 = pos0 + min(rr0 + rt * 16 + r + 8, total - 1) / s.H;
-    const float scale = s.scale * LOG2E;
-    float o[RT][VT][4], m[RT][2], l0 = 0.0f, l1 = 0.0f;
-#pragma unroll
-    for (int x = 0; x < RT; x++) {
-        m[x][0] = m[x][1] = -1e30f;                       // (finite: a row may see nothing of a slice)
-#pragma unroll
-        for (int i = 0; i < VT; i++)
-#pragma unroll
-            for (int j = 0; j < 4; j++) o[x][i][j] = 0.0f;
-    }
-    const uint32_t v_at = (uint32_t)(((lane & 7) + ((lane >> 3) & 1) * 8) * stride + ((lane >> 4) * 8 + c0) * 2);
-    const uint32_t mine = xs + (uint32_t)(warp * 32 + lane) * 16, theirs = xs + (uint32_t)((warp ^ 1) * 32 + lane) * 16;
-    bool ok = true;
-    for (int it = 0; it < ntiles; it++) {
-        ok = pg_mbar_wait(bar + (uint32_t)(it % stages) * 8, (uint32_t)(it / stages) & 1u, &abort_flag, status, limit_ns);
-        const uint32_t kt = ring + (uint32_t)(it % stages) * stage;
-        float sc[2][4] = {};
-        if (KS) {
-#pragma unroll
-            for (int i = 0; i < KS; i++) {
-                uint32_t b[4];
-                pg_ldsm4(b, kt + k_at + (i < sn ? i : 0) * 32);
-                pg_mma_bf16(sc[0], qf[i][0], qf[i][1], qf[i][2], qf[i][3], b[0], b[1]);
-                pg_mma_bf16(sc[1], qf[i][0], qf[i][1], qf[i][2], qf[i][3], b[2], b[3]);
-            }
-        } else {
-            for (int i = 0; i < sn; i++) {
-                uint32_t a[4], b[4];
-                pg_ldsm4(a, q_at + i * 32);
-                pg_ldsm4(b, kt + k_at + i * 32);
-                pg_mma_bf16(sc[0], a[0], a[1], a[2], a[3], b[0], b[1]);
-                pg_mma_bf16(sc[1], a[0], a[1], a[2], a[3], b[2], b[3]);
-            }
-        }
-        // eight keys each: the other half's sums of them from the neighbour
-        {
-            const float (&give)[4] = kh ? sc[0] : sc[1];
-            asm volatile("st.shared.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(mine), "f"(give[0]), "f"(give[1]), "f"(give[2]), "f"(give[3]) : "memory");
-        }
-        // also: every warp is done with the tile before, so its slot can be filled again
-        if (!__syncthreads_and(ok)) {
-            ok = false;
-            break;
-        }
-        if (it > 0 && it - 1 + stages < ntiles) fetch(it - 1 + stages);
-        float sv[4];
-        {
-            const uint4 g = pg_lds128(theirs);
-            const float got[4] = {__uint_as_float(g.x), __uint_as_float(g.y), __uint_as_float(g.z), __uint_as_float(g.w)};
-            const int j0 = t0 + it * LA_KEYS + kq * 16 + kh * 8 + 2 * t;
-#pragma unroll
-            for (int j = 0; j < 4; j++) {
-                const int key = j0 + (j & 1);
-                const bool in = key < t1 && key <= (j < 2 ? lim0 : lim1);
-                sv[j] = in ? ((kh ? sc[1][j] : sc[0][j]) + got[j]) * scale : -INFINITY;
-            }
-        }
-        float b0 = fmaxf(sv[0], sv[1]), b1 = fmaxf(sv[2], sv[3]);
-#pragma unroll
-        for (int x = 1; x < 4; x <<= 1) {
-            b0 = fmaxf(b0, __shfl_xor_sync(0xffffffffu, b0, x));
-            b1 = fmaxf(b1, __shfl_xor_sync(0xffffffffu, b1, x));
-        }
-        if (t == 0) {
-            red[rt][r][kq * 2 + kh] = b0;
-            red[rt][r + 8][kq * 2 + kh] = b1;
-        }
-        __syncthreads();                                  // the maxima are there
-        float f[RT][2];
-        bool moved = false;
-#pragma unroll
-        for (int x = 0; x < RT; x++)
-#pragma unroll
-            for (int e = 0; e < 2; e++) {
-                const float4 u = *reinterpret_cast<const float4 *>(red[x][r + 8 * e]), v = *reinterpret_cast<const float4 *>(red[x][r + 8 * e] + 4);
-                const float top = fmaxf(m[x][e], fmaxf(fmaxf(fmaxf(u.x, u.y), fmaxf(u.z, u.w)), fmaxf(fmaxf(v.x, v.y), fmaxf(v.z, v.w))));
-                f[x][e] = pg_ex2(m[x][e] - top);
-                moved |= top > m[x][e];
-                m[x][e] = top;
-            }
-        float m0 = m[0][0], m1 = m[0][1], f0 = f[0][0], f1 = f[0][1];
-        if (RT == 2 && rt == 1) m0 = m[RT - 1][0], m1 = m[RT - 1][1], f0 = f[RT - 1][0], f1 = f[RT - 1][1];
-        const float p0 = pg_ex2(sv[0] - m0), p1 = pg_ex2(sv[1] - m0), p2 = pg_ex2(sv[2] - m1), p3 = pg_ex2(sv[3] - m1);
-        l0 = fmaf(l0, f0, p0 + p1);
-        l1 = fmaf(l1, f1, p2 + p3);
-        {
-            const uint32_t at = ps + (uint32_t)((rt * 16 + r) * LA_PS + kq * 16 + kh * 8 + 2 * t) * 2;
-            asm volatile("st.shared.u32 [%0], %1;" ::"r"(at), "r"(pg_pack_bf16(p0, p1)) : "memory");
-            asm volatile("st.shared.u32 [%0], %1;" ::"r"(at + 8 * LA_PS * 2), "r"(pg_pack_bf16(p2, p3)) : "memory");
-        }
-        __syncthreads();                                  // the weights are there
-        if (nv == 0) continue;
-        if (__any_sync(0xffffffffu, moved)) {
-#pragma unroll
-            for (int x = 0; x < RT; x++)
-#pragma unroll
-                for (int i = 0; i < VT; i++) {
-                    o[x][i][0] *= f[x][0];
-                    o[x][i][1] *= f[x][0];
-                    o[x][i][2] *= f[x][1];
-                    o[x][i][3] *= f[x][1];
+    if (warp == 4) {
+        // ---------------------------------------------------------------- producer
+        if (lane == 0) {
+            bool ok = true, waited = false;
+            for (int j = 0; ok && j < ntiles; j++) {
+                const int key0 = t0 + j * LA_KEYS;
+                if (!waited && (j > 0 || key0 + LA_KEYS > pos0)) {
+                    // what follows may read what the kernel before has written: the queries, and the cache from pos0 on
+                    asm volatile("griddepcontrol.wait;" ::: "memory");
+                    waited = true;
+                    pg_mbar_expect(bar_q, nb * LA_QBLOCK);
+                    for (int b = 0; b < nb; b++) tma_load_2d(q_at + b * LA_QBLOCK, &map_q, bar_q, b * 64, row0 * s.H + rr0);
                 }
-        }
-#pragma unroll
-        for (int kk = 0; kk < LA_KEYS / 16; kk++) {
-            uint32_t a[RT][4];
-#pragma unroll
-            for (int x = 0; x < RT; x++) pg_ldsm4(a[x], ps + (uint32_t)((x * 16 + (lane & 15)) * LA_PS + kk * 16 + (lane >> 4) * 8) * 2);
-#pragma unroll
-            for (int i = 0; i < VT; i += 2) {
-                uint32_t b[4];
-                pg_ldsm4_t(b, kt + v_at + (uint32_t)(kk * 16 * stride + (i < nv ? i : 0) * 16));
-#pragma unroll
-                for (int x = 0; x < RT; x++) {
-                    pg_mma_bf16(o[x][i], a[x][0], a[x][1], a[x][2], a[x][3], b[0], b[1]);
-                    pg_mma_bf16(o[x][i + 1], a[x][0], a[x][1], a[x][2], a[x][3], b[2], b[3]);
+                for (int b = 0; b < nb; b++) {
+                    if (!(ok = pg_mbar_wait(bar_empty + 8 * b, (j & 1) ^ 1, &abort_flag, status, limit_ns))) break;
+                    pg_mbar_expect(bar_full + 8 * b, LA_BLOCK);
+                    tma_load_3d(keys_at + b * LA_BLOCK, &map_k, bar_full + 8 * b, b * 64, key0, slot);
+                }
+            }
+            if (!waited) {
+                asm volatile("griddepcontrol.wait;" ::: "memory");
+                pg_mbar_expect(bar_q, nb * LA_QBLOCK);
+                for (int b = 0; b < nb; b++) tma_load_2d(q_at + b * LA_QBLOCK, &map_q, bar_q, b * 64, row0 * s.H + rr0);
+            }
+            if (!ok) {
+                // give copies that are still in flight a bounded time to land before the CTA exits
+                const unsigned long long w0 = pg_globaltimer_ns();
+                while (pg_globaltimer_ns() - w0 < 2000000ull) {
                 }
             }
         }
-    }
-    if (!ok) {
-        // copies that are still in flight get a bounded time to land before the shared memory goes
-        const unsigned long long w0 = pg_globaltimer_ns();
-        while (pg_globaltimer_ns() - w0 < 2000000ull) {
-        }
-        return;
-    }
+    } else if (warp == 5) {
+        // ---------------------------------------------------------------- MMA issuer
+        if (lane == 0) {
+            constexpr uint32_t idesc_s = make_idesc(128, LA_ROWS), idesc_o = make_idesc(128, LA_ROWS) | IDESC_A_MN_MAJOR;
+            bool ok = pg_mbar_wait(bar_q, 0, &abort_flag, status, limit_ns);
+            tc_fence_after();
+            for (int j = 0; ok && j < ntiles; j++) {
+                for (int b = 0; b < nb; b++) {
+                    if (!(ok = pg_mbar_wait(bar_full + 8 * b, j & 1, &abort_flag, status, limit_ns))) break;
+                    tc_fence_after();
 #pragma unroll
-    for (int x = 1; x < 4; x <<= 1) {
-        l0 += __shfl_xor_sync(0xffffffffu, l0, x);
-        l1 += __shfl_xor_sync(0xffffffffu, l1, x);
-    }
-    __syncthreads();
-    if (t == 0) {
-        red[rt][r][kq * 2 + kh] = l0;
-        red[rt][r + 8][kq * 2 + kh] = l1;
-    }
-    __syncthreads();
-    const int ms = s.cp + 4;
-    float *dst = part + ((first_tile(s, row0, seq, ROWS, per_seq) + tile) * S + split) * ROWS * ms;
+                    for (int i = 0; i < 4; i++)
+                        umma_f16(tmem_s, make_smem_desc(keys_at + b * LA_BLOCK + i * 32), make_smem_desc(q_at + b * LA_QBLOCK + i * 32), idesc_s, (b | i) != 0);
+                    if (b * 64 >= s.cp) umma_commit(bar_empty + 8 * b);   // no value columns: done with
+                }
+                if (!ok) break;
+                umma_commit(bar_s);
+                if (!(ok = pg_mbar_wait(bar_p, j & 1, &abort_flag, status, limit_ns))) break;
+                tc_fence_after();
+                for (int g = 0; g < ng; g++) {
+                    const uint32_t vt = keys_at + 2 * g * LA_BLOCK;
+                    // (the last group of an odd number of blocks reads one block too many, into rows of O^T that nobody reads)
 #pragma unroll
-    for (int x = 0; x < RT; x++)
-#pragma unroll
-        for (int e = 0; e < 2; e++) {
-            float *row = dst + (size_t)(x * 16 + r + 8 * e) * ms;
-#pragma unroll
-            for (int i = 0; i < VT; i++)
-                if (i < nv) *reinterpret_cast<float2 *>(row + c0 + i * 8 + 2 * t) = make_float2(o[x][i][2 * e], o[x][i][2 * e + 1]);
-            if (warp == 0 && t == 0) {
-                const float *g = red[x][r + 8 * e];
-                *reinterpret_cast<float2 *>(row + s.cp) = make_float2(m[x][e], ((g[0] + g[1]) + (g[2] + g[3])) + ((g[4] + g[5]) + (g[6] + g[7])));
+                    for (int i = 0; i < LA_KEYS / 16; i++)
+                        umma_f16(tmem_o + g * LA_ROWS, make_smem_desc_mn(vt + i * 2048, LA_BLOCK), make_smem_desc(p_at + (i / 4) * LA_QBLOCK + (i % 4) * 32), idesc_o,
+                                 (j | i) != 0);
+                }
+                for (int b = 0; b * 64 < s.cp; b++) umma_commit(bar_empty + 8 * b);
+                umma_commit(bar_o);
             }
         }
+    } else {
+        // ---------------------------------------------------------------- softmax
+        const uint32_t lanes = (uint32_t)(warp * 32) << 16;
+        const float sl2 = s.scale * LOG2E;
+        const int low = lims[0];                              // every row sees the keys up to here
+        float m = -1e30f, l[LA_ROWS];                         // m: of row `lane` (finite: a row may see nothing of a slice)
+#pragma unroll
+        for (int c = 0; c < LA_ROWS; c++) l[c] = 0.0f;
+        bool ok = true;
+        for (int j = 0; j < ntiles; j++) {
+            ok = ok && pg_mbar_wait(bar_s, j & 1, &abort_flag, status, limit_ns);
+            ok = __all_sync(0xffffffffu, ok);
+            tc_fence_after();
+            uint32_t v[32];
+            tmem_ld32(tmem_s + lanes, v);
+            const int key = t0 + j * LA_KEYS + warp * 32 + lane;
+            float x[LA_ROWS];
+#pragma unroll
+            for (int c = 0; c < LA_ROWS; c++) x[c] = __uint_as_float(v[c]) * sl2;
+            if (__any_sync(0xffffffffu, key > low || key >= t1)) {
+#pragma unroll
+                for (int c = 0; c < LA_ROWS; c++)
+                    if (key >= t1 || key > lims[c]) x[c] = -INFINITY;
+            }
+            // lane c ends with row c's maximum over the warp's 32 keys
+            float y[LA_ROWS];
+#pragma unroll
+            for (int c = 0; c < LA_ROWS; c++) y[c] = x[c];
+#pragma unroll
+            for (int w = 16; w > 0; w >>= 1) {
+                const bool upper = lane & w;
+#pragma unroll
+                for (int c = 0; c < w; c++) {
+                    const float give = upper ? y[c] : y[c + w], keep = upper ? y[c + w] : y[c];
+                    y[c] = fmaxf(keep, __shfl_xor_sync(0xffffffffu, give, w));
+                }
+            }
+            red[lane][warp] = y[0];
+            if (!(ok = all_four(ok))) break;                  // (the warps give up together)
+            const float4 r4 = *reinterpret_cast<const float4 *>(red[lane]);
+            const float top = fmaxf(fmaxf(r4.x, r4.y), fmaxf(r4.z, r4.w));
+            const bool behind = j == 0 ? top > m : top > m + 8.0f;
+            const float f = behind ? pg_ex2(m - top) : 1.0f;
+            if (behind) m = top;
+            now[warp][lane] = m;
+            __syncwarp();
+            if (j > 0) {
+                // (the products of the tile before read P and write O^T)
+                ok = pg_mbar_wait(bar_o, (j - 1) & 1, &abort_flag, status, limit_ns);
+                ok = __all_sync(0xffffffffu, ok);
+                tc_fence_after();
+                if (ok && __any_sync(0xffffffffu, behind)) {  // (the same in all four warps)
+                    for (int g = 0; g < ng; g++) {
+                        uint32_t o[32];
+                        tmem_ld32(tmem_o + lanes + g * LA_ROWS, o);
+#pragma unroll
+                        for (int c = 0; c < LA_ROWS; c++) o[c] = __float_as_uint(__uint_as_float(o[c]) * __shfl_sync(0xffffffffu, f, c));
+                        tmem_st32(tmem_o + lanes + g * LA_ROWS, o);
+                    }
+                    tmem_wait_st();
+#pragma unroll
+                    for (int c = 0; c < LA_ROWS; c++) l[c] *= __shfl_sync(0xffffffffu, f, c);
+                }
+            }
+            {
+                // row c's weights: 128 bytes per row and 64 keys, 16-byte pieces exchanged by row as the copies do
+                const uint32_t at = p_at + (warp >> 1) * LA_QBLOCK, col = (uint32_t)(warp & 1) * 4 + (lane >> 3), in = (uint32_t)(lane & 7) * 2;
+#pragma unroll
+                for (int c = 0; c < LA_ROWS; c += 4) {
+                    const float4 mm = *reinterpret_cast<const float4 *>(&now[warp][c]);
+                    const float mc[4] = {mm.x, mm.y, mm.z, mm.w};
+#pragma unroll
+                    for (int i = 0; i < 4; i++) {
+                        const float p = pg_ex2(x[c + i] - mc[i]);
+                        l[c + i] += p;
+                        const bf16 pb = __float2bfloat16_rn(p);
+                        asm volatile("st.shared.u16 [%0], %1;" ::"r"(at + (c + i) * 128 + ((col ^ ((c + i) & 7)) << 4) + in), "h"(*reinterpret_cast<const unsigned short *>(&pb))
+                                     : "memory");
+                    }
+                }
+            }
+            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) pg_mbar_arrive(bar_p);
+            // (`red` is written again behind the next wait for bar_s, which is behind all four arrivals)
+        }
+        if (all_four(ok)) {
+            // lane c ends with row c's sum over the warp's keys
+#pragma unroll
+            for (int w = 16; w > 0; w >>= 1) {
+                const bool upper = lane & w;
+#pragma unroll
+                for (int c = 0; c < w; c++) {
+                    const float give = upper ? l[c] : l[c + w], keep = upper ? l[c + w] : l[c];
+                    l[c] = keep + __shfl_xor_sync(0xffffffffu, give, w);
+                }
+            }
+            asm volatile("bar.sync 1, 128;" ::: "memory");
+            red[lane][warp] = l[0];
+            asm volatile("bar.sync 1, 128;" ::: "memory");
+            const int ms = s.cp + 4;
+            float *dst = part + ((first_tile(s, row0, seq, LA_ROWS, per_seq) + tile) * S + split) * LA_ROWS * ms;
+            if (warp == 0) {
+                const float4 r4 = *reinterpret_cast<const float4 *>(red[lane]);
+                *reinterpret_cast<float2 *>(dst + (size_t)lane * ms + s.cp) = make_float2(m, (r4.x + r4.y) + (r4.z + r4.w));
+            }
+            ok = pg_mbar_wait(bar_o, (ntiles - 1) & 1, &abort_flag, status, limit_ns);
+            ok = __all_sync(0xffffffffu, ok);
+            tc_fence_after();
+            const int rows = min(LA_ROWS, total - rr0);
+            for (int g = 0; ok && g < ng; g++) {
+                uint32_t o[32];
+                tmem_ld32(tmem_o + lanes + g * LA_ROWS, o);
+                const int col = g * 128 + warp * 32 + lane;
+                if (col < s.cp) {
+#pragma unroll
+                    for (int c = 0; c < LA_ROWS; c++)
+                        if (c < rows) dst[(size_t)c * ms + col] = __uint_as_float(o[c]);
+                }
+            }
+        }
+    }
+    __syncwarp();
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 5) {
+        tc_fence_after();
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_s), "r"(TMEM_COLS) : "memory");
+    }
 }
 
-// grid (H, parts of 64 columns, groups of `group` <= 16 rows): adds the slices of its rows, then W_uv of its head, then the gate
-constexpr int LV_T = 256;
+// grid (H, parts of 128 columns, groups of `group` <= 16 rows): adds the slices of its rows, then W_uv of its head, then the gate.
+// `ways` threads share the slices of four columns of a row.
+constexpr int LV_T = 512;
 constexpr int LV_SLICES = 64;
-__global__ void __launch_bounds__(LV_T)
-    latent_value_kernel(const LatentShape s, const pg_batch bt, const float *__restrict__ part, int per_seq, int S, int rows, int group,
+constexpr int LV_AHEAD = 9;
+__global__ void __launch_bounds__(LV_T, 1)
+    latent_value_kernel(const LatentShape s, const pg_batch bt, const float *__restrict__ part, int per_seq, int S, int group, int ways,
                         const float *__restrict__ proj, int64_t ldp, bf16 *__restrict__ out, int64_t ldo)
 {
-    extern __shared__ __align__(128) unsigned char smem[];   // [16][cp + 8]
+    extern __shared__ __align__(128) unsigned char smem[];   // [16][cp + 8] | sums [ways][group][cp]
     __shared__ float weight[16][LV_SLICES];
     __shared__ int64_t base[16];
     __shared__ int used[16];
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     const int h = blockIdx.x, m0 = blockIdx.z * group, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int c = blockIdx.y * 64 + warp * 8;
+    const int c = blockIdx.y * 128 + warp * 8;
+    // weights and the batch's arrays do not depend on the kernel before
     Weights8<16> w;
     // (rows of W_uv behind the head's last one belong to the next head or are padding; their products are dropped)
+    w.pieces = 0;
     if (c < s.V) w.ask(s.uv + ((int64_t)h * s.V + c) * s.cp, s.cp, s.cp, lane);
-    pg_pdl_begin();
     bf16 *sa = reinterpret_cast<bf16 *>(smem);
     const int ld = s.cp + 8, ms = s.cp + 4;
-    for (int x = warp; x < 16; x += LV_T / 32) {
-        // a warp per row: where its slices are, and their weights
-        const int m = m0 + x;
+    float *sums = reinterpret_cast<float *>(smem + (size_t)16 * ld * 2);
+    if (threadIdx.x < 16) {
+        // where the row's slices are
+        const int m = m0 + threadIdx.x;
         int n = 0;
-        if (x < group && m < bt.rows) {
+        int64_t at = 0;
+        if ((int)threadIdx.x < group && m < bt.rows) {
             const int seq = __ldcg(bt.d_row_seq + m), row0 = __ldcg(bt.d_seq_row0 + seq), T = seq_len(bt, seq);
-            const int pos0 = __ldcg(bt.d_pos + row0), rr = (m - row0) * s.H + h, tile = rr / rows;
-            const Slices sl = slices_of(s, pos0, T, tile, rows, S);
+            const int pos0 = __ldcg(bt.d_pos + row0), rr = (m - row0) * s.H + h, tile = rr / LA_ROWS;
+            const Slices sl = slices_of(s, pos0, T, tile, LA_ROWS, S);
             if (T < s.long_from && sl.kmax <= s.cap) {
                 n = sl.used;
-                const int64_t at = ((first_tile(s, row0, seq, rows, per_seq) + tile) * S * rows + rr % rows) * (int64_t)ms;
-                float2 ml[LV_SLICES / 32];
-                float top = -INFINITY, l = 0.0f;
-#pragma unroll
-                for (int i = 0; i < LV_SLICES / 32; i++) {
-                    const int k = i * 32 + lane;
-                    ml[i] = k < n ? __ldcg(reinterpret_cast<const float2 *>(part + at + (int64_t)k * rows * ms + s.cp)) : make_float2(-INFINITY, 0.0f);
-                    top = fmaxf(top, ml[i].x);
-                }
-#pragma unroll
-                for (int y = 16; y > 0; y >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, y));
-#pragma unroll
-                for (int i = 0; i < LV_SLICES / 32; i++) {
-                    ml[i].x = exp2f(ml[i].x - top);
-                    l = fmaf(ml[i].x, ml[i].y, l);
-                }
-                const float inv = __fdiv_rn(1.0f, pg_warp_sum(l));
-#pragma unroll
-                for (int i = 0; i < LV_SLICES / 32; i++) weight[x][i * 32 + lane] = ml[i].x * inv;
-                if (lane == 0) base[x] = at;
+                at = ((first_tile(s, row0, seq, LA_ROWS, per_seq) + tile) * S * LA_ROWS + rr % LA_ROWS) * (int64_t)ms;
             }
         }
-        if (lane == 0) used[x] = n;
+        used[threadIdx.x] = n;
+        base[threadIdx.x] = at;
     }
     __syncthreads();
-    const int quads = s.cp / 4;
-    for (int i = threadIdx.x; i < 16 * quads; i += LV_T) {
-        const int x = i / quads, k4 = (i - x * quads) * 4, n = used[x];
-        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-        const float *src = part + (n ? base[x] : 0) + k4;
-        for (int k0 = 0; k0 < n; k0 += 12) {              // twelve loads in flight; behind the last slice its weight is 0
-            float4 v[12];
-#pragma unroll
-            for (int k = 0; k < 12; k++) v[k] = __ldcg(reinterpret_cast<const float4 *>(src + (int64_t)min(k0 + k, n - 1) * rows * ms));
-#pragma unroll
-            for (int k = 0; k < 12; k++) {
-                const float f = k0 + k < n ? weight[x][k0 + k] : 0.0f;
-                a.x = fmaf(f, v[k].x, a.x), a.y = fmaf(f, v[k].y, a.y), a.z = fmaf(f, v[k].z, a.z), a.w = fmaf(f, v[k].w, a.w);
-            }
-        }
-        *reinterpret_cast<uint2 *>(sa + x * ld + k4) = make_uint2(pg_pack_bf16(a.x, a.y), pg_pack_bf16(a.z, a.w));
-    }
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    const int quads = s.cp / 4, items = group * quads * ways;
+    const int64_t step = (int64_t)LA_ROWS * ms;
     const int r = lane >> 2, t = lane & 3;
+    // the first loads of everything together: sums of slices, their maxima and denominators, gates
+    float4 v[LV_AHEAD];
+    auto ask = [&](int i, int k0) {
+        const int way = i / (group * quads), x = i / quads - way * group, k4 = (i % quads) * 4, n = used[x];
+        const float *src = part + base[x] + k4;
+#pragma unroll
+        for (int k = 0; k < LV_AHEAD; k++) v[k] = n ? __ldcg(reinterpret_cast<const float4 *>(src + (int64_t)min((k0 + k) * ways + way, n - 1) * step)) : make_float4(0.f, 0.f, 0.f, 0.f);
+    };
+    if ((int)threadIdx.x < items) ask(threadIdx.x, 0);
     float gate[2][2];
 #pragma unroll
     for (int half = 0; half < 2; half++)
@@ -495,6 +541,56 @@ __global__ void __launch_bounds__(LV_T)
             const int col = c + 2 * t + j;
             gate[half][j] = used[r + 8 * half] && col < s.V ? __ldcg(proj + (int64_t)(m0 + r + 8 * half) * ldp + s.at_gate + h * s.V + col) : 0.0f;
         }
+    if (warp < group && used[warp]) {
+        // a warp per row: the weights of its slices
+        const int n = used[warp];
+        float2 ml[LV_SLICES / 32];
+        float top = -INFINITY, l = 0.0f;
+#pragma unroll
+        for (int i = 0; i < LV_SLICES / 32; i++) {
+            const int k = i * 32 + lane;
+            ml[i] = k < n ? __ldcg(reinterpret_cast<const float2 *>(part + base[warp] + k * step + s.cp)) : make_float2(-INFINITY, 0.0f);
+            top = fmaxf(top, ml[i].x);
+        }
+#pragma unroll
+        for (int y = 16; y > 0; y >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, y));
+#pragma unroll
+        for (int i = 0; i < LV_SLICES / 32; i++) {
+            ml[i].x = exp2f(ml[i].x - top);
+            l = fmaf(ml[i].x, ml[i].y, l);
+        }
+        const float inv = __fdiv_rn(1.0f, pg_warp_sum(l));
+#pragma unroll
+        for (int i = 0; i < LV_SLICES / 32; i++) weight[warp][i * 32 + lane] = ml[i].x * inv;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < items; i += LV_T) {
+        const int way = i / (group * quads), x = i / quads - way * group, k4 = (i % quads) * 4, n = used[x];
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i != (int)threadIdx.x) ask(i, 0);
+        for (int k0 = 0; k0 * ways < n; k0 += LV_AHEAD) {
+            if (k0 > 0) ask(i, k0);
+#pragma unroll
+            for (int k = 0; k < LV_AHEAD; k++) {
+                const int slice = (k0 + k) * ways + way;
+                const float f = slice < n ? weight[x][slice] : 0.0f;   // (behind the last slice: the last one again, with weight 0)
+                a.x = fmaf(f, v[k].x, a.x), a.y = fmaf(f, v[k].y, a.y), a.z = fmaf(f, v[k].z, a.z), a.w = fmaf(f, v[k].w, a.w);
+            }
+        }
+        *reinterpret_cast<float4 *>(sums + (size_t)(way * group + x) * s.cp + k4) = a;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < 16 * quads; i += LV_T) {
+        const int x = i / quads, k4 = (i - x * quads) * 4;
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (x < group) {
+            for (int way = 0; way < ways; way++) {
+                const float4 u = *reinterpret_cast<const float4 *>(sums + (size_t)(way * group + x) * s.cp + k4);
+                a.x += u.x, a.y += u.y, a.z += u.z, a.w += u.w;
+            }
+        }
+        *reinterpret_cast<uint2 *>(sa + x * ld + k4) = make_uint2(pg_pack_bf16(a.x, a.y), pg_pack_bf16(a.z, a.w));
+    }
     __syncthreads();
     if (c >= s.V) return;
     float d[4] = {};
@@ -606,32 +702,14 @@ LatentShape shape_of(const pg_latent *p)
     return s;
 }
 
-constexpr int LA_SMEM = 220 * 1024;
-int attn_rows(const LatentShape &s) { return s.H > 16 ? 32 : 16; }
-int attn_smem(const LatentShape &s, int stages) { return (stages * LA_KEYS + attn_rows(s)) * (s.ck * 2 + 16) + attn_rows(s) * (LA_PS * 2 + 256); }
+int attn_smem(const LatentShape &s) { return 1024 + (s.ck + 63) / 64 * (LA_BLOCK + LA_QBLOCK) + 2 * LA_QBLOCK; }
 
-// slices of the context: about one CTA per SM, none shorter than 64 positions of a full cache
+// slices of the context: about one CTA per SM, none shorter than 128 positions of a full cache
 int slices(const pg_ctx *ctx, int64_t units, int64_t cap)
 {
     int64_t S = std::max<int64_t>(1, (int64_t)ctx->sm_count / std::max<int64_t>(1, units));
     S = std::min<int64_t>(S, std::max<int64_t>(1, cap / LA_KEYS));
     return (int)std::min<int64_t>(S, LV_SLICES);
-}
-
-template <int RT>
-int32_t launch_attn(pg_ctx *ctx, const LatentShape &s, const pg_batch *batch, dim3 grid, const bf16 *q, const bf16 *cache, float *part, int per_seq, int stages)
-{
-    auto go = [&](auto kern, std::atomic<uint64_t> &set) -> int32_t {
-        PG_CUDA(pg_max_smem_once(kern, LA_SMEM, ctx->device, set));
-        return launch_pdl(ctx, kern, grid, dim3(RT * 256), (size_t)attn_smem(s, stages), s, *batch, q, cache, part, per_seq, stages, ctx->d_status,
-                          ctx->wait_limit_ns);
-    };
-    static std::atomic<uint64_t> set[5] = {};
-    if (s.ck <= 96) return go(latent_attn_kernel<RT, 3>, set[0]);
-    if (s.ck <= 160) return go(latent_attn_kernel<RT, 5>, set[1]);
-    if (s.ck <= 320) return go(latent_attn_kernel<RT, 10>, set[2]);
-    if (s.ck <= 576) return go(latent_attn_kernel<RT, 18>, set[3]);
-    return go(latent_attn_kernel<RT, 0>, set[4]);
 }
 
 int32_t check(const pg_latent *p, const pg_batch *batch, int64_t ldp, int64_t ldo)
@@ -641,7 +719,7 @@ int32_t check(const pg_latent *p, const pg_batch *batch, int64_t ldp, int64_t ld
                    p->cap > 0 && p->heads <= 65534,
                "latent attention: bad shape (dim %d and latent %d at most 512, an even rot_dim %d)", p->dim, p->kv_rank, p->rot_dim);
     const LatentShape s = shape_of(p);
-    PG_REQUIRE(attn_smem(s, 2) <= LA_SMEM, "latent attention: a key of %d and %d columns is too wide", s.C, s.R);
+    PG_REQUIRE(s.ck <= 640, "latent attention: a key of %d and %d columns is too wide", s.C, s.R);
     PG_REQUIRE(ldp >= s.at_gate + (int64_t)s.H * s.V && ldo >= (int64_t)s.H * s.V, "latent attention: rows too short");
     PG_REQUIRE(batch->rows >= 0 && batch->seqs <= 65535, "latent attention: too many sequences");
     return PG_OK;
@@ -657,8 +735,8 @@ PG_API int64_t pg_latent_part_floats(pg_ctx *ctx, const pg_latent *p, int32_t dt
     const LatentShape s = shape_of(p);
     if (dtype == PG_F32) return max_rows * s.H * s.C;
     // tiles x slices: as many as there are tiles, or about one CTA per SM
-    const int64_t tiles = (max_rows * s.H + attn_rows(s) - 1) / attn_rows(s) + max_seqs;
-    return std::max<int64_t>(tiles, 2 * ctx->sm_count) * attn_rows(s) * (s.cp + 4);
+    const int64_t tiles = (max_rows * s.H + LA_ROWS - 1) / LA_ROWS + max_seqs;
+    return std::max<int64_t>(tiles, 2 * ctx->sm_count) * LA_ROWS * (s.cp + 4);
 }
 
 PG_API int32_t pg_latent_run(pg_ctx *ctx, const pg_latent *p, const pg_batch *batch, int64_t long_from, int64_t short_rows, int64_t short_len,
@@ -694,28 +772,40 @@ PG_API int32_t pg_latent_run(pg_ctx *ctx, const pg_latent *p, const pg_batch *ba
     rc = launch_pdl(ctx, latent_query_kernel, dim3((unsigned)(s.H + s.own), (unsigned)parts, row_tiles), dim3(LQ_T), (size_t)(16 * (s.dk + 8) * 2), s, *batch,
                     d_proj, ldp, q, cache, ctx->d_status);
     if (rc != PG_OK) return rc;
-    const int rows = attn_rows(s);
-    const int64_t tiles = (short_len * s.H + rows - 1) / rows;
+    const int64_t tiles = (short_len * s.H + LA_ROWS - 1) / LA_ROWS;
     PG_REQUIRE(tiles <= 65535, "latent attention: too many rows in one sequence");
     // the numbering of tiles that needs fewer of them, and as many slices as then have room
-    const int64_t dense = (int64_t)batch->rows * s.H / rows + batch->seqs, even = tiles * batch->seqs;
+    const int64_t dense = (int64_t)batch->rows * s.H / LA_ROWS + batch->seqs, even = tiles * batch->seqs;
     const int per_seq = even <= dense ? (int)tiles : 0;
-    const int64_t room = p->part_floats / ((int64_t)rows * (s.cp + 4)) / std::min(even, dense);
+    const int64_t room = p->part_floats / ((int64_t)LA_ROWS * (s.cp + 4)) / std::min(even, dense);
     PG_REQUIRE(room >= 1, "latent attention: the step has more rows than d_part has room for");
-    const int S = (int)std::min<int64_t>(room, slices(ctx, std::max<int64_t>(tiles, (short_rows * s.H + rows - 1) / rows), s.cap));
-    int stages = 4;
-    while (stages > 2 && attn_smem(s, stages) > LA_SMEM) stages--;
-    const dim3 grid((unsigned)S, (unsigned)tiles, (unsigned)batch->seqs);
-    rc = rows == 32 ? launch_attn<2>(ctx, s, batch, grid, q, cache, p->d_part, per_seq, stages) : launch_attn<1>(ctx, s, batch, grid, q, cache, p->d_part, per_seq, stages);
-    if (rc != PG_OK) return rc;
+    const int S = (int)std::min<int64_t>(room, slices(ctx, std::max<int64_t>(tiles, (short_rows * s.H + LA_ROWS - 1) / LA_ROWS), s.cap));
+    {
+        CUtensorMap mk, mq;
+        const cuuint64_t dk[3] = {(cuuint64_t)s.ck, (cuuint64_t)s.cap, (cuuint64_t)p->slots}, sk[2] = {(cuuint64_t)s.ck * 2, (cuuint64_t)s.cap * s.ck * 2};
+        const cuuint64_t dq[2] = {(cuuint64_t)s.ck, (cuuint64_t)batch->rows * s.H}, sq[1] = {(cuuint64_t)s.ck * 2};
+        const cuuint32_t bk[3] = {64, LA_KEYS, 1}, bq[2] = {64, LA_ROWS};
+        rc = pg_encode_bf16(&mk, cache, 3, dk, sk, bk);
+        if (rc == PG_OK) rc = pg_encode_bf16(&mq, q, 2, dq, sq, bq);
+        if (rc != PG_OK) return rc;
+        static std::atomic<uint64_t> set{0};
+        PG_CUDA(pg_max_smem_once(latent_attn_kernel, 224 * 1024, ctx->device, set));
+        rc = launch_pdl(ctx, latent_attn_kernel, dim3((unsigned)S, (unsigned)tiles, (unsigned)batch->seqs), dim3(LA_THREADS), (size_t)attn_smem(s), mk, mq, s, *batch,
+                        p->d_part, per_seq, ctx->d_status, ctx->wait_limit_ns);
+        if (rc != PG_OK) return rc;
+    }
     // groups of rows small enough for about one CTA per SM
-    const unsigned parts64 = (unsigned)((s.V + 63) / 64);
+    const unsigned parts128 = (unsigned)((s.V + 127) / 128);
     int group = 16;
-    while (group > 1 && (int64_t)s.H * parts64 * ((batch->rows + group - 1) / group) < ctx->sm_count * 3 / 4) group /= 2;
+    while (group > 1 && (int64_t)s.H * parts128 * ((batch->rows + group - 1) / group) < ctx->sm_count * 3 / 4) group /= 2;
+    const int ways = std::max(1, std::min(8, LV_T / (group * s.cp / 4)));
     const int64_t groups = (batch->rows + group - 1) / group;
-    PG_REQUIRE(groups <= 65535 && parts64 <= 65535, "latent attention: too many rows");
-    return launch_pdl(ctx, latent_value_kernel, dim3((unsigned)s.H, parts64, (unsigned)groups), dim3(LV_T), (size_t)(16 * (s.cp + 8) * 2), s, *batch,
-                      (const float *)p->d_part, per_seq, S, rows, group, d_proj, ldp, (bf16 *)d_out, ldo);
+    PG_REQUIRE(groups <= 65535 && parts128 <= 65535, "latent attention: too many rows");
+    const size_t smem = (size_t)16 * (s.cp + 8) * 2 + (size_t)ways * group * s.cp * 4;
+    static std::atomic<uint64_t> set{0};
+    PG_CUDA(pg_max_smem_once(latent_value_kernel, 64 * 1024, ctx->device, set));
+    return launch_pdl(ctx, latent_value_kernel, dim3((unsigned)s.H, parts128, (unsigned)groups), dim3(LV_T), smem, s, *batch, (const float *)p->d_part, per_seq, S,
+                      group, ways, d_proj, ldp, (bf16 *)d_out, ldo);
 }
 
 PG_API int32_t pg_latent_prompt_supports(const pg_latent *p)

@@ -26,6 +26,28 @@ inline int32_t launch_pdl_cluster(pg_ctx *ctx, K kern, dim3 grid, dim3 block, si
     return PG_OK;
 }
 
+// The same, but started when everything before it has ended.  The first kernel of a step is launched this way, so that the
+// kernels behind it may read the batch's arrays, and what earlier steps left in caches and states, before they wait.
+template <typename K, typename... Args>
+inline int32_t launch_whole_cluster(pg_ctx *ctx, K kern, dim3 grid, dim3 block, size_t smem, int cs, Args... args)
+{
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = (unsigned)cs;
+    attr[0].val.clusterDim.y = 1;
+    attr[0].val.clusterDim.z = 1;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = ctx->stream;
+    cfg.attrs = attr;
+    cfg.numAttrs = cs > 1 ? 1 : 0;
+    PG_CUDA(cudaLaunchKernelEx(&cfg, kern, args...));
+    PG_LAUNCHED();
+    return PG_OK;
+}
+
 // CTAs per row for the row kernels: as many (up to 8) as keep the grid within about two CTAs per SM, divide the row's
 // `units` evenly and leave each CTA at least `min_units`.
 inline int row_cluster(const pg_ctx *ctx, int64_t rows, int64_t units, int64_t min_units)

@@ -176,6 +176,7 @@ int32_t run_rows(pg_ctx *ctx, const RowArgs &a, int64_t rows, int32_t dtype, boo
     {                                                                                                   \
         static std::atomic<uint64_t> set{0};                                                            \
         PG_CUDA(pg_max_smem_once(row_norm_kernel<SRC, VV, T>, 132 * 1024, ctx->device, set));           \
+        if (SRC == SRC_EMBED) return launch_whole_cluster(ctx, row_norm_kernel<SRC, VV, T>, g, dim3(RW_T), smem, cs, a); \
         return launch_pdl_cluster(ctx, row_norm_kernel<SRC, VV, T>, g, dim3(RW_T), smem, cs, a);        \
     }
     if (dtype == PG_BF16) {

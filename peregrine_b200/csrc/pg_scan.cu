@@ -198,7 +198,7 @@ __device__ __forceinline__ float sum2(f32x2 v)
 // grid (ceil(inner / 32), ceil(rows / R)).  NC: quads of states per lane
 constexpr int SS_W = 8;                  // 16-byte pieces of a row of W_dt that a lane asks for ahead (rank up to 256)
 template <int NC, int R, typename TA>
-__global__ void __launch_bounds__(SR_T)
+__global__ void __launch_bounds__(SR_T, NC == 1 ? 6 : 1)
     scan_step_kernel(const ScanShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, const TA *__restrict__ x, int64_t ldx,
                      const float *__restrict__ low, int64_t ldl, float *state, TA *__restrict__ out, int64_t ldo)
 {
@@ -220,15 +220,24 @@ __global__ void __launch_bounds__(SR_T)
     for (int i = 0; i < NC; i++)
         a[i] = quad(live && q + 4 * i < quads ? __ldg(reinterpret_cast<const float4 *>(s.a + (int64_t)c * s.ss) + q + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f));
     const float dt_bias = live ? __ldg(s.dt_bias + c) : 0.0f, skip = live ? __ldg(s.d + c) : 0.0f;
-    asm volatile("griddepcontrol.wait;" ::: "memory");
-    int64_t at[R];
-    bool old[R];
+    // neither do the batch's arrays and what earlier steps left
+    int slot[R];
+    Quad S[R][NC];
+#pragma unroll
+    for (int r = 0; r < R; r++) slot[r] = live && m0 + r < bt.rows ? __ldcg(bt.d_seq_slot + m0 + r) : -1;   // (one row per sequence)
+    auto at = [&](int r) { return reinterpret_cast<float4 *>(state + ((int64_t)slot[r] * s.inner + c) * s.ss) + q; };
 #pragma unroll
     for (int r = 0; r < R; r++) {
-        const int m = m0 + r;
-        const bool on = live && m < bt.rows;
-        at[r] = on ? ((int64_t)__ldcg(bt.d_seq_slot + __ldcg(bt.d_row_seq + m)) * s.inner + c) * s.ss : -1;
-        old[r] = on && __ldcg(bt.d_pos + m) > 0;
+        const bool old = slot[r] >= 0 && __ldcg(bt.d_pos + m0 + r) > 0;
+#pragma unroll
+        for (int i = 0; i < NC; i++) S[r][i] = quad(old && q + 4 * i < quads ? __ldcg(at(r) + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f));
+    }
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    float xv[R], z[R];
+#pragma unroll
+    for (int r = 0; r < R; r++) {
+        xv[r] = slot[r] >= 0 ? pg_get(x + (int64_t)(m0 + r) * ldx + c) : 0.0f;
+        z[r] = slot[r] >= 0 ? __ldcg(proj + (int64_t)(m0 + r) * ldp + s.inner + c) : 0.0f;
     }
 #pragma unroll
     for (int r = 0; r < R; r++) {
@@ -239,16 +248,6 @@ __global__ void __launch_bounds__(SR_T)
             const int which = k / NP, n = k - which * NP;
             sbc[r * 2 * NP + k] = on && n < s.N ? __ldcg(src + s.dtp + which * s.N + n) : 0.0f;
         }
-    }
-    Quad S[R][NC];
-    float xv[R], z[R];
-#pragma unroll
-    for (int r = 0; r < R; r++) {
-#pragma unroll
-        for (int i = 0; i < NC; i++)
-            S[r][i] = quad(old[r] && q + 4 * i < quads ? __ldcg(reinterpret_cast<const float4 *>(state + at[r]) + q + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f));
-        xv[r] = at[r] >= 0 ? pg_get(x + (int64_t)(m0 + r) * ldx + c) : 0.0f;
-        z[r] = at[r] >= 0 ? __ldcg(proj + (int64_t)(m0 + r) * ldp + s.inner + c) : 0.0f;
     }
     __syncthreads();
     float acc[R] = {};
@@ -275,11 +274,11 @@ __global__ void __launch_bounds__(SR_T)
         for (int i = 0; i < NC; i++) {
             const float *b = sbc + r * 2 * NP + (q + 4 * i) * 4;
             y += sum2(update(S[r][i], a[i], pair(dt, dt), pair(du, du), load_quad(b), load_quad(b + NP)));
-            if (at[r] >= 0 && q + 4 * i < quads) reinterpret_cast<float4 *>(state + at[r])[q + 4 * i] = quad4(S[r][i]);
+            if (slot[r] >= 0 && q + 4 * i < quads) at(r)[4 * i] = quad4(S[r][i]);
         }
         y += __shfl_xor_sync(0xffffffffu, y, 1);
         y += __shfl_xor_sync(0xffffffffu, y, 2);
-        if (q == 0 && at[r] >= 0) pg_put(out + (int64_t)(m0 + r) * ldo + c, fmaf(skip, xv[r], y) * pg_silu(z[r]));
+        if (q == 0 && slot[r] >= 0) pg_put(out + (int64_t)(m0 + r) * ldo + c, fmaf(skip, xv[r], y) * pg_silu(z[r]));
     }
 }
 
@@ -401,24 +400,40 @@ __global__ void __launch_bounds__(2 * SR_T)
     for (int i = 0; i < tiles; i++) {
         __syncthreads();
         const int b = i & 1;
+        float y[TT];
 #pragma unroll
         for (int t = 0; t < TT; t += 4) {
-            float y[4];
+            // four tokens: everything that does not depend on the state first, then the chain
+            f32x2 part[4];
 #pragma unroll
-            for (int u = 0; u < 4; u++) {
-                const Quad d = load_quad(reinterpret_cast<const float *>(&sd[b][t + u][cl]));
-                f32x2 part = 0;
+            for (int n = 0; n < NC; n++) {
+                Quad e[4], g[4], c4[4];
 #pragma unroll
-                for (int n = 0; n < NC; n++) {
-                    const f32x2 v = update(S[n], a[n], d.lo, d.hi, load_quad(&sbc[b][t + u][0][(q + 4 * n) * 4]), load_quad(&sbc[b][t + u][1][(q + 4 * n) * 4]));
-                    part = n == 0 ? v : fma2(pair(1.0f, 1.0f), v, part);
+                for (int u = 0; u < 4; u++) {
+                    const Quad d = load_quad(reinterpret_cast<const float *>(&sd[b][t + u][cl])), bb = load_quad(&sbc[b][t + u][0][(q + 4 * n) * 4]);
+                    c4[u] = load_quad(&sbc[b][t + u][1][(q + 4 * n) * 4]);
+                    e[u] = {mul2(d.lo, a[n].lo), mul2(d.lo, a[n].hi)};
+                    g[u] = {mul2(d.hi, bb.lo), mul2(d.hi, bb.hi)};
                 }
-                y[u] = sum2(part);
+#pragma unroll
+                for (int u = 0; u < 4; u++) e[u] = {ex2_pair(e[u].lo), ex2_pair(e[u].hi)};
+#pragma unroll
+                for (int u = 0; u < 4; u++) {
+                    S[n].lo = fma2(e[u].lo, S[n].lo, g[u].lo);
+                    S[n].hi = fma2(e[u].hi, S[n].hi, g[u].hi);
+                    part[u] = n == 0 ? mul2(S[n].lo, c4[u].lo) : fma2(S[n].lo, c4[u].lo, part[u]);
+                    part[u] = fma2(S[n].hi, c4[u].hi, part[u]);
+                }
             }
-            // four tokens' sums over four lanes: lane q ends with token q's
-            const bool odd = q & 1, up = q & 2;
-            const float g0 = __shfl_xor_sync(0xffffffffu, odd ? y[0] : y[1], 1), g1 = __shfl_xor_sync(0xffffffffu, odd ? y[2] : y[3], 1);
-            const float k0 = (odd ? y[1] : y[0]) + g0, k1 = (odd ? y[3] : y[2]) + g1;
+#pragma unroll
+            for (int u = 0; u < 4; u++) y[t + u] = sum2(part[u]);
+        }
+        // four tokens' sums over four lanes: lane q ends with token q's
+        const bool odd = q & 1, up = q & 2;
+#pragma unroll
+        for (int t = 0; t < TT; t += 4) {
+            const float g0 = __shfl_xor_sync(0xffffffffu, odd ? y[t] : y[t + 1], 1), g1 = __shfl_xor_sync(0xffffffffu, odd ? y[t + 2] : y[t + 3], 1);
+            const float k0 = (odd ? y[t + 1] : y[t]) + g0, k1 = (odd ? y[t + 3] : y[t + 2]) + g1;
             const float g2 = __shfl_xor_sync(0xffffffffu, up ? k0 : k1, 2);
             sy[b][t + q][cl] = (up ? k1 : k0) + g2;
         }

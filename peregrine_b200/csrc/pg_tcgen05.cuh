@@ -95,7 +95,7 @@ __device__ __forceinline__ uint64_t make_smem_desc_mn(uint32_t smem_addr, uint32
     d |= (uint64_t)2 << 61;
     return d;
 }
-constexpr uint32_t IDESC_B_MN_MAJOR = 1u << 16;
+constexpr uint32_t IDESC_A_MN_MAJOR = 1u << 15, IDESC_B_MN_MAJOR = 1u << 16;
 // kind::f16: D = f32 (1 at bit 4), A and B = bf16 (1 at bits 7 and 10), both K-major, N >> 3 at bit 17, M >> 4 at bit 24
 __host__ __device__ constexpr uint32_t make_idesc(int m, int n)
 {
