@@ -67,6 +67,15 @@ __device__ __forceinline__ void pg_cp16(uint32_t dst, const void *src)
 {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
 }
+// N = 4, 8 or 16 bytes; zeros where `in` is false.  The short forms go through L1: only for kernels that are launched whole.
+template <int N>
+__device__ __forceinline__ void pg_cp_in(uint32_t dst, const void *src, bool in)
+{
+    if constexpr (N == 16)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? N : 0) : "memory");
+    else
+        asm volatile("cp.async.ca.shared.global [%0], [%1], %2, %3;" ::"r"(dst), "l"(src), "n"(N), "r"(in ? N : 0) : "memory");
+}
 __device__ __forceinline__ void pg_cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N>
 __device__ __forceinline__ void pg_cp_wait()
@@ -76,7 +85,7 @@ __device__ __forceinline__ void pg_cp_wait()
 // D[16 x 8] += A[16 x 16] B[16 x 8], bf16 operands, f32 sums
 __device__ __forceinline__ void pg_mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1)
 {
-    asm volatile(
+    asm(
         "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
         : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
         : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));

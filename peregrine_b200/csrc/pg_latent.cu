@@ -46,39 +46,60 @@ struct LatentShape {
 
 __device__ __forceinline__ int seq_len(const pg_batch &bt, int seq) { return __ldcg(bt.d_seq_row0 + seq + 1) - __ldcg(bt.d_seq_row0 + seq); }
 
-// One warp: the pairs of src rotated for position pos; columns R .. rp are zero.
+// A lane's cosines and sines for position pos: pairs lane + 32 i (rot_dim <= 128).
+struct Turn {
+    float2 r[2];
+    __device__ __forceinline__ void ask(const LatentShape &s, int pos, int lane)
+    {
+        const float2 *cs = reinterpret_cast<const float2 *>(s.rot) + (int64_t)min(max(pos, 0), s.cap - 1) * (s.R / 2);
+#pragma unroll
+        for (int i = 0; i < 2; i++) r[i] = 2 * (lane + 32 * i) < s.R ? __ldg(cs + lane + 32 * i) : make_float2(1.0f, 0.0f);
+    }
+};
+// One warp: the pairs of src rotated; columns R .. rp are zero.
 template <typename TA>
-__device__ __forceinline__ void rotate(const LatentShape &s, const float *src, int pos, TA *dst, int rp, int lane)
+__device__ __forceinline__ void rotate(const LatentShape &s, const float *src, const Turn &turn, TA *dst, int rp, int lane)
 {
-    const float2 *cs = reinterpret_cast<const float2 *>(s.rot) + (int64_t)pos * (s.R / 2);
-    for (int i = lane; i < rp / 2; i += 32) {
-        float u = 0.0f, v = 0.0f;
-        if (2 * i < s.R) {
-            const float a = __ldcg(src + 2 * i), b = __ldcg(src + 2 * i + 1);
-            const float2 r = __ldg(cs + i);
-            u = a * r.x - b * r.y;
-            v = b * r.x + a * r.y;
+    float a[2], b[2];
+#pragma unroll
+    for (int i = 0; i < 2; i++) {
+        const int at = 2 * (lane + 32 * i);
+        a[i] = at < s.R ? __ldcg(src + at) : 0.0f;
+        b[i] = at < s.R ? __ldcg(src + at + 1) : 0.0f;
+    }
+#pragma unroll
+    for (int i = 0; i < 2; i++) {
+        const int at = 2 * (lane + 32 * i);
+        if (at < rp) {
+            pg_put(dst + at, a[i] * turn.r[i].x - b[i] * turn.r[i].y);
+            pg_put(dst + at + 1, b[i] * turn.r[i].x + a[i] * turn.r[i].y);
         }
-        pg_put(dst + 2 * i, u);
-        pg_put(dst + 2 * i + 1, v);
     }
 }
 
 // One warp: the cache row of a token, [c | 0 | rotated key part | 0] (kv_rank <= 512).
+struct NormWeights {
+    float w[16];
+    __device__ __forceinline__ void ask(const LatentShape &s, int lane)
+    {
+#pragma unroll
+        for (int i = 0; i < 16; i++) w[i] = i * 32 + lane < s.C ? __ldg(s.c_norm + i * 32 + lane) : 0.0f;
+    }
+};
 template <typename TA>
-__device__ __forceinline__ void append(const LatentShape &s, const float *kv, int pos, TA *dst, int lane)
+__device__ __forceinline__ void append(const LatentShape &s, const float *kv, const Turn &turn, const NormWeights &nw, TA *dst, int lane)
 {
     float x[16], ss = 0.0f;
 #pragma unroll
     for (int i = 0; i < 16; i++) x[i] = i * 32 + lane < s.C ? __ldcg(kv + i * 32 + lane) : 0.0f;
-    rotate(s, kv + s.C, pos, dst + s.cp, s.rp, lane);
+    rotate(s, kv + s.C, turn, dst + s.cp, s.rp, lane);
 #pragma unroll
     for (int i = 0; i < 16; i++) ss += x[i] * x[i];
     const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(pg_warp_sum(ss), (float)s.C) + s.eps));
 #pragma unroll
     for (int i = 0; i < 16; i++) {
         const int c = i * 32 + lane;
-        if (c < s.cp) pg_put(dst + c, c < s.C ? x[i] * inv * __ldg(s.c_norm + c) : 0.0f);
+        if (c < s.cp) pg_put(dst + c, x[i] * inv * nw.w[i]);
     }
 }
 
@@ -97,12 +118,14 @@ struct Weights8 {
 #pragma unroll
         for (int i = 0; i < PRE; i++) x[i] = i < pieces ? __ldg(at + 4 * i) : make_uint4(0u, 0u, 0u, 0u);
     }
+    // HI: whether rows 8 .. 15 are there
+    template <bool HI>
     __device__ __forceinline__ void times(float (&d)[4], uint32_t a, int ld, int lane)
     {
         const uint32_t a0 = a + (uint32_t)((lane >> 2) * ld + (lane & 3) * 8) * 2, a1 = a0 + (uint32_t)(8 * ld) * 2;
         float e[4] = {};                                  // two sums: shorter chains
         auto step = [&](const uint4 &v, int i) {
-            const uint4 lo = pg_lds128(a0 + i * 64), hi = pg_lds128(a1 + i * 64);
+            const uint4 lo = pg_lds128(a0 + i * 64), hi = HI ? pg_lds128(a1 + i * 64) : make_uint4(0u, 0u, 0u, 0u);
             pg_mma_bf16(d, lo.x, hi.x, lo.y, hi.y, v.x, v.y);
             pg_mma_bf16(e, lo.z, hi.z, lo.w, hi.w, v.z, v.w);
         };
@@ -132,12 +155,16 @@ __global__ void __launch_bounds__(LQ_T)
     if (h < s.H && c < s.cp) w.ask(s.uk + ((int64_t)h * s.cp + c) * s.dk, s.dk, s.dk, lane);
     const int mine = blockIdx.y * NW + warp;                 // the first row that this warp rotates (or appends)
     const int pos_first = mine < n ? __ldcg(bt.d_pos + m0 + mine) : 0;
+    Turn turn;
+    turn.ask(s, pos_first, lane);
     bf16 *sa = reinterpret_cast<bf16 *>(smem);
     const int ld = s.dk + 8;
     if (h == s.H) {
         const int seq_first = mine < n ? __ldcg(bt.d_row_seq + m0 + mine) : 0;
         const int64_t slot_first = __ldcg(bt.d_seq_slot + seq_first);
         const bool skip_first = seq_len(bt, seq_first) >= s.long_from;
+        NormWeights nw;
+        nw.ask(s, lane);
         asm volatile("griddepcontrol.wait;" ::: "memory");
         for (int i = mine; i < n; i += gridDim.y * NW) {
             const int m = m0 + i, pos = i == mine ? pos_first : __ldcg(bt.d_pos + m), seq = i == mine ? seq_first : __ldcg(bt.d_row_seq + m);
@@ -146,7 +173,8 @@ __global__ void __launch_bounds__(LQ_T)
                 if (lane == 0) atomicExch(status, (int32_t)PG_ERR_INVALID);
                 continue;
             }
-            append(s, proj + (int64_t)m * ldp + s.at_kv, pos, cache + ((i == mine ? slot_first : (int64_t)__ldcg(bt.d_seq_slot + seq)) * s.cap + pos) * s.ck, lane);
+            if (i != mine) turn.ask(s, pos, lane);
+            append(s, proj + (int64_t)m * ldp + s.at_kv, turn, nw, cache + ((i == mine ? slot_first : (int64_t)__ldcg(bt.d_seq_slot + seq)) * s.cap + pos) * s.ck, lane);
         }
         return;
     }
@@ -165,7 +193,8 @@ __global__ void __launch_bounds__(LQ_T)
             if (lane == 0) atomicExch(status, (int32_t)PG_ERR_INVALID);
             continue;
         }
-        rotate(s, proj + (int64_t)m * ldp + h * (s.D + s.R) + s.D, pos, qx + ((int64_t)m * s.H + h) * s.ck + s.cp, s.rp, lane);
+        if (i != mine) turn.ask(s, pos, lane);
+        rotate(s, proj + (int64_t)m * ldp + h * (s.D + s.R) + s.D, turn, qx + ((int64_t)m * s.H + h) * s.ck + s.cp, s.rp, lane);
     }
 #pragma unroll
     for (int k = 0; k < AHEAD; k++) {
@@ -182,7 +211,7 @@ __global__ void __launch_bounds__(LQ_T)
     const int r = lane >> 2, t = lane & 3;
     while (c < s.cp) {
         float d[4] = {};
-        w.times(d, pg_smem(sa), ld, lane);
+        w.times<true>(d, pg_smem(sa), ld, lane);
 #pragma unroll
         for (int half = 0; half < 2; half++)
             if (r + 8 * half < n)
@@ -319,15 +348,16 @@ __global__ void __launch_bounds__(LA_THREADS, 1)
         // ---------------------------------------------------------------- MMA issuer
         if (lane == 0) {
             constexpr uint32_t idesc_s = make_idesc(128, LA_ROWS), idesc_o = make_idesc(128, LA_ROWS) | IDESC_A_MN_MAJOR;
+            const uint64_t desc_k = make_smem_desc(keys_at), desc_q = make_smem_desc(q_at), desc_p = make_smem_desc(p_at), desc_v = make_smem_desc_mn(keys_at, LA_BLOCK);
             bool ok = pg_mbar_wait(bar_q, 0, &abort_flag, status, limit_ns);
             tc_fence_after();
             for (int j = 0; ok && j < ntiles; j++) {
                 for (int b = 0; b < nb; b++) {
                     if (!(ok = pg_mbar_wait(bar_full + 8 * b, j & 1, &abort_flag, status, limit_ns))) break;
                     tc_fence_after();
+                    const uint64_t dk = desc_k + (uint64_t)(b * (LA_BLOCK >> 4)), dq = desc_q + (uint64_t)(b * (LA_QBLOCK >> 4));
 #pragma unroll
-                    for (int i = 0; i < 4; i++)
-                        umma_f16(tmem_s, make_smem_desc(keys_at + b * LA_BLOCK + i * 32), make_smem_desc(q_at + b * LA_QBLOCK + i * 32), idesc_s, (b | i) != 0);
+                    for (int i = 0; i < 4; i++) umma_f16(tmem_s, dk + i * 2, dq + i * 2, idesc_s, (b | i) != 0);
                     if (b * 64 >= s.cp) umma_commit(bar_empty + 8 * b);   // no value columns: done with
                 }
                 if (!ok) break;
@@ -335,12 +365,11 @@ __global__ void __launch_bounds__(LA_THREADS, 1)
                 if (!(ok = pg_mbar_wait(bar_p, j & 1, &abort_flag, status, limit_ns))) break;
                 tc_fence_after();
                 for (int g = 0; g < ng; g++) {
-                    const uint32_t vt = keys_at + 2 * g * LA_BLOCK;
+                    const uint64_t dv = desc_v + (uint64_t)(2 * g * (LA_BLOCK >> 4));
                     // (the last group of an odd number of blocks reads one block too many, into rows of O^T that nobody reads)
 #pragma unroll
                     for (int i = 0; i < LA_KEYS / 16; i++)
-                        umma_f16(tmem_o + g * LA_ROWS, make_smem_desc_mn(vt + i * 2048, LA_BLOCK), make_smem_desc(p_at + (i / 4) * LA_QBLOCK + (i % 4) * 32), idesc_o,
-                                 (j | i) != 0);
+                        umma_f16(tmem_o + g * LA_ROWS, dv + i * (2048 >> 4), desc_p + (i / 4) * (LA_QBLOCK >> 4) + (i % 4) * 2, idesc_o, (j | i) != 0);
                 }
                 for (int b = 0; b * 64 < s.cp; b++) umma_commit(bar_empty + 8 * b);
                 umma_commit(bar_o);
@@ -594,7 +623,10 @@ __global__ void __launch_bounds__(LV_T, 1)
     __syncthreads();
     if (c >= s.V) return;
     float d[4] = {};
-    w.times(d, pg_smem(sa), ld, lane);
+    if (group > 8)
+        w.times<true>(d, pg_smem(sa), ld, lane);
+    else
+        w.times<false>(d, pg_smem(sa), ld, lane);
 #pragma unroll
     for (int half = 0; half < 2; half++) {
         const int x = r + 8 * half, m = m0 + x;
@@ -621,15 +653,19 @@ __global__ void __launch_bounds__(256)
         return;
     }
     const float *row = proj + (int64_t)m * ldp;
+    Turn turn;
+    turn.ask(s, pos, lane);
     for (int h = warp; h < s.H + s.own; h += 8) {
         if (h == s.H) {
-            append(s, row + s.at_kv, pos, cache + (slot * s.cap + pos) * s.ck, lane);
+            NormWeights nw;
+            nw.ask(s, lane);
+            append(s, row + s.at_kv, turn, nw, cache + (slot * s.cap + pos) * s.ck, lane);
         } else {
             const float *src = row + h * (s.D + s.R);
             bf16 *dst = q + ((int64_t)m * s.H + h) * qd;
             for (int c = 2 * lane; c < dn; c += 64)
                 *reinterpret_cast<uint32_t *>(dst + c) = pg_pack_bf16(c < s.D ? __ldcg(src + c) : 0.0f, c + 1 < s.D ? __ldcg(src + c + 1) : 0.0f);
-            rotate(s, src + s.D, pos, dst + dn, qd - dn, lane);
+            rotate(s, src + s.D, turn, dst + dn, qd - dn, lane);
         }
     }
 }
@@ -663,13 +699,23 @@ __global__ void __launch_bounds__(128)
     }
     if (h == s.H) {
         const int64_t slot = __ldcg(bt.d_seq_slot + __ldcg(bt.d_row_seq + m));
-        if (threadIdx.x < 32) append(s, proj + (int64_t)m * ldp + s.at_kv, pos, cache + (slot * s.cap + pos) * s.ck, lane);
+        if (threadIdx.x < 32) {
+            Turn turn;
+            NormWeights nw;
+            turn.ask(s, pos, lane);
+            nw.ask(s, lane);
+            append(s, proj + (int64_t)m * ldp + s.at_kv, turn, nw, cache + (slot * s.cap + pos) * s.ck, lane);
+        }
         return;
     }
     const float *src = proj + (int64_t)m * ldp + h * (s.D + s.R);
     float *dst = qx + ((int64_t)m * s.H + h) * s.ck;
     for (int i = threadIdx.x; i < s.dk; i += 128) sm[i] = i < s.D ? __ldcg(src + i) : 0.0f;
-    if (threadIdx.x < 32) rotate(s, src + s.D, pos, dst + s.cp, s.rp, lane);
+    if (threadIdx.x < 32) {
+        Turn turn;
+        turn.ask(s, pos, lane);
+        rotate(s, src + s.D, turn, dst + s.cp, s.rp, lane);
+    }
     __syncthreads();
     for (int n = threadIdx.x; n < s.cp; n += 128) dst[n] = dot_row(s.uk + ((int64_t)h * s.cp + n) * s.dk, sm, s.dk);
 }
@@ -715,9 +761,9 @@ int slices(const pg_ctx *ctx, int64_t units, int64_t cap)
 int32_t check(const pg_latent *p, const pg_batch *batch, int64_t ldp, int64_t ldo)
 {
     PG_REQUIRE(p && batch && p->d_rot && p->d_uk && p->d_uv && p->d_q && (p->d_norm || !p->own), "latent attention: null pointer");
-    PG_REQUIRE(p->heads > 0 && p->dim > 0 && p->dim <= 512 && p->rot_dim >= 0 && p->rot_dim % 2 == 0 && p->vdim > 0 && p->kv_rank > 0 && p->kv_rank <= 512 &&
+    PG_REQUIRE(p->heads > 0 && p->dim > 0 && p->dim <= 512 && p->rot_dim >= 0 && p->rot_dim <= 128 && p->rot_dim % 2 == 0 && p->vdim > 0 && p->kv_rank > 0 && p->kv_rank <= 512 &&
                    p->cap > 0 && p->heads <= 65534,
-               "latent attention: bad shape (dim %d and latent %d at most 512, an even rot_dim %d)", p->dim, p->kv_rank, p->rot_dim);
+               "latent attention: bad shape (dim %d and latent %d at most 512, an even rot_dim %d at most 128)", p->dim, p->kv_rank, p->rot_dim);
     const LatentShape s = shape_of(p);
     PG_REQUIRE(s.ck <= 640, "latent attention: a key of %d and %d columns is too wide", s.C, s.R);
     PG_REQUIRE(ldp >= s.at_gate + (int64_t)s.H * s.V && ldo >= (int64_t)s.H * s.V, "latent attention: rows too short");

@@ -71,6 +71,8 @@ __device__ __forceinline__ float pg_get(const bf16 *p)
     const unsigned short b = __ldcg(reinterpret_cast<const unsigned short *>(p));
     return __uint_as_float((uint32_t)b << 16);
 }
+__device__ __forceinline__ float pg_get_plain(const float *p) { return *p; }   // (shared memory)
+__device__ __forceinline__ float pg_get_plain(const bf16 *p) { return __uint_as_float((uint32_t)*reinterpret_cast<const unsigned short *>(p) << 16); }
 __device__ __forceinline__ uint32_t pg_pack_bf16(float lo, float hi)
 {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);

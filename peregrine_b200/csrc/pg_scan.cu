@@ -7,13 +7,14 @@
 //   scan_step_kernel    one token per sequence: W_dt, softplus, update, read-out and gate in one launch; the state is read and
 //                       written once
 //   scan_run_kernel     portions: a CTA has 32 channels of a sequence, four lanes per channel, whose states stay in registers;
-//                       step sizes, inputs, B and C come in tiles of tokens through shared memory, brought and finished by
-//                       four more warps.  It also stores the convolution inputs that the next portion needs.
+//                       step sizes, inputs, B and C come in tiles of tokens through a ring in shared memory, brought and
+//                       finished by four more warps.  It also stores the convolution inputs that the next portion needs.
 //
 // Convolution inputs are kept per slot in a ring of `taps` entries, position p in entry p mod taps: a single token writes an
 // entry that nobody reads any more.  A sequence starts at position 0: what its slot holds is then taken as zero.
 #include <algorithm>
 
+#include "pg_async.cuh"
 #include "pg_lm.cuh"
 
 namespace {
@@ -239,16 +240,29 @@ __global__ void __launch_bounds__(SR_T, NC == 1 ? 6 : 1)
         xv[r] = slot[r] >= 0 ? pg_get(x + (int64_t)(m0 + r) * ldx + c) : 0.0f;
         z[r] = slot[r] >= 0 ? __ldcg(proj + (int64_t)(m0 + r) * ldp + s.inner + c) : 0.0f;
     }
+    // the low-rank rows, all copies in flight together
+    const uint32_t at_dt = pg_smem(sdt), at_bc = pg_smem(sbc);
+    const bool quads_fit = s.N % 4 == 0 && ldl % 4 == 0;
 #pragma unroll
     for (int r = 0; r < R; r++) {
         const bool on = m0 + r < bt.rows;
-        const float *src = low + (int64_t)(m0 + r) * ldl;
-        for (int k = tid; k < s.dtp; k += SR_T) sdt[r * s.dtp + k] = on ? __ldcg(src + k) : 0.0f;
-        for (int k = tid; k < 2 * NP; k += SR_T) {
-            const int which = k / NP, n = k - which * NP;
-            sbc[r * 2 * NP + k] = on && n < s.N ? __ldcg(src + s.dtp + which * s.N + n) : 0.0f;
+        const float *src = low + (on ? (int64_t)(m0 + r) * ldl : 0);
+        if (quads_fit) {
+            for (int k = tid * 4; k < s.dtp; k += SR_T * 4) pg_cp_in<16>(at_dt + (r * s.dtp + k) * 4, src + k, on);
+            for (int k = tid * 4; k < 2 * NP; k += SR_T * 4) {
+                const int which = k / NP, n = k - which * NP;
+                pg_cp_in<16>(at_bc + (r * 2 * NP + k) * 4, src + (n < s.N ? s.dtp + which * s.N + n : 0), on && n < s.N);
+            }
+        } else {
+            for (int k = tid; k < s.dtp; k += SR_T) sdt[r * s.dtp + k] = on ? __ldcg(src + k) : 0.0f;
+            for (int k = tid; k < 2 * NP; k += SR_T) {
+                const int which = k / NP, n = k - which * NP;
+                sbc[r * 2 * NP + k] = on && n < s.N ? __ldcg(src + s.dtp + which * s.N + n) : 0.0f;
+            }
         }
     }
+    pg_cp_commit();
+    pg_cp_wait<0>();
     __syncthreads();
     float acc[R] = {};
     auto dot = [&](const uint4 &b, int k) {
@@ -282,33 +296,26 @@ __global__ void __launch_bounds__(SR_T, NC == 1 ? 6 : 1)
     }
 }
 
-// an element of a step's type before its conversion
-template <typename TA>
-struct Raw;
-template <>
-struct Raw<float> {
-    float v;
-    __device__ __forceinline__ void load(const float *p, bool in) { v = in ? __ldcg(p) : 0.0f; }
-    __device__ __forceinline__ float value() const { return v; }
-};
-template <>
-struct Raw<bf16> {
-    unsigned short v;
-    __device__ __forceinline__ void load(const bf16 *p, bool in) { v = in ? __ldcg(reinterpret_cast<const unsigned short *>(p)) : (unsigned short)0; }
-    __device__ __forceinline__ float value() const { return __uint_as_float((uint32_t)v << 16); }
+// Bytes of one tile as it is brought: dt and z [TT][32] f32, x [TT][32] in the step's type, B and C [TT][2][16 NC] f32.
+template <int NC, typename TA>
+struct ScanTile {
+    static constexpr int NP = 16 * NC, TT = NC > 4 ? 4 : 16;
+    static constexpr int Z = TT * SR_CH * 4, X = 2 * Z, BC = X + TT * SR_CH * (int)sizeof(TA), BYTES = BC + TT * 2 * NP * 4;
+    static constexpr int DEPTH = 6;      // tiles in shared memory: one being finished, one being run, one being converted, three on their way
 };
 
-// grid (ceil(inner / 32), seqs), eight warps.  Tiles of TT tokens, two buffers: while warps 0 .. 3 run tile i through the
-// states, warps 4 .. 7 finish the outputs of tile i - 1, turn the raw step sizes of tile i + 1 into what the recurrence
-// takes, and ask for the inputs of tile i + 2.
-template <int NC, typename TA>
+// grid (ceil(inner / 32), seqs), eight warps.  While warps 0 .. 3 run tile i through the states, warps 4 .. 7 finish the outputs
+// of tile i - 1, turn the raw step sizes of tile i + 1 into what the recurrence takes, and ask for tile i + 5 where tile i - 1 lay.
+// VEC: rows and channels allow copies of 16 bytes.
+template <int NC, typename TA, bool VEC>
 __global__ void __launch_bounds__(2 * SR_T)
     scan_run_kernel(const ScanShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, float *ring, const TA *__restrict__ x, int64_t ldx,
                     const float *__restrict__ dt, int64_t ldt, const float *__restrict__ bc, int64_t ldb, float *state, TA *__restrict__ out, int64_t ldo)
 {
-    constexpr int NP = 16 * NC, TT = NC > 4 ? 4 : 16, PER = TT * SR_CH / SR_T, PERB = TT * 2 * NP / SR_T;
+    using Tile = ScanTile<NC, TA>;
+    constexpr int NP = Tile::NP, TT = Tile::TT, DEPTH = Tile::DEPTH, PER = TT * SR_CH / SR_T;
+    extern __shared__ __align__(16) float sm[];            // [DEPTH] tiles
     __shared__ __align__(16) float4 sd[2][TT][SR_CH];      // dt, dt, dt x, dt x
-    __shared__ __align__(16) float sbc[2][TT][2][NP];
     __shared__ float sy[2][TT][SR_CH];
     pg_pdl_begin();
     const bool aux = threadIdx.x >= SR_T;
@@ -317,70 +324,91 @@ __global__ void __launch_bounds__(2 * SR_T)
     if (T <= 0) return;
     const int pos0 = __ldcg(bt.d_pos + row0), tiles = (T + TT - 1) / TT;
     const int64_t slot = __ldcg(bt.d_seq_slot + seq);
+    const unsigned char *raw = reinterpret_cast<const unsigned char *>(sm);
     if (aux) {
         // tokens tid / 32 + 4 i of channel tid % 32
-        const int ec = c0 + (tid & 31), et = tid >> 5;
+        const int cx = tid & 31, ec = c0 + cx, et = tid >> 5;
         const bool on = ec < s.inner;
         const float dt_bias = on ? __ldg(s.dt_bias + ec) : 0.0f, skip = on ? __ldg(s.d + ec) : 0.0f;
-        float rdt[PER], rz[PER], rbc[PERB], x1[PER], z1[PER], x2[PER], z2[PER];
-        Raw<TA> rx[PER];                                  // (as loaded: nothing waits for a load before its tile is converted)
-        // (a tile's B and C lie in a fixed order of tokens and states: element tid + i SR_T)
-        auto fetch = [&](int t0) {
+        const uint32_t sm_at = pg_smem(sm);
+        auto fetch = [&](int tile) {
+            const uint32_t at = sm_at + (uint32_t)(tile % DEPTH) * Tile::BYTES;
+            const int t0 = tile * TT;
+            constexpr int V = VEC ? 4 : 1;                 // f32 elements of a copy
 #pragma unroll
-            for (int i = 0; i < PER; i++) {
-                const int t = t0 + et + i * (SR_T / 32);
-                const bool in = on && t < T;
-                const int64_t m = row0 + t;
-                rdt[i] = in ? __ldcg(dt + m * ldt + ec) : 0.0f;
-                rx[i].load(x + m * ldx + ec, in);
-                rz[i] = in ? __ldcg(proj + m * ldp + s.inner + ec) : 0.0f;
+            for (int e = tid * V; e < TT * SR_CH; e += SR_T * V) {
+                const int t = e / SR_CH, c = e % SR_CH;
+                const bool in = t0 + t < T && c0 + c < s.inner;
+                const int64_t m = in ? row0 + t0 + t : row0;
+                const int64_t ch = in ? c0 + c : 0;
+                pg_cp_in<4 * V>(at + e * 4, dt + m * ldt + ch, in);
+                pg_cp_in<4 * V>(at + Tile::Z + e * 4, proj + m * ldp + s.inner + ch, in);
+            }
+            constexpr int VX = VEC ? 16 / (int)sizeof(TA) : 4 / (int)sizeof(TA);
+#pragma unroll
+            for (int e = tid * VX; e < TT * SR_CH; e += SR_T * VX) {
+                const int t = e / SR_CH, c = e % SR_CH;
+                const bool in = t0 + t < T && c0 + c < s.inner;   // (a pair may reach one column behind the last channel: ldx is even)
+                pg_cp_in<VX * (int)sizeof(TA)>(at + Tile::X + e * (int)sizeof(TA), x + (in ? (row0 + t0 + t) * ldx + c0 + c : 0), in);
             }
 #pragma unroll
-            for (int i = 0; i < PERB; i++) {
-                const int e = tid + i * SR_T, t = t0 + e / (2 * NP), k = e % (2 * NP), which = k / NP, n = k - which * NP;
-                rbc[i] = t < T && n < s.N ? __ldcg(bc + (int64_t)(row0 + t) * ldb + which * s.N + n) : 0.0f;
+            for (int e = tid * V; e < TT * 2 * NP; e += SR_T * V) {
+                const int t = e / (2 * NP), k = e % (2 * NP), which = k / NP, n = k - which * NP;
+                const bool in = t0 + t < T && n < s.N;
+                pg_cp_in<4 * V>(at + Tile::BC + e * 4, bc + (in ? (int64_t)(row0 + t0 + t) * ldb + which * s.N + n : 0), in);
             }
+            pg_cp_commit();
         };
+        auto x_of = [&](const unsigned char *at, int t) { return pg_get_plain(reinterpret_cast<const TA *>(at + Tile::X) + t * SR_CH + cx); };
         auto convert = [&](int tile) {
-            const int b = tile & 1;
+            const unsigned char *at = raw + (size_t)(tile % DEPTH) * Tile::BYTES;
 #pragma unroll
             for (int i = 0; i < PER; i++) {
                 const int t = et + i * (SR_T / 32);
                 // (tokens behind the end leave the state alone: exp(0) S + 0)
-                const float d = on && tile * TT + t < T ? softplus(rdt[i] + dt_bias) : 0.0f, xi = rx[i].value(), u = d * xi;
-                sd[b][t][tid & 31] = make_float4(d, d, u, u);
-                x2[i] = xi;
-                z2[i] = rz[i];
+                const float r = reinterpret_cast<const float *>(at)[t * SR_CH + cx];
+                const float d = on && tile * TT + t < T ? softplus(r + dt_bias) : 0.0f, u = d * x_of(at, t);
+                sd[tile & 1][t][cx] = make_float4(d, d, u, u);
             }
-#pragma unroll
-            for (int i = 0; i < PERB; i++) (&sbc[b][0][0][0])[tid + i * SR_T] = rbc[i];
         };
         auto finish = [&](int tile) {
+            const unsigned char *at = raw + (size_t)(tile % DEPTH) * Tile::BYTES;
 #pragma unroll
             for (int i = 0; i < PER; i++) {
                 const int t = et + i * (SR_T / 32);
-                if (on && tile * TT + t < T)
-                    pg_put(out + (int64_t)(row0 + tile * TT + t) * ldo + ec, fmaf(skip, x1[i], sy[tile & 1][t][tid & 31]) * pg_silu(z1[i]));
+                const float z = reinterpret_cast<const float *>(at + Tile::Z)[t * SR_CH + cx];
+                const float y = fmaf(skip, x_of(at, t), sy[tile & 1][t][cx]) * pg_silu(z);
+                if (on && tile * TT + t < T) pg_put(out + (int64_t)(row0 + tile * TT + t) * ldo + ec, y);
             }
         };
-        auto shift = [&]() {
-#pragma unroll
-            for (int i = 0; i < PER; i++) x1[i] = x2[i], z1[i] = z2[i];
+        // (the warps of this half meet on their own where one has copied what another reads)
+        auto landed = [&]() {
+            pg_cp_wait<DEPTH - 3>();
+            asm volatile("bar.sync 1, 128;" ::: "memory");
         };
-        fetch(0);
+        // one group of copies per tile, empty behind the end, so that the wait counts tiles
+        for (int i = 0; i < DEPTH - 1; i++) {
+            if (i < tiles)
+                fetch(i);
+            else
+                pg_cp_commit();
+        }
+        pg_cp_wait<DEPTH - 2>();
+        asm volatile("bar.sync 1, 128;" ::: "memory");
         convert(0);
-        fetch(TT);
         for (int i = 0; i < tiles; i++) {
             __syncthreads();                              // tile i may be run; tile i - 1 has been
             if (i > 0) finish(i - 1);
-            shift();
-            if (i + 1 < tiles) {
-                convert(i + 1);
-                fetch((i + 2) * TT);
-            }
+            landed();                                     // tile i + 1; tile i - 1 is finished everywhere
+            if (i + 1 < tiles) convert(i + 1);
+            if (i + DEPTH - 1 < tiles)
+                fetch(i + DEPTH - 1);
+            else
+                pg_cp_commit();
         }
         __syncthreads();
         finish(tiles - 1);
+        pg_cp_wait<0>();
         // the inputs that the next portion's convolution reads (scan_conv_kernel is done with the old ones)
         if (on)
             for (int t = max(0, T - s.taps) + et; t < T; t += SR_T / 32)
@@ -400,6 +428,7 @@ __global__ void __launch_bounds__(2 * SR_T)
     for (int i = 0; i < tiles; i++) {
         __syncthreads();
         const int b = i & 1;
+        const float *sbc = reinterpret_cast<const float *>(raw + (size_t)(i % DEPTH) * Tile::BYTES + Tile::BC);
         float y[TT];
 #pragma unroll
         for (int t = 0; t < TT; t += 4) {
@@ -410,8 +439,8 @@ __global__ void __launch_bounds__(2 * SR_T)
                 Quad e[4], g[4], c4[4];
 #pragma unroll
                 for (int u = 0; u < 4; u++) {
-                    const Quad d = load_quad(reinterpret_cast<const float *>(&sd[b][t + u][cl])), bb = load_quad(&sbc[b][t + u][0][(q + 4 * n) * 4]);
-                    c4[u] = load_quad(&sbc[b][t + u][1][(q + 4 * n) * 4]);
+                    const Quad d = load_quad(reinterpret_cast<const float *>(&sd[b][t + u][cl])), bb = load_quad(sbc + (t + u) * 2 * NP + (q + 4 * n) * 4);
+                    c4[u] = load_quad(sbc + (t + u) * 2 * NP + NP + (q + 4 * n) * 4);
                     e[u] = {mul2(d.lo, a[n].lo), mul2(d.lo, a[n].hi)};
                     g[u] = {mul2(d.hi, bb.lo), mul2(d.hi, bb.hi)};
                 }
@@ -499,12 +528,24 @@ int32_t run_scan(pg_ctx *ctx, const ScanShape &s, const pg_batch *bt, const floa
                  int64_t ldt, const float *bc, int64_t ldb, float *state, TA *out, int64_t ldo)
 {
     const dim3 grid((unsigned)((s.inner + SR_CH - 1) / SR_CH), (unsigned)bt->seqs);
-#define PG_SR(NC) return launch_whole(ctx, scan_run_kernel<NC, TA>, grid, dim3(2 * SR_T), 0, s, *bt, proj, ldp, ring, x, ldx, dt, ldt, bc, ldb, state, out, ldo)
-    if (s.N <= 16) PG_SR(1);
-    if (s.N <= 32) PG_SR(2);
-    if (s.N <= 64) PG_SR(4);
-    if (s.N <= 128) PG_SR(8);
-    PG_SR(16);
+    PG_REQUIRE(ldx % 2 == 0 && ((uintptr_t)x & 3) == 0, "scan: rows of x start on 4-byte boundaries");
+    const bool vec = s.inner % 8 == 0 && s.N % 4 == 0 && ldt % 4 == 0 && ldp % 4 == 0 && ldb % 4 == 0 && ldx % 8 == 0 &&
+                     (((uintptr_t)dt | (uintptr_t)proj | (uintptr_t)bc | (uintptr_t)x) & 15) == 0;
+    auto go = [&](auto kern, std::atomic<uint64_t> &set, int smem) -> int32_t {
+        PG_CUDA(pg_max_smem_once(kern, smem, ctx->device, set));
+        return launch_whole(ctx, kern, grid, dim3(2 * SR_T), (size_t)smem, s, *bt, proj, ldp, ring, x, ldx, dt, ldt, bc, ldb, state, out, ldo);
+    };
+#define PG_SR(NC, I)                                                                                                    \
+    do {                                                                                                                \
+        constexpr int smem = ScanTile<NC, TA>::DEPTH * ScanTile<NC, TA>::BYTES;                                         \
+        return vec ? go(scan_run_kernel<NC, TA, true>, set[2 * I], smem) : go(scan_run_kernel<NC, TA, false>, set[2 * I + 1], smem); \
+    } while (0)
+    static std::atomic<uint64_t> set[10] = {};
+    if (s.N <= 16) PG_SR(1, 0);
+    if (s.N <= 32) PG_SR(2, 1);
+    if (s.N <= 64) PG_SR(4, 2);
+    if (s.N <= 128) PG_SR(8, 3);
+    PG_SR(16, 4);
 #undef PG_SR
 }
 
