@@ -396,13 +396,14 @@ def bubotar_kernel_figures(torch, gpu, hbm: float, tflops: float) -> dict:
             e.update(tflops=flops / us * 1e-6, frac_of_bf16_peak=flops / us * 1e-6 / tflops)
 
     rnd = lambda *s: torch.randn(*s, device=dev, dtype=torch.bfloat16) * s[-1] ** -0.5
-    for name, n, k, gated in (("scan_in", 16384, N, False), ("scan_low", 288, 8192, False), ("scan_dt", 8192, 256, False), ("latent_proj", 10816, N, False),
+    for name, n, k, gated in (("scan_in", 16384, N, False), ("scan_low", 288, 8192, False), ("scan_low_dt", 256, 8192, False), ("scan_low_bc", 32, 8192, False), ("scan_dt", 8192, 256, False), ("latent_proj", 10816, N, False),
                               ("latent_unfold", 8192, 512, False), ("o", N, 4096, False), ("scan_o", N, 8192, False), ("gate_up", 28672, N, True),
                               ("down", N, 14336, False)):
         ls = [Linear(d, (rnd(n // 2, k), rnd(n // 2, k)) if gated else rnd(n, k), gated=gated) for _ in range(min(80, max(2, int(400e6 / (n * k * 2)) + 1)))]
-        for M in (1, 16, 64, T):
+        # (decoding takes the low-rank product whole, prompts in its two parts)
+        for M in {"scan_low": (1, 16), "scan_low_dt": (64, T), "scan_low_bc": (64, T), "scan_dt": (64, T), "latent_unfold": (T,)}.get(name, (1, 16, 64, T)):
             a = torch.randn(M, k, device=dev).to(torch.bfloat16)
-            narrow = gated or name == "latent_unfold"
+            narrow = gated or name in ("latent_unfold", "scan_low_dt")
             y = torch.zeros(M, n // 2 if gated else n, device=dev, dtype=torch.bfloat16 if narrow else torch.float32)
             torch.cuda.synchronize()
             act = _lib.ACT_CLAMPED_SWISH_GLU if gated else _lib.ACT_NONE

@@ -148,32 +148,37 @@ __global__ void __launch_bounds__(AT_THREADS, 1)
             }
         }
     } else if (warp == 9) {
-        // ---------------------------------------------------------------- MMA issuer
-        if (lane == 0 && most > 0) {
+        // ---------------------------------------------------------------- MMA issuer (the whole warp; one lane's products count)
+        if (most > 0) {
+            const uint32_t on = pg_elect();
             constexpr uint32_t idesc_s = make_idesc(TQ, TKEYS), idesc_o = make_idesc(TQ, DV) | IDESC_B_MN_MAJOR;
             int at = 0, phase = 0;
-            auto wait_full = [&]() { return pg_mbar_wait(bar_full + 8 * at, phase, abort_flag, status, limit_ns); };
+            auto wait = [&](uint32_t bar, uint32_t parity) { return (bool)__all_sync(0xffffffffu, pg_mbar_wait(bar, parity, abort_flag, status, limit_ns)); };
+            auto wait_full = [&]() { return wait(bar_full + 8 * at, phase); };
             auto advance = [&]() {
                 if (++at == SLOTS) {
                     at = 0;
                     phase ^= 1;
                 }
             };
+            // (descriptors of other addresses: only the address field, 16 bytes to one, differs)
+            const uint64_t desc_q = make_smem_desc(sq), desc_ring = make_smem_desc(ring), desc_v = make_smem_desc_mn(ring, BLOCK);
             auto scores = [&](int t, int k_slot) {
-                const uint32_t kt = ring + k_slot * C::SLOT, qt = sq + t * C::Q_BYTES;
+                const uint64_t kt = desc_ring + (uint64_t)(k_slot * (C::SLOT >> 4)), qt = desc_q + (uint64_t)(t * (C::Q_BYTES >> 4));
 #pragma unroll
                 for (int i = 0; i < DK / 16; i++) {
-                    const uint32_t off = (i / 4) * BLOCK + (i % 4) * 32;
-                    umma_f16(tmem + t * 128, make_smem_desc(qt + off), make_smem_desc(kt + off), idesc_s, i != 0);
+                    constexpr int block = BLOCK >> 4;
+                    const uint64_t off = (uint64_t)((i / 4) * block + (i % 4) * 2);
+                    umma_f16(tmem + t * 128, qt + off, kt + off, idesc_s, i != 0, on);
                 }
-                umma_commit(bar_s + 8 * t);
+                umma_commit(bar_s + 8 * t, on);
             };
-            bool ok = pg_mbar_wait(bar_q, 0, abort_flag, status, limit_ns) && wait_full();
+            bool ok = wait(bar_q, 0) && wait_full();
             tc_fence_after();
             if (ok) {
                 for (int t = 0; t < 2; t++)
                     if (tiles[t] > 0) scores(t, at);
-                umma_commit(bar_empty + 8 * at);
+                umma_commit(bar_empty + 8 * at, on);
                 advance();
             }
             for (int j = 0; ok && j < most; j++) {
@@ -184,12 +189,12 @@ __global__ void __launch_bounds__(AT_THREADS, 1)
                 bool next = false;                      // the next keys have arrived
                 for (int t = 0; ok && t < 2; t++) {
                     if (j >= tiles[t]) continue;
-                    if (!(ok = pg_mbar_wait(bar_p + 8 * t, j & 1, abort_flag, status, limit_ns))) break;
+                    if (!(ok = wait(bar_p + 8 * t, j & 1))) break;
                     tc_fence_after();
-                    const uint32_t vt = ring + v_slot * C::SLOT;
+                    const uint64_t vt = desc_v + (uint64_t)(v_slot * (C::SLOT >> 4));
 #pragma unroll
                     for (int i = 0; i < TKEYS / 16; i++)
-                        umma_f16_ta(tmem + 256 + t * 128, tmem + t * 128 + i * 8, make_smem_desc_mn(vt + i * 2048, BLOCK), idesc_o, (j | i) != 0);
+                        umma_f16_ta(tmem + 256 + t * 128, tmem + t * 128 + i * 8, vt + i * (2048 >> 4), idesc_o, (j | i) != 0, on);
                     if (j + 1 < tiles[t]) {
                         if (!next) {
                             if (!(ok = wait_full())) break;
@@ -198,13 +203,13 @@ __global__ void __launch_bounds__(AT_THREADS, 1)
                         }
                         scores(t, at);
                     } else {
-                        umma_commit(bar_o + 8 * t);
+                        umma_commit(bar_o + 8 * t, on);
                     }
                 }
                 if (!ok) break;
-                umma_commit(bar_empty + 8 * v_slot);
+                umma_commit(bar_empty + 8 * v_slot, on);
                 if (next) {
-                    umma_commit(bar_empty + 8 * at);
+                    umma_commit(bar_empty + 8 * at, on);
                     advance();
                 }
             }

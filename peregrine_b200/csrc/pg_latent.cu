@@ -311,7 +311,7 @@ __global__ void __launch_bounds__(LA_THREADS, 1)
     tc_fence_after();
     // (not before the CTA has its TMEM: nothing behind this kernel can then hold what it needs)
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-    const uint32_t tmem_s = tmem_slot, tmem_o = tmem_s + 32;
+    const uint32_t tmem_s = tmem_slot, tmem_o = tmem_s + LA_ROWS;
 
     if (warp == 4) {
         // ---------------------------------------------------------------- producer
@@ -331,6 +331,9 @@ __global__ void __launch_bounds__(LA_THREADS, 1)
                     pg_mbar_expect(bar_full + 8 * b, LA_BLOCK);
                     tma_load_3d(keys_at + b * LA_BLOCK, &map_k, bar_full + 8 * b, b * 64, key0, slot);
                 }
+                // the next tile on its way to L2 meanwhile
+                if (j + 1 < ntiles)
+                    for (int b = 0; b < nb; b++) tma_prefetch_3d(&map_k, b * 64, key0 + LA_KEYS, slot);
             }
             if (!waited) {
                 asm volatile("griddepcontrol.wait;" ::: "memory");
@@ -345,34 +348,36 @@ __global__ void __launch_bounds__(LA_THREADS, 1)
             }
         }
     } else if (warp == 5) {
-        // ---------------------------------------------------------------- MMA issuer
-        if (lane == 0) {
+        // ---------------------------------------------------------------- MMA issuer (the whole warp; one lane's products count)
+        {
+            const uint32_t on = pg_elect();
+            auto wait = [&](uint32_t bar, uint32_t parity) { return (bool)__all_sync(0xffffffffu, pg_mbar_wait(bar, parity, &abort_flag, status, limit_ns)); };
             constexpr uint32_t idesc_s = make_idesc(128, LA_ROWS), idesc_o = make_idesc(128, LA_ROWS) | IDESC_A_MN_MAJOR;
             const uint64_t desc_k = make_smem_desc(keys_at), desc_q = make_smem_desc(q_at), desc_p = make_smem_desc(p_at), desc_v = make_smem_desc_mn(keys_at, LA_BLOCK);
-            bool ok = pg_mbar_wait(bar_q, 0, &abort_flag, status, limit_ns);
+            bool ok = wait(bar_q, 0);
             tc_fence_after();
             for (int j = 0; ok && j < ntiles; j++) {
                 for (int b = 0; b < nb; b++) {
-                    if (!(ok = pg_mbar_wait(bar_full + 8 * b, j & 1, &abort_flag, status, limit_ns))) break;
+                    if (!(ok = wait(bar_full + 8 * b, j & 1))) break;
                     tc_fence_after();
                     const uint64_t dk = desc_k + (uint64_t)(b * (LA_BLOCK >> 4)), dq = desc_q + (uint64_t)(b * (LA_QBLOCK >> 4));
 #pragma unroll
-                    for (int i = 0; i < 4; i++) umma_f16(tmem_s, dk + i * 2, dq + i * 2, idesc_s, (b | i) != 0);
-                    if (b * 64 >= s.cp) umma_commit(bar_empty + 8 * b);   // no value columns: done with
+                    for (int i = 0; i < 4; i++) umma_f16(tmem_s, dk + i * 2, dq + i * 2, idesc_s, (b | i) != 0, on);
+                    if (b * 64 >= s.cp) umma_commit(bar_empty + 8 * b, on);   // no value columns: done with
                 }
                 if (!ok) break;
-                umma_commit(bar_s);
-                if (!(ok = pg_mbar_wait(bar_p, j & 1, &abort_flag, status, limit_ns))) break;
+                umma_commit(bar_s, on);
+                if (!(ok = wait(bar_p, j & 1))) break;
                 tc_fence_after();
                 for (int g = 0; g < ng; g++) {
-                    const uint64_t dv = desc_v + (uint64_t)(2 * g * (LA_BLOCK >> 4));
                     // (the last group of an odd number of blocks reads one block too many, into rows of O^T that nobody reads)
+                    const uint64_t dv = desc_v + (uint64_t)(2 * g * (LA_BLOCK >> 4));
 #pragma unroll
                     for (int i = 0; i < LA_KEYS / 16; i++)
-                        umma_f16(tmem_o + g * LA_ROWS, dv + i * (2048 >> 4), desc_p + (i / 4) * (LA_QBLOCK >> 4) + (i % 4) * 2, idesc_o, (j | i) != 0);
+                        umma_f16(tmem_o + g * LA_ROWS, dv + i * (2048 >> 4), desc_p + (i / 4) * (LA_QBLOCK >> 4) + (i % 4) * 2, idesc_o, (j | i) != 0, on);
+                    for (int b = 2 * g; b < 2 * g + 2 && b * 64 < s.cp; b++) umma_commit(bar_empty + 8 * b, on);
                 }
-                for (int b = 0; b * 64 < s.cp; b++) umma_commit(bar_empty + 8 * b);
-                umma_commit(bar_o);
+                umma_commit(bar_o, on);
             }
         }
     } else {
@@ -388,9 +393,9 @@ __global__ void __launch_bounds__(LA_THREADS, 1)
             ok = ok && pg_mbar_wait(bar_s, j & 1, &abort_flag, status, limit_ns);
             ok = __all_sync(0xffffffffu, ok);
             tc_fence_after();
+            const int key = t0 + j * LA_KEYS + warp * 32 + lane;
             uint32_t v[32];
             tmem_ld32(tmem_s + lanes, v);
-            const int key = t0 + j * LA_KEYS + warp * 32 + lane;
             float x[LA_ROWS];
 #pragma unroll
             for (int c = 0; c < LA_ROWS; c++) x[c] = __uint_as_float(v[c]) * sl2;
@@ -606,21 +611,25 @@ __global__ void __launch_bounds__(LV_T, 1)
                 a.x = fmaf(f, v[k].x, a.x), a.y = fmaf(f, v[k].y, a.y), a.z = fmaf(f, v[k].z, a.z), a.w = fmaf(f, v[k].w, a.w);
             }
         }
-        *reinterpret_cast<float4 *>(sums + (size_t)(way * group + x) * s.cp + k4) = a;
+        if (ways == 1)
+            *reinterpret_cast<uint2 *>(sa + x * ld + k4) = make_uint2(pg_pack_bf16(a.x, a.y), pg_pack_bf16(a.z, a.w));
+        else
+            *reinterpret_cast<float4 *>(sums + (size_t)(way * group + x) * s.cp + k4) = a;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < 16 * quads; i += LV_T) {
-        const int x = i / quads, k4 = (i - x * quads) * 4;
-        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (x < group) {
+    if (ways > 1) {
+        for (int i = threadIdx.x; i < group * quads; i += LV_T) {
+            const int x = i / quads, k4 = (i - x * quads) * 4;
+            float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
             for (int way = 0; way < ways; way++) {
                 const float4 u = *reinterpret_cast<const float4 *>(sums + (size_t)(way * group + x) * s.cp + k4);
                 a.x += u.x, a.y += u.y, a.z += u.z, a.w += u.w;
             }
+            *reinterpret_cast<uint2 *>(sa + x * ld + k4) = make_uint2(pg_pack_bf16(a.x, a.y), pg_pack_bf16(a.z, a.w));
         }
-        *reinterpret_cast<uint2 *>(sa + x * ld + k4) = make_uint2(pg_pack_bf16(a.x, a.y), pg_pack_bf16(a.z, a.w));
+        __syncthreads();
     }
-    __syncthreads();
+    // (rows behind the group are whatever the shared memory held: nobody reads their products)
     if (c >= s.V) return;
     float d[4] = {};
     if (group > 8)
@@ -655,12 +664,36 @@ __global__ void __launch_bounds__(256)
     const float *row = proj + (int64_t)m * ldp;
     Turn turn;
     turn.ask(s, pos, lane);
-    for (int h = warp; h < s.H + s.own; h += 8) {
-        if (h == s.H) {
-            NormWeights nw;
-            nw.ask(s, lane);
-            append(s, row + s.at_kv, turn, nw, cache + (slot * s.cap + pos) * s.ck, lane);
-        } else {
+    if (s.own && warp == 7) {
+        NormWeights nw;
+        nw.ask(s, lane);
+        append(s, row + s.at_kv, turn, nw, cache + (slot * s.cap + pos) * s.ck, lane);
+    }
+    if (s.D % 4 == 0 && s.D <= 128 && s.R % 2 == 0 && s.R <= 64 && (s.D + s.R) % 4 == 0 && ldp % 4 == 0) {
+        // four heads at a time, all their loads in flight
+        for (int h0 = warp; h0 < s.H; h0 += 32) {
+            float4 v[4];
+            float2 p[4];
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                const float *src = row + (h0 + 8 * i) * (s.D + s.R);
+                const bool in = h0 + 8 * i < s.H;
+                v[i] = in && 4 * lane < s.D ? __ldcg(reinterpret_cast<const float4 *>(src) + lane) : make_float4(0.f, 0.f, 0.f, 0.f);
+                p[i] = in && 2 * lane < s.R ? __ldcg(reinterpret_cast<const float2 *>(src + s.D) + lane) : make_float2(0.f, 0.f);
+            }
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                if (h0 + 8 * i >= s.H) break;
+                bf16 *dst = q + ((int64_t)m * s.H + h0 + 8 * i) * qd;
+                if (4 * lane < dn) *reinterpret_cast<uint2 *>(dst + 4 * lane) = make_uint2(pg_pack_bf16(v[i].x, v[i].y), pg_pack_bf16(v[i].z, v[i].w));
+                if (2 * lane < qd - dn)
+                    *reinterpret_cast<uint32_t *>(dst + dn + 2 * lane) = pg_pack_bf16(p[i].x * turn.r[0].x - p[i].y * turn.r[0].y, p[i].y * turn.r[0].x + p[i].x * turn.r[0].y);
+            }
+        }
+        return;
+    }
+    for (int h = warp; h < s.H; h += 8) {
+        {
             const float *src = row + h * (s.D + s.R);
             bf16 *dst = q + ((int64_t)m * s.H + h) * qd;
             for (int c = 2 * lane; c < dn; c += 64)
@@ -847,7 +880,7 @@ PG_API int32_t pg_latent_run(pg_ctx *ctx, const pg_latent *p, const pg_batch *ba
     const int ways = std::max(1, std::min(8, LV_T / (group * s.cp / 4)));
     const int64_t groups = (batch->rows + group - 1) / group;
     PG_REQUIRE(groups <= 65535 && parts128 <= 65535, "latent attention: too many rows");
-    const size_t smem = (size_t)16 * (s.cp + 8) * 2 + (size_t)ways * group * s.cp * 4;
+    const size_t smem = (size_t)16 * (s.cp + 8) * 2 + (ways > 1 ? (size_t)ways * group * s.cp * 4 : 0);
     static std::atomic<uint64_t> set{0};
     PG_CUDA(pg_max_smem_once(latent_value_kernel, 64 * 1024, ctx->device, set));
     return launch_pdl(ctx, latent_value_kernel, dim3((unsigned)s.H, parts128, (unsigned)groups), dim3(LV_T), smem, s, *batch, (const float *)p->d_part, per_seq, S,

@@ -181,32 +181,33 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
             }
         }
     } else if (warp == 1) {
-        // ---------------------------------------------------------------- MMA issuer
-        if (lane == 0) {
+        // ---------------------------------------------------------------- MMA issuer (the whole warp; one lane's products count)
+        {
+            const uint32_t on = pg_elect();
             constexpr uint32_t idesc = make_idesc(BM, BN);
             uint32_t stage = 0, phase = 0, acc = 0, acc_phase = 0;
             bool ok = true;
             for (int u = blockIdx.x; ok && u < total; u += gridDim.x) {
-                if (!(ok = pg_mbar_wait(bar_tempty + 8 * acc, acc_phase ^ 1, abort_flag, status, limit_ns))) break;
+                if (!(ok = __all_sync(0xffffffffu, pg_mbar_wait(bar_tempty + 8 * acc, acc_phase ^ 1, abort_flag, status, limit_ns)))) break;
                 tc_fence_after();
                 const uint32_t d_tmem = tmem_base + acc * BN;
                 const int first = k_first(u), end = k_end(u);
                 for (int kb = first; kb < end; kb++) {
-                    if (!(ok = pg_mbar_wait(bar_full + 8 * stage, phase, abort_flag, status, limit_ns))) break;
+                    if (!(ok = __all_sync(0xffffffffu, pg_mbar_wait(bar_full + 8 * stage, phase, abort_flag, status, limit_ns)))) break;
                     tc_fence_after();
                     const uint32_t sa = base + stage * C::STAGE;
                     const uint64_t da = make_smem_desc(sa), db = make_smem_desc(sa + C::STAGE_A);
 #pragma unroll
                     for (int j = 0; j < BKB / UMMA_KB; j++)
-                        umma_f16(d_tmem, da + (uint64_t)(j * (UMMA_KB >> 4)), db + (uint64_t)(j * (UMMA_KB >> 4)), idesc, kb != first || j != 0 ? 1u : 0u);
-                    umma_commit(bar_empty + 8 * stage);   // stage reusable once these MMAs have read it
+                        umma_f16(d_tmem, da + (uint64_t)(j * (UMMA_KB >> 4)), db + (uint64_t)(j * (UMMA_KB >> 4)), idesc, kb != first || j != 0 ? 1u : 0u, on);
+                    umma_commit(bar_empty + 8 * stage, on);   // stage reusable once these MMAs have read it
                     if (++stage == STAGES) {
                         stage = 0;
                         phase ^= 1;
                     }
                 }
                 if (!ok) break;
-                umma_commit(bar_tfull + 8 * acc);         // accumulator complete
+                umma_commit(bar_tfull + 8 * acc, on);         // accumulator complete
                 if (++acc == 2) {
                     acc = 0;
                     acc_phase ^= 1;
@@ -269,10 +270,16 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
                         float sum[32];
 #pragma unroll
                         for (int j = 0; j < 32; j++) sum[j] = __ldcg(slab + j * 32);
-                        for (int p = 1; p < sp; p++) {
-                            const float *at = slab + (int64_t)p * 4 * BN * 32;
+                        for (int p = 1; p < sp; p += 2) {  // (two slabs at a time: twice the loads in flight)
+                            const float *at = slab + (int64_t)p * 4 * BN * 32, *at2 = at + (p + 1 < sp ? (int64_t)4 * BN * 32 : 0);
+                            const float on = p + 1 < sp ? 1.0f : 0.0f;
+                            float a[32], b[32];
 #pragma unroll
-                            for (int j = 0; j < 32; j++) sum[j] += __ldcg(at + j * 32);
+                            for (int j = 0; j < 32; j++) a[j] = __ldcg(at + j * 32);
+#pragma unroll
+                            for (int j = 0; j < 32; j++) b[j] = __ldcg(at2 + j * 32);
+#pragma unroll
+                            for (int j = 0; j < 32; j++) sum[j] = fmaf(on, b[j], sum[j] + a[j]);
                         }
                         uint32_t v[32];
 #pragma unroll
@@ -344,13 +351,16 @@ int32_t dispatch(pg_ctx *ctx, pg_linear *lin, const bf16 *a, int64_t lda, int64_
     KParts kp = {1, kblocks, nullptr, nullptr};
     if (bn < 128 && rt.blocks == nullptr) {
         // narrow tiles read the rows of a over and over: K in parts of at least four blocks instead, if that fills the GPU too
+        // -- the widest tile that does, else the one with the most parts in all
+        int64_t best = std::min<int64_t>(tiles(bn), ctx->sm_count);
         for (int cand = lin->n > 64 ? 128 : lin->n > 32 ? 64 : 32; cand >= 32; cand /= 2) {
-            const int64_t most = std::min<int64_t>(ctx->sm_count / std::max<int64_t>(1, tiles(cand)), kblocks / 4);
-            if (most < 2 || tiles(cand) * most < ctx->sm_count * 3 / 4) continue;
+            const int64_t most = std::min<int64_t>({ctx->sm_count / std::max<int64_t>(1, tiles(cand)), kblocks / 4, 16});
+            if (most < 2 || (tiles(cand) * most < ctx->sm_count * 3 / 4 && tiles(cand) * most <= best)) continue;
+            best = tiles(cand) * most;
             bn = cand;
             kp.blocks = (kblocks + (int)most - 1) / (int)most;
             kp.parts = (kblocks + kp.blocks - 1) / kp.blocks;
-            break;
+            if (best >= ctx->sm_count * 3 / 4) break;
         }
         const size_t need = PG_LM_TICKET_BYTES + (size_t)tiles(bn) * kp.parts * BM * bn * sizeof(float);
         if (kp.parts > 1 && need > ctx->splitk_bytes) {

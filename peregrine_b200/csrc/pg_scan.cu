@@ -199,7 +199,7 @@ __device__ __forceinline__ float sum2(f32x2 v)
 // grid (ceil(inner / 32), ceil(rows / R)).  NC: quads of states per lane
 constexpr int SS_W = 8;                  // 16-byte pieces of a row of W_dt that a lane asks for ahead (rank up to 256)
 template <int NC, int R, typename TA>
-__global__ void __launch_bounds__(SR_T, NC == 1 ? 6 : 1)
+__global__ void __launch_bounds__(SR_T, NC == 1 ? (R == 8 ? 4 : 6) : 1)
     scan_step_kernel(const ScanShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, const TA *__restrict__ x, int64_t ldx,
                      const float *__restrict__ low, int64_t ldl, float *state, TA *__restrict__ out, int64_t ldo)
 {
@@ -516,6 +516,8 @@ template <typename TA>
 int32_t run_step(pg_ctx *ctx, const ScanShape &s, const pg_batch *bt, const float *proj, int64_t ldp, const TA *x, int64_t ldx, const float *low, int64_t ldl,
                  float *state, TA *out, int64_t ldo)
 {
+    // (a single wave of CTAs also for many channels)
+    if (s.N <= 16 && bt->rows > 4) return launch_step<1, 8, TA>(ctx, s, bt, proj, ldp, x, ldx, low, ldl, state, out, ldo);
     if (s.N <= 16) return launch_step<1, 4, TA>(ctx, s, bt, proj, ldp, x, ldx, low, ldl, state, out, ldo);
     if (s.N <= 32) return launch_step<2, 4, TA>(ctx, s, bt, proj, ldp, x, ldx, low, ldl, state, out, ldo);
     if (s.N <= 64) return launch_step<4, 2, TA>(ctx, s, bt, proj, ldp, x, ldx, low, ldl, state, out, ldo);
