@@ -50,10 +50,48 @@ __device__ __forceinline__ void head_norm(const float *src, const float *__restr
     }
 }
 
-// a CTA per token
+// four columns per lane, four heads per warp with their loads in flight together (widths up to 128, all multiples of four)
+__device__ __forceinline__ void put4(float *p, const float4 &v) { *reinterpret_cast<float4 *>(p) = v; }
+__device__ __forceinline__ void put4(bf16 *p, const float4 &v) { *reinterpret_cast<uint2 *>(p) = make_uint2(pg_pack_bf16(v.x, v.y), pg_pack_bf16(v.z, v.w)); }
+template <typename TA>
+__device__ __forceinline__ void prep_heads4(const AttnShape &s, const float *row, int64_t q_at, int64_t kv_at, float mul, TA *q, TA *kc, TA *vc, int warp, int lane)
+{
+    const int n = s.H + 2 * s.G, c = 4 * lane;
+    auto norm4 = [&](const float *w, bool in) { return w && in && c < s.D ? __ldg(reinterpret_cast<const float4 *>(w) + lane) : make_float4(1.f, 1.f, 1.f, 1.f); };
+    const float4 wq = norm4(s.qn, true), wk = norm4(s.kn, true);
+    for (int i0 = warp; i0 < n; i0 += 32) {
+        float4 x[4];
+#pragma unroll
+        for (int u = 0; u < 4; u++) {
+            const int i = i0 + 8 * u;
+            const float *src = i < s.H + s.G ? row + i * s.D : row + (int64_t)(s.H + s.G) * s.D + (int64_t)(i - s.H - s.G) * s.V;
+            x[u] = i < n && c < (i < s.H + s.G ? s.D : s.V) ? __ldcg(reinterpret_cast<const float4 *>(src) + lane) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int u = 0; u < 4; u++) {
+            const int i = i0 + 8 * u;
+            if (i >= n) break;
+            if (i >= s.H + s.G) {
+                if (c < s.vp) put4(vc + (kv_at + (int64_t)(i - s.H - s.G) * s.cap) * s.vp + c, x[u]);
+                continue;
+            }
+            const bool query = i < s.H;
+            float f = query ? mul : 1.0f;
+            float4 w = make_float4(1.f, 1.f, 1.f, 1.f);
+            if (query ? s.qn : s.kn) {
+                f *= __fdiv_rn(1.0f, sqrtf(__fdiv_rn(pg_warp_sum((x[u].x * x[u].x + x[u].y * x[u].y) + (x[u].z * x[u].z + x[u].w * x[u].w)), (float)s.D) + s.eps));
+                w = query ? wq : wk;
+            }
+            const float4 y = make_float4(x[u].x * f * w.x, x[u].y * f * w.y, x[u].z * f * w.z, x[u].w * f * w.w);
+            if (c < s.dp) put4(query ? q + (q_at + i) * s.dp + c : kc + (kv_at + (int64_t)(i - s.H) * s.cap) * s.dp + c, y);
+        }
+    }
+}
+
+// a CTA per token; wide: prep_heads4 fits
 template <typename TA>
 __global__ void __launch_bounds__(256)
-    attn_prep_kernel(const AttnShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, TA *__restrict__ q, TA *kc, TA *vc, int32_t *status)
+    attn_prep_kernel(const AttnShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, TA *__restrict__ q, TA *kc, TA *vc, int wide, int32_t *status)
 {
     pg_pdl_begin();
     const int m = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -66,6 +104,10 @@ __global__ void __launch_bounds__(256)
     const float *row = proj + (int64_t)m * ldp;
     const float mul = temperature(s, pos);
     const int at = attn_row(s, pos);
+    if (wide) {
+        prep_heads4(s, row, (int64_t)m * s.H, slot * s.G * s.cap + at, mul, q, kc, vc, warp, lane);
+        return;
+    }
     for (int i = warp; i < s.H + 2 * s.G; i += 8) {
         if (i < s.H) {
             head_norm(row + i * s.D, s.qn, s.D, s.dp, s.eps, mul, q + ((int64_t)m * s.H + i) * s.dp, lane);
@@ -719,16 +761,17 @@ PG_API int32_t pg_attention_run(pg_ctx *ctx, const pg_attention *p, const pg_bat
     PG_REQUIRE(s.G <= 65535 && batch->rows >= 0 && batch->seqs <= 65535, "attention: too many heads or sequences");
     if (batch->rows == 0) return PG_OK;
     const int M = batch->rows;
+    const int wide = s.D % 4 == 0 && s.V % 4 == 0 && s.D <= 128 && s.V <= 128 && ldp % 4 == 0 && ((uintptr_t)d_proj & 15) == 0;
     if (dtype == PG_F32) {
         int32_t rc = launch_pdl(ctx, attn_prep_kernel<float>, dim3((unsigned)M), dim3(256), 0, s, *batch, d_proj, ldp, (float *)p->d_q, (float *)d_kcache,
-                                (float *)d_vcache, ctx->d_status);
+                                (float *)d_vcache, wide, ctx->d_status);
         if (rc != PG_OK) return rc;
         return pgk_attention_f32(ctx, s, batch, (const float *)p->d_q, (const float *)d_kcache, (const float *)d_vcache, (float *)d_out, ldo);
     }
     bf16 *q = (bf16 *)p->d_q, *kc = (bf16 *)d_kcache, *vc = (bf16 *)d_vcache, *out = (bf16 *)d_out;
     const bool step = batch->max_len == 1, fused = step && s.rep <= 16;
     if (!fused) {
-        const int32_t rc = launch_pdl(ctx, attn_prep_kernel<bf16>, dim3((unsigned)M), dim3(256), 0, s, *batch, d_proj, ldp, q, kc, vc, ctx->d_status);
+        const int32_t rc = launch_pdl(ctx, attn_prep_kernel<bf16>, dim3((unsigned)M), dim3(256), 0, s, *batch, d_proj, ldp, q, kc, vc, wide, ctx->d_status);
         if (rc != PG_OK) return rc;
     }
     if (!step && pgk_attention_prompt_tc_supports(s, batch, p->slots, ldo, out)) return pgk_attention_prompt_tc(ctx, s, batch, p->slots, q, kc, vc, out, ldo);

@@ -37,13 +37,6 @@ struct AtCfg {
     static constexpr int SMEM = 2 * Q_BYTES + SLOTS * SLOT + 1024 + 256;
 };
 
-__device__ __forceinline__ float ex2(float x)
-{
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-
 // what the split form has beyond the plain one
 struct SplitArgs {
     int seq0, k_blocks;      // 64-column blocks of a key that come from map_k; the others come from map_s
@@ -262,7 +255,7 @@ __global__ void __launch_bounds__(AT_THREADS, 1)
                 const bool behind = top > m + 8.0f;
                 if (__any_sync(0xffffffffu, behind)) {
                     // (these scores were committed behind the previous keys' sums: O is at rest)
-                    const float f = behind ? ex2(m - top) : 1.0f;
+                    const float f = behind ? pg_ex2(m - top) : 1.0f;
                     if (behind) m = top;
                     l0 *= f;
                     l1 *= f;
@@ -283,7 +276,7 @@ __global__ void __launch_bounds__(AT_THREADS, 1)
 #pragma unroll
                 for (int i = 0; i < 32; i++) {
                     const int c = h * 2 + (i >> 4), e = (i & 15) * 2;
-                    const float a = ex2(fmaf(__uint_as_float(v[c][e]), sx, -m)), b = ex2(fmaf(__uint_as_float(v[c][e + 1]), sx, -m));
+                    const float a = pg_ex2(fmaf(__uint_as_float(v[c][e]), sx, -m)), b = pg_ex2(fmaf(__uint_as_float(v[c][e + 1]), sx, -m));
                     l0 += a;
                     l1 += b;
                     p[i] = pg_pack_bf16(a, b);
@@ -300,7 +293,7 @@ __global__ void __launch_bounds__(AT_THREADS, 1)
             ok = __all_sync(0xffffffffu, ok);
             tc_fence_after();
             float l = l0 + l1;
-            if (s.sink) l += ex2(-m);
+            if (s.sink) l += pg_ex2(-m);
             const float inv = __fdiv_rn(1.0f, l);
             const int head_at = (g * s.rep + rc % s.rep) * s.V;
             bf16 *dst = out + (int64_t)(row0 + rc / s.rep) * ldo + head_at;

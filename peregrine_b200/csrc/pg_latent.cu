@@ -24,13 +24,6 @@ namespace {
 
 constexpr float LOG2E = 1.4426950408889634f;
 
-__device__ __forceinline__ float pg_ex2(float x)
-{
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-
 struct LatentShape {
     int H, D, R, V, C;           // heads, unrotated and rotated query widths, value width, latent width
     int cp, rp, ck;              // C up to 64, R up to 16, and both: a row of the cache

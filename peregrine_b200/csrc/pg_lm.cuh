@@ -104,6 +104,13 @@ __device__ __forceinline__ float pg_glu(float g, float u, float limit)
     u = fminf(fmaxf(u, -limit), limit);
     return g * pg_sigmoid(1.702f * g) * (u + 1.0f);
 }
+// 2^x, within two units in the last place (results below 2^-126 become 0)
+__device__ __forceinline__ float pg_ex2(float x)
+{
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 __device__ __forceinline__ float pg_warp_sum(float v)
 {
 #pragma unroll

@@ -25,18 +25,11 @@ struct ScanShape {
     const bf16 *dt;
 };
 
-__device__ __forceinline__ float ex2(float x)
-{
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-
 // ln(1 + e^x) = max(x, 0) + ln(1 + e) with e = e^-|x| in (0, 1], and ln(1 + e) = 2 artanh(e / (2 + e)) by its power series:
 // the argument is at most 1/3, and what is left out is below 2^-26 of the sum.
 __device__ __forceinline__ float softplus(float x)
 {
-    const float e = ex2(-1.4426950408889634f * fabsf(x)), z = __fdividef(e, 2.0f + e), w = z * z;
+    const float e = pg_ex2(-1.4426950408889634f * fabsf(x)), z = __fdividef(e, 2.0f + e), w = z * z;
     float p = 1.0f / 15.0f;
     p = fmaf(p, w, 1.0f / 13.0f);
     p = fmaf(p, w, 1.0f / 11.0f);
@@ -180,7 +173,7 @@ __device__ __forceinline__ Quad load_quad(const float *p)   // shared memory
 __device__ __forceinline__ f32x2 ex2_pair(f32x2 v)
 {
     const float2 h = halves(v);
-    return pair(ex2(h.x), ex2(h.y));
+    return pair(pg_ex2(h.x), pg_ex2(h.y));
 }
 
 // A quad of states takes a token (dt and dt x in both halves); returns its part of the read-out.
