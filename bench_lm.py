@@ -424,7 +424,7 @@ def bubotar_kernel_figures(torch, gpu, hbm: float, tflops: float) -> dict:
     f32 = torch.float32
 
     # scan
-    mx = [SelectiveScan(d, cfg["layers"][0]["mixer"], Below(W, "l0.mix."), N) for _ in range(4)]
+    mx = [SelectiveScan(d, cfg["layers"][0]["mixer"], Below(W, "l0.mix."), N) for _ in range(16)]
     states = [m.new_state(pool) for m in mx]
     proj, mixed = torch.randn(T, mx[0].proj.n, device=dev), d.buffer("mixed", mx[0].out.k)
     x, low = d.buffer("scan.x", mx[0].low.k), d.buffer("scan.low", mx[0].low.n, dtype=f32)
@@ -444,7 +444,7 @@ def bubotar_kernel_figures(torch, gpu, hbm: float, tflops: float) -> dict:
     def scan(m, s, b):
         ck(lib.pg_scan_run(gh, C.byref(m.c), C.byref(b.c), ptr(proj), proj.stride(0), ptr(s["ring"]), ptr(x), x.stride(0), ptr(dt), dt.stride(0), ptr(bc),
                            bc.stride(0), ptr(s["state"]), ptr(mixed), d.code, mixed.stride(0)))
-    pairs = list(zip(mx, states)) * 3
+    pairs = list(zip(mx, states))
     for B, b in steps.items():
         note(f"scan.conv.b{B}", time_us([(lambda m=m, s=s: conv(m, s, b)) for m, s in pairs]), nbytes=B * I * (4 * 4 + 4 + 2))
         note(f"scan.step.b{B}", time_us([(lambda m=m, s=s: step(m, s, b)) for m, s in pairs]), nbytes=B * I * (2 * S * 4 + 8) + I * (256 * 2 + S * 4))

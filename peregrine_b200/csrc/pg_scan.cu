@@ -223,8 +223,12 @@ __global__ void __launch_bounds__(SR_T, NC == 1 ? (R == 8 ? 4 : 6) : 1)
 #pragma unroll
     for (int r = 0; r < R; r++) {
         const bool old = slot[r] >= 0 && __ldcg(bt.d_pos + m0 + r) > 0;
+        // (asked for before the position is there: at position 0 it is dropped)
 #pragma unroll
-        for (int i = 0; i < NC; i++) S[r][i] = quad(old && q + 4 * i < quads ? __ldcg(at(r) + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f));
+        for (int i = 0; i < NC; i++) {
+            const float4 v = slot[r] >= 0 && q + 4 * i < quads ? __ldcg(at(r) + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            S[r][i] = quad(old ? v : make_float4(0.f, 0.f, 0.f, 0.f));
+        }
     }
     asm volatile("griddepcontrol.wait;" ::: "memory");
     float xv[R], z[R];
@@ -257,24 +261,32 @@ __global__ void __launch_bounds__(SR_T, NC == 1 ? (R == 8 ? 4 : 6) : 1)
     pg_cp_commit();
     pg_cp_wait<0>();
     __syncthreads();
-    float acc[R] = {};
+    f32x2 sums[R];
+#pragma unroll
+    for (int r = 0; r < R; r++) sums[r] = pair(0.0f, 0.0f);
     auto dot = [&](const uint4 &b, int k) {
+        const f32x2 b0 = pair(pg_bf16_lo(b.x), pg_bf16_hi(b.x)), b1 = pair(pg_bf16_lo(b.y), pg_bf16_hi(b.y)), b2 = pair(pg_bf16_lo(b.z), pg_bf16_hi(b.z)),
+                    b3 = pair(pg_bf16_lo(b.w), pg_bf16_hi(b.w));
 #pragma unroll
         for (int r = 0; r < R; r++) {
-            const float4 *v = reinterpret_cast<const float4 *>(sdt + r * s.dtp + k * 32 + q * 8);
-            const float4 u0 = v[0], u1 = v[1];
-            acc[r] += (fmaf(pg_bf16_lo(b.x), u0.x, pg_bf16_hi(b.x) * u0.y) + fmaf(pg_bf16_lo(b.y), u0.z, pg_bf16_hi(b.y) * u0.w)) +
-                      (fmaf(pg_bf16_lo(b.z), u1.x, pg_bf16_hi(b.z) * u1.y) + fmaf(pg_bf16_lo(b.w), u1.z, pg_bf16_hi(b.w) * u1.w));
+            const float *v = sdt + r * s.dtp + k * 32 + q * 8;
+            const Quad u0 = load_quad(v), u1 = load_quad(v + 4);
+            sums[r] = fma2(b0, u0.lo, fma2(b1, u0.hi, fma2(b2, u1.lo, fma2(b3, u1.hi, sums[r]))));
         }
     };
     // (all in one stretch: behind the rank's last piece the weights are zero)
 #pragma unroll
     for (int k = 0; k < SS_W; k++) dot(w[k], k < pieces ? k : 0);
     for (int k = SS_W; k < pieces; k++) dot(__ldg(wrow + 4 * k), k);
+    float acc[R];
+#pragma unroll
+    for (int r = 0; r < R; r++) acc[r] = sum2(sums[r]);
+#pragma unroll
+    for (int r = 0; r < R; r++) acc[r] += __shfl_xor_sync(0xffffffffu, acc[r], 1);
+#pragma unroll
+    for (int r = 0; r < R; r++) acc[r] += __shfl_xor_sync(0xffffffffu, acc[r], 2);
 #pragma unroll
     for (int r = 0; r < R; r++) {
-        acc[r] += __shfl_xor_sync(0xffffffffu, acc[r], 1);
-        acc[r] += __shfl_xor_sync(0xffffffffu, acc[r], 2);
         const float dt = softplus(acc[r] + dt_bias), du = dt * xv[r];
         float y = 0.0f;
 #pragma unroll
