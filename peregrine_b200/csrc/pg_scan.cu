@@ -190,9 +190,9 @@ __device__ __forceinline__ float sum2(f32x2 v)
 }
 
 // grid (ceil(inner / 32), ceil(rows / R)).  NC: quads of states per lane
-constexpr int SS_W = 8;                  // 16-byte pieces of a row of W_dt that a lane asks for ahead (rank up to 256)
+constexpr int SS_W = 4;                  // 16-byte pieces of a row of W_dt that a lane has in flight together
 template <int NC, int R, typename TA>
-__global__ void __launch_bounds__(SR_T, NC == 1 ? (R == 8 ? 4 : 6) : 1)
+__global__ void __launch_bounds__(SR_T, NC == 1 ? 7 : 1)
     scan_step_kernel(const ScanShape s, const pg_batch bt, const float *__restrict__ proj, int64_t ldp, const TA *__restrict__ x, int64_t ldx,
                      const float *__restrict__ low, int64_t ldl, float *state, TA *__restrict__ out, int64_t ldo)
 {
@@ -277,7 +277,12 @@ __global__ void __launch_bounds__(SR_T, NC == 1 ? (R == 8 ? 4 : 6) : 1)
     // (all in one stretch: behind the rank's last piece the weights are zero)
 #pragma unroll
     for (int k = 0; k < SS_W; k++) dot(w[k], k < pieces ? k : 0);
-    for (int k = SS_W; k < pieces; k++) dot(__ldg(wrow + 4 * k), k);
+    for (int k0 = SS_W; k0 < pieces; k0 += SS_W) {
+#pragma unroll
+        for (int k = 0; k < SS_W; k++) w[k] = k0 + k < pieces ? __ldg(wrow + 4 * (k0 + k)) : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+        for (int k = 0; k < SS_W; k++) dot(w[k], k0 + k < pieces ? k0 + k : 0);
+    }
     float acc[R];
 #pragma unroll
     for (int r = 0; r < R; r++) acc[r] = sum2(sums[r]);
@@ -521,8 +526,6 @@ template <typename TA>
 int32_t run_step(pg_ctx *ctx, const ScanShape &s, const pg_batch *bt, const float *proj, int64_t ldp, const TA *x, int64_t ldx, const float *low, int64_t ldl,
                  float *state, TA *out, int64_t ldo)
 {
-    // (a single wave of CTAs also for many channels)
-    if (s.N <= 16 && bt->rows > 4) return launch_step<1, 8, TA>(ctx, s, bt, proj, ldp, x, ldx, low, ldl, state, out, ldo);
     if (s.N <= 16) return launch_step<1, 4, TA>(ctx, s, bt, proj, ldp, x, ldx, low, ldl, state, out, ldo);
     if (s.N <= 32) return launch_step<2, 4, TA>(ctx, s, bt, proj, ldp, x, ldx, low, ldl, state, out, ldo);
     if (s.N <= 64) return launch_step<4, 2, TA>(ctx, s, bt, proj, ldp, x, ldx, low, ldl, state, out, ldo);
