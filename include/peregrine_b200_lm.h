@@ -6,6 +6,9 @@
  * Conventions (beyond those of peregrine_b200.h)
  *   - A step runs the rows (tokens) of one or more sequences, all rows of a sequence next to each other; pg_batch says
  *     which row is which position of which sequence, and in which slot that sequence keeps its cache or state.
+ *   - A step starts with pg_embed_norm or pg_embed_prenorm (or with a copy), which wait for everything before them.  The
+ *     kernels behind may read the batch's arrays, and what earlier steps left in caches and states, while the kernel in
+ *     front of them still runs.
  *   - Activations that enter a product are [rows, K] in the step's type (PG_F32 or PG_BF16) with K a multiple of 64:
  *     columns behind a matrix's true width are zero in the weights and zero in the activations.
  *   - The residual stream, norms, routers, scores, decays and recurrent states are f32 in both types.
